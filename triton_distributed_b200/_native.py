@@ -16,7 +16,10 @@ _ERR = None
 
 
 def lib_path() -> Path:
-    return Path(__file__).resolve().parent / "_C.so"
+    """The full library, or the decoder subset when only that has been built (``build.ensure``)."""
+    here = Path(__file__).resolve().parent
+    full, decoder = here / "_C.so", here / "_C_decoder.so"
+    return decoder if decoder.exists() and not full.exists() else full
 
 
 def load(required: bool = False):

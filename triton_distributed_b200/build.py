@@ -5,6 +5,9 @@ file by ``g++``; objects land in ``csrc/build/`` and the shared object next to t
 with the source tree.  Nothing is compiled at import time: ``python -m triton_distributed_b200.build``
 (or ``build()`` below) is the only entry point that runs a compiler.
 
+``build("decoder")`` compiles a subset into ``_C_decoder.so``: what a layered decoder needs on one GPU (no collectives, expert
+parallelism, megakernel, fp8 or gated-delta-rule kernels); ``ensure`` builds it when no library is there yet.
+
 Stands in for the reference's CMake + setup.py build of its plugin and ``csrc`` library
 (CMakeLists.txt:183-227, python/setup.py); here there is no compiler plugin to build, only kernels.
 """
@@ -22,12 +25,16 @@ ROOT = Path(__file__).resolve().parent
 CSRC = ROOT / "csrc"
 OBJ = CSRC / "build"
 LIB_NAME = "_C"
+DECODER_LIB_NAME = "_C_decoder"
+# sources outside the decoder subset; what the remaining bindings say about them is compiled out by TDB_DECODER_ONLY
+NOT_DECODER = {"collectives.cu", "ep_a2a.cu", "gdn.cu", "gdn_chunk.cu", "gemm_fp8_sm100.cu", "megakernel.cu", "scheduler.cc",
+               "bind_ep.cc", "bind_mega.cc"}
 
 NVCC_ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
 
 
-def lib_path() -> Path:
-    return ROOT / f"{LIB_NAME}.so"
+def lib_path(subset: str = "full") -> Path:
+    return ROOT / f"{DECODER_LIB_NAME if subset == 'decoder' else LIB_NAME}.so"
 
 
 def _cuda_home() -> str:
@@ -76,14 +83,29 @@ def _compile(cmd, src: Path, obj: Path, verbose: bool):
     return out
 
 
-def build(verbose: bool = False, ptxas_info: bool = False, jobs: int | None = None) -> Path:
-    """Compile every source for sm_100a and link ``_C.so`` in-tree.  Returns its path."""
+def ensure(subset: str = "full") -> Path:
+    """Path of a library with at least ``subset``; compiles when there is none (one process at a time)."""
+    import fcntl
+
+    if lib_path().exists():
+        return lib_path()
     OBJ.mkdir(parents=True, exist_ok=True)
+    with open(OBJ / ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return build(subset=subset)
+
+
+def build(verbose: bool = False, ptxas_info: bool = False, jobs: int | None = None, subset: str = "full") -> Path:
+    """Compile every source (of the subset) for sm_100a and link the library in-tree.  Returns its path."""
+    OBJ.mkdir(parents=True, exist_ok=True)
+    decoder = subset == "decoder"
     cuda = _cuda_home()
     nvcc = f"{cuda}/bin/nvcc"
     inc, torch_lib, defs = _torch_flags()
     common_inc = [f"-I{CSRC / 'include'}", f"-I{cuda}/include"]
     cu, cc = _sources()
+    if decoder:
+        cu, cc = ([s for s in src if s.name not in NOT_DECODER] for src in (cu, cc))
     tasks = []
     for src in cu:
         obj = OBJ / (src.stem + ".cu.o")
@@ -93,10 +115,11 @@ def build(verbose: bool = False, ptxas_info: bool = False, jobs: int | None = No
             cmd.insert(1, "-Xptxas=-v")
         tasks.append((cmd, src, obj))
     for src in cc:
-        obj = OBJ / (src.stem + ".cc.o")
+        bind = src.name.startswith("bind")
+        obj = OBJ / (src.stem + (".decoder" if bind and decoder else "") + ".cc.o")
         cmd = ["g++", "-O2", "-std=c++17", "-fPIC", "-Wall", "-Wno-unused-function", *common_inc]
-        if src.name.startswith("bind"):
-            cmd += inc + defs + ["-fvisibility=hidden"]
+        if bind:
+            cmd += inc + defs + ["-fvisibility=hidden"] + (["-DTDB_DECODER_ONLY"] if decoder else [])
         cmd += ["-c", str(src), "-o", str(obj)]
         tasks.append((cmd, src, obj))
     with ThreadPoolExecutor(max_workers=jobs or os.cpu_count() or 4) as ex:
@@ -104,7 +127,7 @@ def build(verbose: bool = False, ptxas_info: bool = False, jobs: int | None = No
             if verbose or ptxas_info:
                 print(msg, flush=True)
     objs = [str(t[2]) for t in tasks]
-    out = lib_path()
+    out = lib_path(subset)
     newest = max(os.path.getmtime(o) for o in objs)
     if not out.exists() or os.path.getmtime(out) < newest:
         link = ["g++", "-shared", "-o", str(out), *objs, f"-L{torch_lib}", "-ltorch_python", "-ltorch", "-ltorch_cpu",

@@ -48,9 +48,10 @@ struct PrefillParams {
   int causal;
   float scale, softcap;
   int64_t total_q;
+  HeadEpilogue epi;
 };
 
-template <int D>
+template <int D, bool TIED>
 __global__ void __launch_bounds__(kAttnThreads) flash_fwd_kernel(const PrefillParams p) {
   extern __shared__ __align__(16) uint8_t smem[];
   using T = Tiles<D>;
@@ -78,15 +79,15 @@ __global__ void __launch_bounds__(kAttnThreads) flash_fwd_kernel(const PrefillPa
   const int warp_lim = p.causal ? min(kv_len, pos0 + row0 + warp * 16 + 16) : kv_len;
   const int nblk = (kv_end + kBlockN - 1) / kBlockN;
   if (nblk > 0) {
-    load_kv_block<D>(p.kv, b, hkv, 0, kv_end, smem, smem + T::kTileBytes);
+    load_kv_block<D, TIED>(p.kv, b, hkv, 0, kv_end, smem, smem + T::kTileBytes);
     cp_async_commit();
   }
   for (int i = 0; i < nblk; ++i) {
-    uint8_t* sK = smem + (i & 1) * 2 * T::kTileBytes;
-    uint8_t* sV = sK + T::kTileBytes;
+    uint8_t* sK = smem + (i & 1) * stage_bytes<D, TIED>();
+    uint8_t* sV = TIED ? sK : sK + T::kTileBytes;
     if (i + 1 < nblk) {
-      uint8_t* nK = smem + ((i + 1) & 1) * 2 * T::kTileBytes;
-      load_kv_block<D>(p.kv, b, hkv, (i + 1) * kBlockN, kv_end, nK, nK + T::kTileBytes);
+      uint8_t* nK = smem + ((i + 1) & 1) * stage_bytes<D, TIED>();
+      load_kv_block<D, TIED>(p.kv, b, hkv, (i + 1) * kBlockN, kv_end, nK, nK + T::kTileBytes);
       cp_async_commit();
       cp_async_wait<1>();
     } else {
@@ -94,7 +95,9 @@ __global__ void __launch_bounds__(kAttnThreads) flash_fwd_kernel(const PrefillPa
     }
     __syncthreads();
     // skip blocks that are fully masked for this warp's rows
-    if (i * kBlockN < warp_lim) w.template step<8>(sK, sV, i * kBlockN, 0, lim_lo, lim_hi, p.scale, p.softcap);
+    if (i * kBlockN < warp_lim)
+      w.template step<8, TIED>(sK, sV, i * kBlockN, 0, lim_lo, lim_hi, p.scale, p.softcap,
+                               reinterpret_cast<const float*>(sK + T::kTileBytes));
     __syncthreads();
   }
   float inv[2], lse[2];
@@ -105,9 +108,14 @@ __global__ void __launch_bounds__(kAttnThreads) flash_fwd_kernel(const PrefillPa
     const int row = r ? r_hi : r_lo;
     if (row >= q_len) continue;
     __nv_bfloat16* orow = p.out + ((static_cast<int64_t>(q_begin) + row) * p.Hq + head) * D;
+    const float f = inv[r] * p.epi.sink_factor(head, lse[r]);
+    const __nv_bfloat16* grow = p.epi.gate_row(static_cast<int64_t>(q_begin) + row, head, D);
 #pragma unroll
-    for (int jd = 0; jd < D / 8; ++jd)
-      *reinterpret_cast<uint32_t*>(orow + 8 * jd + c) = pack_bf16x2(w.o[jd][2 * r] * inv[r], w.o[jd][2 * r + 1] * inv[r]);
+    for (int jd = 0; jd < D / 8; ++jd) {
+      const float2 gt = gate2(grow, 8 * jd + c);
+      *reinterpret_cast<uint32_t*>(orow + 8 * jd + c) =
+          pack_bf16x2(w.o[jd][2 * r] * f * gt.x, w.o[jd][2 * r + 1] * f * gt.y);
+    }
     if (p.lse && (lane & 3) == 0) p.lse[static_cast<int64_t>(head) * p.total_q + q_begin + row] = lse[r];
   }
 }
@@ -194,20 +202,24 @@ __device__ void merge_chunk(const DecodeParams& p, uint8_t* smem, Emit emit) {
   }
 }
 
-template <int D, int S>
+template <int D, int S, bool TIED = false>
 __global__ void __launch_bounds__(kAttnThreads) decode_splitkv_kernel(const DecodeParams p) {
   extern __shared__ __align__(16) uint8_t smem[];
   pdl_wait();   // q and the cache rows of the new token come from the previous kernel
   auto sync = [] { __syncthreads(); };
-  decode_splitkv_body<D, decltype(sync), S>(p, blockIdx.x, blockIdx.y, blockIdx.z, smem, sync);
+  decode_splitkv_body<D, decltype(sync), S, TIED>(p, blockIdx.x, blockIdx.y, blockIdx.z, smem, sync);
   if (p.fuse_counters == nullptr) return;
   // ---- fused combine
   pdl_launch_dependents();
   if (!splits_arrive_last(p)) return;
-  merge_chunk<D>(p, smem, [&](int, int64_t bh, int dv, float4 o, float) {
+  merge_chunk<D>(p, smem, [&](int, int64_t bh, int dv, float4 o, float lse) {
+    const int b = blockIdx.z, head = static_cast<int>(bh - static_cast<int64_t>(b) * p.Hq);
+    const float f = p.epi.sink_factor(head, lse);
+    const __nv_bfloat16* grow = p.epi.gate_row(b, head, D);
+    const float2 g0 = gate2(grow, dv * 4), g1 = gate2(grow, dv * 4 + 2);
     uint2 r;
-    r.x = pack_bf16x2(o.x, o.y);
-    r.y = pack_bf16x2(o.z, o.w);
+    r.x = pack_bf16x2(o.x * f * g0.x, o.y * f * g0.y);
+    r.y = pack_bf16x2(o.z * f * g1.x, o.w * f * g1.y);
     *reinterpret_cast<uint2*>(p.fuse_out + bh * D + dv * 4) = r;
   });
 }
@@ -486,13 +498,21 @@ PagedKV make_kv(const AttnKV& kv) {
   r.max_pages = kv.max_pages;
   r.page_size = kv.page_size;
   r.Hkv = kv.num_kv_heads;
+  r.k_scale = kv.k_scale;
+  return r;
+}
+HeadEpilogue make_epi(const AttnEpilogue& e) {
+  HeadEpilogue r;
+  r.sink = e.sink;
+  r.gate = reinterpret_cast<const __nv_bfloat16*>(e.gate);
+  r.ld_gate = e.ld_gate;
   return r;
 }
 
 }  // namespace
 
 cudaError_t launch_flash_fwd(const FlashFwdArgs& a, cudaStream_t stream) {
-  if (a.head_dim != 64 && a.head_dim != 128) return cudaErrorInvalidValue;
+  const bool tied = a.kv.k_scale != nullptr;
   if (a.num_q_heads % a.kv.num_kv_heads != 0) return cudaErrorInvalidValue;
   PrefillParams p;
   p.q = reinterpret_cast<const __nv_bfloat16*>(a.q);
@@ -509,19 +529,29 @@ cudaError_t launch_flash_fwd(const FlashFwdArgs& a, cudaStream_t stream) {
   p.softcap = a.softcap;
   p.total_q = a.total_q;
   if (a.batch == 0 || a.max_q_len == 0) return cudaSuccess;
+  p.epi = make_epi(a.epi);
   dim3 grid((a.max_q_len + 63) / 64, a.num_q_heads, a.batch);
-  if (a.head_dim == 128) {
-    static SmemOptIn set;
-    cudaError_t e = ensure_smem(flash_fwd_kernel<128>, Tiles<128>::kSmem, &set);
+  auto launch = [&](auto kernel, int smem, SmemOptIn* set) -> cudaError_t {
+    cudaError_t e = ensure_smem(kernel, smem, set);
     if (e != cudaSuccess) return e;
-    flash_fwd_kernel<128><<<grid, kAttnThreads, Tiles<128>::kSmem, stream>>>(p);
-  } else {
-    static SmemOptIn set;
-    cudaError_t e = ensure_smem(flash_fwd_kernel<64>, Tiles<64>::kSmem, &set);
-    if (e != cudaSuccess) return e;
-    flash_fwd_kernel<64><<<grid, kAttnThreads, Tiles<64>::kSmem, stream>>>(p);
+    kernel<<<grid, kAttnThreads, smem, stream>>>(p);
+    return cudaGetLastError();
+  };
+  static SmemOptIn s128, s64, t32, t64, t128, t256;
+  if (tied) {
+    switch (a.head_dim) {
+      case 32: return launch(flash_fwd_kernel<32, true>, 2 * Tiles<32>::kTiedStage, &t32);
+      case 64: return launch(flash_fwd_kernel<64, true>, 2 * Tiles<64>::kTiedStage, &t64);
+      case 128: return launch(flash_fwd_kernel<128, true>, 2 * Tiles<128>::kTiedStage, &t128);
+      case 256: return launch(flash_fwd_kernel<256, true>, 2 * Tiles<256>::kTiedStage, &t256);
+      default: return cudaErrorInvalidValue;
+    }
   }
-  return cudaGetLastError();
+  switch (a.head_dim) {
+    case 64: return launch(flash_fwd_kernel<64, false>, Tiles<64>::kSmem, &s64);
+    case 128: return launch(flash_fwd_kernel<128, false>, Tiles<128>::kSmem, &s128);
+    default: return cudaErrorInvalidValue;
+  }
 }
 
 int decode_workspace_floats(int batch, int num_q_heads, int head_dim, int splits) {
@@ -531,8 +561,12 @@ int decode_workspace_floats(int batch, int num_q_heads, int head_dim, int splits
 namespace {
 // Shared by the local and the one-launch distributed form.  `tail` == nullptr: local.
 cudaError_t launch_splitkv_impl(const DecodeArgs& a, const DistTail* tail, cudaStream_t stream) {
-  if (a.head_dim != 64 && a.head_dim != 128) return cudaErrorInvalidValue;
+  const bool tied = a.kv.k_scale != nullptr;
+  if (!tied && a.head_dim != 64 && a.head_dim != 128) return cudaErrorInvalidValue;
   if (a.num_q_heads % a.kv.num_kv_heads != 0 || a.splits < 1) return cudaErrorInvalidValue;
+  // the epilogue belongs to the fused combine; the distributed tail has neither it nor the tied form
+  const bool plain = !tied && a.epi.sink == nullptr && a.epi.gate == nullptr && a.chunk == 0;
+  if (!plain && (tail != nullptr || a.fuse_counters == nullptr || a.fuse_out == nullptr)) return cudaErrorInvalidValue;
   if (a.batch == 0) return cudaSuccess;
   DecodeParams p;
   p.q = reinterpret_cast<const __nv_bfloat16*>(a.q);
@@ -548,6 +582,8 @@ cudaError_t launch_splitkv_impl(const DecodeArgs& a, const DistTail* tail, cudaS
   p.softcap = a.softcap;
   p.fuse_counters = (a.fuse_counters != nullptr && a.fuse_out != nullptr) ? a.fuse_counters : nullptr;
   p.fuse_out = reinterpret_cast<__nv_bfloat16*>(a.fuse_out);
+  p.epi = make_epi(a.epi);
+  p.chunk = a.chunk;
   dim3 grid(a.splits, a.kv.num_kv_heads * p.head_chunks, a.batch);
   // A grid of at most one CTA per SM is latency-bound: four stages (three blocks in flight per CTA) instead of two.
   int dev = 0, sms = 0;
@@ -575,6 +611,25 @@ cudaError_t launch_splitkv_impl(const DecodeArgs& a, const DistTail* tail, cudaS
     if (e != cudaSuccess) return e;
     return launch_pdl(kernel, grid, dim3(kAttnThreads), static_cast<size_t>(smem), stream, p);
   };
+  if (tied) {
+    // the tied stage is half as large, so the deep pipeline fits for every head dim
+    static SmemOptIn t32_2, t32_4, t64_2, t64_4, t128_2, t128_4, t256_2, t256_4;
+    switch (a.head_dim) {
+      case 32:
+        return deep ? launch(decode_splitkv_kernel<32, 4, true>, 4 * Tiles<32>::kTiedStage, &t32_4)
+                    : launch(decode_splitkv_kernel<32, 2, true>, 2 * Tiles<32>::kTiedStage, &t32_2);
+      case 64:
+        return deep ? launch(decode_splitkv_kernel<64, 4, true>, 4 * Tiles<64>::kTiedStage, &t64_4)
+                    : launch(decode_splitkv_kernel<64, 2, true>, 2 * Tiles<64>::kTiedStage, &t64_2);
+      case 128:
+        return deep ? launch(decode_splitkv_kernel<128, 4, true>, 4 * Tiles<128>::kTiedStage, &t128_4)
+                    : launch(decode_splitkv_kernel<128, 2, true>, 2 * Tiles<128>::kTiedStage, &t128_2);
+      case 256:
+        return deep ? launch(decode_splitkv_kernel<256, 4, true>, 4 * Tiles<256>::kTiedStage, &t256_4)
+                    : launch(decode_splitkv_kernel<256, 2, true>, 2 * Tiles<256>::kTiedStage, &t256_2);
+      default: return cudaErrorInvalidValue;
+    }
+  }
   static SmemOptIn set128_2, set128_4, set64_2, set64_4;
   if (a.head_dim == 128) {
     return deep ? launch(decode_splitkv_kernel<128, 4>, 2 * Tiles<128>::kSmem, &set128_4)

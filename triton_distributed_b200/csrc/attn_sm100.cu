@@ -74,6 +74,7 @@ struct FwdParams {
   float scale_log2;            // scale * log2(e)
   int64_t total_q;
   int* error_flag;             // device int, set on a timeout
+  AttnEpilogue epi;            // sink / output gate of the rows
 };
 
 // ------------------------------------------------------------------------------------------------------------------
@@ -87,8 +88,10 @@ struct PackParams {
   int max_pages, page_size, Hkv, Lp;
   __nv_bfloat16* k_out;        // [B * Hkv][Lp][D]
   __nv_bfloat16* vt_out;       // [B * Hkv][D][Lp]
+  const float* k_scale;        // tied form (see AttnKV): V is the raw key, K the key times its factor
 };
 
+template <bool TIED>
 __global__ void __launch_bounds__(256) attn_pack_kv_kernel(const PackParams p) {
   __shared__ __align__(16) __nv_bfloat16 vs[kBN][kD + 8];
   const int t0 = blockIdx.x * kBN, h = blockIdx.y, b = blockIdx.z;
@@ -102,7 +105,18 @@ __global__ void __launch_bounds__(256) attn_pack_kv_kernel(const PackParams p) {
       const int page = p.block_table[static_cast<int64_t>(b) * p.max_pages + tok / p.page_size];
       const int64_t off = ((static_cast<int64_t>(page) * p.page_size + tok % p.page_size) * p.Hkv + h) * kD + c;
       kv = *reinterpret_cast<const uint4*>(p.k_cache + off);
-      vv = *reinterpret_cast<const uint4*>(p.v_cache + off);
+      if constexpr (TIED) {
+        vv = kv;
+        const float f = p.k_scale[static_cast<int64_t>(page) * p.page_size + tok % p.page_size];
+        uint32_t* w = reinterpret_cast<uint32_t*>(&kv);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float2 x = unpack_bf16x2(w[i]);
+          w[i] = pack_bf16x2(x.x * f, x.y * f);
+        }
+      } else {
+        vv = *reinterpret_cast<const uint4*>(p.v_cache + off);
+      }
     }
     *reinterpret_cast<uint4*>(p.k_out + (bh * p.Lp + tok) * kD + c) = kv;
     *reinterpret_cast<uint4*>(&vs[r][c]) = vv;
@@ -248,8 +262,28 @@ __device__ __forceinline__ void softmax_tile(const FwdParams& p, const TileCtx& 
   }
   if (!ok) *abort_flag = 1;
   if (ok && row_ok) {
-    const float inv = l > 0.f ? 1.f / l : 0.f;
-    __nv_bfloat16* orow = p.out + ((static_cast<int64_t>(q_begin) + row0 + row) * p.Hq + head) * kD;
+    float inv = l > 0.f ? 1.f / l : 0.f;
+    const int64_t tok = static_cast<int64_t>(q_begin) + row0 + row;
+    if (p.epi.sink != nullptr && l > 0.f) {
+      const float lse = (m + log2f(l)) * 0.6931471805599453f;
+      inv /= 1.f + __expf(p.epi.sink[head] - lse);
+    }
+    if (p.epi.gate != nullptr) {
+      const uint4* g4 = reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(p.epi.gate) +
+                                                       tok * p.epi.ld_gate + static_cast<int64_t>(head) * kD);
+#pragma unroll
+      for (int c = 0; c < kD / 8; ++c) {
+        const uint4 u = g4[c];
+        const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 z = unpack_bf16x2(w[e]);
+          o[8 * c + 2 * e] *= 1.f / (1.f + __expf(-z.x));
+          o[8 * c + 2 * e + 1] *= 1.f / (1.f + __expf(-z.y));
+        }
+      }
+    }
+    __nv_bfloat16* orow = p.out + (tok * p.Hq + head) * kD;
 #pragma unroll
     for (int c = 0; c < kD / 8; ++c) {
       uint4 v;
@@ -599,7 +633,12 @@ cudaError_t launch_flash_fwd_sm100(const FlashFwdSm100Args& a, cudaStream_t stre
   pk.Lp = a.Lp;
   pk.k_out = reinterpret_cast<__nv_bfloat16*>(a.k_dense);
   pk.vt_out = reinterpret_cast<__nv_bfloat16*>(a.vt_dense);
-  attn_pack_kv_kernel<<<dim3(a.Lp / kBN, a.num_kv_heads, a.batch), 256, 0, stream>>>(pk);
+  pk.k_scale = a.kv.k_scale;
+  const dim3 pack_grid(a.Lp / kBN, a.num_kv_heads, a.batch);
+  if (pk.k_scale != nullptr)
+    attn_pack_kv_kernel<true><<<pack_grid, 256, 0, stream>>>(pk);
+  else
+    attn_pack_kv_kernel<false><<<pack_grid, 256, 0, stream>>>(pk);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return e;
 
@@ -628,6 +667,9 @@ cudaError_t launch_flash_fwd_sm100(const FlashFwdSm100Args& a, cudaStream_t stre
   p.scale_log2 = a.scale * 1.4426950408889634f;
   p.total_q = a.total_q;
   p.error_flag = a.error_flag;
+  p.epi = a.epi;
+  if (p.epi.gate != nullptr && (p.epi.ld_gate % 8 != 0 || (reinterpret_cast<uintptr_t>(p.epi.gate) & 15u) != 0))
+    return cudaErrorInvalidValue;
   dim3 grid((a.max_q_len + kBM - 1) / kBM, a.num_q_heads, a.batch);
   CUtensorMap mq, mk, mv;
   memcpy(&mq, tq.bytes, sizeof(mq));

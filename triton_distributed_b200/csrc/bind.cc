@@ -284,6 +284,7 @@ void gemm_rs_bf16(SymmHeap& h, const at::Tensor& a, const at::Tensor& b, at::Ten
   check_cuda(tdb::launch_gemm(g, cur_stream()), "launch_gemm(reduce-scatter)");
 }
 
+#ifndef TDB_DECODER_ONLY
 // ------------------------------------------------------------------ block-scaled fp8 GEMM family
 void check_fp8_operands(const at::Tensor& a_q, const at::Tensor& a_s, const at::Tensor& b_q, const at::Tensor& b_s,
                         const char* name) {
@@ -414,6 +415,8 @@ void gemm_rs_fp8(SymmHeap& h, const at::Tensor& a_q, const at::Tensor& a_s, cons
   g.stats = stats_ptr(stats, g.num_ctas);
   check_cuda(tdb::launch_gemm_fp8(g, cur_stream()), "launch_gemm_fp8(reduce-scatter)");
 }
+
+#endif  // TDB_DECODER_ONLY
 
 // Small-M GEMM (decode): out[M,N] = x[M,K] @ w[N,K]^T with split-K; acc / counters are caller-kept scratch.
 void skinny_gemm_bf16(const at::Tensor& x, const at::Tensor& w, at::Tensor& out, at::Tensor& acc, at::Tensor& counters,
@@ -629,6 +632,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm_rs_bf16", &gemm_rs_bf16, py::arg("heap"), py::arg("a"), py::arg("b"), py::arg("out"), py::arg("slots"),
         py::arg("flags"), py::arg("ctx"), py::arg("max_seg_rows"), py::arg("max_tiles"), py::arg("block_n"),
         py::arg("num_ctas"), py::arg("timeout_s"), py::arg("stats") = py::none());
+#ifndef TDB_DECODER_ONLY
   m.def("gemm_fp8", &gemm_fp8, py::arg("a_q"), py::arg("a_s"), py::arg("b_q"), py::arg("b_s"), py::arg("c"),
         py::arg("num_ctas") = 0, py::arg("stats") = py::none());
   m.def("ag_gemm_fp8", &ag_gemm_fp8, py::arg("heap"), py::arg("a_q"), py::arg("a_s"), py::arg("b_q"), py::arg("b_s"),
@@ -637,6 +641,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm_rs_fp8", &gemm_rs_fp8, py::arg("heap"), py::arg("a_q"), py::arg("a_s"), py::arg("b_q"), py::arg("b_s"),
         py::arg("out"), py::arg("slots"), py::arg("flags"), py::arg("ctx"), py::arg("max_seg_rows"), py::arg("max_tiles"),
         py::arg("num_ctas"), py::arg("timeout_s"), py::arg("stats") = py::none());
+#endif
   m.def("gemm_smem_bytes", &tdb::gemm_smem_bytes);
   m.def("skinny_gemm_bf16", &skinny_gemm_bf16, py::arg("x"), py::arg("w"), py::arg("out"), py::arg("acc"),
         py::arg("counters"), py::arg("splits"), py::arg("num_ctas"), py::arg("cluster_nt") = 0, py::arg("cluster_s") = 0,

@@ -34,10 +34,37 @@ void check_i32(const at::Tensor& t, const char* name) {
   TORCH_CHECK(t.is_cuda() && t.scalar_type() == at::kInt && t.is_contiguous(), name, ": contiguous int32 CUDA tensor expected");
 }
 
+// Tied form: k_scale [pages, page_size] fp32 (see tdb::AttnKV).
+void set_k_scale(tdb::AttnKV& kv, const at::Tensor& k_cache, const c10::optional<at::Tensor>& k_scale) {
+  if (!k_scale.has_value()) return;
+  TORCH_CHECK(k_scale->is_cuda() && k_scale->scalar_type() == at::kFloat && k_scale->is_contiguous() &&
+                  k_scale->numel() == k_cache.size(0) * k_cache.size(1), "k_scale: contiguous fp32 [pages, page_size]");
+  kv.k_scale = k_scale->data_ptr<float>();
+}
+
+// Sink [Hq] fp32 and output gate [tokens, Hq * D] (rows may be strided).
+tdb::AttnEpilogue make_epilogue(const at::Tensor& q, const c10::optional<at::Tensor>& sink, const c10::optional<at::Tensor>& gate) {
+  tdb::AttnEpilogue e;
+  if (sink.has_value()) {
+    TORCH_CHECK(sink->is_cuda() && sink->scalar_type() == at::kFloat && sink->is_contiguous() && sink->numel() == q.size(1),
+                "sink: contiguous fp32 [Hq]");
+    e.sink = sink->data_ptr<float>();
+  }
+  if (gate.has_value()) {
+    TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == q.scalar_type() && gate->dim() == 2 && gate->stride(1) == 1 &&
+                    gate->size(0) == q.size(0) && gate->size(1) == q.size(1) * q.size(2) && gate->stride(0) % 2 == 0,
+                "gate: [tokens, Hq * D] of q's dtype, even row stride");
+    e.gate = gate->data_ptr();
+    e.ld_gate = gate->stride(0);
+  }
+  return e;
+}
+
 at::Tensor flash_fwd(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache,
                      const at::Tensor& block_table, const at::Tensor& cu_seqlens_q, const at::Tensor& kv_lens,
                      c10::optional<at::Tensor> q_pos0, int64_t max_q_len, bool causal, double scale, double softcap,
-                     c10::optional<at::Tensor> lse) {
+                     c10::optional<at::Tensor> lse, c10::optional<at::Tensor> k_scale, c10::optional<at::Tensor> sink,
+                     c10::optional<at::Tensor> gate) {
   TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && q.scalar_type() == at::kBFloat16, "q must be contiguous bf16 [T, Hq, D]");
   check_i32(cu_seqlens_q, "cu_seqlens_q");
   check_i32(kv_lens, "kv_lens");
@@ -68,6 +95,8 @@ at::Tensor flash_fwd(const at::Tensor& q, const at::Tensor& k_cache, const at::T
   a.causal = causal ? 1 : 0;
   a.scale = scale;
   a.softcap = softcap;
+  set_k_scale(a.kv, k_cache, k_scale);
+  a.epi = make_epilogue(q, sink, gate);
   TORCH_CHECK(k_cache.size(3) == a.head_dim, "head_dim mismatch between q and the cache");
   check_cuda(tdb::launch_flash_fwd(a, cur_stream()), "launch_flash_fwd");
   return out;
@@ -78,7 +107,8 @@ at::Tensor flash_fwd(const at::Tensor& q, const at::Tensor& k_cache, const at::T
 std::vector<at::Tensor> flash_fwd_sm100(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache,
                                         const at::Tensor& block_table, const at::Tensor& cu_seqlens_q, const at::Tensor& kv_lens,
                                         c10::optional<at::Tensor> q_pos0, int64_t max_q_len, int64_t max_kv_len, bool causal,
-                                        double scale, c10::optional<at::Tensor> lse) {
+                                        double scale, c10::optional<at::Tensor> lse, c10::optional<at::Tensor> k_scale,
+                                        c10::optional<at::Tensor> sink, c10::optional<at::Tensor> gate) {
   TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && q.scalar_type() == at::kBFloat16 && q.size(2) == 128,
               "flash_fwd_sm100: q must be contiguous bf16 [T, Hq, 128]");
   TORCH_CHECK(k_cache.scalar_type() == at::kBFloat16 && v_cache.scalar_type() == at::kBFloat16 && k_cache.is_contiguous() &&
@@ -122,6 +152,8 @@ std::vector<at::Tensor> flash_fwd_sm100(const at::Tensor& q, const at::Tensor& k
   a.k_dense = kd.data_ptr();
   a.vt_dense = vt.data_ptr();
   a.error_flag = err.data_ptr<int32_t>();
+  set_k_scale(a.kv, k_cache, k_scale);
+  a.epi = make_epilogue(q, sink, gate);
   check_cuda(tdb::launch_flash_fwd_sm100(a, cur_stream()), "launch_flash_fwd_sm100");
   return {out, err};
 }
@@ -153,9 +185,13 @@ tdb::DecodeArgs decode_args(const at::Tensor& q, const at::Tensor& k_cache, cons
 void decode_attn(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache, const at::Tensor& block_table,
                  const at::Tensor& kv_lens, at::Tensor& workspace, int64_t splits, double scale, double softcap,
                  c10::optional<at::Tensor> out, c10::optional<at::Tensor> out_lse, c10::optional<at::Tensor> out_f32,
-                 c10::optional<at::Tensor> counters) {
+                 c10::optional<at::Tensor> counters, c10::optional<at::Tensor> k_scale, c10::optional<at::Tensor> sink,
+                 c10::optional<at::Tensor> gate, int64_t chunk) {
   c10::cuda::CUDAGuard guard(q.device());
   tdb::DecodeArgs a = decode_args(q, k_cache, v_cache, block_table, kv_lens, workspace, splits, scale, softcap);
+  set_k_scale(a.kv, k_cache, k_scale);
+  a.epi = make_epilogue(q, sink, gate);
+  a.chunk = static_cast<int>(chunk);
   if (counters.has_value() && out.has_value() && !out_lse.has_value() && !out_f32.has_value()) {
     // one launch: the last split CTA of every (sequence, KV head) merges the partials
     const int64_t group = a.num_q_heads / k_cache.size(2);
@@ -209,12 +245,54 @@ int64_t dist_decode_attn(SymmHeap& h, const at::Tensor& q, const at::Tensor& k_c
   return 2;
 }
 
+// Attention of every token over rows [row0, row0 + n_keys) of a tied cache, fp32 arithmetic (fp32 or bf16 tensors).
+at::Tensor tied_attn_simple(const at::Tensor& q, const at::Tensor& k, const at::Tensor& k_scale, const at::Tensor& row0,
+                            const at::Tensor& n_keys, c10::optional<at::Tensor> sink, c10::optional<at::Tensor> gate) {
+  TORCH_CHECK(q.is_cuda() && q.dim() == 3 && q.is_contiguous() && (q.scalar_type() == at::kFloat || q.scalar_type() == at::kBFloat16),
+              "tied_attn_simple: contiguous q [T, Hq, D], fp32 or bf16");
+  TORCH_CHECK(k.dim() >= 3 && k.is_contiguous() && k.scalar_type() == q.scalar_type() && k.size(-1) == q.size(2),
+              "tied_attn_simple: contiguous k [..., Hkv, D] of q's dtype");
+  TORCH_CHECK(k_scale.scalar_type() == at::kFloat && k_scale.is_contiguous() &&
+                  k_scale.numel() * k.size(-1) * k.size(-2) == k.numel(), "tied_attn_simple: fp32 k_scale, one per row of k");
+  TORCH_CHECK(row0.is_cuda() && row0.scalar_type() == at::kLong && row0.is_contiguous() && row0.numel() == q.size(0),
+              "tied_attn_simple: int64 row0 [T]");
+  check_i32(n_keys, "n_keys");
+  TORCH_CHECK(n_keys.numel() == q.size(0), "tied_attn_simple: n_keys [T]");
+  c10::cuda::CUDAGuard guard(q.device());
+  at::Tensor out = at::empty_like(q);
+  tdb::TiedSimpleArgs a;
+  a.q = q.data_ptr();
+  a.k = k.data_ptr();
+  a.k_scale = k_scale.data_ptr<float>();
+  a.row0 = row0.data_ptr<int64_t>();
+  a.n_keys = n_keys.data_ptr<int32_t>();
+  a.out = out.data_ptr();
+  a.T = q.size(0);
+  a.Hq = q.size(1);
+  a.Hkv = k.size(-2);
+  a.D = q.size(2);
+  a.is_f32 = q.scalar_type() == at::kFloat;
+  a.epi = make_epilogue(q, sink, gate);
+  check_cuda(tdb::launch_tied_attn_simple(a, cur_stream()), "launch_tied_attn_simple");
+  return out;
+}
+
 }  // namespace
 
 void bind_attn(py::module_& m) {
-  m.def("flash_fwd", &flash_fwd);
-  m.def("flash_fwd_sm100", &flash_fwd_sm100);
-  m.def("decode_attn", &decode_attn);
+  m.def("flash_fwd", &flash_fwd, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_table"),
+        py::arg("cu_seqlens_q"), py::arg("kv_lens"), py::arg("q_pos0"), py::arg("max_q_len"), py::arg("causal"),
+        py::arg("scale"), py::arg("softcap"), py::arg("lse"), py::arg("k_scale") = py::none(), py::arg("sink") = py::none(),
+        py::arg("gate") = py::none());
+  m.def("flash_fwd_sm100", &flash_fwd_sm100, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_table"),
+        py::arg("cu_seqlens_q"), py::arg("kv_lens"), py::arg("q_pos0"), py::arg("max_q_len"), py::arg("max_kv_len"),
+        py::arg("causal"), py::arg("scale"), py::arg("lse"), py::arg("k_scale") = py::none(), py::arg("sink") = py::none(),
+        py::arg("gate") = py::none());
+  m.def("decode_attn", &decode_attn, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_table"),
+        py::arg("kv_lens"), py::arg("workspace"), py::arg("splits"), py::arg("scale"), py::arg("softcap"), py::arg("out"),
+        py::arg("out_lse"), py::arg("out_f32"), py::arg("counters"), py::arg("k_scale") = py::none(),
+        py::arg("sink") = py::none(), py::arg("gate") = py::none(), py::arg("chunk") = 0);
+  m.def("tied_attn_simple", &tied_attn_simple);
   m.def("dist_decode_attn", &dist_decode_attn, py::arg("heap"), py::arg("q"), py::arg("k_cache"), py::arg("v_cache"),
         py::arg("block_table"), py::arg("kv_lens"), py::arg("workspace"), py::arg("splits"), py::arg("scale"),
         py::arg("softcap"), py::arg("out"), py::arg("staging"), py::arg("ctx"), py::arg("timeout_s"),

@@ -29,6 +29,7 @@ tdb::DType to_dtype(at::ScalarType t) {
   }
 }
 
+#ifndef TDB_DECODER_ONLY
 uint64_t ns(double seconds) { return static_cast<uint64_t>(seconds * 1e9); }
 
 void all_reduce(SymmHeap& h, const at::Tensor& in, at::Tensor& out, at::Tensor& ws, at::Tensor& flags, at::Tensor& ctx,
@@ -124,6 +125,8 @@ void p2p_copy(at::Tensor& dst, const at::Tensor& src, int64_t num_ctas, int64_t 
   TORCH_CHECK(static_cast<uint64_t>(dst.numel()) * dst.element_size() >= bytes, "p2p_copy: destination too small");
   check_cuda(tdb::launch_p2p_copy(dst.data_ptr(), src.data_ptr(), bytes, num_ctas, mode, cur_stream()), "launch_p2p_copy");
 }
+
+#endif  // TDB_DECODER_ONLY
 
 // ------------------------------------------------------------------ elementwise
 void check_bf16(const at::Tensor& t, const char* name) {
@@ -237,6 +240,7 @@ void abs_sum(const at::Tensor& x, at::Tensor& out) {
   check_cuda(tdb::launch_abs_sum(x.data_ptr(), x.numel(), out.data_ptr<float>(), cur_stream()), "launch_abs_sum");
 }
 
+#ifndef TDB_DECODER_ONLY
 // Gated delta rule forward (variable length).  q, k [T, H, 128]; v [T, H, V]; g fp32 [T, H]; beta [T, H];
 // cu_seqlens int32 [N + 1] on the device.  Returns (o [T, H, V] bf16, final_state fp32 [N, H, K, V] or an empty tensor).
 std::tuple<at::Tensor, at::Tensor> gdn_fwd(const at::Tensor& q, const at::Tensor& k, const at::Tensor& v, const at::Tensor& g,
@@ -326,6 +330,7 @@ std::vector<at::Tensor> gdn_chunk_fwd(const at::Tensor& q, const at::Tensor& k, 
   return {o, gc, A, ht};
 }
 
+#endif  // TDB_DECODER_ONLY
 }  // namespace
 
 
@@ -333,10 +338,13 @@ void bind_attn(py::module_& m);
 void bind_moe(py::module_& m);
 void bind_ep(py::module_& m);
 void bind_mega(py::module_& m);
+void bind_hybrid(py::module_& m);
 
 void bind_more(py::module_& m) {
   bind_attn(m);
   bind_moe(m);
+  bind_hybrid(m);
+#ifndef TDB_DECODER_ONLY
   bind_ep(m);
   bind_mega(m);
   m.def("all_reduce", &all_reduce);
@@ -348,6 +356,9 @@ void bind_more(py::module_& m) {
         py::arg("cmp") = 1);
   m.def("bounds_probe", &bounds_probe);
   m.def("p2p_copy", &p2p_copy);
+  m.def("gdn_fwd", &gdn_fwd);
+  m.def("gdn_chunk_fwd", &gdn_chunk_fwd);
+#endif
   m.def("rmsnorm", &rmsnorm, py::arg("x"), py::arg("w"), py::arg("eps"), py::arg("residual") = py::none());
   m.def("silu_mul", &silu_mul);
   m.def("add", &add);
@@ -355,6 +366,4 @@ void bind_more(py::module_& m) {
   m.def("embedding", &embedding);
   m.def("argmax", &argmax);
   m.def("abs_sum", &abs_sum);
-  m.def("gdn_fwd", &gdn_fwd);
-  m.def("gdn_chunk_fwd", &gdn_chunk_fwd);
 }

@@ -13,6 +13,18 @@ struct AttnKV {
   int max_pages;
   int page_size;
   int num_kv_heads;
+  // Tied form: the values are the raw (un-normed) keys.  k_cache holds them, v_cache is unused, and k_scale
+  // [num_pages, page_size] fp32 is the factor of a token's score (the reciprocal root mean square of its key row; the
+  // norm's weight is folded into q).
+  const float* k_scale = nullptr;
+};
+
+// Applied to every output row after the softmax (all kernels with `epi`): sink adds exp(sink[head]) to the denominator,
+// gate multiplies by sigmoid(gate[token, head * head_dim + d]).
+struct AttnEpilogue {
+  const float* sink = nullptr;    // [Hq]
+  const void* gate = nullptr;     // bf16, row stride ld_gate elements
+  int64_t ld_gate = 0;
 };
 
 struct FlashFwdArgs {
@@ -27,6 +39,7 @@ struct FlashFwdArgs {
   int64_t total_q;
   int causal;
   float scale, softcap;
+  AttnEpilogue epi;
 };
 cudaError_t launch_flash_fwd(const FlashFwdArgs& a, cudaStream_t stream);
 
@@ -50,6 +63,7 @@ struct FlashFwdSm100Args {
   void* k_dense;
   void* vt_dense;
   int* error_flag;
+  AttnEpilogue epi;
 };
 cudaError_t launch_flash_fwd_sm100(const FlashFwdSm100Args& a, cudaStream_t stream);
 
@@ -64,7 +78,26 @@ struct DecodeArgs {
   // partials of its query heads into fuse_out (bf16 [batch, Hq, D]) and no combine launch is needed.
   uint32_t* fuse_counters = nullptr;   // [batch * Hkv * head_chunks], zero between calls (the kernel leaves them zero)
   void* fuse_out = nullptr;
+  AttnEpilogue epi;                    // needs the fused combine
+  int chunk = 0;                       // > 0: block-local attention, see DecodeParams
 };
+
+// Attention in plain fp32 arithmetic over the tied form, for any head dim up to 512 and fp32 or bf16 tensors: one warp
+// per (token, head).  Token t sees the rows [row0[t], row0[t] + n_keys[t]) of k (viewed as [rows, Hkv, D]).
+struct TiedSimpleArgs {
+  const void* q;               // [T, Hq, D]
+  const void* k;               // [rows, Hkv, D]
+  const float* k_scale;        // [rows]
+  const int64_t* row0;         // [T]
+  const int32_t* n_keys;       // [T]
+  void* out;                   // [T, Hq, D]
+  int64_t T;
+  int Hq, Hkv, D;
+  int is_f32;                  // dtype of q / k / gate / out
+  AttnEpilogue epi;
+};
+cudaError_t launch_tied_attn_simple(const TiedSimpleArgs& a, cudaStream_t stream);
+
 int decode_workspace_floats(int batch, int num_q_heads, int head_dim, int splits);
 cudaError_t launch_decode_splitkv(const DecodeArgs& a, cudaStream_t stream);
 // out_bf16 [B,Hq,D] and/or out_lse [B,Hq] and/or out_f32 [B,Hq,D+1] (out || LSE); any may be null.

@@ -37,7 +37,13 @@ struct Tiles {
   static constexpr int kPitch = D * 2 + 16;        // bytes per token row in shared memory (conflict-free)
   static constexpr int kTileBytes = kBlockN * kPitch;
   static constexpr int kSmem = 4 * kTileBytes;     // K and V, double buffered
+  // Tied form (the value of a token is its raw key): one tile per stage serves both products, followed by the 64
+  // per-token score factors.
+  static constexpr int kTiedStage = kTileBytes + kBlockN * 4;
 };
+// Bytes of one pipeline stage, and where its V tile lives.
+template <int D, bool TIED>
+TDB_DEVICE constexpr int stage_bytes() { return TIED ? Tiles<D>::kTiedStage : 2 * Tiles<D>::kTileBytes; }
 
 // Physical address of token `tok` of sequence `b`, KV head `h` in a paged cache [pages, page_size, Hkv, D].
 struct PagedKV {
@@ -47,14 +53,38 @@ struct PagedKV {
   int max_pages;
   int page_size;
   int Hkv;
-  TDB_DEVICE int64_t token_offset(int b, int tok, int h, int D) const {
+  // Tied form: v is unused, k holds the keys as projected, and k_scale [pages, page_size] the factor that turns a score
+  // against the raw key into the score against the normed one (the norm's weight is folded into the query).
+  const float* k_scale = nullptr;
+  TDB_DEVICE int64_t token_row(int b, int tok) const {
     const int page = block_table[static_cast<int64_t>(b) * max_pages + tok / page_size];
-    return ((static_cast<int64_t>(page) * page_size + tok % page_size) * Hkv + h) * D;
+    return static_cast<int64_t>(page) * page_size + tok % page_size;
   }
+  TDB_DEVICE int64_t token_offset(int b, int tok, int h, int D) const { return (token_row(b, tok) * Hkv + h) * D; }
 };
 
+// What happens to a head's output row after the softmax: a sink (one more term exp(sink) in the denominator, without a
+// value) and an output gate (multiply by sigmoid(gate) element by element).  Either may be absent.
+struct HeadEpilogue {
+  const float* sink = nullptr;             // [Hq]
+  const __nv_bfloat16* gate = nullptr;     // [tokens, ld_gate], head h at columns [h * D, (h + 1) * D)
+  int64_t ld_gate = 0;
+  // Factor of a row whose softmax over the keys alone has the log-sum-exp `lse`.
+  TDB_DEVICE float sink_factor(int head, float lse) const {
+    return sink == nullptr ? 1.f : 1.f / (1.f + __expf(sink[head] - lse));
+  }
+  TDB_DEVICE const __nv_bfloat16* gate_row(int64_t token, int head, int D) const {
+    return gate == nullptr ? nullptr : gate + token * ld_gate + static_cast<int64_t>(head) * D;
+  }
+};
+TDB_DEVICE float2 gate2(const __nv_bfloat16* row, int d) {
+  if (row == nullptr) return make_float2(1.f, 1.f);
+  const float2 z = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(row + d));
+  return make_float2(1.f / (1.f + __expf(-z.x)), 1.f / (1.f + __expf(-z.y)));
+}
+
 // Cooperative load of one 64-token K and V block (tokens [t0, t0+64) of the sequence) into shared memory.
-template <int D>
+template <int D, bool TIED = false>
 TDB_DEVICE void load_kv_block(const PagedKV& kv, int b, int h, int t0, int kv_end, uint8_t* sK, uint8_t* sV) {
   constexpr int kChunksPerRow = D / 8;
   constexpr int kPitch = Tiles<D>::kPitch;
@@ -64,7 +94,12 @@ TDB_DEVICE void load_kv_block(const PagedKV& kv, int b, int h, int t0, int kv_en
     const bool valid = tok < kv_end;
     const int64_t off = valid ? kv.token_offset(b, tok, h, D) + ch * 8 : 0;
     cp_async16(sK + r * kPitch + ch * 16, kv.k + off, valid);
-    cp_async16(sV + r * kPitch + ch * 16, kv.v + off, valid);
+    if constexpr (!TIED) cp_async16(sV + r * kPitch + ch * 16, kv.v + off, valid);
+  }
+  if constexpr (TIED) {   // plain stores: visible to the CTA after the barrier that publishes the block
+    float* sc = reinterpret_cast<float*>(sK + Tiles<D>::kTileBytes);
+    for (int r = threadIdx.x; r < kBlockN; r += kAttnThreads)
+      sc[r] = t0 + r < kv_end ? kv.k_scale[kv.token_row(b, t0 + r)] : 0.f;
   }
 }
 
@@ -95,10 +130,11 @@ struct WarpTile {
     }
   }
   // One step over NT 8-token tiles that start at row `tok_in_block` of the shared-memory block whose first token
-  // is global token `t0`.  Scores of tokens >= limit_lo / limit_hi (per row) are masked.
-  template <int NT>
+  // is global token `t0`.  Scores of tokens >= limit_lo / limit_hi (per row) are masked.  tok_scale (TIED): the block's
+  // per-token score factors.
+  template <int NT, bool TIED = false>
   TDB_DEVICE void step(const uint8_t* sK, const uint8_t* sV, int t0, int tok_in_block, int limit_lo, int limit_hi,
-                       float scale, float softcap) {
+                       float scale, float softcap, const float* tok_scale = nullptr) {
     constexpr int kPitch = Tiles<D>::kPitch;
     const int lane = lane_id();
     const int g = lane >> 2, c = 2 * (lane & 3);
@@ -122,6 +158,7 @@ struct WarpTile {
       for (int e = 0; e < 4; ++e) {
         const int tok = t0 + tok_in_block + 8 * j + c + (e & 1);
         float v = s[j][e] * scale;
+        if constexpr (TIED) v *= tok_scale[tok_in_block + 8 * j + c + (e & 1)];
         if (softcap > 0.f) v = softcap * tanhf(v / softcap);
         v *= kLog2e;
         const int lim = (e < 2) ? limit_lo : limit_hi;
@@ -203,16 +240,24 @@ struct DecodeParams {
   float scale, softcap;
   uint32_t* fuse_counters = nullptr;    // fused combine (see DecodeArgs); null = partials only
   __nv_bfloat16* fuse_out = nullptr;
+  HeadEpilogue epi;                     // applied by the fused combine
+  int chunk = 0;                        // > 0: the query sees only its own block of `chunk` positions, which the cache row
+                                        // position % chunk of its page holds (kv_lens stays the sequence length)
 };
+// Number of cached tokens the query at the end of a sequence of kv_len tokens sees.
+TDB_DEVICE int decode_kv_len(const DecodeParams& p, int b) {
+  const int n = p.kv_lens[b];
+  return p.chunk > 0 && n > 0 ? (n - 1) % p.chunk + 1 : n;
+}
 
 // Body of the split-KV decode step for one (split, kv head x head chunk, sequence).  Executed by 128 threads
 // (threadIdx.x < 128); `sync` is a barrier over exactly those threads.
 // S = shared-memory stages of (K, V) blocks: S - 1 blocks are in flight while one is computed.
-template <int D, typename Sync, int S = 2>
+template <int D, typename Sync, int S = 2, bool TIED = false>
 TDB_DEVICE void decode_splitkv_body(const DecodeParams& p, int split, int yidx, int b, uint8_t* smem, Sync sync) {
   using T = Tiles<D>;
   const int hkv = yidx / p.head_chunks, hc = yidx - hkv * p.head_chunks;
-  const int kv_len = p.kv_lens[b];
+  const int kv_len = decode_kv_len(p, b);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2;
   // split boundaries in units of 64-token blocks
@@ -233,23 +278,24 @@ TDB_DEVICE void decode_splitkv_body(const DecodeParams& p, int split, int yidx, 
 #pragma unroll
   for (int j = 0; j < S - 1; ++j) {
     if (j < nblk) {
-      uint8_t* nK = smem + j * 2 * T::kTileBytes;
-      load_kv_block<D>(p.kv, b, hkv, (blk0 + j) * kBlockN, kv_len, nK, nK + T::kTileBytes);
+      uint8_t* nK = smem + j * stage_bytes<D, TIED>();
+      load_kv_block<D, TIED>(p.kv, b, hkv, (blk0 + j) * kBlockN, kv_len, nK, nK + T::kTileBytes);
     }
     cp_async_commit();
   }
   for (int i = 0; i < nblk; ++i) {
-    uint8_t* sK = smem + (i % S) * 2 * T::kTileBytes;
-    uint8_t* sV = sK + T::kTileBytes;
+    uint8_t* sK = smem + (i % S) * stage_bytes<D, TIED>();
+    uint8_t* sV = TIED ? sK : sK + T::kTileBytes;
     if (i + S - 1 < nblk) {
-      uint8_t* nK = smem + ((i + S - 1) % S) * 2 * T::kTileBytes;
-      load_kv_block<D>(p.kv, b, hkv, (blk0 + i + S - 1) * kBlockN, kv_len, nK, nK + T::kTileBytes);
+      uint8_t* nK = smem + ((i + S - 1) % S) * stage_bytes<D, TIED>();
+      load_kv_block<D, TIED>(p.kv, b, hkv, (blk0 + i + S - 1) * kBlockN, kv_len, nK, nK + T::kTileBytes);
     }
     cp_async_commit();
     cp_async_wait<S - 1>();
     sync();
     // each warp takes 16 of the block's 64 tokens
-    w.template step<2>(sK, sV, (blk0 + i) * kBlockN, warp * 16, kv_len, kv_len, p.scale, p.softcap);
+    w.template step<2, TIED>(sK, sV, (blk0 + i) * kBlockN, warp * 16, kv_len, kv_len, p.scale, p.softcap,
+                             reinterpret_cast<const float*>(sK + T::kTileBytes));
     sync();
   }
   // merge the 4 warps (different token subsets, same rows) through shared memory

@@ -1,0 +1,50 @@
+// Eight-element vector access to bf16 or fp32 rows as fp32 values, for kernels templated on the activation type.
+#pragma once
+#include "ptx.cuh"
+
+namespace tdb {
+
+TDB_DEVICE void load8(const __nv_bfloat16* p, float (&f)[8]) {
+  const uint4 v = *reinterpret_cast<const uint4*>(p);
+  const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y), c = unpack_bf16x2(v.z), d = unpack_bf16x2(v.w);
+  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y; f[4] = c.x; f[5] = c.y; f[6] = d.x; f[7] = d.y;
+}
+TDB_DEVICE void load8(const float* p, float (&f)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+TDB_DEVICE void store8(__nv_bfloat16* p, const float (&f)[8]) {
+  uint4 o;
+  o.x = pack_bf16x2(f[0], f[1]); o.y = pack_bf16x2(f[2], f[3]);
+  o.z = pack_bf16x2(f[4], f[5]); o.w = pack_bf16x2(f[6], f[7]);
+  *reinterpret_cast<uint4*>(p) = o;
+}
+TDB_DEVICE void store8(float* p, const float (&f)[8]) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(f[0], f[1], f[2], f[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
+}
+TDB_DEVICE float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+TDB_DEVICE float to_f32(float v) { return v; }
+template <typename T>
+TDB_DEVICE T from_f32(float v);
+template <>
+TDB_DEVICE __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+template <>
+TDB_DEVICE float from_f32<float>(float v) { return v; }
+
+// Sum over the block; `red` holds 32 floats.  Every thread gets the result.
+TDB_DEVICE float block_reduce_sum(float v, float* red) {
+  v = warp_sum(v);
+  const int w = threadIdx.x >> 5, l = threadIdx.x & 31;
+  if (l == 0) red[w] = v;
+  __syncthreads();
+  const int nw = (blockDim.x + 31) >> 5;
+  float t = 0.f;
+  for (int i = 0; i < nw; ++i) t += red[i];
+  __syncthreads();
+  return t;
+}
+
+TDB_DEVICE float sigmoid_f32(float z) { return 1.f / (1.f + expf(-z)); }
+
+}  // namespace tdb

@@ -1,0 +1,182 @@
+// Experts of the form y = W_down relu(W_up (w h))^2 with a per-(token, expert) input weight w, without gate projection.
+// The up projection has no bias, so the weight can scale its OUTPUT: relu2 takes it on the way.
+//
+//   relu2_kernel        (relu(w * in))^2 over rows, between the two grouped GEMMs of a prefill
+//   expert_up_kernel    few tokens: one (token, chosen expert or shared expert) pair per blockIdx.y, weight rows streamed
+//                       once with 16-byte loads, four rows per warp, activation fused
+//   expert_down_kernel  sum over the token's experts and the gated shared expert in one pass, fp32 output
+//
+// A decode step is bound by the weights of the experts it touches; experts shared by tokens of the batch come from L2.
+#include "tdb/hybrid.h"
+#include "tdb/launch.cuh"
+#include "tdb/vec.cuh"
+
+namespace tdb {
+
+namespace {
+
+TDB_DEVICE float relu2(float v) {
+  v = fmaxf(v, 0.f);
+  return v * v;
+}
+
+template <typename T>
+__global__ void relu2_kernel(const T* in, const float* __restrict__ w, T* out, int64_t rows, int F) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int nv = F >> 3;
+  for (int64_t v = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; v < rows * nv;
+       v += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    const float s = w != nullptr ? w[v / nv] : 1.f;
+    float f[8];
+    load8(in + v * 8, f);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) f[i] = relu2(s * f[i]);
+    store8(out + v * 8, f);
+  }
+}
+
+constexpr int kWarps = 8;
+
+// acc[r] += row r of w (R rows, n columns) . xs over the warp's lanes (not reduced)
+template <typename T, int R>
+TDB_DEVICE void rows_dot(const T* w, int64_t ldw, const T* xs, int n, int rows, float (&acc)[R]) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll 2
+  for (int c = lane * 8; c < n; c += 256) {
+    float x[8];
+    load8(xs + c, x);
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      if (r >= rows) break;
+      float v[8];
+      load8(w + r * ldw + c, v);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) acc[r] = fmaf(v[i], x[i], acc[r]);
+    }
+  }
+}
+
+constexpr int kUpRows = 4;
+template <typename T>
+__global__ void __launch_bounds__(kWarps * 32) expert_up_kernel(const ExpertGemvArgs p) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  T* xs = reinterpret_cast<T*>(smem);          // [K]
+  const int slots = p.top + (p.shared_up != nullptr ? 1 : 0);
+  const int64_t t = blockIdx.y / slots;
+  const int s = blockIdx.y - static_cast<int>(t) * slots;
+  const bool shared = s == p.top;
+  const int F = shared ? p.Fs : p.F;
+  const int r0 = (blockIdx.x * kWarps + (threadIdx.x >> 5)) * kUpRows;
+  pdl_wait();
+  pdl_launch_dependents();
+  if (blockIdx.x * kWarps * kUpRows >= F) return;
+  const T* x = reinterpret_cast<const T*>(p.x) + t * p.K;
+  for (int c = threadIdx.x * 8; c < p.K; c += kWarps * 256) {
+    float f[8];
+    load8(x + c, f);
+    store8(xs + c, f);
+  }
+  int e = 0;
+  float wgt = 1.f;
+  if (!shared) {
+    e = p.ids[t * p.top + s];
+    wgt = p.weights[t * p.top + s];
+    if (e < 0 || e >= p.E) e = 0, wgt = 0.f;
+  }
+  const T* w = shared ? reinterpret_cast<const T*>(p.shared_up) : reinterpret_cast<const T*>(p.up) + static_cast<int64_t>(e) * p.F * p.K;
+  __syncthreads();
+  if (r0 >= F) return;
+  const int rows = min(kUpRows, F - r0);
+  float acc[kUpRows] = {};
+  if (rows == kUpRows) rows_dot<T, kUpRows>(w + static_cast<int64_t>(r0) * p.K, p.K, xs, p.K, kUpRows, acc);
+  else rows_dot<T, kUpRows>(w + static_cast<int64_t>(r0) * p.K, p.K, xs, p.K, rows, acc);
+  T* act = reinterpret_cast<T*>(p.act) + t * (static_cast<int64_t>(p.top) * p.F + p.Fs) + static_cast<int64_t>(s) * p.F;
+#pragma unroll
+  for (int r = 0; r < kUpRows; ++r) {
+    const float v = warp_sum(acc[r]);
+    if ((threadIdx.x & 31) == r && r < rows) act[r0 + r] = from_f32<T>(relu2(wgt * v));
+  }
+}
+
+constexpr int kDownRows = 2;
+template <typename T>
+__global__ void __launch_bounds__(kWarps * 32) expert_down_kernel(const ExpertGemvArgs p) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  T* as = reinterpret_cast<T*>(smem);          // [top * F + Fs]
+  const int64_t t = blockIdx.y;
+  const int n_act = p.top * p.F + p.Fs;
+  pdl_wait();
+  pdl_launch_dependents();
+  const T* act = reinterpret_cast<const T*>(p.act) + t * n_act;
+  for (int c = threadIdx.x * 8; c < n_act; c += kWarps * 256) {
+    float f[8];
+    load8(act + c, f);
+    store8(as + c, f);
+  }
+  __syncthreads();
+  const int r0 = (blockIdx.x * kWarps + (threadIdx.x >> 5)) * kDownRows;
+  if (r0 >= p.K) return;
+  const int rows = min(kDownRows, p.K - r0);
+  float acc[kDownRows] = {}, sh[kDownRows] = {};
+  for (int s = 0; s < p.top; ++s) {
+    const int e = p.ids[t * p.top + s];
+    if (e < 0 || e >= p.E) continue;
+    const T* w = reinterpret_cast<const T*>(p.down) + (static_cast<int64_t>(e) * p.K + r0) * p.F;
+    rows_dot<T, kDownRows>(w, p.F, as + s * p.F, p.F, rows, acc);
+  }
+  float gate = 0.f;
+  if (p.shared_down != nullptr) {
+    gate = p.shared_gate != nullptr ? p.shared_gate[t] : 1.f;
+    rows_dot<T, kDownRows>(reinterpret_cast<const T*>(p.shared_down) + static_cast<int64_t>(r0) * p.Fs, p.Fs,
+                           as + p.top * p.F, p.Fs, rows, sh);
+  }
+#pragma unroll
+  for (int r = 0; r < kDownRows; ++r) {
+    const float v = warp_sum(acc[r] + gate * sh[r]);
+    if ((threadIdx.x & 31) == r && r < rows) p.y[t * p.K + r0 + r] = v;
+  }
+}
+
+template <typename T>
+cudaError_t launch_experts(const ExpertGemvArgs& a, cudaStream_t s) {
+  const int slots = a.top + (a.shared_up != nullptr ? 1 : 0);
+  const size_t smem_up = static_cast<size_t>(a.K) * sizeof(T);
+  const size_t smem_dn = static_cast<size_t>(a.top * a.F + a.Fs) * sizeof(T);
+  if (smem_up > 200 * 1024 || smem_dn > 200 * 1024) return cudaErrorInvalidValue;
+  static SmemOptIn up, dn;
+  cudaError_t e = up.ensure(expert_up_kernel<T>, 200 * 1024);
+  if (e != cudaSuccess) return e;
+  e = dn.ensure(expert_down_kernel<T>, 200 * 1024);
+  if (e != cudaSuccess) return e;
+  const int fmax = a.F > a.Fs ? a.F : a.Fs;
+  const int per_up = kWarps * kUpRows, per_dn = kWarps * kDownRows;
+  e = launch_pdl(expert_up_kernel<T>, dim3((fmax + per_up - 1) / per_up, static_cast<unsigned>(a.T * slots)),
+                 dim3(kWarps * 32), smem_up, s, a);
+  if (e != cudaSuccess) return e;
+  return launch_pdl(expert_down_kernel<T>, dim3((a.K + per_dn - 1) / per_dn, static_cast<unsigned>(a.T)), dim3(kWarps * 32),
+                    smem_dn, s, a);
+}
+
+}  // namespace
+
+cudaError_t launch_relu2(const void* in, const float* row_weight, void* out, int64_t rows, int F, int is_f32, cudaStream_t s) {
+  if (F % 8 != 0) return cudaErrorInvalidValue;
+  if (rows == 0) return cudaSuccess;
+  const int64_t blocks = (rows * (F / 8) + 255) / 256;
+  const dim3 grid(static_cast<unsigned>(blocks < 148 * 16 ? blocks : 148 * 16));
+  return is_f32 ? launch_pdl(relu2_kernel<float>, grid, dim3(256), 0, s, reinterpret_cast<const float*>(in), row_weight,
+                             reinterpret_cast<float*>(out), rows, F)
+                : launch_pdl(relu2_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, reinterpret_cast<const __nv_bfloat16*>(in),
+                             row_weight, reinterpret_cast<__nv_bfloat16*>(out), rows, F);
+}
+
+cudaError_t launch_expert_gemv(const ExpertGemvArgs& a, cudaStream_t s) {
+  if (a.K % 8 != 0 || a.F % 8 != 0 || a.Fs % 8 != 0 || a.top < 1) return cudaErrorInvalidValue;
+  if ((a.shared_up == nullptr) != (a.shared_down == nullptr) || (a.shared_up == nullptr && a.Fs != 0)) return cudaErrorInvalidValue;
+  if (a.T * (a.top + 1) > 65535) return cudaErrorInvalidValue;
+  if (a.T == 0) return cudaSuccess;
+  return a.is_f32 ? launch_experts<float>(a, s) : launch_experts<__nv_bfloat16>(a, s);
+}
+
+}  // namespace tdb

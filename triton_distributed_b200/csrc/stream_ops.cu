@@ -1,0 +1,172 @@
+// Residual-stream kernels of decoders that keep the stream in fp32 and norm a sublayer's OUTPUT before adding it:
+// embedding into the stream, x += RMSNorm(y) * w (y summed over a token's expert rows and a gated shared row on the
+// way), and the norm in front of the head.  The stream has a bf16 copy that the next sublayer's GEMMs read.
+// One block per token, 32-byte accesses, the row is kept in shared memory between the two passes.
+#include "tdb/hybrid.h"
+#include "tdb/launch.cuh"
+#include "tdb/vec.cuh"
+
+namespace tdb {
+
+namespace {
+
+template <typename T>
+__global__ void embed_stream_kernel(const int64_t* __restrict__ ids, const T* __restrict__ table, float* __restrict__ x,
+                                    T* __restrict__ xb, int W, int64_t vocab) {
+  const int64_t t = blockIdx.x;
+  int64_t id = ids[t];
+  if (id < 0 || id >= vocab) id = 0;
+  for (int c = threadIdx.x * 8; c < W; c += blockDim.x * 8) {
+    float f[8];
+    load8(table + id * W + c, f);
+    store8(x + t * W + c, f);
+    if (xb != nullptr) store8(xb + t * W + c, f);
+  }
+}
+
+// Sum of a token's contributions, columns [c, c + 8).
+template <typename TY>
+TDB_DEVICE void token_sum(const TY* y, int rows, const TY* shared, float gate, int64_t t, int W, int c, float (&acc)[8]) {
+  load8(y + t * rows * W + c, acc);
+  for (int r = 1; r < rows; ++r) {
+    float f[8];
+    load8(y + (t * rows + r) * W + c, f);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) acc[i] += f[i];
+  }
+  if (shared != nullptr) {
+    float f[8];
+    load8(shared + t * W + c, f);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) acc[i] += gate * f[i];
+  }
+}
+
+template <typename TY>
+__global__ void postnorm_add_kernel(const PostNormArgs p) {
+  __shared__ float red[32];
+  extern __shared__ float row[];       // [W]
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t t = blockIdx.x;
+  const TY* y = reinterpret_cast<const TY*>(p.y);
+  const TY* sh = reinterpret_cast<const TY*>(p.shared);
+  const float gate = (sh != nullptr && p.shared_gate != nullptr) ? p.shared_gate[t] : 1.f;
+  float ss = 0.f;
+  for (int c = threadIdx.x * 8; c < p.W; c += blockDim.x * 8) {
+    float a[8];
+    token_sum(y, p.rows_per_token, sh, gate, t, p.W, c, a);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss += a[i] * a[i];
+    store8(row + c, a);
+  }
+  const float inv = 1.f / sqrtf(block_reduce_sum(ss, red) / p.n_real + p.eps);
+  __nv_bfloat16* xb = reinterpret_cast<__nv_bfloat16*>(p.xb);
+  for (int c = threadIdx.x * 8; c < p.W; c += blockDim.x * 8) {
+    float a[8], w[8], x[8];
+    load8(row + c, a);
+    load8(p.w + c, w);
+    load8(p.x + t * p.W + c, x);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) x[i] += a[i] * inv * w[i];
+    store8(p.x + t * p.W + c, x);
+    if (xb != nullptr) store8(xb + t * p.W + c, x);
+  }
+}
+
+template <typename TY>
+__global__ void combine_rows_kernel(const PostNormArgs p, TY* out) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t t = blockIdx.x;
+  const TY* sh = reinterpret_cast<const TY*>(p.shared);
+  const float gate = (sh != nullptr && p.shared_gate != nullptr) ? p.shared_gate[t] : 1.f;
+  for (int c = threadIdx.x * 8; c < p.W; c += blockDim.x * 8) {
+    float a[8];
+    token_sum(reinterpret_cast<const TY*>(p.y), p.rows_per_token, sh, gate, t, p.W, c, a);
+    store8(out + t * p.W + c, a);
+  }
+}
+
+template <typename TO>
+__global__ void stream_norm_kernel(const float* __restrict__ x, const int64_t* __restrict__ rows, const float* __restrict__ w,
+                                   TO* __restrict__ out, int W, int n_real, float eps) {
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t i = blockIdx.x;
+  const float* xr = x + (rows != nullptr ? rows[i] : i) * W;
+  float ss = 0.f;
+  for (int c = threadIdx.x * 8; c < W; c += blockDim.x * 8) {
+    float a[8];
+    load8(xr + c, a);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss += a[j] * a[j];
+  }
+  const float inv = 1.f / sqrtf(block_reduce_sum(ss, red) / n_real + eps);
+  for (int c = threadIdx.x * 8; c < W; c += blockDim.x * 8) {
+    float a[8], g[8];
+    load8(xr + c, a);
+    load8(w + c, g);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) a[j] *= inv * g[j];
+    store8(out + i * W + c, a);
+  }
+}
+
+int row_threads(int W) {
+  const int vec = W / 8;
+  return vec >= 512 ? 512 : vec >= 256 ? 256 : vec >= 128 ? 128 : 64;
+}
+
+}  // namespace
+
+cudaError_t launch_embed_stream(const int64_t* ids, const void* table, float* x, void* xb, int64_t T, int W, int64_t vocab,
+                                int is_f32, cudaStream_t s) {
+  if (W % 8 != 0) return cudaErrorInvalidValue;
+  if (T == 0) return cudaSuccess;
+  if (is_f32)
+    embed_stream_kernel<float><<<static_cast<unsigned>(T), row_threads(W), 0, s>>>(
+        ids, reinterpret_cast<const float*>(table), x, nullptr, W, vocab);
+  else
+    embed_stream_kernel<__nv_bfloat16><<<static_cast<unsigned>(T), row_threads(W), 0, s>>>(
+        ids, reinterpret_cast<const __nv_bfloat16*>(table), x, reinterpret_cast<__nv_bfloat16*>(xb), W, vocab);
+  return cudaGetLastError();
+}
+
+cudaError_t launch_postnorm_add(const PostNormArgs& a, cudaStream_t s) {
+  if (a.W % 8 != 0 || a.n_real < 1 || a.rows_per_token < 1) return cudaErrorInvalidValue;
+  if (a.T == 0) return cudaSuccess;
+  const size_t smem = static_cast<size_t>(a.W) * 4;
+  if (smem > 200 * 1024) return cudaErrorInvalidValue;
+  static SmemOptIn f, b;
+  if (smem > 40 * 1024) {
+    cudaError_t e = a.y_f32 ? f.ensure(postnorm_add_kernel<float>, 200 * 1024)
+                            : b.ensure(postnorm_add_kernel<__nv_bfloat16>, 200 * 1024);
+    if (e != cudaSuccess) return e;
+  }
+  const dim3 grid(static_cast<unsigned>(a.T)), block(row_threads(a.W));
+  return a.y_f32 ? launch_pdl(postnorm_add_kernel<float>, grid, block, smem, s, a)
+                 : launch_pdl(postnorm_add_kernel<__nv_bfloat16>, grid, block, smem, s, a);
+}
+
+cudaError_t launch_combine_rows(const PostNormArgs& a, void* out, cudaStream_t s) {
+  if (a.W % 8 != 0 || a.rows_per_token < 1) return cudaErrorInvalidValue;
+  if (a.T == 0) return cudaSuccess;
+  const dim3 grid(static_cast<unsigned>(a.T)), block(row_threads(a.W));
+  return a.y_f32 ? launch_pdl(combine_rows_kernel<float>, grid, block, 0, s, a, reinterpret_cast<float*>(out))
+                 : launch_pdl(combine_rows_kernel<__nv_bfloat16>, grid, block, 0, s, a, reinterpret_cast<__nv_bfloat16*>(out));
+}
+
+cudaError_t launch_stream_norm(const float* x, const int64_t* rows, const float* w, void* out, int64_t n, int W, int n_real,
+                               float eps, int out_f32, cudaStream_t s) {
+  if (W % 8 != 0 || n_real < 1) return cudaErrorInvalidValue;
+  if (n == 0) return cudaSuccess;
+  const dim3 grid(static_cast<unsigned>(n)), block(row_threads(W));
+  return out_f32 ? launch_pdl(stream_norm_kernel<float>, grid, block, 0, s, x, rows, w, reinterpret_cast<float*>(out), W,
+                              n_real, eps)
+                 : launch_pdl(stream_norm_kernel<__nv_bfloat16>, grid, block, 0, s, x, rows, w,
+                              reinterpret_cast<__nv_bfloat16*>(out), W, n_real, eps);
+}
+
+}  // namespace tdb

@@ -1,10 +1,19 @@
 """Models, KV caches, weight loading and the serving engine (the reference's ``triton_dist.models``)."""
 from .config import ArchConfig, ModelConfig, PRESETS  # noqa: F401
-from .kv_cache import KV_Cache, PagedKVCache  # noqa: F401
+from .kv_cache import HybridCache, KV_Cache, PagedKVCache, StateSpec, StepPlan, TiedKVSpec  # noqa: F401
 from .safetensors_io import SafetensorsFile, ShardedCheckpoint, save_file  # noqa: F401
 from .dense import DenseLLM, DenseLLMLayer  # noqa: F401
 from .engine import Engine  # noqa: F401
 from .qwen_moe import Qwen3MoE, Qwen3MoELayer  # noqa: F401
+from .vasolix import VASOLIX_PRESETS, VasolixConfig, VasolixLLM  # noqa: F401
+
+# "architecture" of a config.json -> (configuration class, model class); configurations without that key are read as
+# Hugging Face ones (DenseLLM / Qwen3MoE).
+ARCHITECTURES = {"Vasolix": (VasolixConfig, VasolixLLM)}
+
+
+def all_presets() -> dict:
+    return {**PRESETS, **VASOLIX_PRESETS}
 
 
 class AutoLLM:
@@ -13,6 +22,9 @@ class AutoLLM:
     @staticmethod
     def from_pretrained(model_config: ModelConfig, group=None):
         arch = model_config.arch()
+        for config_cls, model_cls in ARCHITECTURES.values():
+            if isinstance(arch, config_cls):
+                return model_cls(model_config, group)
         if arch.is_moe:
             from .qwen_moe import Qwen3MoE
             return Qwen3MoE(model_config, group)

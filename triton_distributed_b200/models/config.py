@@ -87,14 +87,24 @@ class ModelConfig:
     num_layers_override: Optional[int] = None
     seed: int = 0
 
-    def arch(self) -> ArchConfig:
+    def arch(self):
+        """The architecture: a checkpoint's ``config.json`` (read by the class its ``architecture`` names in
+        ``ARCHITECTURES``, else as a Hugging Face configuration), or a preset."""
+        from . import ARCHITECTURES, all_presets
+        presets = all_presets()
         if self.checkpoint_dir and os.path.exists(os.path.join(self.checkpoint_dir, "config.json")):
-            a = ArchConfig.from_hf_json(self.checkpoint_dir)
-        elif self.model_name in PRESETS:
-            a = PRESETS[self.model_name]
+            with open(os.path.join(self.checkpoint_dir, "config.json")) as f:
+                name = json.load(f).get("architecture")
+            if name is not None and name not in ARCHITECTURES:
+                raise KeyError(f"unknown architecture {name}; known: {sorted(ARCHITECTURES)}")
+            a = ARCHITECTURES[name][0].from_json(self.checkpoint_dir) if name else ArchConfig.from_hf_json(self.checkpoint_dir)
+        elif self.model_name in presets:
+            a = presets[self.model_name]
         else:
-            raise KeyError(f"unknown model {self.model_name}; known: {sorted(PRESETS)}")
+            raise KeyError(f"unknown model {self.model_name}; known: {sorted(presets)}")
         if self.num_layers_override is not None:
+            if hasattr(a, "with_num_layers"):
+                return a.with_num_layers(self.num_layers_override)
             import dataclasses
             a = dataclasses.replace(a, num_hidden_layers=self.num_layers_override)
         return a

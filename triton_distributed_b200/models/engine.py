@@ -6,7 +6,7 @@ API of the reference: ``Engine`` (python/triton_dist/models/engine.py:37-189): a
 from __future__ import annotations
 
 import time
-from typing import Optional
+from typing import Dict, List, Optional, Sequence
 
 import torch
 
@@ -41,8 +41,13 @@ class Engine:
         self._sample_gen = torch.Generator(device=self.rt.device)
         self._sample_gen.manual_seed(int(seed))
         self._ctx_key = None      # (backend, max_M) the model's communication contexts were built for
+        self.step_cache = None    # cache of the packed steps (see step()), apart from serve()'s
+        self._step_slots: Dict[object, int] = {}
 
     def _init_kv_cache(self, bsz: int):
+        if hasattr(self.model, "new_cache"):
+            self.kv_cache = self.model.new_cache(bsz, self.model_config.max_length)
+            return
         a = self.model.arch
         kv_heads = max(1, a.num_key_value_heads // self.rt.world_size)
         self.kv_cache = KV_Cache(a.num_hidden_layers, bsz, self.model_config.max_length, kv_heads, a.head_dim,
@@ -55,6 +60,7 @@ class Engine:
     def _init_cuda_graph(self):
         """Three warm-up steps on a side stream, then capture one whole decode step."""
         off = self.kv_cache.kv_offset.clone()
+        snap = self.kv_cache.snapshot() if hasattr(self.kv_cache, "snapshot") else None   # recurrent states
         s = torch.cuda.Stream()
         s.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(s):
@@ -67,10 +73,12 @@ class Engine:
         with torch.cuda.graph(self.graph):
             self._decode_step()
         self.kv_cache.kv_offset.copy_(off)
+        if snap is not None:
+            self.kv_cache.restore(snap)
         torch.cuda.synchronize()
         self.rt.host_barrier()
 
-    def validate_request(self, input_ids: torch.Tensor, gen_len: int):
+    def validate_request(self, input_ids: torch.Tensor, gen_len: int, seq_lens: Optional[Sequence[int]] = None):
         """Host-side check of a request against the model's limits; raises ``ValueError``.  Cache rows are addressed as
         ``batch * max_length + position``, so a prompt plus generation longer than ``max_length`` (or a token id outside
         the vocabulary) would index past the sequence's rows: such requests never reach a kernel."""
@@ -89,7 +97,12 @@ class Engine:
         lo, hi = int(input_ids.min()), int(input_ids.max())
         if lo < 0 or hi >= vocab:
             raise ValueError(f"token ids must lie in [0, {vocab}), got [{lo}, {hi}]")
-        if self.backend in ("triton_dist", "ag_rs") and B % max(self.rt.world_size, 1) != 0:
+        if seq_lens is not None:
+            if not hasattr(self.model, "forward_step"):
+                raise ValueError("this model serves prompts of one length per batch")
+            if len(seq_lens) != B or min(seq_lens) < 1 or max(seq_lens) > S:
+                raise ValueError(f"seq_lens must give a length in [1, {S}] for each of the {B} prompts")
+        elif self.backend in ("triton_dist", "ag_rs") and B % max(self.rt.world_size, 1) != 0:
             raise ValueError(f"backend {self.backend} shards the batch: {B} is not a multiple of {self.rt.world_size}")
 
     def _sample(self, logits: torch.Tensor) -> torch.Tensor:
@@ -114,11 +127,63 @@ class Engine:
         self.model.init_ctx_for(self.backend, max_M)
         self._ctx_key = key
 
+    # -- packed steps: the caller decides which tokens go in -----------------------------------------------------
     @torch.no_grad()
-    def serve(self, input_ids: torch.Tensor, gen_len: int) -> torch.Tensor:
+    def step(self, entries: Sequence[tuple]) -> torch.Tensor:
+        """One step over given tokens: ``entries`` is a list of ``(request id, token ids, wanted places)``; a new id starts a
+        sequence, a known one continues it.  All tokens of the step run as one packed batch through the model's
+        ``forward_step``; returns fp32 logits [wanted, vocab] in the order of the entries.  :meth:`end` gives a sequence's
+        slot back.  Prompts run with the torch backend and single-token steps with ``self.backend``, as in :meth:`serve`."""
+        if not hasattr(self.model, "forward_step"):
+            raise NotImplementedError(f"{type(self.model).__name__} has no packed steps")
+        vocab, max_len = self.model.arch.vocab_size, int(self.model_config.max_length)
+        ids_seen, held = set(), {}
+        for rid, tokens, want in entries:
+            if rid in ids_seen or not len(tokens):
+                raise ValueError("a step needs distinct requests with at least one token each")
+            ids_seen.add(rid)
+            if min(tokens) < 0 or max(tokens) >= vocab:
+                raise ValueError(f"token ids must lie in [0, {vocab})")
+            if len(want) and (min(want) < 0 or max(want) >= len(tokens)):
+                raise ValueError("a wanted place lies outside the step's tokens")
+            held[rid] = self.step_cache.lens[self._step_slots[rid]] if rid in self._step_slots else 0
+            if held[rid] + len(tokens) > max_len:
+                raise ValueError(f"request {rid!r} would exceed max_length ({max_len})")
+        if not entries:
+            raise ValueError("empty step")
+        if self.step_cache is None:
+            self.step_cache = self.model.new_cache(len(entries), max_len, allocate=False)
+        for rid, _, _ in entries:
+            if rid not in self._step_slots:
+                self._step_slots[rid] = self.step_cache.alloc()
+        slots = [self._step_slots[rid] for rid, _, _ in entries]
+        lens = [len(t) for _, t, _ in entries]
+        plan = self.step_cache.plan(slots, lens)
+        if plan.decode:
+            self._ensure_ctx(len(entries))
+        self.model.set_fwd(self.backend if plan.decode else "torch")
+        flat, rows, base = [], [], 0
+        for _, tokens, want in entries:
+            flat += [int(t) for t in tokens]
+            rows += [base + int(w) for w in want]
+            base += len(tokens)
+        dev = self.rt.device
+        logits = self.model.forward_step(torch.tensor(flat, dtype=torch.int64).to(dev), plan,
+                                         torch.tensor(rows, dtype=torch.int64).to(dev), wo_lm_head=not rows)
+        self.step_cache.advance(slots, lens)
+        return logits
+
+    def end(self, request_ids: Sequence):
+        """Requests that are finished: their cache rows and states go back."""
+        for rid in request_ids:
+            self.step_cache.free(self._step_slots.pop(rid))
+
+    @torch.no_grad()
+    def serve(self, input_ids: torch.Tensor, gen_len: int, seq_lens: Optional[Sequence[int]] = None) -> torch.Tensor:
         """Prefill ``input_ids`` [B, S] with the torch backend, then generate ``gen_len`` tokens with ``self.backend``.
-        Requests that do not fit the model (see :meth:`validate_request`) raise ``ValueError`` before any launch."""
-        self.validate_request(input_ids, gen_len)
+        Requests that do not fit the model (see :meth:`validate_request`) raise ``ValueError`` before any launch.
+        ``seq_lens``: lengths of right-padded prompts (models with packed steps)."""
+        self.validate_request(input_ids, gen_len, seq_lens)
         B, S = input_ids.shape
         self._bsz = B
         input_ids = input_ids.to(self.rt.device)
@@ -129,8 +194,12 @@ class Engine:
             self.kv_cache.clear()
         pos = torch.arange(S, device=self.rt.device, dtype=torch.int64).unsqueeze(0).expand(B, S).contiguous()
         self.model.set_fwd("torch")
-        logits = self.model.inference(input_ids, pos, self.kv_cache)
-        self.kv_cache.inc_offset(S)
+        if seq_lens is None:
+            logits = self.model.inference(input_ids, pos, self.kv_cache)
+            self.kv_cache.inc_offset(S)
+        else:
+            logits = self.model.inference(input_ids, pos, self.kv_cache, seq_lens=seq_lens)
+            self.kv_cache.inc_offset([int(n) for n in seq_lens])
         nxt = self._sample(logits)
         out = [nxt]
         self.step_logits = [logits.float().clone()] if self.keep_logits else []

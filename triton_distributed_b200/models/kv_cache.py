@@ -4,11 +4,13 @@ kernels take: ``layer(i) -> (k, v) [pages, page_size, Hkv, D]`` plus an int32 ``
 Offsets live on the device so a CUDA graph of one decode step can be replayed while they advance."""
 from __future__ import annotations
 
-from typing import Optional, Tuple
+from dataclasses import dataclass
+from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
 from ..ops.attention import decode_workspace, pick_kv_splits
+from ..ops.gla import gla_chunk_tables
 
 
 class KV_Cache:
@@ -113,3 +115,247 @@ class PagedKVCache:
         self.k_cache.normal_()
         self.v_cache.normal_()
         self.kv_offset.fill_(length)
+
+
+# ------------------------------------------------------------------ layered decoders: per-layer storage, packed steps
+@dataclass(frozen=True)
+class TiedKVSpec:
+    """A layer that caches raw keys (which are also its values) and one fp32 factor per token.  ``block`` > 0: attention is
+    local to blocks of that many positions, so a sequence keeps ``block`` rows, position p at row ``p % block``."""
+    kv_heads: int
+    head_dim: int
+    block: int = 0
+
+    def rows(self, max_length: int) -> int:
+        return min(self.block, max_length) if self.block > 0 else max_length
+
+
+@dataclass(frozen=True)
+class StateSpec:
+    """A recurrent layer: fp32 state [heads, dk, dv] per sequence."""
+    heads: int
+    dk: int
+    dv: int
+
+
+@dataclass
+class BlockPlan:
+    """What a tied-KV layer needs to know about a step (see ``StepPlan.blocks``); ``rows`` is the page size of its cache."""
+    home_rows: torch.Tensor                         # int64 [T] cache row of every token, -1 = not kept after the step
+    block_table: torch.Tensor                       # int32 [virtual sequences, 1]
+    row0: torch.Tensor                              # int64 [T] first visible row of every token (of the page pool used)
+    n_keys: torch.Tensor                            # int32 [T]
+    kv_lens: torch.Tensor                           # int32 [virtual sequences]
+    # prompts only: every (sequence, block) pair is a virtual sequence of its own with a page of a scratch pool
+    scratch_rows: Optional[torch.Tensor] = None     # int64 [T]
+    cu: Optional[torch.Tensor] = None               # int32 [virtual sequences + 1]
+    q_pos0: Optional[torch.Tensor] = None           # int32 [virtual sequences] position of the first query in its block
+    pages: int = 0
+    page_rows: int = 0
+    max_q: int = 0
+    max_kv: int = 0
+    carry_src: Optional[torch.Tensor] = None        # cache rows of earlier steps that a continued block still needs ...
+    carry_dst: Optional[torch.Tensor] = None        # ... and where they go in the scratch pool
+
+
+class StepPlan:
+    """The tokens of one step, packed sequence after sequence.  Built by the cache; the per-layer tables are derived once
+    per distinct block size.  A decode plan (one token per sequence) is made of device tensors only, so it can be captured
+    in a CUDA graph."""
+
+    def __init__(self, cache: "HybridCache", slots: torch.Tensor, positions: torch.Tensor, pos0: torch.Tensor,
+                 host: Optional[Tuple[List[int], List[int], List[int]]] = None):
+        self.cache, self.slots, self.positions, self.pos0, self.host = cache, slots, positions, pos0, host
+        self.num_seqs, self.num_tokens = slots.numel(), positions.numel()
+        self.decode = host is None
+        self.cu = None
+        self._blocks: Dict[int, BlockPlan] = {}
+        self._chunks = None
+        if not self.decode:
+            cu = [0]
+            for n in host[2]:
+                cu.append(cu[-1] + n)
+            self.cu_host = cu
+            self.cu = torch.tensor(cu, dtype=torch.int32).to(slots.device)
+            self.last_rows = torch.tensor([c - 1 for c in cu[1:]], dtype=torch.int64).to(slots.device)
+
+    def chunk_tables(self):
+        """Chunks of the gated-linear-attention kernels (None for a decode step)."""
+        if self._chunks is None and not self.decode:
+            self._chunks = gla_chunk_tables(self.cu_host, self.slots.device)
+        return self._chunks
+
+    def blocks(self, spec: TiedKVSpec) -> BlockPlan:
+        rows = spec.rows(self.cache.max_length)
+        if rows not in self._blocks:
+            self._blocks[rows] = self._decode_blocks(rows) if self.decode else self._prompt_blocks(rows)
+        return self._blocks[rows]
+
+    def _decode_blocks(self, rows: int) -> BlockPlan:
+        base = self.slots.to(torch.int64) * rows
+        off = self.positions % rows
+        return BlockPlan(home_rows=base + off, block_table=self.slots.unsqueeze(1).contiguous(), row0=base,
+                         n_keys=(off + 1).to(torch.int32), kv_lens=(self.positions + 1).to(torch.int32))
+
+    def _prompt_blocks(self, rows: int) -> BlockPlan:
+        slots, starts, lens = self.host
+        virt = []                                    # (first token, tokens, position inside the block, slot or -1 = not last)
+        tok = 0
+        for slot, start, n in zip(slots, starts, lens):
+            at, left = start, n
+            while left > 0:
+                take = min(left, rows - at % rows)
+                virt.append((tok, take, at % rows, slot, left == take))
+                tok, at, left = tok + take, at + take, left - take
+        max_kv = max(off + n for _, n, off, _, _ in virt)
+        page_rows = min(rows, (max_kv + 7) // 8 * 8)
+        home, scratch, row0, keys = [], [], [], []
+        src, dst = [], []
+        for i, (_, n, off, slot, last) in enumerate(virt):
+            r = torch.arange(off, off + n)
+            home.append(r + slot * rows if last else torch.full((n,), -1))
+            scratch.append(r + i * page_rows)
+            row0.append(torch.full((n,), i * page_rows))
+            keys.append(r + 1)
+            if off > 0:                              # the block began in an earlier step
+                src.append(torch.arange(off) + slot * rows)
+                dst.append(torch.arange(off) + i * page_rows)
+        dev = self.slots.device
+        T = self.num_tokens
+        big = torch.cat([torch.cat(x) for x in (home, scratch, row0)] + src + dst).to(torch.int64).to(dev)
+        nv, nc = len(virt), sum(int(x.numel()) for x in src)
+        small = torch.tensor([v[0] for v in virt] + [T] + [v[2] for v in virt] + [v[2] + v[1] for v in virt] + list(range(nv)),
+                             dtype=torch.int32)
+        small = torch.cat([small, torch.cat(keys).to(torch.int32)]).to(dev)
+        return BlockPlan(home_rows=big[:T], scratch_rows=big[T:2 * T], row0=big[2 * T:3 * T],
+                         carry_src=big[3 * T:3 * T + nc] if nc else None, carry_dst=big[3 * T + nc:] if nc else None,
+                         cu=small[:nv + 1], q_pos0=small[nv + 1:2 * nv + 1], kv_lens=small[2 * nv + 1:3 * nv + 1],
+                         block_table=small[3 * nv + 1:4 * nv + 1].unsqueeze(1), n_keys=small[4 * nv + 1:], pages=nv,
+                         page_rows=page_rows, max_q=max(v[1] for v in virt), max_kv=max_kv)
+
+
+class HybridCache:
+    """Cache of a layered decoder: one storage per layer (``TiedKVSpec`` or ``StateSpec``), indexed by a sequence's slot.
+
+    Slots are handed out by ``alloc`` and given back by ``free``; nothing is cleared in between, because a sequence that
+    starts at position 0 neither reads its state row nor any row it has not written.  ``kv_offset`` (device) and ``lens``
+    (host) count the tokens each slot holds; a step's plan starts there.  The first ``batch_size`` slots are allocated at
+    construction, which is what :class:`Engine` uses for a rectangular batch."""
+
+    def __init__(self, specs: Sequence, batch_size: int, max_length: int, dtype: torch.dtype = torch.bfloat16, device=None,
+                 allocate: bool = True):
+        self.specs, self.batch_size, self.max_length, self.dtype = list(specs), batch_size, max_length, dtype
+        self.device = device or "cuda"
+        self.capacity = 0
+        self.layers: List[dict] = [{} for _ in self.specs]
+        self.kv_offset = torch.zeros(0, dtype=torch.int32, device=self.device)
+        self.lens: List[int] = []
+        self._free: List[int] = []
+        self._grow(max(1, batch_size))
+        if allocate:
+            for _ in range(batch_size):
+                self.alloc()
+        self.batch_slots = torch.arange(batch_size, dtype=torch.int32, device=self.device)
+
+    # -- slots ------------------------------------------------------------------------------------------------
+    def _grow(self, capacity: int):
+        def widen(t, *shape, dtype):
+            new = torch.zeros(capacity, *shape, dtype=dtype, device=self.device)
+            if t is not None:
+                new[:self.capacity] = t
+            return new
+
+        for spec, st in zip(self.specs, self.layers):
+            if isinstance(spec, TiedKVSpec):
+                rows = spec.rows(self.max_length)
+                st["k"] = widen(st.get("k"), rows, spec.kv_heads, spec.head_dim, dtype=self.dtype)
+                st["scale"] = widen(st.get("scale"), rows, dtype=torch.float32)
+            else:
+                st["state"] = widen(st.get("state"), spec.heads, spec.dk, spec.dv, dtype=torch.float32)
+        self.kv_offset = widen(self.kv_offset, dtype=torch.int32)
+        self._free = list(range(capacity - 1, self.capacity - 1, -1)) + self._free
+        self.lens += [0] * (capacity - self.capacity)
+        self.capacity = capacity
+
+    def alloc(self) -> int:
+        """A slot for a new sequence (the storage doubles when none is free; captured graphs do not survive that)."""
+        if not self._free:
+            self._grow(2 * self.capacity)
+        slot = self._free.pop()
+        self._set_len(slot, 0)
+        return slot
+
+    def free(self, slot: int):
+        if slot in self._free or not 0 <= slot < self.capacity:
+            raise ValueError(f"slot {slot} is not in use")
+        self._free.append(slot)
+
+    def _set_len(self, slot: int, n: int):
+        self.lens[slot] = n
+        self.kv_offset[slot] = n
+
+    # -- step plans -------------------------------------------------------------------------------------------
+    def plan(self, slots: Sequence[int], lens: Sequence[int]) -> StepPlan:
+        """A step that brings ``lens[i]`` new tokens of the sequence in ``slots[i]``.  Raises ``ValueError`` when a sequence
+        would outgrow ``max_length``."""
+        slots, lens = list(slots), list(lens)
+        if not slots or len(slots) != len(lens) or min(lens) < 1 or len(set(slots)) != len(slots):
+            raise ValueError("a step needs distinct sequences with at least one token each")
+        starts = [self.lens[s] for s in slots]
+        for s, a, n in zip(slots, starts, lens):
+            if a + n > self.max_length:
+                raise ValueError(f"sequence of {a + n} tokens exceeds max_length ({self.max_length})")
+        dev_slots = torch.tensor(slots, dtype=torch.int32).to(self.device)
+        pos0 = torch.tensor(starts, dtype=torch.int64).to(self.device)
+        if max(lens) == 1:
+            return StepPlan(self, dev_slots, pos0, pos0)
+        pos = torch.cat([torch.arange(a, a + n) for a, n in zip(starts, lens)]).to(self.device)
+        return StepPlan(self, dev_slots, pos, pos0, (slots, starts, lens))
+
+    def decode_plan(self, positions: torch.Tensor) -> StepPlan:
+        """One token for each of the first ``len(positions)`` slots; ``positions`` int64 on the device."""
+        pos = positions.reshape(-1).to(torch.int64)
+        return StepPlan(self, self.batch_slots[:pos.numel()], pos, pos)
+
+    def advance(self, slots: Sequence[int], lens: Sequence[int]):
+        """The tokens of a step have been computed."""
+        for s, n in zip(slots, lens):
+            self.lens[s] += n
+        idx = torch.tensor(list(slots), dtype=torch.int64).to(self.device)
+        self.kv_offset[idx] += torch.tensor(list(lens), dtype=torch.int32).to(self.device)
+
+    # -- the rectangular-batch interface of the engine ----------------------------------------------------------
+    def inc_offset(self, n=1):
+        """Advance the engine's batch by ``n`` tokens (one number, or one per sequence)."""
+        per = [n] * self.batch_size if isinstance(n, int) else list(n)
+        for s, k in enumerate(per):
+            self.lens[s] += k
+        if isinstance(n, int):
+            self.kv_offset[:self.batch_size] += n
+        else:
+            self.kv_offset[:self.batch_size] += torch.tensor(per, dtype=torch.int32).to(self.device)
+
+    def clear(self):
+        self.kv_offset.zero_()
+        self.lens = [0] * self.capacity
+
+    def snapshot(self):
+        """Copies of what a decode step changes besides the row it writes (recurrent states): a step run for warm-up must
+        not count."""
+        return [st["state"].clone() if "state" in st else None for st in self.layers]
+
+    def restore(self, snap):
+        for st, old in zip(self.layers, snap):
+            if old is not None:
+                st["state"].copy_(old)
+
+    def rand_fill(self, length: int):
+        """Pretend ``length`` tokens are cached (random contents): used by decode benchmarks."""
+        for st in self.layers:
+            for name, t in st.items():
+                if name == "scale":
+                    t.fill_(1.0)
+                else:
+                    t.normal_()
+        self.kv_offset.fill_(length)
+        self.lens = [length] * self.capacity

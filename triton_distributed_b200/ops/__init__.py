@@ -17,7 +17,8 @@ from .elementwise import (rmsnorm, silu_mul, residual_add, qk_norm_rope_kv, embe
                           abs_sum)
 from .attention import (flash_attn_varlen, gqa_fwd_batch_decode, gqa_fwd_batch_decode_intra_rank,  # noqa: F401
                         gqa_fwd_batch_decode_persistent, attention_reference, merge_attention_partials,
-                        dense_block_table, decode_workspace, pick_kv_splits)
+                        dense_block_table, decode_workspace, pick_kv_splits, tied_attention_simple, tied_attn_varlen,
+                        tied_attn_decode, TIED_TENSOR_CORE_DIMS)
 from .gemv import (GemvARContext, create_gemv_ar_context, gemv_fused, gemv_reference, gemv_supported,  # noqa: F401
                    GEMV_FAST_M, GEMV_MAX_M)
 from .gemm_ar import (GemmARContext, LLGemmARContext, create_gemm_ar_context, create_ll_gemm_ar_context,  # noqa: F401
@@ -38,3 +39,6 @@ from .fp8 import (ag_gemm_fp8, dequantize_act_1x128, dequantize_weight_128x128, 
                   gemm_rs_fp8_reference, AGGemmFp8Context, GemmRSFp8Context)
 from .moe import (tile_arrival_order, tile_schedule, sort_topk_ids_staged, group_gemm_gather,  # noqa: F401,E402
                   MoESort, MoEAgScatterGroupGemmContext, MoEReduceRSContext)
+from .stream import (embed_stream, postnorm_add, combine_rows, stream_norm, qk_sumsq, qk_norm_tied)  # noqa: F401,E402
+from .gla import gated_linear_attention, gla_chunk_tables, GLA_CHUNK  # noqa: F401,E402
+from .moe import (narrow_linear, sigmoid_router, relu2, relu2_experts_gemv, EXPERT_GEMV_MAX_T)  # noqa: F401,E402

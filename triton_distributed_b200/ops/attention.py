@@ -192,3 +192,65 @@ def merge_attention_partials(outs: torch.Tensor, lses: torch.Tensor) -> torch.Te
     tot = w.sum(dim=0)
     res = (w.unsqueeze(-1) * outs.float()).sum(dim=0) / tot.clamp_min(1e-30).unsqueeze(-1)
     return res
+
+
+# ------------------------------------------------------------------ tied KV: values are the raw keys
+TIED_TENSOR_CORE_DIMS = (32, 64, 128, 256)      # head dims of the mma.sync / tcgen05 kernels in tied form
+
+
+def _tied_attention_restatement(q, k, k_scale, row0, n_keys, sink, gate):
+    T, Hq, D = q.shape
+    Hkv = k.shape[-2]
+    kf, sf = k.reshape(-1, Hkv, D), k_scale.reshape(-1)
+    out = torch.empty(T, Hq, D)
+    for t in range(T):
+        lo, hi = int(row0[t]), int(row0[t]) + int(n_keys[t])
+        kk = kf[lo:hi].float().repeat_interleave(Hq // Hkv, dim=1)
+        s = torch.einsum("hd,nhd->hn", q[t].float(), kk) * sf[lo:hi]
+        if sink is not None:
+            s = torch.cat([s, sink.float().unsqueeze(1)], dim=1)
+        out[t] = torch.einsum("hn,nhd->hd", torch.softmax(s, dim=-1)[:, :hi - lo], kk)
+    if gate is not None:
+        out *= torch.sigmoid(gate.float()).reshape(T, Hq, D)
+    return out.to(q.dtype)
+
+
+def tied_attention_simple(q, k, k_scale, row0, n_keys, sink=None, gate=None):
+    """fp32-arithmetic attention over a tied cache, any head dim up to 512: token t sees rows ``row0[t] .. + n_keys[t]`` of
+    ``k`` (viewed as [rows, Hkv, D]); its score is ``q . k[row] * k_scale[row]``, its value ``k[row]``."""
+    if _native.use_native(q, k):
+        return _native.load(True).tied_attn_simple(q, k, k_scale, row0, n_keys, sink, gate)
+    return _tied_attention_restatement(q, k, k_scale, row0, n_keys, sink, gate)
+
+
+def tied_attn_varlen(q: torch.Tensor, k: torch.Tensor, k_scale: torch.Tensor, block_table: torch.Tensor,
+                     cu_seqlens_q: torch.Tensor, q_pos0: torch.Tensor, kv_lens: torch.Tensor, max_q_len: int, max_kv_len: int,
+                     sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, impl: str = "auto"):
+    """Causal prefill over a tied cache ``k`` [pages, page_size, Hkv, D] / ``k_scale`` [pages, page_size] (GPU, bf16, head dim
+    in ``TIED_TENSOR_CORE_DIMS``): ``q`` [T, Hq, D] carries the score scale.  ``sink`` fp32 [Hq] adds exp(sink) to every
+    denominator, ``gate`` [T, Hq D] multiplies the output by its sigmoid.  tcgen05 for head dim 128 from
+    ``SM100_PREFILL_MIN_Q`` rows on, else mma.sync (``impl``: "auto" / "sm100" / "mma")."""
+    lib = _native.load(True)
+    if impl == "sm100" or (impl == "auto" and q.shape[-1] == 128 and max_q_len >= SM100_PREFILL_MIN_Q):
+        out, err = lib.flash_fwd_sm100(q, k, k, block_table, cu_seqlens_q, kv_lens, q_pos0, int(max_q_len), int(max_kv_len),
+                                       True, 1.0, None, k_scale, sink, gate)
+        _PENDING_ERRORS.append(err)
+        if len(_PENDING_ERRORS) > 64:
+            check_attention_errors()
+        return out
+    return lib.flash_fwd(q, k, k, block_table, cu_seqlens_q, kv_lens, q_pos0, int(max_q_len), True, 1.0, 0.0, None, k_scale,
+                         sink, gate)
+
+
+def tied_attn_decode(q: torch.Tensor, k: torch.Tensor, k_scale: torch.Tensor, block_table: torch.Tensor, kv_lens: torch.Tensor,
+                     block: int, splits: int, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None):
+    """One query token per sequence over a tied cache (split-KV, merge, sink and gate in one launch).  ``block`` > 0: the
+    query sees only its own block of ``block`` positions, kept at row ``position % block`` of its page."""
+    B, Hq, D = q.shape
+    Hkv = k.shape[2]
+    ws = decode_workspace(B, Hq, D, splits, q.device)
+    out = torch.empty_like(q)
+    counters = _decode_counters(q.device, B * Hkv * ((Hq // Hkv + 15) // 16))
+    _native.load(True).decode_attn(q, k, k, block_table, kv_lens, ws, int(splits), 1.0, 0.0, out, None, None, counters, k_scale,
+                                   sink, gate, int(block))
+    return out

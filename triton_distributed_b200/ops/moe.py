@@ -71,6 +71,79 @@ def topk_router(logits: torch.Tensor, k: int, normalize: bool = True):
     return topk_router_reference(logits, k, normalize)
 
 
+_ROUTER_COUNTERS = {}
+
+
+def _router_counters(device, n: int) -> torch.Tensor:
+    """Zeroed arrival counters of the router's selection, one buffer per device (the kernel leaves them zero)."""
+    key = (device.type, device.index)
+    buf = _ROUTER_COUNTERS.get(key)
+    if buf is None or buf.numel() < n:
+        if buf is not None:
+            _ROUTER_COUNTERS.setdefault("old", []).append(buf)    # a captured graph may still count in it
+        buf = torch.zeros(max(n, 4096), dtype=torch.int32, device=device)
+        _ROUTER_COUNTERS[key] = buf
+    return buf
+
+
+def narrow_linear(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """``x`` [T, K] @ ``w`` [N, K]^T with fp32 accumulation AND fp32 output, for a few to a few hundred columns."""
+    if _native.use_native(x, w):
+        return _native.load(True).narrow_linear(x, w)
+    return x.float() @ w.float().t()
+
+
+def sigmoid_router(x: torch.Tensor, w: torch.Tensor, k: int, shared_gate: bool = False):
+    """Router with independent scores: ``sigmoid(x @ w^T)`` in fp32, the ``k`` largest with their scores as weights (not
+    renormalised).  With ``shared_gate`` the last row of ``w`` is a gate: its sigmoid comes back as a third tensor [T].
+    Returns (ids int32 [T, k], weights fp32 [T, k], gate or None); projection and selection are one launch
+    (``csrc/router.cu``)."""
+    if _native.use_native(x, w):
+        ids, wts, gate = _native.load(True).sigmoid_router(x, w, int(k), bool(shared_gate),
+                                                           _router_counters(x.device, (x.shape[0] + 15) // 16))
+        return ids, wts, (gate if shared_gate else None)
+    s = torch.sigmoid(x.float() @ w.float().t())
+    gate = s[:, -1].contiguous() if shared_gate else None
+    wts, ids = torch.topk(s[:, :-1] if shared_gate else s, k, dim=-1)
+    return ids.to(torch.int32), wts, gate
+
+
+def relu2(x: torch.Tensor, row_weight: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``relu(row_weight * x) ** 2`` (``row_weight`` fp32 per row: a scale of the input of the bias-free projection that
+    produced ``x``)."""
+    if _native.use_native(x):
+        return _native.load(True).relu2(x.contiguous(), row_weight)
+    f = x.float() if row_weight is None else x.float() * row_weight.float().reshape(-1, 1)
+    return f.clamp_min(0).pow(2).to(x.dtype)
+
+
+EXPERT_GEMV_MAX_T = 16     # up to here streaming the chosen experts per token beats sorting into 128-row GEMM tiles
+
+
+def relu2_experts_gemv(x: torch.Tensor, up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
+                       shared_up: Optional[torch.Tensor] = None, shared_down: Optional[torch.Tensor] = None,
+                       shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """fp32 [T, K]: sum over the chosen experts of ``down relu2(up (w x))`` plus the gated shared expert, every (token,
+    expert) pair streamed on its own (two launches, ``csrc/moe_gemv.cu``): decode steps, and fp32 models of any length."""
+    T = x.shape[0]
+    if _native.use_native(x, up):
+        lib = _native.load(True)
+        step = 65535 // (ids.shape[1] + 1)
+        if T <= step:
+            return lib.expert_gemv(x, up, down, ids, weights, shared_up, shared_down, shared_gate)
+        return torch.cat([lib.expert_gemv(x[i:i + step], up, down, ids[i:i + step], weights[i:i + step], shared_up, shared_down,
+                                          None if shared_gate is None else shared_gate[i:i + step]) for i in range(0, T, step)])
+    y = torch.zeros(T, x.shape[1])
+    for e in ids.unique().tolist():
+        t, s = (ids == e).nonzero(as_tuple=True)
+        h = relu2((x[t].float() @ up[e].float().t()), weights[t, s]).to(x.dtype)
+        y.index_add_(0, t, h.float() @ down[e].float().t())
+    if shared_up is not None:
+        h = relu2(x.float() @ shared_up.float().t()).to(x.dtype).float() @ shared_down.float().t()
+        y += h if shared_gate is None else shared_gate.float().reshape(T, 1) * h
+    return y
+
+
 @dataclass
 class MoESort:
     sorted_ids: torch.Tensor    # [cap] flat (token*k+slot) per sorted row, -1 = padding

@@ -3,6 +3,10 @@
 from .tp_mlp import TP_MLP  # noqa: F401
 from .tp_attn import TP_Attn  # noqa: F401
 from .tp_moe import TP_MoE  # noqa: F401
+from .tp_layer import TPLayer  # noqa: F401
+from .tp_block_attn import TP_BlockAttn  # noqa: F401
+from .tp_gla import TP_GLA  # noqa: F401
+from .tp_sigmoid_moe import TP_SigmoidMoE  # noqa: F401
 from .ep_layer import EPAll2AllLayer, EP_MoE  # noqa: F401
 from .sp_flash_decode import SpGQAFlashDecodeAttention  # noqa: F401
 from .sp_attention import (SPAllGatherAttentionContextIntraNode, create_sp_ag_attention_context_intra_node,  # noqa: F401
