@@ -168,7 +168,8 @@ def test_tied_decode(rt, D, Hq, Hkv, splits):
 
 # ------------------------------------------------------------------ router and experts
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("T,K,E,top,gated", [(1, 64, 5, 2, True), (17, 72, 33, 1, False), (150, 512, 128, 8, True), (65, 256, 511, 32, True)])
+@pytest.mark.parametrize("T,K,E,top,gated", [(1, 64, 5, 2, True), (17, 72, 33, 1, False), (150, 512, 128, 8, True), (65, 256, 511, 32, True), (2077, 136, 130, 5, True),
+                                             (2100, 200, 300, 4, False), (4096, 64, 16, 16, True)])
 def test_sigmoid_router(rt, dtype, T, K, E, top, gated):
     from triton_distributed_b200 import ops
 

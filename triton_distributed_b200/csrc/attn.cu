@@ -78,8 +78,9 @@ __global__ void __launch_bounds__(kAttnThreads) flash_fwd_kernel(const PrefillPa
   // warp-uniform bound of the visible tokens (the branch around step() must not diverge inside a warp)
   const int warp_lim = p.causal ? min(kv_len, pos0 + row0 + warp * 16 + 16) : kv_len;
   const int nblk = (kv_end + kBlockN - 1) / kBlockN;
+  const int64_t kv_row0 = TIED ? p.kv.token_row(b, 0) : 0;
   if (nblk > 0) {
-    load_kv_block<D, TIED>(p.kv, b, hkv, 0, kv_end, smem, smem + T::kTileBytes);
+    load_kv_block<D, TIED>(p.kv, b, hkv, 0, kv_end, smem, smem + T::kTileBytes, kv_row0);
     cp_async_commit();
   }
   for (int i = 0; i < nblk; ++i) {
@@ -87,7 +88,7 @@ __global__ void __launch_bounds__(kAttnThreads) flash_fwd_kernel(const PrefillPa
     uint8_t* sV = TIED ? sK : sK + T::kTileBytes;
     if (i + 1 < nblk) {
       uint8_t* nK = smem + ((i + 1) & 1) * stage_bytes<D, TIED>();
-      load_kv_block<D, TIED>(p.kv, b, hkv, (i + 1) * kBlockN, kv_end, nK, nK + T::kTileBytes);
+      load_kv_block<D, TIED>(p.kv, b, hkv, (i + 1) * kBlockN, kv_end, nK, nK + T::kTileBytes, kv_row0);
       cp_async_commit();
       cp_async_wait<1>();
     } else {
@@ -513,7 +514,7 @@ HeadEpilogue make_epi(const AttnEpilogue& e) {
 
 cudaError_t launch_flash_fwd(const FlashFwdArgs& a, cudaStream_t stream) {
   const bool tied = a.kv.k_scale != nullptr;
-  if (a.num_q_heads % a.kv.num_kv_heads != 0) return cudaErrorInvalidValue;
+  if (a.num_q_heads % a.kv.num_kv_heads != 0 || (tied && a.kv.max_pages != 1)) return cudaErrorInvalidValue;
   PrefillParams p;
   p.q = reinterpret_cast<const __nv_bfloat16*>(a.q);
   p.out = reinterpret_cast<__nv_bfloat16*>(a.out);
@@ -562,6 +563,7 @@ namespace {
 // Shared by the local and the one-launch distributed form.  `tail` == nullptr: local.
 cudaError_t launch_splitkv_impl(const DecodeArgs& a, const DistTail* tail, cudaStream_t stream) {
   const bool tied = a.kv.k_scale != nullptr;
+  if (tied && a.kv.max_pages != 1) return cudaErrorInvalidValue;
   if (!tied && a.head_dim != 64 && a.head_dim != 128) return cudaErrorInvalidValue;
   if (a.num_q_heads % a.kv.num_kv_heads != 0 || a.splits < 1) return cudaErrorInvalidValue;
   // the epilogue belongs to the fused combine; the distributed tail has neither it nor the tied form

@@ -21,9 +21,10 @@ namespace tdb {
 namespace {
 
 constexpr int kDecodeThreads = 512;
+constexpr int kMaxParts = 16;
 
 template <typename T>
-__global__ void __launch_bounds__(kDecodeThreads) gla_decode_kernel(const GlaArgs p) {
+__global__ void __launch_bounds__(kDecodeThreads, 1) gla_decode_kernel(const GlaArgs p) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[32];
   float* s_q = sm;                 // [dk]
@@ -31,36 +32,55 @@ __global__ void __launch_bounds__(kDecodeThreads) gla_decode_kernel(const GlaArg
   float* s_d = s_k + p.dk;         // [dk] decay
   float* s_v = s_d + p.dk;         // [dv]
   float* s_o = s_v + p.dv;         // [row groups][dv]
+  float* s_z = s_o;                // [parts][dk], before s_o is used
   const int h = blockIdx.x, n = blockIdx.y;
   pdl_wait();
   pdl_launch_dependents();
-  const T* row = reinterpret_cast<const T*>(p.qkvg) + n * p.ld;
-  const int Hk = p.H * p.dk, Hv = p.H * p.dv;
-  for (int c = threadIdx.x; c < p.dk; c += kDecodeThreads) {
-    s_q[c] = to_f32(row[h * p.dk + c]) * p.q_scale;
-    s_k[c] = to_f32(row[Hk + h * p.dk + c]);
-    float z = p.a2_b[h * p.dk + c];
-    for (int r = 0; r < p.R; ++r) z = fmaf(p.a2[static_cast<int64_t>(r) * Hk + h * p.dk + c], p.a[static_cast<int64_t>(n) * p.R + r], z);
-    s_d[c] = expf(gla_log_decay(z, p.inv_tau));
-  }
-  for (int c = threadIdx.x; c < p.dv; c += kDecodeThreads) s_v[c] = to_f32(row[2 * Hk + h * p.dv + c]);
-  __syncthreads();
+  // the state rows this thread starts with are requested first: the decays are computed while they travel
   const int dv4 = p.dv >> 2;
   const int groups = kDecodeThreads / dv4;           // rows processed side by side
   const int c4 = threadIdx.x % dv4, rg = threadIdx.x / dv4;
   const bool fresh = p.pos0[n] == 0;
   float4* S = reinterpret_cast<float4*>(p.state + ((static_cast<int64_t>(p.slots[n]) * p.H + h) * p.dk) * p.dv) + c4;
+  constexpr int U = 8;
+  float4 s[U];
+  auto fetch = [&](int r0) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int r = r0 + u * groups;
+      s[u] = (r < p.dk && !fresh) ? S[static_cast<int64_t>(r) * dv4] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  };
+  if (rg < groups) fetch(rg);
+  const T* row = reinterpret_cast<const T*>(p.qkvg) + n * p.ld;
+  const int Hk = p.H * p.dk, Hv = p.H * p.dv;
+  // z = a2^T a + b: the threads of a channel share the low-rank dimension, so its loads are all in flight at once
+  const int parts = max(1, min(kDecodeThreads / p.dk, kMaxParts));
+  for (int i = threadIdx.x; i < parts * p.dk; i += kDecodeThreads) {
+    const int c = i % p.dk, part = i / p.dk;
+    float z = 0.f;
+#pragma unroll 4
+    for (int r = part; r < p.R; r += parts)
+      z = fmaf(p.a2[static_cast<int64_t>(r) * Hk + h * p.dk + c], p.a[static_cast<int64_t>(n) * p.R + r], z);
+    s_z[part * p.dk + c] = z;
+  }
+  for (int c = threadIdx.x; c < p.dk; c += kDecodeThreads) {
+    s_q[c] = to_f32(row[h * p.dk + c]) * p.q_scale;
+    s_k[c] = to_f32(row[Hk + h * p.dk + c]);
+  }
+  for (int c = threadIdx.x; c < p.dv; c += kDecodeThreads) s_v[c] = to_f32(row[2 * Hk + h * p.dv + c]);
+  __syncthreads();
+  for (int c = threadIdx.x; c < p.dk; c += kDecodeThreads) {
+    float z = p.a2_b[h * p.dk + c];
+    for (int i = 0; i < parts; ++i) z += s_z[i * p.dk + c];
+    s_d[c] = expf(gla_log_decay(z, p.inv_tau));
+  }
+  __syncthreads();
   float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
   if (rg < groups) {
     const float4 v = reinterpret_cast<const float4*>(s_v)[c4];
-    constexpr int U = 8;
     for (int r0 = rg; r0 < p.dk; r0 += groups * U) {
-      float4 s[U];
-#pragma unroll
-      for (int u = 0; u < U; ++u) {
-        const int r = r0 + u * groups;
-        s[u] = (r < p.dk && !fresh) ? S[static_cast<int64_t>(r) * dv4] : make_float4(0.f, 0.f, 0.f, 0.f);
-      }
+      if (r0 != rg) fetch(r0);
 #pragma unroll
       for (int u = 0; u < U; ++u) {
         const int r = r0 + u * groups;
@@ -238,7 +258,8 @@ cudaError_t launch_gla_decode(const GlaArgs& a, cudaStream_t s) {
   if (!args_ok(a)) return cudaErrorInvalidValue;
   if (a.N == 0) return cudaSuccess;
   const int groups = kDecodeThreads / (a.dv / 4);
-  const size_t smem = static_cast<size_t>(3 * a.dk + a.dv + groups * a.dv) * 4;
+  const int tail = groups * a.dv > kDecodeThreads + a.dk ? groups * a.dv : kDecodeThreads + a.dk;   // s_o, or s_z before it
+  const size_t smem = static_cast<size_t>(3 * a.dk + a.dv + tail) * 4;
   const dim3 grid(a.H, a.N), block(kDecodeThreads);
   return a.is_f32 ? launch_pdl(gla_decode_kernel<float>, grid, block, smem, s, a)
                   : launch_pdl(gla_decode_kernel<__nv_bfloat16>, grid, block, smem, s, a);

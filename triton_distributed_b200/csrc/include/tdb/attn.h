@@ -13,7 +13,7 @@ struct AttnKV {
   int max_pages;
   int page_size;
   int num_kv_heads;
-  // Tied form: the values are the raw (un-normed) keys.  k_cache holds them, v_cache is unused, and k_scale
+  // Tied form (mma.sync kernels: every sequence in one page, max_pages = 1): the values are the raw (un-normed) keys.  k_cache holds them, v_cache is unused, and k_scale
   // [num_pages, page_size] fp32 is the factor of a token's score (the reciprocal root mean square of its key row; the
   // norm's weight is folded into q).
   const float* k_scale = nullptr;

@@ -15,6 +15,10 @@ TDB_DEVICE void cp_async16(void* smem_dst, const void* gsrc, bool valid) {
   const uint32_t sz = valid ? 16u : 0u;  // src-size 0 -> 16 bytes of zeros
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(smem_dst)), "l"(gsrc), "r"(sz) : "memory");
 }
+TDB_DEVICE void cp_async4(void* smem_dst, const void* gsrc, bool valid) {
+  const uint32_t sz = valid ? 4u : 0u;
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_u32(smem_dst)), "l"(gsrc), "r"(sz) : "memory");
+}
 TDB_DEVICE void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N>
 TDB_DEVICE void cp_async_wait() {
@@ -53,7 +57,7 @@ struct PagedKV {
   int max_pages;
   int page_size;
   int Hkv;
-  // Tied form: v is unused, k holds the keys as projected, and k_scale [pages, page_size] the factor that turns a score
+  // Tied form (every sequence in one page: max_pages = 1): v is unused, k holds the keys as projected, and k_scale [pages, page_size] the factor that turns a score
   // against the raw key into the score against the normed one (the norm's weight is folded into the query).
   const float* k_scale = nullptr;
   TDB_DEVICE int64_t token_row(int b, int tok) const {
@@ -84,22 +88,27 @@ TDB_DEVICE float2 gate2(const __nv_bfloat16* row, int d) {
 }
 
 // Cooperative load of one 64-token K and V block (tokens [t0, t0+64) of the sequence) into shared memory.
+// TIED: row0 = kv.token_row(b, 0), looked up once by the caller.
 template <int D, bool TIED = false>
-TDB_DEVICE void load_kv_block(const PagedKV& kv, int b, int h, int t0, int kv_end, uint8_t* sK, uint8_t* sV) {
+TDB_DEVICE void load_kv_block(const PagedKV& kv, int b, int h, int t0, int kv_end, uint8_t* sK, uint8_t* sV, int64_t row0 = 0) {
   constexpr int kChunksPerRow = D / 8;
   constexpr int kPitch = Tiles<D>::kPitch;
   for (int c = threadIdx.x; c < kBlockN * kChunksPerRow; c += kAttnThreads) {
     const int r = c / kChunksPerRow, ch = c - r * kChunksPerRow;
     const int tok = t0 + r;
     const bool valid = tok < kv_end;
-    const int64_t off = valid ? kv.token_offset(b, tok, h, D) + ch * 8 : 0;
+    int64_t off = 0;
+    if constexpr (TIED) off = valid ? ((row0 + tok) * kv.Hkv + h) * D + ch * 8 : 0;
+    else off = valid ? kv.token_offset(b, tok, h, D) + ch * 8 : 0;
     cp_async16(sK + r * kPitch + ch * 16, kv.k + off, valid);
     if constexpr (!TIED) cp_async16(sV + r * kPitch + ch * 16, kv.v + off, valid);
   }
-  if constexpr (TIED) {   // plain stores: visible to the CTA after the barrier that publishes the block
+  if constexpr (TIED) {
     float* sc = reinterpret_cast<float*>(sK + Tiles<D>::kTileBytes);
-    for (int r = threadIdx.x; r < kBlockN; r += kAttnThreads)
-      sc[r] = t0 + r < kv_end ? kv.k_scale[kv.token_row(b, t0 + r)] : 0.f;
+    for (int r = threadIdx.x; r < kBlockN; r += kAttnThreads) {
+      const bool valid = t0 + r < kv_end;
+      cp_async4(sc + r, kv.k_scale + (valid ? row0 + t0 + r : 0), valid);
+    }
   }
 }
 
@@ -273,13 +282,14 @@ TDB_DEVICE void decode_splitkv_body(const DecodeParams& p, int split, int yidx, 
   w.load_q(h_lo < p.group ? qb + static_cast<int64_t>(head0 + h_lo) * D : nullptr,
            h_hi < p.group ? qb + static_cast<int64_t>(head0 + h_hi) * D : nullptr);
   const int nblk = blk1 - blk0;
+  const int64_t row0 = TIED ? p.kv.token_row(b, 0) : 0;
   // one commit group per block, empty when there is no block left, so that "all but the newest S - 1 groups are
   // complete" always means "block i has landed"
 #pragma unroll
   for (int j = 0; j < S - 1; ++j) {
     if (j < nblk) {
       uint8_t* nK = smem + j * stage_bytes<D, TIED>();
-      load_kv_block<D, TIED>(p.kv, b, hkv, (blk0 + j) * kBlockN, kv_len, nK, nK + T::kTileBytes);
+      load_kv_block<D, TIED>(p.kv, b, hkv, (blk0 + j) * kBlockN, kv_len, nK, nK + T::kTileBytes, row0);
     }
     cp_async_commit();
   }
@@ -288,7 +298,7 @@ TDB_DEVICE void decode_splitkv_body(const DecodeParams& p, int split, int yidx, 
     uint8_t* sV = TIED ? sK : sK + T::kTileBytes;
     if (i + S - 1 < nblk) {
       uint8_t* nK = smem + ((i + S - 1) % S) * stage_bytes<D, TIED>();
-      load_kv_block<D, TIED>(p.kv, b, hkv, (blk0 + i + S - 1) * kBlockN, kv_len, nK, nK + T::kTileBytes);
+      load_kv_block<D, TIED>(p.kv, b, hkv, (blk0 + i + S - 1) * kBlockN, kv_len, nK, nK + T::kTileBytes, row0);
     }
     cp_async_commit();
     cp_async_wait<S - 1>();

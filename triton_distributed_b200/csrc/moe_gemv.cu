@@ -36,23 +36,52 @@ __global__ void relu2_kernel(const T* in, const float* __restrict__ w, T* out, i
   }
 }
 
+// Eight weights on their way from global memory.
+template <typename T>
+struct Raw8;
+template <>
+struct Raw8<__nv_bfloat16> {
+  uint4 v;
+  TDB_DEVICE void load(const __nv_bfloat16* p) { v = ld_nc_v4(p); }
+  TDB_DEVICE float dot(const float (&x)[8]) const {
+    const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y), c = unpack_bf16x2(v.z), d = unpack_bf16x2(v.w);
+    return fmaf(a.x, x[0], fmaf(a.y, x[1], fmaf(b.x, x[2], b.y * x[3]))) + fmaf(c.x, x[4], fmaf(c.y, x[5], fmaf(d.x, x[6], d.y * x[7])));
+  }
+};
+template <>
+struct Raw8<float> {
+  float4 a, b;
+  TDB_DEVICE void load(const float* p) {
+    a = reinterpret_cast<const float4*>(p)[0];
+    b = reinterpret_cast<const float4*>(p)[1];
+  }
+  TDB_DEVICE float dot(const float (&x)[8]) const {
+    return fmaf(a.x, x[0], fmaf(a.y, x[1], fmaf(a.z, x[2], a.w * x[3]))) + fmaf(b.x, x[4], fmaf(b.y, x[5], fmaf(b.z, x[6], b.w * x[7])));
+  }
+};
+
 constexpr int kWarps = 8;
+constexpr int kMaxTop = 64;
 
 // acc[r] += row r of w (R rows, n columns) . xs over the warp's lanes (not reduced)
 template <typename T, int R>
 TDB_DEVICE void rows_dot(const T* w, int64_t ldw, const T* xs, int n, int rows, float (&acc)[R]) {
   const int lane = threadIdx.x & 31;
-#pragma unroll 2
-  for (int c = lane * 8; c < n; c += 256) {
-    float x[8];
-    load8(xs + c, x);
+  constexpr int U = sizeof(T) == 2 ? 4 : 2;     // steps whose weight loads are in flight together
+  for (int c0 = lane * 8; c0 < n; c0 += 256 * U) {
+    Raw8<T> v[U][R];
 #pragma unroll
-    for (int r = 0; r < R; ++r) {
-      if (r >= rows) break;
-      float v[8];
-      load8(w + r * ldw + c, v);
+    for (int u = 0; u < U; ++u)
 #pragma unroll
-      for (int i = 0; i < 8; ++i) acc[r] = fmaf(v[i], x[i], acc[r]);
+      for (int r = 0; r < R; ++r)
+        if (c0 + u * 256 < n) v[u][r].load(w + (r < rows ? r : 0) * ldw + c0 + u * 256);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      if (c0 + u * 256 >= n) break;
+      float x[8];
+      load8(xs + c0 + u * 256, x);
+#pragma unroll
+      for (int r = 0; r < R; ++r) acc[r] += v[u][r].dot(x);
     }
   }
 }
@@ -71,12 +100,6 @@ __global__ void __launch_bounds__(kWarps * 32) expert_up_kernel(const ExpertGemv
   pdl_wait();
   pdl_launch_dependents();
   if (blockIdx.x * kWarps * kUpRows >= F) return;
-  const T* x = reinterpret_cast<const T*>(p.x) + t * p.K;
-  for (int c = threadIdx.x * 8; c < p.K; c += kWarps * 256) {
-    float f[8];
-    load8(x + c, f);
-    store8(xs + c, f);
-  }
   int e = 0;
   float wgt = 1.f;
   if (!shared) {
@@ -84,13 +107,18 @@ __global__ void __launch_bounds__(kWarps * 32) expert_up_kernel(const ExpertGemv
     wgt = p.weights[t * p.top + s];
     if (e < 0 || e >= p.E) e = 0, wgt = 0.f;
   }
+  const T* x = reinterpret_cast<const T*>(p.x) + t * p.K;
+  for (int c = threadIdx.x * 8; c < p.K; c += kWarps * 256) {
+    float f[8];
+    load8(x + c, f);
+    store8(xs + c, f);
+  }
   const T* w = shared ? reinterpret_cast<const T*>(p.shared_up) : reinterpret_cast<const T*>(p.up) + static_cast<int64_t>(e) * p.F * p.K;
   __syncthreads();
   if (r0 >= F) return;
   const int rows = min(kUpRows, F - r0);
   float acc[kUpRows] = {};
-  if (rows == kUpRows) rows_dot<T, kUpRows>(w + static_cast<int64_t>(r0) * p.K, p.K, xs, p.K, kUpRows, acc);
-  else rows_dot<T, kUpRows>(w + static_cast<int64_t>(r0) * p.K, p.K, xs, p.K, rows, acc);
+  rows_dot<T, kUpRows>(w + static_cast<int64_t>(r0) * p.K, p.K, xs, p.K, rows, acc);
   T* act = reinterpret_cast<T*>(p.act) + t * (static_cast<int64_t>(p.top) * p.F + p.Fs) + static_cast<int64_t>(s) * p.F;
 #pragma unroll
   for (int r = 0; r < kUpRows; ++r) {
@@ -104,10 +132,15 @@ template <typename T>
 __global__ void __launch_bounds__(kWarps * 32) expert_down_kernel(const ExpertGemvArgs p) {
   extern __shared__ __align__(16) uint8_t smem[];
   T* as = reinterpret_cast<T*>(smem);          // [top * F + Fs]
+  __shared__ int s_ids[kMaxTop];
   const int64_t t = blockIdx.y;
   const int n_act = p.top * p.F + p.Fs;
   pdl_wait();
   pdl_launch_dependents();
+  if (threadIdx.x < p.top) {
+    const int e = p.ids[t * p.top + threadIdx.x];
+    s_ids[threadIdx.x] = (e >= 0 && e < p.E) ? e : 0;     // an id out of range got the activation zero
+  }
   const T* act = reinterpret_cast<const T*>(p.act) + t * n_act;
   for (int c = threadIdx.x * 8; c < n_act; c += kWarps * 256) {
     float f[8];
@@ -118,22 +151,40 @@ __global__ void __launch_bounds__(kWarps * 32) expert_down_kernel(const ExpertGe
   const int r0 = (blockIdx.x * kWarps + (threadIdx.x >> 5)) * kDownRows;
   if (r0 >= p.K) return;
   const int rows = min(kDownRows, p.K - r0);
-  float acc[kDownRows] = {}, sh[kDownRows] = {};
-  for (int s = 0; s < p.top; ++s) {
-    const int e = p.ids[t * p.top + s];
-    if (e < 0 || e >= p.E) continue;
-    const T* w = reinterpret_cast<const T*>(p.down) + (static_cast<int64_t>(e) * p.K + r0) * p.F;
-    rows_dot<T, kDownRows>(w, p.F, as + s * p.F, p.F, rows, acc);
-  }
-  float gate = 0.f;
-  if (p.shared_down != nullptr) {
-    gate = p.shared_gate != nullptr ? p.shared_gate[t] : 1.f;
-    rows_dot<T, kDownRows>(reinterpret_cast<const T*>(p.shared_down) + static_cast<int64_t>(r0) * p.Fs, p.Fs,
-                           as + p.top * p.F, p.Fs, rows, sh);
+  const float gate = p.shared_gate != nullptr ? p.shared_gate[t] : 1.f;
+  const int n_routed = p.top * p.F;
+  float acc[kDownRows] = {};
+  // one loop over the activations of all experts of the token, so that the loads of several experts are in flight together
+  // (a vector of eight never crosses an expert: F is a multiple of eight)
+  constexpr int U = 4;
+  for (int c0 = (threadIdx.x & 31) * 8; c0 < n_act; c0 += 256 * U) {
+    Raw8<T> v[U][kDownRows];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int c = c0 + u * 256;
+      if (c >= n_act) break;
+      const bool routed = c < n_routed;
+      const int s = routed ? c / p.F : 0;
+      const T* w = routed ? reinterpret_cast<const T*>(p.down) + (static_cast<int64_t>(s_ids[s]) * p.K + r0) * p.F + (c - s * p.F)
+                          : reinterpret_cast<const T*>(p.shared_down) + static_cast<int64_t>(r0) * p.Fs + (c - n_routed);
+      const int64_t ldw = routed ? p.F : p.Fs;
+#pragma unroll
+      for (int r = 0; r < kDownRows; ++r) v[u][r].load(w + (r < rows ? r : 0) * ldw);
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int c = c0 + u * 256;
+      if (c >= n_act) break;
+      const float f = c < n_routed ? 1.f : gate;
+      float x[8];
+      load8(as + c, x);
+#pragma unroll
+      for (int r = 0; r < kDownRows; ++r) acc[r] = fmaf(f, v[u][r].dot(x), acc[r]);
+    }
   }
 #pragma unroll
   for (int r = 0; r < kDownRows; ++r) {
-    const float v = warp_sum(acc[r] + gate * sh[r]);
+    const float v = warp_sum(acc[r]);
     if ((threadIdx.x & 31) == r && r < rows) p.y[t * p.K + r0 + r] = v;
   }
 }
@@ -172,7 +223,7 @@ cudaError_t launch_relu2(const void* in, const float* row_weight, void* out, int
 }
 
 cudaError_t launch_expert_gemv(const ExpertGemvArgs& a, cudaStream_t s) {
-  if (a.K % 8 != 0 || a.F % 8 != 0 || a.Fs % 8 != 0 || a.top < 1) return cudaErrorInvalidValue;
+  if (a.K % 8 != 0 || a.F % 8 != 0 || a.Fs % 8 != 0 || a.top < 1 || a.top > kMaxTop) return cudaErrorInvalidValue;
   if ((a.shared_up == nullptr) != (a.shared_down == nullptr) || (a.shared_up == nullptr && a.Fs != 0)) return cudaErrorInvalidValue;
   if (a.T * (a.top + 1) > 65535) return cudaErrorInvalidValue;
   if (a.T == 0) return cudaSuccess;

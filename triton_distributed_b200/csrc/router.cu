@@ -8,7 +8,9 @@
 //
 // Router mode: the last column CTA of a 16-token tile to arrive reads the tile's logits back and does the selection, one
 // warp per token: scores sigmoid(z), the `top` largest (ties to the lower index) with their scores as weights, not
-// renormalised, and sigmoid of the extra column that gates a shared expert.  One launch from activations to routing.
+// renormalised, and sigmoid of the extra column that gates a shared expert.  One launch from activations to routing; from
+// 2048 tokens on, where the selection wants more warps than the projection has CTAs, two.
+#include "tdb/attn_device.cuh"
 #include "tdb/hybrid.h"
 #include "tdb/launch.cuh"
 #include "tdb/vec.cuh"
@@ -82,40 +84,35 @@ TDB_DEVICE void tile_partial(const NarrowLinearArgs& p, const float* x, const fl
   }
 }
 
+// Selection of one token by one warp; PER = experts per lane.
+template <int PER>
 TDB_DEVICE void select_token(const NarrowLinearArgs& p, int64_t t) {
   const int lane = threadIdx.x & 31;
   const float* z = p.out + t * p.N;
-  float v[kMaxPerLane];
+  uint32_t key[PER];       // scores are >= 0, so their bit patterns order like them; key = bits + 1, 0 = not a candidate
 #pragma unroll
-  for (int i = 0; i < kMaxPerLane; ++i) {
+  for (int i = 0; i < PER; ++i) {
     const int e = lane + 32 * i;
-    v[i] = e < p.E ? sigmoid_f32(__ldcg(z + e)) : -1.f;    // scores are >= 0, -1 = not a candidate
+    key[i] = e < p.E ? __float_as_uint(sigmoid_f32(__ldcg(z + e))) + 1u : 0u;
   }
   float my_w = 0.f;
   int my_id = 0;
   for (int j = 0; j < p.top; ++j) {
-    float best = -1.f;
-    int bi = 0x7fffffff;
+    uint32_t best = 0u;
 #pragma unroll
-    for (int i = 0; i < kMaxPerLane; ++i)
-      if (v[i] > best) {
-        best = v[i];
-        bi = lane + 32 * i;
-      }
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (ob > best || (ob == best && oi < bi)) {
-        best = ob;
-        bi = oi;
-      }
-    }
+    for (int i = 0; i < PER; ++i) best = max(best, key[i]);
+    best = __reduce_max_sync(0xffffffffu, best);
+    uint32_t mine = 0xffffffffu;
 #pragma unroll
-    for (int i = 0; i < kMaxPerLane; ++i)
-      if (lane + 32 * i == bi) v[i] = -1.f;
+    for (int i = PER - 1; i >= 0; --i)
+      if (key[i] == best) mine = lane + 32 * i;
+    const uint32_t id = __reduce_min_sync(0xffffffffu, mine);      // ties to the lower index
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (lane + 32 * i == static_cast<int>(id)) key[i] = 0u;
     if (lane == j) {
-      my_w = best;
-      my_id = bi;
+      my_w = __uint_as_float(best - 1u);
+      my_id = static_cast<int>(id);
     }
   }
   if (lane < p.top) {
@@ -123,6 +120,35 @@ TDB_DEVICE void select_token(const NarrowLinearArgs& p, int64_t t) {
     p.weights[t * p.top + lane] = my_w;
   }
   if (p.has_gate && lane == 0) p.gate[t] = sigmoid_f32(__ldcg(z + p.E));
+}
+TDB_DEVICE void select_any(const NarrowLinearArgs& p, int64_t t) {
+  if (p.E <= 32) select_token<1>(p, t);
+  else if (p.E <= 64) select_token<2>(p, t);
+  else if (p.E <= 128) select_token<4>(p, t);
+  else select_token<kMaxPerLane>(p, t);
+}
+
+// The selection as a launch of its own, one warp per token, after the many-token projection.
+__global__ void __launch_bounds__(256) select_kernel(const NarrowLinearArgs p) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t t = static_cast<int64_t>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  if (t < p.T) select_any(p, t);
+}
+
+// Counts this column CTA of token tile `tile` in; true for the last one, whose view of the others' outputs is then complete.
+TDB_DEVICE bool columns_arrive_last(const NarrowLinearArgs& p, int tile, int* s_last) {
+  __threadfence();
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    const uint32_t prev = atomicAdd(p.counters + tile, 1u);
+    *s_last = prev == gridDim.x - 1;
+    if (*s_last) p.counters[tile] = 0;      // every arrival has been counted: clean for the next call
+  }
+  __syncthreads();
+  if (!*s_last) return false;
+  __threadfence();
+  return true;
 }
 
 template <typename T, int NT, int WARPS>
@@ -145,18 +171,81 @@ __global__ void __launch_bounds__(WARPS * 32) narrow_linear_kernel(const NarrowL
     if (tok < p.T && col < p.N) p.out[tok * p.N + col] = s;
   }
   if (p.top < 1) return;
-  __threadfence();
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    const uint32_t prev = atomicAdd(p.counters + blockIdx.y, 1u);
-    s_last = prev == gridDim.x - 1;
-    if (s_last) p.counters[blockIdx.y] = 0;      // every arrival has been counted: clean for the next call
-  }
-  __syncthreads();
-  if (!s_last) return;
-  __threadfence();
+  if (!columns_arrive_last(p, blockIdx.y, &s_last)) return;
   for (int i = threadIdx.x >> 5; i < kTok; i += WARPS)
-    if (t0 + i < p.T) select_token(p, t0 + i);
+    if (t0 + i < p.T) select_any(p, t0 + i);
+}
+
+// ---- many tokens: 64 tokens x up to 136 columns per CTA, both operands through shared memory (cp.async, two stages of 64
+// elements of K), so that the weights are read once per 64 tokens and x once.  Each of the four warps owns 16 tokens.
+constexpr int kWideTok = 64, kWideTiles = 17, kWideCols = 8 * kWideTiles, kWideK = 64;
+constexpr int kWidePitch = kWideK + 32;     // elements: 16-byte reads of eight rows spread over all banks
+constexpr int kWideStage = (kWideTok + kWideCols) * kWidePitch * 2;
+
+__global__ void __launch_bounds__(128) narrow_linear_wide_kernel(const NarrowLinearArgs p, int cols_per_cta) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const int64_t t0 = static_cast<int64_t>(blockIdx.y) * kWideTok;
+  const int n0 = blockIdx.x * cols_per_cta, nc = min(cols_per_cta, p.N - n0);
+  const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(p.x);
+  const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(p.w);
+  pdl_wait();
+  pdl_launch_dependents();
+  auto load = [&](int slab) {
+    __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(smem + (slab & 1) * kWideStage);
+    __nv_bfloat16* ws = xs + kWideTok * kWidePitch;
+    const int k0 = slab * kWideK;
+    for (int i = threadIdx.x; i < (kWideTok + nc) * (kWideK / 8); i += 128) {
+      const int r = i / (kWideK / 8), k = k0 + (i % (kWideK / 8)) * 8;
+      if (r < kWideTok) {
+        const bool ok = k < p.K && t0 + r < p.T;
+        attn::cp_async16(xs + r * kWidePitch + (k - k0), x + (ok ? (t0 + r) * p.ldx + k : 0), ok);
+      } else {
+        const bool ok = k < p.K;
+        attn::cp_async16(ws + (r - kWideTok) * kWidePitch + (k - k0), w + (ok ? static_cast<int64_t>(n0 + r - kWideTok) * p.K + k : 0), ok);
+      }
+    }
+    attn::cp_async_commit();
+  };
+  float c[kWideTiles][4];
+#pragma unroll
+  for (int i = 0; i < kWideTiles; ++i) c[i][0] = c[i][1] = c[i][2] = c[i][3] = 0.f;
+  const int slabs = (p.K + kWideK - 1) / kWideK, tiles = (nc + 7) / 8;
+  load(0);
+  for (int s = 0; s < slabs; ++s) {
+    if (s + 1 < slabs) {
+      load(s + 1);
+      attn::cp_async_wait<1>();
+    } else {
+      attn::cp_async_wait<0>();
+    }
+    __syncthreads();
+    const __nv_bfloat16* xs = reinterpret_cast<const __nv_bfloat16*>(smem + (s & 1) * kWideStage);
+    const __nv_bfloat16* ws = xs + kWideTok * kWidePitch;
+#pragma unroll
+    for (int kb = 0; kb < kWideK / 32; ++kb) {
+      const uint4 al = *reinterpret_cast<const uint4*>(xs + (warp * 16 + g) * kWidePitch + kb * 32 + t * 8);
+      const uint4 ah = *reinterpret_cast<const uint4*>(xs + (warp * 16 + g + 8) * kWidePitch + kb * 32 + t * 8);
+#pragma unroll
+      for (int i = 0; i < kWideTiles; ++i) {
+        if (i < tiles) {     // columns of the last tile beyond nc hold stale data: their products are not stored
+          const uint4 bv = *reinterpret_cast<const uint4*>(ws + (i * 8 + g) * kWidePitch + kb * 32 + t * 8);
+          mma_16816(c[i], al.x, ah.x, al.y, ah.y, bv.x, bv.y);
+          mma_16816(c[i], al.z, ah.z, al.w, ah.w, bv.z, bv.w);
+        }
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < kWideTiles; ++i) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int64_t tok = t0 + warp * 16 + g + (e >> 1) * 8;
+      const int col = i * 8 + 2 * t + (e & 1);
+      if (tok < p.T && col < nc) p.out[tok * p.N + n0 + col] = c[i][e];
+    }
+  }
 }
 
 template <typename T, int NT, int WARPS>
@@ -177,6 +266,17 @@ cudaError_t launch_narrow_linear(const NarrowLinearArgs& a, cudaStream_t s) {
   // few tokens: as many CTAs and as much split K as the columns allow; many: wider column tiles re-read x less often
   if (a.is_f32) return launch_t<float, 1, 8>(a, s);
   if (a.T <= 64) return launch_t<__nv_bfloat16, 1, 8>(a, s);
+  if (a.T >= 2048) {
+    static SmemOptIn opt;
+    cudaError_t e = opt.ensure(narrow_linear_wide_kernel, 2 * kWideStage);
+    if (e != cudaSuccess) return e;
+    const int tiles = (a.N + 7) / 8, groups = (tiles + kWideTiles - 1) / kWideTiles;
+    const int cols = 8 * ((tiles + groups - 1) / groups);
+    e = launch_pdl(narrow_linear_wide_kernel, dim3((a.N + cols - 1) / cols, static_cast<unsigned>((a.T + kWideTok - 1) / kWideTok)),
+                      dim3(128), static_cast<size_t>(2 * kWideStage), s, a, cols);
+    if (e != cudaSuccess || a.top < 1) return e;
+    return launch_pdl(select_kernel, dim3(static_cast<unsigned>((a.T + 7) / 8)), dim3(256), 0, s, a);
+  }
   return launch_t<__nv_bfloat16, 4, 4>(a, s);
 }
 

@@ -111,3 +111,11 @@ class Qwen3MoE(DenseLLM):
         for l in self.layers[1:]:
             l.attn.gemm_ar_ctx = l0.attn.gemm_ar_ctx
             l.mlp.ag_ctx, l.mlp.rs_ctx, l.mlp.ll_ctx = l0.mlp.ag_ctx, l0.mlp.rs_ctx, l0.mlp.ll_ctx
+
+    def finalize(self):
+        l0 = self.layers[0]
+        l0.attn.finalize()
+        l0.mlp.finalize()
+        for l in self.layers[1:]:
+            l.attn.ag_ctx = l.attn.rs_ctx = l.attn.ar_ctx = l.attn.gemm_ar_ctx = None
+            l.mlp.ag_ctx = l.mlp.rs_ctx = l.mlp.ll_ctx = None

@@ -242,6 +242,14 @@ def tied_attn_varlen(q: torch.Tensor, k: torch.Tensor, k_scale: torch.Tensor, bl
                          sink, gate)
 
 
+def pick_tied_splits(batch: int, num_kv_heads: int, head_dim_chunks: int, rows: int, num_sms: int = 148) -> int:
+    """KV splits of :func:`tied_attn_decode`: like :func:`pick_kv_splits` with a walk over blocks that is twice as fast
+    (one tile per block, one page per sequence), so that a merge pays later: about sqrt(2 x blocks)."""
+    blocks = max(1, (rows + 63) // 64)
+    one_wave = max(1, (3 * num_sms) // max(1, batch * num_kv_heads * head_dim_chunks))
+    return int(max(1, min(math.ceil(math.sqrt(2.0 * blocks)), one_wave, blocks, 64)))
+
+
 def tied_attn_decode(q: torch.Tensor, k: torch.Tensor, k_scale: torch.Tensor, block_table: torch.Tensor, kv_lens: torch.Tensor,
                      block: int, splits: int, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None):
     """One query token per sequence over a tied cache (split-KV, merge, sink and gate in one launch).  ``block`` > 0: the

@@ -12,7 +12,6 @@ import torch
 import torch.distributed as dist
 
 from .. import ops
-from ..ops.attention import pick_kv_splits
 from .tp_layer import TPLayer, pad8, pad_heads, pad_rows, shard
 
 
@@ -69,7 +68,7 @@ class TP_BlockAttn(TPLayer):
             q = ops.qk_norm_tied(*norm, home, None, sumsq).reshape(T, self.q_heads, D)
             if tensor_cores:
                 rows = storage["k"].shape[1]
-                splits = pick_kv_splits(T, self.kv_heads, (self.q_heads // self.kv_heads + 15) // 16, rows)
+                splits = ops.pick_tied_splits(T, self.kv_heads, (self.q_heads // self.kv_heads + 15) // 16, rows)
                 o = ops.tied_attn_decode(q, storage["k"], storage["scale"], bp.block_table, bp.kv_lens, rows, splits, self.sink, gate)
             else:
                 o = ops.tied_attention_simple(q, storage["k"], storage["scale"], bp.row0, bp.n_keys, self.sink, gate)
