@@ -5,7 +5,7 @@
 //
 //   gla_decode_kernel     one token per sequence: decay, state update, output, norm and gate in one launch; the state is
 //                         read and written once with 16-byte accesses (what the step is bound by)
-//   gla_log_decay_kernel  log alpha of every token and channel, for the forms below
+//   gla_log_decay_kernel  log alpha of every token and channel, for the recurrent form
 //   gla_recurrent_kernel  token by token with the state in registers (a CTA owns 32 columns of one head of one sequence;
 //                         every column is shared by four lanes): the 32-bit path
 //   gla_norm_gate_kernel  norm and gate of its outputs
@@ -245,14 +245,14 @@ bool args_ok(const GlaArgs& a) {
          a.R >= 1 && a.R <= 512;
 }
 
-}  // namespace
-
 cudaError_t launch_gla_log_decay(const GlaArgs& a, cudaStream_t s) {
   const int64_t tiles = (a.T + kDecayTok - 1) / kDecayTok;
   if (tiles > 65535) return cudaErrorInvalidValue;
   return launch_pdl(gla_log_decay_kernel, dim3((a.H * a.dk + 255) / 256, static_cast<unsigned>(tiles)), dim3(256),
                     static_cast<size_t>(kDecayTok * a.R * 4), s, a);
 }
+
+}  // namespace
 
 cudaError_t launch_gla_decode(const GlaArgs& a, cudaStream_t s) {
   if (!args_ok(a)) return cudaErrorInvalidValue;

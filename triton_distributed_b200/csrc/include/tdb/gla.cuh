@@ -8,7 +8,4 @@ namespace tdb {
 // log of sigmoid(z)^(1 / tau), stable for any z.
 TDB_DEVICE float gla_log_decay(float z, float inv_tau) { return (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau; }
 
-// log_decay[T, H, dk] from the low-rank input (gla.cu).
-cudaError_t launch_gla_log_decay(const GlaArgs& a, cudaStream_t s);
-
 }  // namespace tdb
