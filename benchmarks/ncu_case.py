@@ -7,6 +7,8 @@
   python benchmarks/ncu_case.py gemm_fp8  # block-scaled e4m3 GEMM 8192 x 3584 x 8192 (pair kernel, ~150 MB)
   python benchmarks/ncu_case.py moe       # grouped GEMM with in-kernel row gather: 8192 tokens, top-2 of 16 experts, 2048 x 2048
   python benchmarks/ncu_case.py gdn       # chunk-parallel gated delta rule, 8192 tokens x 16 heads
+  python benchmarks/ncu_case.py gla       # chunk-parallel gated linear attention, 8192 tokens x 16 heads, 128 x 128 states
+  python benchmarks/ncu_case.py tied      # tied-KV block decode attention, 64 seqs x 4096 positions, 32 q heads / 4 kv heads
 """
 import sys
 
@@ -61,6 +63,26 @@ def main():
         g = F.logsigmoid(torch.rand(1, T, H, device="cuda"))
         for _ in range(2):
             ops.chunk_gated_delta_rule_fwd(q, kk, v, g, beta, K ** -0.5, impl="chunk")
+    elif case == "gla":
+        T, H, dk, dv = 8192, 16, 128, 128
+        qkvg = torch.randn(T, 2 * H * (dk + dv), device="cuda", dtype=torch.bfloat16)
+        low, a2 = torch.randn(T, 16, device="cuda"), torch.randn(16, H * dk, device="cuda")
+        bias, norm = torch.full((H * dk,), 2.0, device="cuda"), torch.ones(dv, device="cuda")
+        state = torch.zeros(1, H, dk, dv, device="cuda")
+        slot, pos0 = torch.zeros(1, dtype=torch.int32, device="cuda"), torch.zeros(1, dtype=torch.int64, device="cuda")
+        cu = torch.tensor([0, T], dtype=torch.int32, device="cuda")
+        tabs = ops.gla_chunk_tables([0, T], "cuda")
+        for _ in range(2):
+            ops.gated_linear_attention(qkvg, low, a2, bias, 16.0, norm, state, slot, pos0, cu, dv, dk ** -0.5, 1e-5, tabs)
+    elif case == "tied":
+        B, Hq, Hkv, D, L = 64, 32, 4, 128, 4096
+        k = torch.randn(B, L, Hkv, D, device="cuda", dtype=torch.bfloat16)
+        scale = torch.ones(B, L, device="cuda")
+        q = torch.randn(B, Hq, D, device="cuda", dtype=torch.bfloat16)
+        bt, lens = ops.dense_block_table(B, "cuda"), torch.full((B,), L, dtype=torch.int32, device="cuda")
+        sink = torch.zeros(Hq, device="cuda")
+        for _ in range(3):
+            ops.tied_attn_decode(q, k, scale, bt, lens, L, ops.pick_tied_splits(B, Hkv, 1, L), sink)
     elif case == "decode":
         B, Hq, Hkv, D, L = 16, 8, 1, 128, 4096
         k = torch.randn(B, L, Hkv, D, device="cuda", dtype=torch.bfloat16)

@@ -128,7 +128,7 @@ __global__ void __launch_bounds__(kWarps * 32) expert_up_kernel(const ExpertGemv
 }
 
 constexpr int kDownRows = 2;
-template <typename T>
+template <typename T, int U>     // U vectors of eight weights per row in flight: 8 for one or two tokens, where CTAs are few
 __global__ void __launch_bounds__(kWarps * 32) expert_down_kernel(const ExpertGemvArgs p) {
   extern __shared__ __align__(16) uint8_t smem[];
   T* as = reinterpret_cast<T*>(smem);          // [top * F + Fs]
@@ -156,7 +156,6 @@ __global__ void __launch_bounds__(kWarps * 32) expert_down_kernel(const ExpertGe
   float acc[kDownRows] = {};
   // one loop over the activations of all experts of the token, so that the loads of several experts are in flight together
   // (a vector of eight never crosses an expert: F is a multiple of eight)
-  constexpr int U = 4;
   for (int c0 = (threadIdx.x & 31) * 8; c0 < n_act; c0 += 256 * U) {
     Raw8<T> v[U][kDownRows];
 #pragma unroll
@@ -195,18 +194,20 @@ cudaError_t launch_experts(const ExpertGemvArgs& a, cudaStream_t s) {
   const size_t smem_up = static_cast<size_t>(a.K) * sizeof(T);
   const size_t smem_dn = static_cast<size_t>(a.top * a.F + a.Fs) * sizeof(T);
   if (smem_up > 200 * 1024 || smem_dn > 200 * 1024) return cudaErrorInvalidValue;
-  static SmemOptIn up, dn;
+  const bool few = a.T <= 2 && sizeof(T) == 2;
+  static SmemOptIn up, dn, dn8;
   cudaError_t e = up.ensure(expert_up_kernel<T>, 200 * 1024);
   if (e != cudaSuccess) return e;
-  e = dn.ensure(expert_down_kernel<T>, 200 * 1024);
+  e = few ? dn8.ensure(expert_down_kernel<T, 8>, 200 * 1024) : dn.ensure(expert_down_kernel<T, 4>, 200 * 1024);
   if (e != cudaSuccess) return e;
   const int fmax = a.F > a.Fs ? a.F : a.Fs;
   const int per_up = kWarps * kUpRows, per_dn = kWarps * kDownRows;
   e = launch_pdl(expert_up_kernel<T>, dim3((fmax + per_up - 1) / per_up, static_cast<unsigned>(a.T * slots)),
                  dim3(kWarps * 32), smem_up, s, a);
   if (e != cudaSuccess) return e;
-  return launch_pdl(expert_down_kernel<T>, dim3((a.K + per_dn - 1) / per_dn, static_cast<unsigned>(a.T)), dim3(kWarps * 32),
-                    smem_dn, s, a);
+  const dim3 grid_dn((a.K + per_dn - 1) / per_dn, static_cast<unsigned>(a.T));
+  return few ? launch_pdl(expert_down_kernel<T, 8>, grid_dn, dim3(kWarps * 32), smem_dn, s, a)
+             : launch_pdl(expert_down_kernel<T, 4>, grid_dn, dim3(kWarps * 32), smem_dn, s, a);
 }
 
 }  // namespace

@@ -42,7 +42,7 @@ TDB_DEVICE void tile_partial(const NarrowLinearArgs& p, const __nv_bfloat16* x, 
   for (int i = 0; i < NT; ++i) c[i][0] = c[i][1] = c[i][2] = c[i][3] = 0.f;
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
   const int nb = (p.K + 31) >> 5;
-#pragma unroll 4
+#pragma unroll(NT == 1 ? 8 : 4)
   for (int b = warp; b < nb; b += WARPS) {
     const int kk = b * 32 + t * 8;
     const bool ok = kk < p.K;

@@ -32,15 +32,16 @@ class AutoLLM:
 
 
 def smoke_decode():
-    """One prefill + two decode steps of a tiny Qwen3-shaped model on the current device."""
+    """One prefill + two decode steps of a tiny Qwen3-shaped model, and of a tiny layered one, on the current device."""
     import torch
 
     from ..runtime import get_runtime
 
     rt = get_runtime()
-    cfg = ModelConfig(model_name="tiny-dense", max_length=64, rank=rt.rank, world_size=rt.world_size)
-    eng = Engine(cfg)
-    eng.backend = "triton_dist_gemm_ar"
-    ids = torch.randint(0, 1000, (2, 8), device=rt.device)
-    out = eng.serve(ids, 3)
-    assert out.shape == (2, 3)
+    for name in ("tiny-dense", "tiny-vasolix"):
+        cfg = ModelConfig(model_name=name, max_length=64, rank=rt.rank, world_size=rt.world_size)
+        eng = Engine(cfg)
+        eng.backend = "triton_dist_gemm_ar"
+        ids = torch.randint(0, 1000, (2, 8), device=rt.device)
+        out = eng.serve(ids, 3)
+        assert out.shape == (2, 3)
