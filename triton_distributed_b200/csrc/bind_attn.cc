@@ -246,24 +246,28 @@ int64_t dist_decode_attn(SymmHeap& h, const at::Tensor& q, const at::Tensor& k_c
 }
 
 // Attention of every token over rows [row0, row0 + n_keys) of a tied cache, fp32 arithmetic (fp32 or bf16 tensors).
-at::Tensor tied_attn_simple(const at::Tensor& q, const at::Tensor& k, const at::Tensor& k_scale, const at::Tensor& row0,
-                            const at::Tensor& n_keys, c10::optional<at::Tensor> sink, c10::optional<at::Tensor> gate) {
+at::Tensor tied_attn_simple(const at::Tensor& q, const at::Tensor& k, c10::optional<at::Tensor> k_scale, const at::Tensor& row0,
+                            const at::Tensor& n_keys, c10::optional<at::Tensor> sink, c10::optional<at::Tensor> gate, double scale,
+                            int64_t dv, bool out_f32) {
   TORCH_CHECK(q.is_cuda() && q.dim() == 3 && q.is_contiguous() && (q.scalar_type() == at::kFloat || q.scalar_type() == at::kBFloat16),
               "tied_attn_simple: contiguous q [T, Hq, D], fp32 or bf16");
   TORCH_CHECK(k.dim() >= 3 && k.is_contiguous() && k.scalar_type() == q.scalar_type() && k.size(-1) == q.size(2),
               "tied_attn_simple: contiguous k [..., Hkv, D] of q's dtype");
-  TORCH_CHECK(k_scale.scalar_type() == at::kFloat && k_scale.is_contiguous() &&
-                  k_scale.numel() * k.size(-1) * k.size(-2) == k.numel(), "tied_attn_simple: fp32 k_scale, one per row of k");
+  TORCH_CHECK(!k_scale.has_value() || (k_scale->scalar_type() == at::kFloat && k_scale->is_contiguous() &&
+                                       k_scale->numel() * k.size(-1) * k.size(-2) == k.numel()),
+              "tied_attn_simple: fp32 k_scale, one per row of k");
   TORCH_CHECK(row0.is_cuda() && row0.scalar_type() == at::kLong && row0.is_contiguous() && row0.numel() == q.size(0),
               "tied_attn_simple: int64 row0 [T]");
   check_i32(n_keys, "n_keys");
   TORCH_CHECK(n_keys.numel() == q.size(0), "tied_attn_simple: n_keys [T]");
   c10::cuda::CUDAGuard guard(q.device());
-  at::Tensor out = at::empty_like(q);
+  const int64_t Dv = dv > 0 ? dv : q.size(2);
+  TORCH_CHECK(Dv == q.size(2) || !gate.has_value(), "tied_attn_simple: a gate needs values as wide as keys");
+  at::Tensor out = at::empty({q.size(0), q.size(1), Dv}, out_f32 ? q.options().dtype(at::kFloat) : q.options());
   tdb::TiedSimpleArgs a;
   a.q = q.data_ptr();
   a.k = k.data_ptr();
-  a.k_scale = k_scale.data_ptr<float>();
+  a.k_scale = k_scale.has_value() ? k_scale->data_ptr<float>() : nullptr;
   a.row0 = row0.data_ptr<int64_t>();
   a.n_keys = n_keys.data_ptr<int32_t>();
   a.out = out.data_ptr();
@@ -271,7 +275,10 @@ at::Tensor tied_attn_simple(const at::Tensor& q, const at::Tensor& k, const at::
   a.Hq = q.size(1);
   a.Hkv = k.size(-2);
   a.D = q.size(2);
+  a.Dv = Dv;
+  a.scale = scale;
   a.is_f32 = q.scalar_type() == at::kFloat;
+  a.out_f32 = out.scalar_type() == at::kFloat;
   a.epi = make_epilogue(q, sink, gate);
   check_cuda(tdb::launch_tied_attn_simple(a, cur_stream()), "launch_tied_attn_simple");
   return out;
@@ -292,7 +299,9 @@ void bind_attn(py::module_& m) {
         py::arg("kv_lens"), py::arg("workspace"), py::arg("splits"), py::arg("scale"), py::arg("softcap"), py::arg("out"),
         py::arg("out_lse"), py::arg("out_f32"), py::arg("counters"), py::arg("k_scale") = py::none(),
         py::arg("sink") = py::none(), py::arg("gate") = py::none(), py::arg("chunk") = 0);
-  m.def("tied_attn_simple", &tied_attn_simple);
+  m.def("tied_attn_simple", &tied_attn_simple, py::arg("q"), py::arg("k"), py::arg("k_scale"), py::arg("row0"), py::arg("n_keys"),
+        py::arg("sink") = py::none(), py::arg("gate") = py::none(), py::arg("scale") = 1.0, py::arg("dv") = 0,
+        py::arg("out_f32") = false);
   m.def("dist_decode_attn", &dist_decode_attn, py::arg("heap"), py::arg("q"), py::arg("k_cache"), py::arg("v_cache"),
         py::arg("block_table"), py::arg("kv_lens"), py::arg("workspace"), py::arg("splits"), py::arg("scale"),
         py::arg("softcap"), py::arg("out"), py::arg("staging"), py::arg("ctx"), py::arg("timeout_s"),

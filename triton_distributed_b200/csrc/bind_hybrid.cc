@@ -4,6 +4,7 @@
 #include <torch/extension.h>
 
 #include "tdb/hybrid.h"
+#include "tdb/latent.h"
 
 namespace py = pybind11;
 using OptTensor = c10::optional<at::Tensor>;
@@ -18,6 +19,7 @@ int act_f32(const at::Tensor& t, const char* name) {
   TORCH_CHECK(t.is_cuda() && (t.scalar_type() == at::kFloat || t.scalar_type() == at::kBFloat16), name, ": fp32 or bf16 CUDA tensor");
   return t.scalar_type() == at::kFloat ? 1 : 0;
 }
+int act_f32_of(const at::Tensor& t) { return act_f32(t, "y"); }
 void check_same(const at::Tensor& t, const at::Tensor& like, const char* name) {
   TORCH_CHECK(t.is_cuda() && t.scalar_type() == like.scalar_type() && t.is_contiguous(), name, ": contiguous CUDA tensor of the activation dtype");
 }
@@ -37,18 +39,18 @@ int64_t* i64(const at::Tensor& t, int64_t numel, const char* name) {
   return t.data_ptr<int64_t>();
 }
 
-void embed_stream(const at::Tensor& ids, const at::Tensor& table, at::Tensor& x, const OptTensor& xb) {
+void embed_stream(const at::Tensor& ids, const at::Tensor& table, at::Tensor& x, const OptTensor& xb, double scale) {
   const int fp = act_f32(table, "table");
   TORCH_CHECK(table.dim() == 2 && table.is_contiguous(), "embed_stream: contiguous table [V, W]");
   const int64_t T = ids.numel(), W = table.size(1);
   c10::cuda::CUDAGuard guard(table.device());
   void* b = nullptr;
-  if (!fp) {
-    TORCH_CHECK(xb.has_value() && xb->numel() == T * W, "embed_stream: bf16 copy missing");
+  if (!fp && xb.has_value()) {
+    TORCH_CHECK(xb->numel() == T * W, "embed_stream: bf16 copy [T, W]");
     check_same(*xb, table, "xb");
     b = xb->data_ptr();
   }
-  check_cuda(tdb::launch_embed_stream(i64(ids, T, "ids"), table.data_ptr(), f32(x, T * W, "x"), b, T, W, table.size(0), fp, cur_stream()),
+  check_cuda(tdb::launch_embed_stream(i64(ids, T, "ids"), table.data_ptr(), f32(x, T * W, "x"), b, T, W, table.size(0), scale, fp, cur_stream()),
              "launch_embed_stream");
 }
 
@@ -84,6 +86,63 @@ void postnorm_add(at::Tensor& x, const OptTensor& xb, const at::Tensor& y, const
   a.n_real = n_real;
   a.eps = eps;
   check_cuda(tdb::launch_postnorm_add(a, cur_stream()), "launch_postnorm_add");
+}
+
+// x += mix + (rows of y) + shared + bias and up to two norms of the new x: (h1, h2), empty where not asked for.  sum_only: the
+// sum alone, fp32 [T, W].
+std::vector<at::Tensor> parallel_add(at::Tensor& x, const OptTensor& mix, const OptTensor& y, int64_t rows, const OptTensor& ids,
+                                     const OptTensor& weights, int64_t experts, const OptTensor& hin, const OptTensor& shared,
+                                     const OptTensor& bias, const OptTensor& w1, const OptTensor& w2, int64_t n_real, double eps,
+                                     bool act_f32, bool sum_only) {
+  TORCH_CHECK(x.dim() == 2, "parallel_add: x [T, W]");
+  const int64_t T = x.size(0), W = x.size(1);
+  c10::cuda::CUDAGuard guard(x.device());
+  tdb::ParallelAddArgs a = {};
+  const auto act = x.options().dtype(act_f32 ? at::kFloat : at::kBFloat16);
+  auto in = [&](const OptTensor& t, const char* name) -> const void* {
+    if (!t.has_value()) return nullptr;
+    TORCH_CHECK(t->is_cuda() && t->scalar_type() == act.dtype() && t->is_contiguous() && t->numel() == T * W, name,
+                ": contiguous [T, W] of the activation dtype");
+    return t->data_ptr();
+  };
+  a.x = f32(x, T * W, "x");
+  a.mix = in(mix, "mix");
+  a.shared = in(shared, "shared");
+  a.hin = in(hin, "hin");
+  a.rows = rows;
+  if (y.has_value()) {
+    a.y_f32 = act_f32_of(*y);
+    TORCH_CHECK(y->is_contiguous() && y->numel() == T * rows * W, "y: contiguous [T * rows, W]");
+    a.y = y->data_ptr();
+  }
+  if (ids.has_value()) {
+    TORCH_CHECK(weights.has_value(), "parallel_add: weights missing");
+    a.ids = i32(*ids, T * rows, "ids");
+    a.weights = f32(*weights, T * rows, "weights");
+    a.experts = experts;
+  }
+  if (bias.has_value()) a.bias = f32(*bias, W, "bias");
+  a.act_f32 = act_f32 ? 1 : 0;
+  a.T = T; a.W = W; a.n_real = n_real; a.eps = eps;
+  std::vector<at::Tensor> out;
+  if (sum_only) {
+    out.push_back(at::empty({T, W}, x.options()));
+    a.sum_out = out[0].data_ptr<float>();
+  } else {
+    if (w1.has_value()) {
+      out.push_back(at::empty({T, W}, act));
+      a.w1 = f32(*w1, W, "w1");
+      a.h1 = out[0].data_ptr();
+    }
+    if (w2.has_value()) {
+      TORCH_CHECK(w1.has_value(), "parallel_add: w2 without w1");
+      out.push_back(at::empty({T, W}, act));
+      a.w2 = f32(*w2, W, "w2");
+      a.h2 = out[1].data_ptr();
+    }
+  }
+  check_cuda(tdb::launch_parallel_add(a, cur_stream()), "launch_parallel_add");
+  return out;
 }
 
 at::Tensor combine_rows(const at::Tensor& y, int64_t T, int64_t rows, const OptTensor& shared, const OptTensor& gate) {
@@ -197,24 +256,54 @@ std::vector<at::Tensor> sigmoid_router(const at::Tensor& x, const at::Tensor& w,
   return {ids, wts, gate};
 }
 
-at::Tensor relu2(const at::Tensor& in, const OptTensor& row_weight) {
+// softmax scores over all columns of w: returns (ids int32 [T, top], scores fp32 [T, top]).
+std::vector<at::Tensor> softmax_router(const at::Tensor& x, const at::Tensor& w, const at::Tensor& correction, int64_t top, int64_t groups,
+                                       int64_t keep, const at::Tensor& counters) {
+  c10::cuda::CUDAGuard guard(x.device());
+  tdb::NarrowLinearArgs a = narrow_args(x, w);
+  auto fo = x.options().dtype(at::kFloat);
+  at::Tensor z = at::empty({a.T, a.N}, fo);
+  at::Tensor ids = at::empty({a.T, top}, x.options().dtype(at::kInt));
+  at::Tensor wts = at::empty({a.T, top}, fo);
+  a.out = z.data_ptr<float>();
+  a.top = top;
+  a.E = a.N;
+  a.softmax = 1;
+  a.correction = f32(correction, a.N, "correction");
+  a.groups = groups;
+  a.keep = keep;
+  a.ids = ids.data_ptr<int32_t>();
+  a.weights = wts.data_ptr<float>();
+  a.counters = reinterpret_cast<uint32_t*>(i32(counters, (a.T + 15) / 16, "counters"));
+  check_cuda(tdb::launch_narrow_linear(a, cur_stream()), "launch_narrow_linear(softmax router)");
+  return {ids, wts};
+}
+
+at::Tensor relu2(const at::Tensor& in, const OptTensor& row_weight, const OptTensor& bias) {
   const int fp = act_f32(in, "in");
   TORCH_CHECK(in.dim() == 2 && in.is_contiguous(), "relu2: contiguous [rows, F]");
   c10::cuda::CUDAGuard guard(in.device());
   at::Tensor out = at::empty_like(in);
   const float* w = row_weight.has_value() ? f32(*row_weight, in.size(0), "row_weight") : nullptr;
-  check_cuda(tdb::launch_relu2(in.data_ptr(), w, out.data_ptr(), in.size(0), in.size(1), fp, cur_stream()), "launch_relu2");
+  const float* b = bias.has_value() ? f32(*bias, in.size(1), "bias") : nullptr;
+  check_cuda(tdb::launch_relu2(in.data_ptr(), w, b, out.data_ptr(), in.size(0), in.size(1), fp, cur_stream()), "launch_relu2");
   return out;
 }
 
 at::Tensor expert_gemv(const at::Tensor& x, const at::Tensor& up, const at::Tensor& down, const at::Tensor& ids, const at::Tensor& weights,
-                       const OptTensor& shared_up, const OptTensor& shared_down, const OptTensor& shared_gate) {
+                       const OptTensor& shared_up, const OptTensor& shared_down, const OptTensor& shared_gate, bool gated, int64_t identity,
+                       bool skip_identity) {
   tdb::ExpertGemvArgs a = {};
   a.is_f32 = act_f32(x, "x");
   TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && up.dim() == 3 && down.dim() == 3, "expert_gemv: x [T, K], up [E, F, K], down [E, K, F]");
   check_same(up, x, "up");
   check_same(down, x, "down");
-  a.T = x.size(0); a.K = x.size(1); a.E = up.size(0); a.F = up.size(1);
+  a.gated = gated ? 1 : 0;
+  a.identity = identity;
+  a.skip_identity = skip_identity ? 1 : 0;
+  const int64_t rows = gated ? 2 : 1;
+  TORCH_CHECK(up.size(1) % rows == 0, "expert_gemv: gated weights come in pairs of rows");
+  a.T = x.size(0); a.K = x.size(1); a.E = up.size(0); a.F = up.size(1) / rows;
   TORCH_CHECK(up.size(2) == a.K && down.size(0) == a.E && down.size(1) == a.K && down.size(2) == a.F, "expert_gemv: shape mismatch");
   TORCH_CHECK(ids.dim() == 2 && ids.size(0) == a.T, "expert_gemv: ids [T, top]");
   a.top = ids.size(1);
@@ -224,8 +313,8 @@ at::Tensor expert_gemv(const at::Tensor& x, const at::Tensor& up, const at::Tens
     TORCH_CHECK(shared_down.has_value(), "expert_gemv: shared_down missing");
     check_same(*shared_up, x, "shared_up");
     check_same(*shared_down, x, "shared_down");
-    a.Fs = shared_up->size(0);
-    TORCH_CHECK(shared_up->size(1) == a.K && shared_down->size(0) == a.K && shared_down->size(1) == a.Fs, "expert_gemv: shared shapes");
+    a.Fs = shared_up->size(0) / rows;
+    TORCH_CHECK(shared_up->size(1) == a.K && shared_down->size(0) == a.K && shared_down->size(1) == a.Fs && shared_up->size(0) == a.Fs * rows, "expert_gemv: shared shapes");
     a.shared_up = shared_up->data_ptr();
     a.shared_down = shared_down->data_ptr();
     if (shared_gate.has_value()) a.shared_gate = f32(*shared_gate, a.T, "shared_gate");
@@ -238,6 +327,85 @@ at::Tensor expert_gemv(const at::Tensor& x, const at::Tensor& up, const at::Tens
   a.y = y.data_ptr<float>();
   check_cuda(tdb::launch_expert_gemv(a, cur_stream()), "launch_expert_gemv");
   return y;
+}
+
+// ---- latent attention
+tdb::LatentPrepArgs latent_args(const at::Tensor& z, int64_t H, int64_t d, int64_t r, const OptTensor& norm_w, int64_t R, int64_t R_real,
+                                double eps, const at::Tensor& cos_sin, const at::Tensor& pos, const OptTensor& cache, const OptTensor& rows,
+                                const OptTensor& ctx, const OptTensor& ctx_rows) {
+  tdb::LatentPrepArgs a = {};
+  a.is_f32 = act_f32(z, "z");
+  TORCH_CHECK(z.dim() == 2 && z.stride(1) == 1, "latent: z [T, columns]");
+  a.z = z.data_ptr();
+  a.ld = z.stride(0);
+  a.T = z.size(0);
+  a.H = H; a.d = d; a.r = r; a.R = R; a.R_real = R_real;
+  a.eps = eps;
+  a.n_pos = cos_sin.size(0);
+  TORCH_CHECK(cos_sin.dim() == 2 && cos_sin.size(1) == r, "latent: cos_sin [positions, r]");
+  a.cos_sin = f32(cos_sin, a.n_pos * r, "cos_sin");
+  a.pos = i64(pos, a.T, "pos");
+  a.own_kv = norm_w.has_value() ? 1 : 0;
+  TORCH_CHECK(z.size(1) >= H * (d + r) + (a.own_kv ? R + r : 0), "latent: z has too few columns");
+  auto dest = [&](const OptTensor& c, const OptTensor& ri, void*& base, const int64_t*& rp, int64_t& cap, const char* name) {
+    check_same(*c, z, name);
+    TORCH_CHECK(c->size(-1) == R + r && ri.has_value(), name, ": rows of R + r");
+    base = c->data_ptr();
+    cap = c->numel() / (R + r);
+    rp = i64(*ri, a.T, "rows");
+  };
+  if (a.own_kv) {
+    TORCH_CHECK(cache.has_value(), "latent: cache missing");
+    a.norm_w = f32(*norm_w, R, "norm_w");
+    dest(cache, rows, a.cache, a.rows, a.cap, "cache");
+    if (ctx.has_value()) dest(ctx, ctx_rows, a.ctx, a.ctx_rows, a.ctx_cap, "ctx");
+  }
+  return a;
+}
+
+void latent_rotate(at::Tensor& z, int64_t H, int64_t d, int64_t r, const OptTensor& norm_w, int64_t R, int64_t R_real, double eps,
+                   const at::Tensor& cos_sin, const at::Tensor& pos, const OptTensor& cache, const OptTensor& rows, const OptTensor& ctx,
+                   const OptTensor& ctx_rows) {
+  c10::cuda::CUDAGuard guard(z.device());
+  tdb::LatentPrepArgs a = latent_args(z, H, d, r, norm_w, R, R_real, eps, cos_sin, pos, cache, rows, ctx, ctx_rows);
+  check_cuda(tdb::launch_latent_rotate(a, cur_stream()), "launch_latent_rotate");
+}
+
+at::Tensor latent_absorb(const at::Tensor& z, const at::Tensor& uk_t, int64_t r, const OptTensor& norm_w, int64_t R_real, double eps,
+                         const at::Tensor& cos_sin, const at::Tensor& pos, const OptTensor& cache, const OptTensor& rows) {
+  TORCH_CHECK(uk_t.dim() == 3, "latent_absorb: uk_t [H, R, d]");
+  check_same(uk_t, z, "uk_t");
+  const int64_t H = uk_t.size(0), R = uk_t.size(1);
+  c10::cuda::CUDAGuard guard(z.device());
+  tdb::LatentPrepArgs a = latent_args(z, H, uk_t.size(2), r, norm_w, R, R_real, eps, cos_sin, pos, cache, rows, c10::nullopt, c10::nullopt);
+  at::Tensor q = at::empty({a.T, H, R + r}, z.options());
+  a.uk_t = uk_t.data_ptr();
+  a.q_eff = q.data_ptr();
+  check_cuda(tdb::launch_latent_absorb(a, cur_stream()), "launch_latent_absorb");
+  return q;
+}
+
+at::Tensor latent_out(const at::Tensor& o, const OptTensor& ml, const at::Tensor& uv, const at::Tensor& gate) {
+  tdb::LatentOutArgs a = {};
+  TORCH_CHECK(uv.dim() == 3 && o.dim() >= 3, "latent_out: uv [H, dv, R], o [T, H, splits, R]");
+  a.is_f32 = act_f32(uv, "uv");
+  check_same(uv, uv, "uv");
+  a.H = uv.size(0); a.dv = uv.size(1); a.R = uv.size(2);
+  a.T = o.size(0);
+  a.splits = o.dim() == 4 ? o.size(2) : 1;
+  a.o = f32(o, a.T * a.H * static_cast<int64_t>(a.splits) * a.R, "o");
+  TORCH_CHECK(o.size(1) == a.H && o.size(-1) == a.R, "latent_out: o does not fit uv");
+  if (ml.has_value()) a.ml = f32(*ml, a.T * a.H * static_cast<int64_t>(a.splits) * 2, "ml");
+  TORCH_CHECK(gate.is_cuda() && gate.scalar_type() == uv.scalar_type() && gate.dim() == 2 && gate.stride(1) == 1 && gate.size(0) == a.T &&
+                  gate.size(1) >= static_cast<int64_t>(a.H) * a.dv, "latent_out: gate [T, H * dv]");
+  a.uv = uv.data_ptr();
+  a.gate = gate.data_ptr();
+  a.ld_gate = gate.stride(0);
+  c10::cuda::CUDAGuard guard(o.device());
+  at::Tensor out = at::empty({a.T, static_cast<int64_t>(a.H) * a.dv}, uv.options());
+  a.out = out.data_ptr();
+  check_cuda(tdb::launch_latent_out(a, cur_stream()), "launch_latent_out");
+  return out;
 }
 
 // form: 0 decode (one token per sequence), 1 recurrent, 2 chunk-parallel
@@ -310,8 +478,15 @@ void bind_hybrid(py::module_& m) {
   m.def("qk_sumsq", &qk_sumsq);
   m.def("narrow_linear", &narrow_linear);
   m.def("sigmoid_router", &sigmoid_router);
-  m.def("relu2", &relu2);
-  m.def("expert_gemv", &expert_gemv);
+  m.def("softmax_router", &softmax_router);
+  m.def("relu2", &relu2, py::arg("in"), py::arg("row_weight"), py::arg("bias") = py::none());
+  m.def("expert_gemv", &expert_gemv, py::arg("x"), py::arg("up"), py::arg("down"), py::arg("ids"), py::arg("weights"), py::arg("shared_up"),
+        py::arg("shared_down"), py::arg("shared_gate"), py::arg("gated") = false, py::arg("identity") = 0,
+        py::arg("skip_identity") = false);
+  m.def("parallel_add", &parallel_add);
+  m.def("latent_rotate", &latent_rotate);
+  m.def("latent_absorb", &latent_absorb);
+  m.def("latent_out", &latent_out);
   m.def("gla_forward", &gla_forward);
   m.def("gla_chunk_supported", &tdb::gla_chunk_supported);
 }

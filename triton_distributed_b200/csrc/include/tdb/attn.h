@@ -82,18 +82,21 @@ struct DecodeArgs {
   int chunk = 0;                       // > 0: block-local attention, see DecodeParams
 };
 
-// Attention in plain fp32 arithmetic over the tied form, for any head dim up to 512 and fp32 or bf16 tensors: one warp
-// per (token, head).  Token t sees the rows [row0[t], row0[t] + n_keys[t]) of k (viewed as [rows, Hkv, D]).
+// Attention in plain fp32 arithmetic over the tied form, for any head dim up to 1024 and fp32 or bf16 tensors: one warp
+// per (token, head).  Token t sees the rows [row0[t], row0[t] + n_keys[t]) of k (viewed as [rows, Hkv, D]); its value is the
+// first Dv elements of a row (a row may end in a part that is key only).
 struct TiedSimpleArgs {
   const void* q;               // [T, Hq, D]
   const void* k;               // [rows, Hkv, D]
-  const float* k_scale;        // [rows]
+  const float* k_scale;        // [rows], null = 1
   const int64_t* row0;         // [T]
   const int32_t* n_keys;       // [T]
-  void* out;                   // [T, Hq, D]
+  void* out;                   // [T, Hq, Dv]
   int64_t T;
-  int Hq, Hkv, D;
-  int is_f32;                  // dtype of q / k / gate / out
+  int Hq, Hkv, D, Dv;
+  float scale;                 // of the scores, beside k_scale
+  int is_f32;                  // dtype of q / k / gate
+  int out_f32;                 // dtype of out
   AttnEpilogue epi;
 };
 cudaError_t launch_tied_attn_simple(const TiedSimpleArgs& a, cudaStream_t stream);

@@ -1,6 +1,6 @@
 // Host API of the kernels that layered ("hybrid") decoders add: an fp32 residual stream with norms on the sublayers'
-// outputs, whole-projection q / k norms over a tied KV cache, sigmoid routers, pair-wise expert GEMV, gated linear
-// attention.  `is_f32` selects fp32 activations / weights, else bf16; everything that says fp32 is fp32 in both.
+// outputs or on the stream itself (parallel layers), whole-projection q / k norms over a tied KV cache, routers, pair-wise
+// expert GEMV, gated linear attention.  `is_f32` selects fp32 activations / weights, else bf16; everything that says fp32 is fp32 in both.
 #pragma once
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -8,9 +8,9 @@
 namespace tdb {
 
 // ---- residual stream (stream_ops.cu); W a multiple of 8, columns >= n_real are zero and do not count in the norms
-// x[t] = table[ids[t]] in fp32, and its bf16 copy xb (null when is_f32).
+// x[t] = scale * table[ids[t]] in fp32, and its bf16 copy xb (null = none).
 cudaError_t launch_embed_stream(const int64_t* ids, const void* table, float* x, void* xb, int64_t T, int W, int64_t vocab,
-                                int is_f32, cudaStream_t s);
+                                float scale, int is_f32, cudaStream_t s);
 struct PostNormArgs {
   float* x;               // [T, W] residual stream, updated in place: x += rmsnorm(y) * w
   void* xb;               // [T, W] bf16 copy of the new x, null = none
@@ -28,6 +28,29 @@ cudaError_t launch_postnorm_add(const PostNormArgs& a, cudaStream_t s);
 // out[t] = sum of the token's rows + gate * shared, without norm (what tensor-parallel ranks exchange).
 cudaError_t launch_combine_rows(const PostNormArgs& a, void* out, cudaStream_t s);
 // out[i] = rmsnorm(x[rows[i]]) * w (rows null: identity), fp32 or bf16 output.
+// Parallel layers, x += mixer + feed-forward, and the two norms of the new x that the next layer reads.
+struct ParallelAddArgs {
+  float* x;               // [T, W]
+  const void* mix;        // [T, W] activation dtype, null = none
+  const void* y;          // [T * rows, W]: rows of a token are summed; null = none
+  int y_f32, rows;
+  const int32_t* ids;     // [T, rows] experts of the rows (null = all rows count): a row with an id outside [0, experts) is
+  const float* weights;   // not read, weights * hin stands in for it
+  int experts;
+  const void* hin;        // [T, W] activation dtype
+  const void* shared;     // [T, W] activation dtype, null = none
+  const float* bias;      // [W] fp32, null = none
+  float* sum_out;         // non-null: the sum goes there and nothing else happens (what tensor-parallel ranks exchange)
+  const float* w1;        // [W] fp32: h1 = rmsnorm(x) * w1 ...
+  void* h1;               // activation dtype; null = no norm
+  const float* w2;        // ... and h2 (null = one norm only)
+  void* h2;
+  int act_f32;
+  int64_t T;
+  int W, n_real;
+  float eps;
+};
+cudaError_t launch_parallel_add(const ParallelAddArgs& a, cudaStream_t s);
 cudaError_t launch_stream_norm(const float* x, const int64_t* rows, const float* w, void* out, int64_t n, int W, int n_real,
                                float eps, int out_f32, cudaStream_t s);
 
@@ -69,19 +92,29 @@ struct NarrowLinearArgs {
   int32_t* ids;           // [T, top]
   float* weights;         // [T, top] sigmoid scores of the chosen experts
   float* gate;            // [T] sigmoid of the gate logit
+  // scores: independent sigmoids, or a softmax over the E logits; the choice is by score + correction[e] (null = 0), only
+  // inside the `keep` best of `groups` equal groups of neighbours (a group counts as its best choice score; 0 = no groups).
+  // The weights are the scores without the correction.
+  int softmax;
+  const float* correction;
+  int groups, keep;
   uint32_t* counters;     // one per 16 tokens, zero; left zero
 };
 cudaError_t launch_narrow_linear(const NarrowLinearArgs& a, cudaStream_t s);
 
-// ---- experts y = W_down relu(W_up (w h))^2 (moe_gemv.cu)
-// in place or to out: out = (relu(w[row] * in))^2; weight null = 1
-cudaError_t launch_relu2(const void* in, const float* row_weight, void* out, int64_t rows, int F, int is_f32, cudaStream_t s);
+// ---- experts (moe_gemv.cu): y = W_down relu(W_up (w h))^2, or gated y = w W_down (silu(W_gate h) * (W_up h))
+// in place or to out: out = (relu(w[row] * in + bias))^2; weight null = 1, bias null = 0
+cudaError_t launch_relu2(const void* in, const float* row_weight, const float* bias, void* out, int64_t rows, int F, int is_f32,
+                         cudaStream_t s);
 struct ExpertGemvArgs {
   const void* x;          // [T, K]
+  int gated;              // up then holds [E, 2 F, K]: gate rows before up rows (shared_up likewise)
   const void* up;         // [E, F, K]
   const void* down;       // [E, K, F]
   const int32_t* ids;     // [T, top]
-  const float* weights;   // [T, top]: multiplies the expert's input
+  const float* weights;   // [T, top]: multiplies the expert's input (gated: its output)
+  int identity;           // ids E .. E + identity - 1 are experts whose output is x itself (gated form) ...
+  int skip_identity;      // ... and that another rank adds
   const void* shared_up;  // [Fs, K] or null
   const void* shared_down;  // [K, Fs]
   const float* shared_gate; // [T]

@@ -7,9 +7,10 @@
 // loads deliver them, so both operands stream straight from global memory (the x tile is re-read from L2 per column tile).
 //
 // Router mode: the last column CTA of a 16-token tile to arrive reads the tile's logits back and does the selection, one
-// warp per token: scores sigmoid(z), the `top` largest (ties to the lower index) with their scores as weights, not
-// renormalised, and sigmoid of the extra column that gates a shared expert.  One launch from activations to routing; from
-// 2048 tokens on, where the selection wants more warps than the projection has CTAs, two.
+// warp per token: scores sigmoid(z) or softmax(z), the `top` largest choice scores (score + correction, inside the best
+// groups; ties to the lower index) with their scores as weights, not renormalised, and sigmoid of the extra column that gates
+// a shared expert.  One launch from activations to routing; from 2048 tokens on, where the selection wants more warps than the
+// projection has CTAs, two.
 #include "tdb/attn_device.cuh"
 #include "tdb/hybrid.h"
 #include "tdb/launch.cuh"
@@ -84,34 +85,87 @@ TDB_DEVICE void tile_partial(const NarrowLinearArgs& p, const float* x, const fl
   }
 }
 
+// Bit pattern that orders like the float (negative ones too), never 0 for a number.
+TDB_DEVICE uint32_t order_key(float v) {
+  const uint32_t b = __float_as_uint(v);
+  return (b & 0x80000000u) != 0u ? ~b : b | 0x80000000u;
+}
+
+// Index of the largest key of the warp, ties to the lower index; lane l holds the keys l, l + 32, ...
+template <int PER>
+TDB_DEVICE uint32_t best_of(const uint32_t (&key)[PER]) {
+  uint32_t best = 0u, mine = 0xffffffffu;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) best = max(best, key[i]);
+  best = __reduce_max_sync(0xffffffffu, best);
+#pragma unroll
+  for (int i = PER - 1; i >= 0; --i)
+    if (key[i] == best) mine = (threadIdx.x & 31) + 32 * i;
+  return __reduce_min_sync(0xffffffffu, mine);
+}
+
 // Selection of one token by one warp; PER = experts per lane.
 template <int PER>
 TDB_DEVICE void select_token(const NarrowLinearArgs& p, int64_t t) {
   const int lane = threadIdx.x & 31;
   const float* z = p.out + t * p.N;
-  uint32_t key[PER];       // scores are >= 0, so their bit patterns order like them; key = bits + 1, 0 = not a candidate
+  float score[PER];
+  uint32_t key[PER];       // orders like the choice score; 0 = not a candidate
+  if (p.softmax) {
+    float m = -INFINITY, l = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      score[i] = lane + 32 * i < p.E ? __ldcg(z + lane + 32 * i) : -INFINITY;
+      m = fmaxf(m, score[i]);
+    }
+    m = warp_max(m);
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      score[i] = expf(score[i] - m);
+      l += score[i];
+    }
+    l = warp_sum(l);
+#pragma unroll
+    for (int i = 0; i < PER; ++i) score[i] /= l;
+  } else {
+#pragma unroll
+    for (int i = 0; i < PER; ++i) score[i] = lane + 32 * i < p.E ? sigmoid_f32(__ldcg(z + lane + 32 * i)) : 0.f;
+  }
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     const int e = lane + 32 * i;
-    key[i] = e < p.E ? __float_as_uint(sigmoid_f32(__ldcg(z + e))) + 1u : 0u;
+    key[i] = e < p.E ? order_key(score[i] + (p.correction != nullptr ? p.correction[e] : 0.f)) : 0u;
+  }
+  if (p.groups > 0 && p.keep < p.groups) {
+    // the group of the best expert outside the groups found so far is the next best group
+    const int size = p.E / p.groups;
+    uint32_t open[PER];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) open[i] = key[i];
+    for (int j = 0; j < p.keep; ++j) {
+      const int grp = static_cast<int>(best_of<PER>(open)) / size;
+#pragma unroll
+      for (int i = 0; i < PER; ++i)
+        if ((lane + 32 * i) / size == grp) open[i] = 0u;
+    }
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (open[i] != 0u) key[i] = 0u;
   }
   float my_w = 0.f;
   int my_id = 0;
   for (int j = 0; j < p.top; ++j) {
-    uint32_t best = 0u;
-#pragma unroll
-    for (int i = 0; i < PER; ++i) best = max(best, key[i]);
-    best = __reduce_max_sync(0xffffffffu, best);
-    uint32_t mine = 0xffffffffu;
-#pragma unroll
-    for (int i = PER - 1; i >= 0; --i)
-      if (key[i] == best) mine = lane + 32 * i;
-    const uint32_t id = __reduce_min_sync(0xffffffffu, mine);      // ties to the lower index
+    const uint32_t id = best_of<PER>(key);
+    float w = 0.f;
 #pragma unroll
     for (int i = 0; i < PER; ++i)
-      if (lane + 32 * i == static_cast<int>(id)) key[i] = 0u;
+      if (lane + 32 * i == static_cast<int>(id)) {
+        key[i] = 0u;
+        w = score[i];
+      }
+    w = __shfl_sync(0xffffffffu, w, id & 31);
     if (lane == j) {
-      my_w = __uint_as_float(best - 1u);
+      my_w = w;
       my_id = static_cast<int>(id);
     }
   }
@@ -260,7 +314,8 @@ cudaError_t launch_narrow_linear(const NarrowLinearArgs& a, cudaStream_t s) {
   if (a.K % 8 != 0 || a.ldx % 8 != 0 || a.N < 1) return cudaErrorInvalidValue;
   if ((a.T + kTok - 1) / kTok > 65535) return cudaErrorInvalidValue;
   if (a.top > 0 && (a.top > 32 || a.top > a.E || a.E > 32 * kMaxPerLane || a.counters == nullptr ||
-                    a.N != a.E + (a.has_gate ? 1 : 0)))
+                    a.N != a.E + (a.has_gate ? 1 : 0) ||
+                    (a.groups > 0 && (a.E % a.groups != 0 || a.keep < 1 || a.keep > a.groups || a.top > a.E / a.groups * a.keep))))
     return cudaErrorInvalidValue;
   if (a.T == 0) return cudaSuccess;
   // few tokens: as many CTAs and as much split K as the columns allow; many: wider column tiles re-read x less often

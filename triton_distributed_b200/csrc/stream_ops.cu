@@ -1,6 +1,7 @@
 // Residual-stream kernels of decoders that keep the stream in fp32 and norm a sublayer's OUTPUT before adding it:
 // embedding into the stream, x += RMSNorm(y) * w (y summed over a token's expert rows and a gated shared row on the
-// way), and the norm in front of the head.  The stream has a bf16 copy that the next sublayer's GEMMs read.
+// way), and the norm in front of the head.  Of parallel layers that norm the stream itself: x += mixer + feed-forward and both
+// norms of the next layer in one pass.  The stream has a bf16 copy that the next sublayer's GEMMs read.
 // One block per token, 32-byte accesses, the row is kept in shared memory between the two passes.
 #include "tdb/hybrid.h"
 #include "tdb/launch.cuh"
@@ -12,13 +13,15 @@ namespace {
 
 template <typename T>
 __global__ void embed_stream_kernel(const int64_t* __restrict__ ids, const T* __restrict__ table, float* __restrict__ x,
-                                    T* __restrict__ xb, int W, int64_t vocab) {
+                                    T* __restrict__ xb, int W, int64_t vocab, float scale) {
   const int64_t t = blockIdx.x;
   int64_t id = ids[t];
   if (id < 0 || id >= vocab) id = 0;
   for (int c = threadIdx.x * 8; c < W; c += blockDim.x * 8) {
     float f[8];
     load8(table + id * W + c, f);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) f[i] *= scale;
     store8(x + t * W + c, f);
     if (xb != nullptr) store8(xb + t * W + c, f);
   }
@@ -114,6 +117,76 @@ __global__ void stream_norm_kernel(const float* __restrict__ x, const int64_t* _
   }
 }
 
+// One block per token; the new row stays in shared memory between the two passes.
+template <typename TA, typename TY>
+__global__ void parallel_add_kernel(const ParallelAddArgs p) {
+  __shared__ float red[32];
+  extern __shared__ float row[];       // [W]
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t t = blockIdx.x, at = t * p.W;
+  const TA* mix = reinterpret_cast<const TA*>(p.mix);
+  const TA* shared = reinterpret_cast<const TA*>(p.shared);
+  const TA* hin = reinterpret_cast<const TA*>(p.hin);
+  const TY* y = reinterpret_cast<const TY*>(p.y) + at * p.rows;
+  float ss = 0.f;
+  for (int c = threadIdx.x * 8; c < p.W; c += blockDim.x * 8) {
+    float a[8] = {}, f[8];
+    auto add = [&](float w) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) a[i] = fmaf(w, f[i], a[i]);
+    };
+    if (mix != nullptr) {
+      load8(mix + at + c, f);
+      add(1.f);
+    }
+    if (p.y != nullptr)
+      for (int r = 0; r < p.rows; ++r) {
+        const int e = p.ids != nullptr ? p.ids[t * p.rows + r] : 0;
+        if (p.ids == nullptr || (e >= 0 && e < p.experts)) {
+          load8(y + static_cast<int64_t>(r) * p.W + c, f);
+          add(1.f);
+        } else if (hin != nullptr) {
+          load8(hin + at + c, f);
+          add(p.weights[t * p.rows + r]);
+        }
+      }
+    if (shared != nullptr) {
+      load8(shared + at + c, f);
+      add(1.f);
+    }
+    if (p.bias != nullptr) {
+      load8(p.bias + c, f);
+      add(1.f);
+    }
+    if (p.sum_out != nullptr) {
+      store8(p.sum_out + at + c, a);
+      continue;
+    }
+    load8(p.x + at + c, f);
+    add(1.f);
+    if (mix != nullptr || p.y != nullptr) store8(p.x + at + c, a);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss += a[i] * a[i];
+    store8(row + c, a);
+  }
+  if (p.sum_out != nullptr || p.h1 == nullptr) return;
+  const float inv = 1.f / sqrtf(block_reduce_sum(ss, red) / p.n_real + p.eps);
+  for (int c = threadIdx.x * 8; c < p.W; c += blockDim.x * 8) {
+    float a[8], w[8], o[8];
+    load8(row + c, a);
+    load8(p.w1 + c, w);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) o[i] = a[i] * inv * w[i];
+    store8(reinterpret_cast<TA*>(p.h1) + at + c, o);
+    if (p.h2 == nullptr) continue;
+    load8(p.w2 + c, w);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) o[i] = a[i] * inv * w[i];
+    store8(reinterpret_cast<TA*>(p.h2) + at + c, o);
+  }
+}
+
 int row_threads(int W) {
   const int vec = W / 8;
   return vec >= 512 ? 512 : vec >= 256 ? 256 : vec >= 128 ? 128 : 64;
@@ -122,15 +195,15 @@ int row_threads(int W) {
 }  // namespace
 
 cudaError_t launch_embed_stream(const int64_t* ids, const void* table, float* x, void* xb, int64_t T, int W, int64_t vocab,
-                                int is_f32, cudaStream_t s) {
+                                float scale, int is_f32, cudaStream_t s) {
   if (W % 8 != 0) return cudaErrorInvalidValue;
   if (T == 0) return cudaSuccess;
   if (is_f32)
     embed_stream_kernel<float><<<static_cast<unsigned>(T), row_threads(W), 0, s>>>(
-        ids, reinterpret_cast<const float*>(table), x, nullptr, W, vocab);
+        ids, reinterpret_cast<const float*>(table), x, nullptr, W, vocab, scale);
   else
     embed_stream_kernel<__nv_bfloat16><<<static_cast<unsigned>(T), row_threads(W), 0, s>>>(
-        ids, reinterpret_cast<const __nv_bfloat16*>(table), x, reinterpret_cast<__nv_bfloat16*>(xb), W, vocab);
+        ids, reinterpret_cast<const __nv_bfloat16*>(table), x, reinterpret_cast<__nv_bfloat16*>(xb), W, vocab, scale);
   return cudaGetLastError();
 }
 
@@ -156,6 +229,26 @@ cudaError_t launch_combine_rows(const PostNormArgs& a, void* out, cudaStream_t s
   const dim3 grid(static_cast<unsigned>(a.T)), block(row_threads(a.W));
   return a.y_f32 ? launch_pdl(combine_rows_kernel<float>, grid, block, 0, s, a, reinterpret_cast<float*>(out))
                  : launch_pdl(combine_rows_kernel<__nv_bfloat16>, grid, block, 0, s, a, reinterpret_cast<__nv_bfloat16*>(out));
+}
+
+cudaError_t launch_parallel_add(const ParallelAddArgs& a, cudaStream_t s) {
+  if (a.W % 8 != 0 || a.n_real < 1 || (a.y != nullptr && a.rows < 1) || (a.act_f32 && a.y != nullptr && !a.y_f32) ||
+      (a.ids != nullptr && a.weights == nullptr) || (a.h1 != nullptr && a.w1 == nullptr) || (a.h2 != nullptr && a.w2 == nullptr))
+    return cudaErrorInvalidValue;
+  if (a.T == 0) return cudaSuccess;
+  const size_t smem = static_cast<size_t>(a.W) * 4;
+  if (smem > 200 * 1024) return cudaErrorInvalidValue;
+  static SmemOptIn ff, bf, bb;
+  if (smem > 40 * 1024) {
+    cudaError_t e = a.act_f32 ? ff.ensure(parallel_add_kernel<float, float>, 200 * 1024)
+                    : a.y_f32 ? bf.ensure(parallel_add_kernel<__nv_bfloat16, float>, 200 * 1024)
+                              : bb.ensure(parallel_add_kernel<__nv_bfloat16, __nv_bfloat16>, 200 * 1024);
+    if (e != cudaSuccess) return e;
+  }
+  const dim3 grid(static_cast<unsigned>(a.T)), block(row_threads(a.W));
+  return a.act_f32 ? launch_pdl(parallel_add_kernel<float, float>, grid, block, smem, s, a)
+         : a.y_f32 ? launch_pdl(parallel_add_kernel<__nv_bfloat16, float>, grid, block, smem, s, a)
+                   : launch_pdl(parallel_add_kernel<__nv_bfloat16, __nv_bfloat16>, grid, block, smem, s, a);
 }
 
 cudaError_t launch_stream_norm(const float* x, const int64_t* rows, const float* w, void* out, int64_t n, int W, int n_real,

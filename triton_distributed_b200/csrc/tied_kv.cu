@@ -5,8 +5,9 @@
 //
 //   qk_norm_tied_kernel     one block per token: both sums of squares, the scaled query, the raw key row and its factor
 //                           into up to two cache destinations
-//   tied_attn_simple_kernel fp32 arithmetic, one warp per (token, head), any head dim up to 512, fp32 or bf16 tensors:
-//                           the 32-bit path and the check of the tensor-core kernels in attn.cu / attn_sm100.cu
+//   tied_attn_simple_kernel fp32 arithmetic, one warp per (token, head), any head dim up to 1024, fp32 or bf16 tensors:
+//                           the 32-bit path and the check of the tensor-core kernels in attn.cu / attn_sm100.cu; values
+//                           may be a leading part of the row (latent attention)
 #include "tdb/attn.h"
 #include "tdb/hybrid.h"
 #include "tdb/launch.cuh"
@@ -85,11 +86,10 @@ __global__ void qk_sumsq_kernel(const QkNormArgs p, float* out) {
   }
 }
 
-constexpr int kSimpleMaxD = 512;
+constexpr int kSimpleMaxD = 1024;
 
-template <typename T>
+template <typename T, typename TO, int kPer>     // kPer elements of a row per lane
 __global__ void __launch_bounds__(128) tied_attn_simple_kernel(const TiedSimpleArgs p) {
-  constexpr int kPer = kSimpleMaxD / 32;
   pdl_wait();
   pdl_launch_dependents();
   const int64_t wid = static_cast<int64_t>(blockIdx.x) * 4 + (threadIdx.x >> 5);
@@ -122,7 +122,7 @@ __global__ void __launch_bounds__(128) tied_attn_simple_kernel(const TiedSimpleA
       kf[i] = (i < per && d < p.D) ? to_f32(kr[d]) : 0.f;
       s = fmaf(qf[i], kf[i], s);
     }
-    s = warp_sum(s) * p.k_scale[row0 + j];
+    s = warp_sum(s) * (p.k_scale != nullptr ? p.k_scale[row0 + j] * p.scale : p.scale);
     const float mn = fmaxf(m, s);
     const float corr = expf(m - mn), e = expf(s - mn);   // m = -inf -> 0
     l = l * corr + e;
@@ -131,18 +131,26 @@ __global__ void __launch_bounds__(128) tied_attn_simple_kernel(const TiedSimpleA
     for (int i = 0; i < kPer; ++i) o[i] = fmaf(e, kf[i], o[i] * corr);
   }
   const float inv = l > 0.f ? 1.f / l : 0.f;
-  T* out = reinterpret_cast<T*>(p.out) + wid * p.D;
+  TO* out = reinterpret_cast<TO*>(p.out) + wid * p.Dv;
   const T* gate = p.epi.gate != nullptr
-                      ? reinterpret_cast<const T*>(p.epi.gate) + t * p.epi.ld_gate + static_cast<int64_t>(h) * p.D
+                      ? reinterpret_cast<const T*>(p.epi.gate) + t * p.epi.ld_gate + static_cast<int64_t>(h) * p.Dv
                       : nullptr;
 #pragma unroll
   for (int i = 0; i < kPer; ++i) {
     const int d = lane + 32 * i;
-    if (i < per && d < p.D) {
+    if (i < per && d < p.Dv) {
       const float g = gate != nullptr ? sigmoid_f32(to_f32(gate[d])) : 1.f;
-      out[d] = from_f32<T>(o[i] * inv * g);
+      out[d] = from_f32<TO>(o[i] * inv * g);
     }
   }
+}
+
+template <typename T, typename TO>
+cudaError_t launch_simple(const TiedSimpleArgs& a, cudaStream_t s) {
+  const dim3 grid(static_cast<unsigned>((a.T * a.Hq + 3) / 4));
+  return a.D <= 256   ? launch_pdl(tied_attn_simple_kernel<T, TO, 8>, grid, dim3(128), 0, s, a)
+         : a.D <= 512 ? launch_pdl(tied_attn_simple_kernel<T, TO, 16>, grid, dim3(128), 0, s, a)
+                      : launch_pdl(tied_attn_simple_kernel<T, TO, kSimpleMaxD / 32>, grid, dim3(128), 0, s, a);
 }
 
 int norm_threads(int n) { return n >= 2048 ? 256 : n >= 1024 ? 128 : 64; }
@@ -172,11 +180,10 @@ cudaError_t launch_qk_sumsq(const QkNormArgs& a, float* out, cudaStream_t s) {
 }
 
 cudaError_t launch_tied_attn_simple(const TiedSimpleArgs& a, cudaStream_t s) {
-  if (a.D < 1 || a.D > kSimpleMaxD || a.Hkv < 1 || a.Hq % a.Hkv != 0) return cudaErrorInvalidValue;
+  if (a.D < 1 || a.D > kSimpleMaxD || a.Dv < 1 || a.Dv > a.D || a.Hkv < 1 || a.Hq % a.Hkv != 0) return cudaErrorInvalidValue;
   if (a.T == 0) return cudaSuccess;
-  const dim3 grid(static_cast<unsigned>((a.T * a.Hq + 3) / 4));
-  return a.is_f32 ? launch_pdl(tied_attn_simple_kernel<float>, grid, dim3(128), 0, s, a)
-                  : launch_pdl(tied_attn_simple_kernel<__nv_bfloat16>, grid, dim3(128), 0, s, a);
+  if (a.is_f32) return launch_simple<float, float>(a, s);
+  return a.out_f32 ? launch_simple<__nv_bfloat16, float>(a, s) : launch_simple<__nv_bfloat16, __nv_bfloat16>(a, s);
 }
 
 }  // namespace tdb

@@ -1,19 +1,20 @@
 """Models, KV caches, weight loading and the serving engine (the reference's ``triton_dist.models``)."""
 from .config import ArchConfig, ModelConfig, PRESETS  # noqa: F401
-from .kv_cache import HybridCache, KV_Cache, PagedKVCache, StateSpec, StepPlan, TiedKVSpec  # noqa: F401
+from .kv_cache import HybridCache, KV_Cache, LatentSpec, PagedKVCache, SharedSpec, StateSpec, StepPlan, TiedKVSpec  # noqa: F401
 from .safetensors_io import SafetensorsFile, ShardedCheckpoint, save_file  # noqa: F401
 from .dense import DenseLLM, DenseLLMLayer  # noqa: F401
 from .engine import Engine  # noqa: F401
 from .qwen_moe import Qwen3MoE, Qwen3MoELayer  # noqa: F401
+from .lisenex import LISENEX_PRESETS, LisenexConfig, LisenexLLM  # noqa: F401
 from .vasolix import VASOLIX_PRESETS, VasolixConfig, VasolixLLM  # noqa: F401
 
 # "architecture" of a config.json -> (configuration class, model class); configurations without that key are read as
 # Hugging Face ones (DenseLLM / Qwen3MoE).
-ARCHITECTURES = {"Vasolix": (VasolixConfig, VasolixLLM)}
+ARCHITECTURES = {"Vasolix": (VasolixConfig, VasolixLLM), "Lisenex": (LisenexConfig, LisenexLLM)}
 
 
 def all_presets() -> dict:
-    return {**PRESETS, **VASOLIX_PRESETS}
+    return {**PRESETS, **VASOLIX_PRESETS, **LISENEX_PRESETS}
 
 
 class AutoLLM:
@@ -32,13 +33,13 @@ class AutoLLM:
 
 
 def smoke_decode():
-    """One prefill + two decode steps of a tiny Qwen3-shaped model, and of a tiny layered one, on the current device."""
+    """One prefill + two decode steps of a tiny Qwen3-shaped model, and of tiny layered ones, on the current device."""
     import torch
 
     from ..runtime import get_runtime
 
     rt = get_runtime()
-    for name in ("tiny-dense", "tiny-vasolix"):
+    for name in ("tiny-dense", "tiny-vasolix", "tiny-lisenex"):
         cfg = ModelConfig(model_name=name, max_length=64, rank=rt.rank, world_size=rt.world_size)
         eng = Engine(cfg)
         eng.backend = "triton_dist_gemm_ar"

@@ -138,6 +138,37 @@ class StateSpec:
     dv: int
 
 
+@dataclass(frozen=True)
+class LatentSpec:
+    """A layer that caches one row per token, shared by all heads: ``rank`` elements of a latent and ``rot`` of a rotated key
+    part."""
+    rank: int
+    rot: int
+
+
+@dataclass(frozen=True)
+class SharedSpec:
+    """A layer without storage of its own: it reads that of layer ``source``."""
+    source: int
+
+
+@dataclass
+class LatentPlan:
+    """What the latent-attention layers need to know about a step (see ``StepPlan.latent``)."""
+    home_rows: torch.Tensor                         # int64 [T] cache row of every token (slot * max_length + position)
+    row0: torch.Tensor                              # int64 [T] cache row of the sequence's first token
+    n_keys: torch.Tensor                            # int32 [T]
+    kv_lens: torch.Tensor                           # int32 [sequences]
+    # prompts only: the visible rows of all sequences packed one after the other, each start a multiple of 64
+    ctx_len: int = 0
+    ctx_rows: Optional[torch.Tensor] = None         # int64 [T] packed row of every token
+    ctx0: Optional[torch.Tensor] = None             # int32 [sequences]
+    q_pos0: Optional[torch.Tensor] = None           # int32 [sequences]
+    max_q: int = 0
+    carry_src: Optional[torch.Tensor] = None        # cache rows of earlier steps ...
+    carry_dst: Optional[torch.Tensor] = None        # ... and their packed rows
+
+
 @dataclass
 class BlockPlan:
     """What a tied-KV layer needs to know about a step (see ``StepPlan.blocks``); ``rows`` is the page size of its cache."""
@@ -171,6 +202,8 @@ class StepPlan:
         self.cu = None
         self._blocks: Dict[int, BlockPlan] = {}
         self._chunks = None
+        self._latent: Optional[LatentPlan] = None
+        self.contexts: Dict[int, torch.Tensor] = {}  # packed rows of the layers that later layers of the step read as well
         if not self.decode:
             cu = [0]
             for n in host[2]:
@@ -184,6 +217,38 @@ class StepPlan:
         if self._chunks is None and not self.decode:
             self._chunks = gla_chunk_tables(self.cu_host, self.slots.device)
         return self._chunks
+
+    def latent(self) -> LatentPlan:
+        if self._latent is None:
+            self._latent = self._decode_latent() if self.decode else self._prompt_latent()
+        return self._latent
+
+    def _decode_latent(self) -> LatentPlan:
+        row0 = self.slots.to(torch.int64) * self.cache.max_length
+        n = (self.positions + 1).to(torch.int32)
+        return LatentPlan(home_rows=row0 + self.positions, row0=row0, n_keys=n, kv_lens=n)
+
+    def _prompt_latent(self) -> LatentPlan:
+        slots, starts, lens = self.host
+        M, at = self.cache.max_length, 0
+        home, row0, ctx_rows, src, dst, ctx0 = [], [], [], [], [], []
+        for slot, start, n in zip(slots, starts, lens):
+            r = torch.arange(start, start + n)
+            home.append(r + slot * M)
+            row0.append(torch.full((n,), slot * M))
+            ctx_rows.append(r + at)
+            if start > 0:
+                src.append(torch.arange(start) + slot * M)
+                dst.append(torch.arange(start) + at)
+            ctx0.append(at)
+            at += (start + n + 63) // 64 * 64
+        T, N = self.num_tokens, len(lens)
+        nc = sum(starts)
+        big = torch.cat(home + row0 + ctx_rows + src + dst).to(torch.int64).to(self.slots.device)
+        small = torch.tensor([a + n for a, n in zip(starts, lens)] + ctx0 + list(starts), dtype=torch.int32).to(self.slots.device)
+        return LatentPlan(home_rows=big[:T], row0=big[T:2 * T], ctx_rows=big[2 * T:3 * T], n_keys=(self.positions + 1).to(torch.int32),
+                          carry_src=big[3 * T:3 * T + nc] if nc else None, carry_dst=big[3 * T + nc:] if nc else None,
+                          kv_lens=small[:N], ctx0=small[N:2 * N], q_pos0=small[2 * N:], ctx_len=at, max_q=max(lens))
 
     def blocks(self, spec: TiedKVSpec) -> BlockPlan:
         rows = spec.rows(self.cache.max_length)
@@ -235,7 +300,8 @@ class StepPlan:
 
 
 class HybridCache:
-    """Cache of a layered decoder: one storage per layer (``TiedKVSpec`` or ``StateSpec``), indexed by a sequence's slot.
+    """Cache of a layered decoder: one storage per layer (``TiedKVSpec``, ``LatentSpec`` or ``StateSpec``; ``SharedSpec`` layers
+    share another layer's), indexed by a sequence's slot.
 
     Slots are handed out by ``alloc`` and given back by ``free``; nothing is cleared in between, because a sequence that
     starts at position 0 neither reads its state row nor any row it has not written.  ``kv_offset`` (device) and ``lens``
@@ -265,8 +331,14 @@ class HybridCache:
                 new[:self.capacity] = t
             return new
 
-        for spec, st in zip(self.specs, self.layers):
-            if isinstance(spec, TiedKVSpec):
+        for i, (spec, st) in enumerate(zip(self.specs, self.layers)):
+            if isinstance(spec, SharedSpec):
+                if not 0 <= spec.source < i or isinstance(self.specs[spec.source], SharedSpec):
+                    raise ValueError(f"layer {i} cannot share the cache of layer {spec.source}")
+                self.layers[i] = self.layers[spec.source]
+            elif isinstance(spec, LatentSpec):
+                st["latent"] = widen(st.get("latent"), self.max_length, spec.rank + spec.rot, dtype=self.dtype)
+            elif isinstance(spec, TiedKVSpec):
                 rows = spec.rows(self.max_length)
                 st["k"] = widen(st.get("k"), rows, spec.kv_heads, spec.head_dim, dtype=self.dtype)
                 st["scale"] = widen(st.get("scale"), rows, dtype=torch.float32)

@@ -12,23 +12,18 @@ torch.float32``, fp32 throughout.
 """
 from __future__ import annotations
 
-import dataclasses
-import json
-import os
 from dataclasses import dataclass
-from typing import List, Optional, Sequence, Tuple
+from typing import Optional, Tuple
 
 import torch
 
 from .. import ops
 from ..parallel.tp_block_attn import TP_BlockAttn
 from ..parallel.tp_gla import TP_GLA
-from ..parallel.tp_sigmoid_moe import TP_SigmoidMoE
 from ..parallel.tp_layer import pad8, pad_rows
-from ..runtime import get_runtime
-from .config import ModelConfig
-from .kv_cache import HybridCache, StepPlan
-from .safetensors_io import ShardedCheckpoint
+from ..parallel.tp_sigmoid_moe import TP_SigmoidMoE
+from .kv_cache import StepPlan
+from .layered import LayeredConfig, LayeredLLM, RandomWeights, read_config
 
 
 # ------------------------------------------------------------------ configuration
@@ -97,7 +92,7 @@ class LayerSpec:
 
 
 @dataclass(frozen=True)
-class VasolixConfig:
+class VasolixConfig(LayeredConfig):
     name: str
     vocab_size: int
     hidden_size: int
@@ -105,23 +100,12 @@ class VasolixConfig:
     layers: Tuple[LayerSpec, ...]
 
     @property
-    def num_hidden_layers(self) -> int:
-        return len(self.layers)
-
-    @property
     def is_moe(self) -> bool:
         return any(l.mlp is not None for l in self.layers)
 
-    def with_num_layers(self, n: int) -> "VasolixConfig":
-        """The first ``n`` layers (the list is repeated when it is shorter)."""
-        return dataclasses.replace(self, layers=tuple(self.layers[i % len(self.layers)] for i in range(n)))
-
     @staticmethod
     def from_json(path: str) -> "VasolixConfig":
-        if os.path.isdir(path):
-            path = os.path.join(path, "config.json")
-        with open(path) as f:
-            c = json.load(f)
+        c = read_config(path)
         return VasolixConfig(c["architecture"], c["vocab"], c["width"], float(c["norm"]["eps"]),
                              tuple(LayerSpec.from_json(l) for l in c["layers"]))
 
@@ -175,111 +159,23 @@ class VasolixLayer:
             ops.postnorm_add(x, xb, y, self.norm2, self.width, self.eps, rows, shared, gate)
 
 
-class VasolixLLM:
-    """Same interface as :class:`DenseLLM` (``set_fwd``, ``init_ctx_for``, ``inference``, ``finalize``), plus packed steps
-    (``forward_step``) over a :class:`HybridCache` made by ``new_cache``."""
+class VasolixLLM(LayeredLLM):
+    def make_layers(self):
+        return [VasolixLayer(i, s, self.rank, self.world_size, self.group) for i, s in enumerate(self.arch.layers)]
 
-    def __init__(self, model_config: ModelConfig, group=None):
-        self.rt = get_runtime()
-        self.model_config = model_config
-        self.arch: VasolixConfig = model_config.arch()
-        self.rank, self.world_size = self.rt.rank, self.rt.world_size
-        self.group = group if group is not None else self.rt.group
-        self.dtype, self.device = model_config.dtype, self.rt.device
-        if self.dtype not in (torch.bfloat16, torch.float32):
-            raise ValueError("Vasolix runs in bfloat16 or float32")
-        if self.dtype == torch.float32 and self.rt.is_cuda:
-            torch.backends.cuda.matmul.allow_tf32 = False      # 32-bit means 32-bit
-        self.mode = "torch"
-        self.layers = [VasolixLayer(i, s, self.rank, self.world_size, self.group) for i, s in enumerate(self.arch.layers)]
-        self.init_parameters()
-        self.set_fwd("torch")
+    def load_head(self, get):
+        self.embed_tokens, self.lm_head = self.table(get, "embed"), self.table(get, "head")
 
-    # -- parameters -------------------------------------------------------------------------------------------
-    def init_parameters(self):
-        a, mc = self.arch, self.model_config
-        if mc.checkpoint_dir:
-            ckpt = ShardedCheckpoint(mc.checkpoint_dir)
-            get = ckpt.get
-        else:
-            ckpt, get = None, RandomWeights(a, mc.seed, self.device)
-        w8 = pad8(a.hidden_size)
-        table = lambda n: pad_rows(get(n), pad8(a.vocab_size), w8).to(self.dtype).to(self.device).contiguous()   # noqa: E731
-        self.embed_tokens = table("embed")
-        self.lm_head = table("head")
-        self.final_norm_w = pad_rows(get("final.norm").float(), w8).to(self.device)
-        for l in self.layers:
-            l.load(get, a.hidden_size, a.rms_norm_eps, self.dtype, self.device)
-        if ckpt is not None:
-            ckpt.close()
-
-    # -- modes ------------------------------------------------------------------------------------------------
-    def set_fwd(self, mode: str = "torch"):
-        self.mode = mode
-        for l in self.layers:
-            for part in l.parts():
-                part.set_fwd(mode)
-
-    def init_ctx_for(self, mode: str, max_M: int):
-        """Communication contexts of the row-parallel projections, one set for all layers (nothing to do on one rank).
-        The batch-sharded mode of the dense models runs as the all-reduce mode here."""
-        if mode == "torch" or self.world_size == 1:
-            return
-        w8 = pad8(self.arch.hidden_size)
-        first = self.layers[0].mixer
-        first.init_ctx(mode, max_M, w8)
-        for l in self.layers:
-            for part in l.parts():
-                part.ar_ctx, part.gemm_ar_ctx = first.ar_ctx, first.gemm_ar_ctx
-
-    def finalize(self):
-        self.layers[0].mixer.finalize()
-        for l in self.layers:
-            for part in l.parts():
-                part.ar_ctx = part.gemm_ar_ctx = None
-
-    def new_cache(self, batch_size: int, max_length: int, allocate: bool = True) -> HybridCache:
-        return HybridCache([l.mixer.cache_spec() for l in self.layers], batch_size, max_length, self.dtype, self.device, allocate)
-
-    # -- forward ----------------------------------------------------------------------------------------------
-    @torch.no_grad()
-    def forward_step(self, ids: torch.Tensor, plan: StepPlan, rows: Optional[torch.Tensor] = None,
-                     wo_lm_head: bool = False, streams: Optional[List[torch.Tensor]] = None) -> torch.Tensor:
-        """One step over packed tokens ``ids`` [T]: fp32 logits [len(rows), vocab] of the given token rows (None: all), or
-        the normed hidden rows.  The caller advances the cache.  ``streams`` collects the residual stream after every
-        layer (a debugging aid)."""
+    def hidden(self, ids, plan, streams):
         x, xb = ops.embed_stream(ids, self.embed_tokens)
         for l, storage in zip(self.layers, plan.cache.layers):
             l.fwd(x, xb, plan, storage)
             if streams is not None:
                 streams.append(x[:, :self.arch.hidden_size].clone())
-        h = ops.stream_norm(x, self.final_norm_w, self.arch.hidden_size, self.arch.rms_norm_eps, self.dtype, rows)
-        if wo_lm_head:
-            return h
-        logits = torch.matmul(h, self.lm_head.t()) if self.mode == "torch" else ops.gemm(h, self.lm_head)
-        return logits[:, :self.arch.vocab_size].float()
-
-    def inference(self, input_ids: torch.Tensor, position_ids: torch.Tensor, kv_cache: HybridCache, wo_lm_head: bool = False,
-                  seq_lens: Optional[Sequence[int]] = None) -> torch.Tensor:
-        """``input_ids`` [B, S] -> fp32 logits [B, vocab] of every sequence's last token.  S = 1 is a decode step at
-        ``position_ids`` (device values, graph-capturable); longer inputs continue every sequence where the cache stands,
-        right-padded to S when ``seq_lens`` gives their lengths (padding is dropped before the first layer)."""
-        B, S = input_ids.shape
-        if S == 1:
-            return self.forward_step(input_ids.reshape(-1), kv_cache.decode_plan(position_ids), None, wo_lm_head)
-        lens = [S] * B if seq_lens is None else [int(n) for n in seq_lens]
-        ids = input_ids.reshape(-1) if min(lens) == S else torch.cat([input_ids[b, :n] for b, n in enumerate(lens)])
-        plan = kv_cache.plan(range(B), lens)
-        return self.forward_step(ids, plan, None if plan.decode else plan.last_rows, wo_lm_head)
+        return x
 
 
-class RandomWeights:
-    """Random tensors with the shapes of the checkpoint format (weights ~ N(0, 1/fan_in), norms near 1)."""
-
-    def __init__(self, arch: VasolixConfig, seed: int, device):
-        self.arch, self.device = arch, device
-        self.gen = torch.Generator(device=device).manual_seed(seed)
-
+class VasolixRandomWeights(RandomWeights):
     def shape(self, name: str):
         a = self.arch
         if name in ("embed", "head"):
@@ -303,15 +199,10 @@ class RandomWeights:
         ff = spec.mlp.shared_ff if rest.startswith("shared.") else spec.mlp.ff
         return (ff, W) if rest.endswith(".up") else (W, ff)
 
-    def __call__(self, name: str) -> torch.Tensor:
-        shape = self.shape(name)
-        t = torch.randn(*shape, generator=self.gen, device=self.device)
-        if name.endswith("norm") or name.endswith(("norm1", "norm2")):
-            return (1.0 + 0.1 * t).to(torch.bfloat16)
-        if name == "embed":
-            return t.to(torch.bfloat16)
+    def value(self, name, t):
         if name.endswith("a2.b"):
-            return (t + 2.0).to(torch.bfloat16)
-        if name.endswith("sink"):
-            return t.to(torch.bfloat16)
-        return (t * shape[-1] ** -0.5).to(torch.bfloat16)
+            return t + 2.0
+        return t if name.endswith("sink") else super().value(name, t)
+
+
+VasolixLLM.random_weights = VasolixRandomWeights

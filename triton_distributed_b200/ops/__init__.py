@@ -39,6 +39,11 @@ from .fp8 import (ag_gemm_fp8, dequantize_act_1x128, dequantize_weight_128x128, 
                   gemm_rs_fp8_reference, AGGemmFp8Context, GemmRSFp8Context)
 from .moe import (tile_arrival_order, tile_schedule, sort_topk_ids_staged, group_gemm_gather,  # noqa: F401,E402
                   MoESort, MoEAgScatterGroupGemmContext, MoEReduceRSContext)
-from .stream import (embed_stream, postnorm_add, combine_rows, stream_norm, qk_sumsq, qk_norm_tied)  # noqa: F401,E402
+from .stream import (embed_stream, postnorm_add, combine_rows, stream_norm, qk_sumsq, qk_norm_tied, FeedForward,  # noqa: F401,E402
+                     parallel_add, parallel_sum)
 from .gla import gated_linear_attention, gla_chunk_tables, GLA_CHUNK  # noqa: F401,E402
-from .moe import (narrow_linear, sigmoid_router, relu2, relu2_experts_gemv, EXPERT_GEMV_MAX_T)  # noqa: F401,E402
+from .moe import (narrow_linear, sigmoid_router, softmax_router, relu2, relu2_experts_gemv, gated_experts_gemv,  # noqa: F401,E402
+                  EXPERT_GEMV_MAX_T)
+from .latent import (rope_table, latent_rotate, latent_absorb, latent_out, latent_attention, latent_prefill,  # noqa: F401,E402
+                     latent_decode, latent_prefill_supported, latent_decode_supported, pick_latent_splits,
+                     check_latent_errors)

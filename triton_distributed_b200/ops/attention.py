@@ -198,29 +198,33 @@ def merge_attention_partials(outs: torch.Tensor, lses: torch.Tensor) -> torch.Te
 TIED_TENSOR_CORE_DIMS = (32, 64, 128, 256)      # head dims of the mma.sync / tcgen05 kernels in tied form
 
 
-def _tied_attention_restatement(q, k, k_scale, row0, n_keys, sink, gate):
+def _tied_attention_restatement(q, k, k_scale, row0, n_keys, sink, gate, scale=1.0, dv=0):
     T, Hq, D = q.shape
     Hkv = k.shape[-2]
-    kf, sf = k.reshape(-1, Hkv, D), k_scale.reshape(-1)
-    out = torch.empty(T, Hq, D)
+    kf = k.reshape(-1, Hkv, D)
+    sf = torch.full((kf.shape[0],), float(scale)) if k_scale is None else k_scale.reshape(-1) * scale
+    dv = dv or D
+    out = torch.empty(T, Hq, dv)
     for t in range(T):
         lo, hi = int(row0[t]), int(row0[t]) + int(n_keys[t])
         kk = kf[lo:hi].float().repeat_interleave(Hq // Hkv, dim=1)
         s = torch.einsum("hd,nhd->hn", q[t].float(), kk) * sf[lo:hi]
         if sink is not None:
             s = torch.cat([s, sink.float().unsqueeze(1)], dim=1)
-        out[t] = torch.einsum("hn,nhd->hd", torch.softmax(s, dim=-1)[:, :hi - lo], kk)
+        out[t] = torch.einsum("hn,nhd->hd", torch.softmax(s, dim=-1)[:, :hi - lo], kk[..., :dv])
     if gate is not None:
         out *= torch.sigmoid(gate.float()).reshape(T, Hq, D)
     return out.to(q.dtype)
 
 
-def tied_attention_simple(q, k, k_scale, row0, n_keys, sink=None, gate=None):
-    """fp32-arithmetic attention over a tied cache, any head dim up to 512: token t sees rows ``row0[t] .. + n_keys[t]`` of
-    ``k`` (viewed as [rows, Hkv, D]); its score is ``q . k[row] * k_scale[row]``, its value ``k[row]``."""
+def tied_attention_simple(q, k, k_scale, row0, n_keys, sink=None, gate=None, scale: float = 1.0, dv: int = 0, out_f32: bool = False):
+    """fp32-arithmetic attention over a tied cache, any head dim up to 1024: token t sees rows ``row0[t] .. + n_keys[t]`` of
+    ``k`` (viewed as [rows, Hkv, D]); its score is ``q . k[row] * k_scale[row] * scale`` (``k_scale`` None: 1), its value the
+    first ``dv`` elements of ``k[row]`` (0: all).  ``out_f32``: the output stays in fp32."""
     if _native.use_native(q, k):
-        return _native.load(True).tied_attn_simple(q, k, k_scale, row0, n_keys, sink, gate)
-    return _tied_attention_restatement(q, k, k_scale, row0, n_keys, sink, gate)
+        return _native.load(True).tied_attn_simple(q, k, k_scale, row0, n_keys, sink, gate, float(scale), int(dv), bool(out_f32))
+    o = _tied_attention_restatement(q, k, k_scale, row0, n_keys, sink, gate, scale, dv)
+    return o.float() if out_f32 else o
 
 
 def tied_attn_varlen(q: torch.Tensor, k: torch.Tensor, k_scale: torch.Tensor, block_table: torch.Tensor,

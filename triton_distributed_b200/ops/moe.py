@@ -108,12 +108,33 @@ def sigmoid_router(x: torch.Tensor, w: torch.Tensor, k: int, shared_gate: bool =
     return ids.to(torch.int32), wts, gate
 
 
-def relu2(x: torch.Tensor, row_weight: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """``relu(row_weight * x) ** 2`` (``row_weight`` fp32 per row: a scale of the input of the bias-free projection that
-    produced ``x``)."""
+def softmax_router(x: torch.Tensor, w: torch.Tensor, correction: torch.Tensor, k: int, groups: int = 0, keep: int = 0):
+    """Router with a softmax over all rows of ``w`` (identity experts included), in fp32.  The ``k`` largest of score +
+    ``correction`` (fp32 [E]) are chosen, only inside the ``keep`` best of ``groups`` equal groups of neighbours when there are
+    groups (a group counts as its best member); the weights are the scores themselves, not renormalised.  Returns (ids int32
+    [T, k], weights fp32 [T, k]); projection and selection are one launch (``csrc/router.cu``)."""
+    if _native.use_native(x, w):
+        return tuple(_native.load(True).softmax_router(x, w, correction, int(k), int(groups), int(keep),
+                                                       _router_counters(x.device, (x.shape[0] + 15) // 16)))
+    s = torch.softmax(x.float() @ w.float().t(), dim=-1)
+    choice = s + correction
+    if groups > 0:
+        T, E = s.shape
+        best = torch.topk(choice.reshape(T, groups, -1).amax(-1), keep, dim=-1).indices
+        kept = torch.zeros(T, groups, dtype=torch.bool).scatter_(1, best, True).repeat_interleave(E // groups, dim=1)
+        choice = choice.masked_fill(~kept, float("-inf"))
+    ids = torch.topk(choice, k, dim=-1).indices
+    return ids.to(torch.int32), torch.gather(s, 1, ids)
+
+
+def relu2(x: torch.Tensor, row_weight: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``relu(row_weight * x + bias) ** 2`` (``row_weight`` fp32 per row: a scale of the input of the bias-free projection that
+    produced ``x``; ``bias`` fp32 per column)."""
     if _native.use_native(x):
-        return _native.load(True).relu2(x.contiguous(), row_weight)
+        return _native.load(True).relu2(x.contiguous(), row_weight, bias)
     f = x.float() if row_weight is None else x.float() * row_weight.float().reshape(-1, 1)
+    if bias is not None:
+        f = f + bias
     return f.clamp_min(0).pow(2).to(x.dtype)
 
 
@@ -141,6 +162,38 @@ def relu2_experts_gemv(x: torch.Tensor, up: torch.Tensor, down: torch.Tensor, id
     if shared_up is not None:
         h = relu2(x.float() @ shared_up.float().t()).to(x.dtype).float() @ shared_down.float().t()
         y += h if shared_gate is None else shared_gate.float().reshape(T, 1) * h
+    return y
+
+
+def gated_experts_gemv(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
+                       shared_gate_up: Optional[torch.Tensor] = None, shared_down: Optional[torch.Tensor] = None,
+                       identity: int = 0, skip_identity: bool = False) -> torch.Tensor:
+    """fp32 [T, K]: sum over the chosen experts of ``weight * down (silu(gate x) * (up x))`` plus the shared expert; ``gate_up``
+    [E, 2 F, K] holds the gate rows before the up rows.  Ids E .. E + ``identity`` - 1 are identity experts, ``weight * x``
+    (``skip_identity``: left to another rank).  Same launches and uses as :func:`relu2_experts_gemv`."""
+    T = x.shape[0]
+    if _native.use_native(x, gate_up):
+        lib = _native.load(True)
+        step = 65535 // (ids.shape[1] + 1)
+        if T <= step:
+            return lib.expert_gemv(x, gate_up, down, ids, weights, shared_gate_up, shared_down, None, True, int(identity), skip_identity)
+        return torch.cat([lib.expert_gemv(x[i:i + step], gate_up, down, ids[i:i + step], weights[i:i + step], shared_gate_up,
+                                          shared_down, None, True, int(identity), skip_identity) for i in range(0, T, step)])
+
+    def act(h, w):
+        g, u = (h.float() @ w.float().t()).chunk(2, dim=-1)
+        return torch.nn.functional.silu(g) * u
+
+    y = torch.zeros(T, x.shape[1])
+    for e in ids.unique().tolist():
+        t, s = (ids == e).nonzero(as_tuple=True)
+        wt = weights[t, s].unsqueeze(1)
+        if e < gate_up.shape[0]:
+            y.index_add_(0, t, (wt * act(x[t], gate_up[e])).to(x.dtype).float() @ down[e].float().t())
+        elif not skip_identity:
+            y.index_add_(0, t, wt * x[t].float())
+    if shared_gate_up is not None:
+        y += act(x, shared_gate_up).to(x.dtype).float() @ shared_down.float().t()
     return y
 
 

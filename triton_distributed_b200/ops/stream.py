@@ -1,5 +1,6 @@
-"""fp32 residual stream of decoders that norm a sublayer's output: embedding, ``x += RMSNorm(y) * w``, the norm before
-the head, and the whole-projection q / k norm that writes a tied KV cache.
+"""fp32 residual stream of layered decoders: embedding, ``x += RMSNorm(y) * w`` (norm on a sublayer's output) or ``x += mixer +
+feed-forward`` with the next layer's norms (parallel layers), the norm before the head, and the whole-projection q / k norm that
+writes a tied KV cache.
 
 The stream ``x`` [T, W] stays in fp32 for every activation dtype; ``xb`` is its bf16 copy that the next sublayer's GEMMs
 read (for fp32 models ``xb`` IS ``x``).  W may be padded: columns from ``n_real`` on are zero and do not count in means.
@@ -7,6 +8,7 @@ GPU tensors run ``csrc/stream_ops.cu`` / ``csrc/tied_kv.cu``; CPU tensors run th
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Optional, Tuple
 
 import torch
@@ -26,17 +28,16 @@ def _token_sum(y, T, rows, shared, shared_gate):
     return s
 
 
-def embed_stream(ids: torch.Tensor, table: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
-    """``(x, xb)`` of token ids [T]."""
+def embed_stream(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0, copy: bool = True):
+    """``(x, xb)`` of token ids [T]: ``x = scale * table[ids]`` in fp32 (without ``copy``, ``xb`` is None)."""
     ids = ids.reshape(-1)
     if _native.use_native(ids, table):
         x = torch.empty(ids.numel(), table.shape[1], dtype=torch.float32, device=table.device)
-        xb = x if table.dtype == torch.float32 else torch.empty_like(x, dtype=table.dtype)
-        _native.load(True).embed_stream(ids.to(torch.int64).contiguous(), table, x, None if xb is x else xb)
+        xb = None if not copy else x if table.dtype == torch.float32 else torch.empty_like(x, dtype=table.dtype)
+        _native.load(True).embed_stream(ids.to(torch.int64).contiguous(), table, x, None if xb is x else xb, float(scale))
         return x, xb
-    rows = table[ids.long()]
-    x = rows.float().clone()
-    return x, (x if table.dtype == torch.float32 else rows.clone())
+    x = table[ids.long()].float() * scale
+    return x, (None if not copy else x if table.dtype == torch.float32 else x.to(table.dtype))
 
 
 def postnorm_add(x: torch.Tensor, xb: torch.Tensor, y: torch.Tensor, w: torch.Tensor, n_real: int, eps: float,
@@ -52,6 +53,59 @@ def postnorm_add(x: torch.Tensor, xb: torch.Tensor, y: torch.Tensor, w: torch.Te
     x += s * _rms_factor(s, n_real, eps) * w
     if xb is not x:
         xb.copy_(x)
+
+
+@dataclass
+class FeedForward:
+    """What a feed-forward adds to the stream, left in pieces for :func:`parallel_add` to sum: ``rows`` rows of ``y`` per token,
+    of which those of an expert id outside [0, ``experts``) stand for ``weight * hin`` (identity experts; ``hin`` None: nothing),
+    a shared expert's rows and a bias."""
+    y: torch.Tensor
+    rows: int = 1
+    ids: Optional[torch.Tensor] = None
+    weights: Optional[torch.Tensor] = None
+    experts: int = 0
+    hin: Optional[torch.Tensor] = None
+    shared: Optional[torch.Tensor] = None
+    bias: Optional[torch.Tensor] = None
+
+
+def parallel_sum(x: torch.Tensor, mix: Optional[torch.Tensor], ff: Optional[FeedForward]) -> torch.Tensor:
+    """fp32 [T, W]: what :func:`parallel_add` would add to the stream (what tensor-parallel ranks exchange)."""
+    return _parallel(x, mix, ff, None, None, 1, 0.0, torch.float32 if mix is None else mix.dtype, True)[0]
+
+
+def parallel_add(x: torch.Tensor, mix: Optional[torch.Tensor], ff: Optional[FeedForward], w1: Optional[torch.Tensor],
+                 w2: Optional[torch.Tensor], n_real: int, eps: float, dtype: torch.dtype):
+    """In place ``x += mix + ff``; returns ``(RMSNorm(x) * w1, RMSNorm(x) * w2)`` in ``dtype``, None where the weight is None."""
+    out = _parallel(x, mix, ff, w1, w2, n_real, eps, dtype, False)
+    return tuple(out) + (None,) * (2 - len(out))
+
+
+def _parallel(x, mix, ff, w1, w2, n_real, eps, dtype, sum_only):
+    f = ff if ff is not None else FeedForward(None)
+    if _native.use_native(x):
+        return _native.load(True).parallel_add(x, mix, f.y, int(f.rows), f.ids, f.weights, int(f.experts), f.hin, f.shared, f.bias,
+                                               w1, w2, int(n_real), float(eps), dtype == torch.float32, sum_only)
+    s = torch.zeros_like(x)
+    if mix is not None:
+        s += mix.float()
+    if f.y is not None:
+        y = f.y.float().reshape(x.shape[0], f.rows, -1)
+        if f.ids is not None:
+            own = (f.ids >= 0) & (f.ids < f.experts)
+            y = torch.where(own.unsqueeze(-1), y, torch.zeros_like(y))
+            if f.hin is not None:
+                y = y + (~own).unsqueeze(-1) * f.weights.unsqueeze(-1) * f.hin.float().unsqueeze(1)
+        s += y.sum(1)
+    for t in (f.shared, f.bias):
+        if t is not None:
+            s += t.float()
+    if sum_only:
+        return [s]
+    x += s
+    r = x * _rms_factor(x, n_real, eps)
+    return [(r * w).to(dtype) for w in (w1, w2) if w is not None]
 
 
 def combine_rows(y: torch.Tensor, T: int, rows_per_token: int, shared: Optional[torch.Tensor] = None,

@@ -7,6 +7,8 @@ from .tp_layer import TPLayer  # noqa: F401
 from .tp_block_attn import TP_BlockAttn  # noqa: F401
 from .tp_gla import TP_GLA  # noqa: F401
 from .tp_sigmoid_moe import TP_SigmoidMoE  # noqa: F401
+from .tp_latent_attn import TP_LatentAttn  # noqa: F401
+from .tp_routed_ff import TP_DenseFF, TP_RoutedMoE  # noqa: F401
 from .ep_layer import EPAll2AllLayer, EP_MoE  # noqa: F401
 from .sp_flash_decode import SpGQAFlashDecodeAttention  # noqa: F401
 from .sp_attention import (SPAllGatherAttentionContextIntraNode, create_sp_ag_attention_context_intra_node,  # noqa: F401
