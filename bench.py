@@ -13,7 +13,8 @@ Arms:
                     needs the patched Triton submodule, which is empty in the mounted checkout), so this arm
                     prints an "unavailable" line
 
-``--workload hybrid`` runs another measurement instead (see benchmarks/bench_hybrid.py).
+``--workload hybrid`` and ``--workload latent`` run other measurements instead (see benchmarks/bench_hybrid.py and
+benchmarks/bench_latent.py).
 
 Prints ONE JSON line on rank 0.  Device times come from CUDA events around exactly --steps steps, max over ranks.
 """
@@ -43,10 +44,11 @@ def parse():
     ap.add_argument("--e2e-return", default="metric", choices=["metric", "full"],
                     help="what the host reads back every step: the 4-byte checksum of the output (default), or the "
                          "whole output tensor as well (PCIe-bound at small N: 128 MB per step and direction at N=1)")
-    ap.add_argument("--workload", default="tp_mlp", choices=["tp_mlp", "hybrid"],
+    ap.add_argument("--workload", default="tp_mlp", choices=["tp_mlp", "hybrid", "latent"],
                     help="tp_mlp: the headline above (default); hybrid: prefill and decode throughput of the layered decoder "
-                         "(Vasolix) beside Qwen3-MoE at equal layer sizes, one GPU, one JSON line per measurement")
-    ap.add_argument("--hybrid-size", default="30b-a3b,1b")
+                         "(Vasolix) beside Qwen3-MoE at equal layer sizes, one GPU, one JSON line per measurement; latent: the same "
+                         "for Lisenex beside Vasolix")
+    ap.add_argument("--hybrid-size", default="30b-a3b,1b", help="sizes of the hybrid / latent workloads")
     ap.add_argument("--hybrid-parts", default="prefill,decode,kernels")
     return ap.parse_args()
 
@@ -58,23 +60,23 @@ def reference_unavailable():
     return 0
 
 
-def hybrid_workload(args):
+def layered_workload(args):
     import triton_distributed_b200 as tdb
-    from benchmarks import bench_hybrid
+    from benchmarks import bench_hybrid, bench_latent
     from triton_distributed_b200.utils import ClockSampler
 
     if args.impl != "ours":
-        print(json.dumps({"impl": args.impl, "unavailable": "the hybrid workload has one arm"}))
+        print(json.dumps({"impl": args.impl, "unavailable": f"the {args.workload} workload has one arm"}))
         return 0
     tdb.initialize_distributed(seed=0)
     sampler = ClockSampler(gpu_index=tdb.get_runtime().local_rank).start()
     sampler.wait_first_sample(5.0)
     sampler.begin_window()
-    recs = bench_hybrid.run(args.hybrid_size.split(","), args.hybrid_parts.split(","))
+    recs = (bench_hybrid if args.workload == "hybrid" else bench_latent).run(args.hybrid_size.split(","), args.hybrid_parts.split(","))
     sampler.end_window()
     for r in recs:
         print(json.dumps(r), flush=True)
-    print(json.dumps({"workload": "hybrid", "records": len(recs), "data": "synthetic", "dtype": "bf16", "clocks": sampler.stop()}), flush=True)
+    print(json.dumps({"workload": args.workload, "records": len(recs), "data": "synthetic", "dtype": "bf16", "clocks": sampler.stop()}), flush=True)
     tdb.finalize_distributed()
     return 0
 
@@ -90,8 +92,8 @@ def main():
     args = parse()
     if args.impl == "reference":
         return reference_unavailable()
-    if args.workload == "hybrid":
-        return hybrid_workload(args)
+    if args.workload in ("hybrid", "latent"):
+        return layered_workload(args)
     if args.warmup < 3:
         args.warmup = 3
 

@@ -408,6 +408,69 @@ at::Tensor latent_out(const at::Tensor& o, const OptTensor& ml, const at::Tensor
   return out;
 }
 
+// Expanded form on tcgen05.  z holds the (rotated) queries, k [L, H d], ctx [L, R + r], vt [H dv, L].
+at::Tensor latent_prefill(const at::Tensor& z, const at::Tensor& k, const at::Tensor& ctx, const at::Tensor& vt, const at::Tensor& cu,
+                          const at::Tensor& q_pos0, const at::Tensor& kv_lens, const at::Tensor& ctx0, int64_t max_q, int64_t H, int64_t d,
+                          int64_t r, int64_t R, int64_t dv, double scale, const at::Tensor& gate, at::Tensor& error) {
+  TORCH_CHECK(z.is_cuda() && z.scalar_type() == at::kBFloat16 && z.dim() == 2 && z.stride(1) == 1 && z.size(1) >= H * (d + r), "latent_prefill: z");
+  check_same(k, z, "k");
+  check_same(ctx, z, "ctx");
+  check_same(vt, z, "vt");
+  tdb::LatentPrefillArgs a = {};
+  a.T = z.size(0);
+  a.L = ctx.size(0);
+  TORCH_CHECK(ctx.dim() == 2 && ctx.size(1) == R + r && k.numel() == a.L * H * d && vt.dim() == 2 && vt.size(0) == H * dv && vt.size(1) == a.L,
+              "latent_prefill: shapes");
+  TORCH_CHECK(gate.is_cuda() && gate.scalar_type() == at::kBFloat16 && gate.dim() == 2 && gate.stride(1) == 1 && gate.size(0) == a.T &&
+                  gate.size(1) >= H * dv, "latent_prefill: gate [T, H * dv]");
+  a.B = kv_lens.numel();
+  a.q = z.data_ptr();
+  a.ld_q = z.stride(0);
+  a.k = k.data_ptr();
+  a.ctx = ctx.data_ptr();
+  a.vt = vt.data_ptr();
+  a.cu = i32(cu, a.B + 1, "cu");
+  a.q_pos0 = i32(q_pos0, a.B, "q_pos0");
+  a.kv_lens = i32(kv_lens, a.B, "kv_lens");
+  a.ctx0 = i32(ctx0, a.B, "ctx0");
+  a.gate = gate.data_ptr();
+  a.ld_gate = gate.stride(0);
+  a.H = H; a.d = d; a.r = r; a.R = R; a.dv = dv; a.max_q = max_q;
+  a.scale = scale;
+  a.error_flag = i32(error, 1, "error");
+  c10::cuda::CUDAGuard guard(z.device());
+  at::Tensor out = at::empty({a.T, H * dv}, z.options());
+  a.out = out.data_ptr();
+  check_cuda(tdb::launch_latent_prefill(a, cur_stream()), "launch_latent_prefill");
+  return out;
+}
+
+// Absorbed form on tcgen05, one token per sequence: (partials fp32 [B, H, splits, R], their maxima and sums [B, H, splits, 2]).
+std::vector<at::Tensor> latent_decode(const at::Tensor& q, const at::Tensor& cache, const at::Tensor& slots, const at::Tensor& kv_lens,
+                                      int64_t R, double scale, int64_t splits, at::Tensor& error) {
+  TORCH_CHECK(q.is_cuda() && q.scalar_type() == at::kBFloat16 && q.dim() == 3 && q.is_contiguous(), "latent_decode: q [B, H, R + r] bf16");
+  check_same(cache, q, "cache");
+  TORCH_CHECK(cache.dim() == 3 && cache.size(2) == q.size(2), "latent_decode: cache [slots, max_len, R + r]");
+  tdb::LatentDecodeArgs a = {};
+  a.B = q.size(0); a.H = q.size(1); a.R = R; a.r = q.size(2) - R;
+  a.q_eff = q.data_ptr();
+  a.cache = cache.data_ptr();
+  a.slots = i32(slots, a.B, "slots");
+  a.kv_lens = i32(kv_lens, a.B, "kv_lens");
+  a.num_slots = cache.size(0);
+  a.max_len = cache.size(1);
+  a.splits = splits;
+  a.scale = scale;
+  a.error_flag = i32(error, 1, "error");
+  c10::cuda::CUDAGuard guard(q.device());
+  auto fo = q.options().dtype(at::kFloat);
+  at::Tensor o = at::empty({a.B, a.H, splits, R}, fo), ml = at::empty({a.B, a.H, splits, 2}, fo);
+  a.o = o.data_ptr<float>();
+  a.ml = ml.data_ptr<float>();
+  check_cuda(tdb::launch_latent_decode(a, cur_stream()), "launch_latent_decode");
+  return {o, ml};
+}
+
 // form: 0 decode (one token per sequence), 1 recurrent, 2 chunk-parallel
 at::Tensor gla_forward(const at::Tensor& qkvg, const at::Tensor& lowrank, const at::Tensor& a2, const at::Tensor& a2_b, double inv_tau,
                        const at::Tensor& norm_w, at::Tensor& state, const at::Tensor& slots, const at::Tensor& pos0,
@@ -487,6 +550,8 @@ void bind_hybrid(py::module_& m) {
   m.def("latent_rotate", &latent_rotate);
   m.def("latent_absorb", &latent_absorb);
   m.def("latent_out", &latent_out);
+  m.def("latent_prefill", &latent_prefill);
+  m.def("latent_decode", &latent_decode);
   m.def("gla_forward", &gla_forward);
   m.def("gla_chunk_supported", &tdb::gla_chunk_supported);
 }

@@ -13,7 +13,7 @@ rows of their own) [R latent | r key part].  All sizes are padded to multiples o
 """
 from __future__ import annotations
 
-from typing import List, Optional, Tuple
+from typing import Optional, Tuple
 
 import torch
 
@@ -21,7 +21,7 @@ from .. import _native
 from .attention import tied_attention_simple
 
 _TABLES = {}
-_PENDING: List[torch.Tensor] = []      # error flags of tcgen05 launches that have not been looked at yet
+_FLAGS = {}         # one error flag per device, set by a tcgen05 launch whose waits gave up
 
 
 def rope_table(base: float, dims: int, width: int, positions: int, device) -> torch.Tensor:
@@ -105,27 +105,56 @@ def latent_attention(q_eff: torch.Tensor, cache: torch.Tensor, row0: torch.Tenso
     return tied_attention_simple(q_eff, cache.view(-1, 1, cache.shape[-1]), None, row0, n_keys, None, None, scale, rank, True)
 
 
-def latent_prefill_supported(d: int, r: int, dv: int) -> bool:
+def latent_prefill_supported(d: int, r: int, dv: int, scale: float = 1.0) -> bool:
     """Sizes of the tcgen05 prompt kernel."""
-    return False
+    return d <= 128 and r <= 64 and dv <= 128 and scale > 0
 
 
-def latent_decode_supported(R: int, r: int) -> bool:
+def latent_decode_supported(R: int, r: int, scale: float = 1.0) -> bool:
     """Sizes of the tcgen05 decode kernel."""
-    return False
+    return R <= 512 and r <= 64 and scale > 0
+
+
+def _error_flag(device) -> torch.Tensor:
+    key = str(device)
+    if key not in _FLAGS:
+        _FLAGS[key] = torch.zeros(1, dtype=torch.int32, device=device)
+    return _FLAGS[key]
 
 
 def check_latent_errors() -> None:
-    pass
+    """Raise if a bounded wait inside a tcgen05 latent-attention kernel gave up since the last check (synchronises)."""
+    for flag in _FLAGS.values():
+        if int(flag.item()) != 0:
+            flag.zero_()
+            raise RuntimeError("latent attention: a wait inside the kernel timed out")
 
 
-def latent_prefill(*a, **k):
-    raise NotImplementedError
+def latent_prefill(z: torch.Tensor, k: torch.Tensor, ctx: torch.Tensor, vt: torch.Tensor, cu: torch.Tensor, q_pos0: torch.Tensor,
+                   kv_lens: torch.Tensor, ctx0: torch.Tensor, max_q: int, heads: int, d: int, r: int, dv: int, scale: float,
+                   gate: torch.Tensor) -> torch.Tensor:
+    """Causal prompt attention in the expanded form with the output gate, [T, H dv] (GPU, bf16, tcgen05): queries in ``z``
+    (rotated), keys ``k`` [L, H d] and the rotated part in the packed rows ``ctx`` [L, R + r], values ``vt`` [H dv, L].  Sequence b's
+    queries are rows ``cu[b] .. cu[b + 1]`` from position ``q_pos0[b]`` on, its ``kv_lens[b]`` visible tokens start at packed row
+    ``ctx0[b]`` (a multiple of 64, like L)."""
+    return _native.load(True).latent_prefill(z, k, ctx, vt, cu, q_pos0, kv_lens, ctx0, int(max_q), int(heads), int(d), int(r),
+                                             ctx.shape[1] - int(r), int(dv), float(scale), gate, _error_flag(z.device))
 
 
-def latent_decode(*a, **k):
-    raise NotImplementedError
+DECODE_TILE, DECODE_HEADS = 128, 32     # tokens per tile and heads per CTA of the decode kernel
 
 
-def pick_latent_splits(*a, **k):
-    raise NotImplementedError
+def pick_latent_splits(batch: int, heads: int, rows: int, num_sms: int = 148) -> int:
+    """KV splits of :func:`latent_decode`, one CTA per SM: as many as one wave holds, at most one per tile of tokens."""
+    tiles = max(1, (rows + DECODE_TILE - 1) // DECODE_TILE)
+    ctas = batch * ((heads + DECODE_HEADS - 1) // DECODE_HEADS)
+    return int(max(1, min(num_sms // max(1, ctas), tiles, 64)))
+
+
+def latent_decode(q_eff: torch.Tensor, cache: torch.Tensor, slots: torch.Tensor, kv_lens: torch.Tensor, rank: int, scale: float,
+                  splits: int = 0) -> Tuple[torch.Tensor, torch.Tensor]:
+    """Absorbed attention of one token per sequence over ``cache`` [slots, max_len, R + r] (GPU, bf16, tcgen05): split partials
+    and their (maximum, sum) for :func:`latent_out`."""
+    splits = splits or pick_latent_splits(q_eff.shape[0], q_eff.shape[1], cache.shape[1])
+    return tuple(_native.load(True).latent_decode(q_eff, cache, slots, kv_lens, int(rank), float(scale), int(splits),
+                                                  _error_flag(q_eff.device)))

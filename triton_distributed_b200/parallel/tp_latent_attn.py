@@ -71,10 +71,10 @@ class TP_LatentAttn(TPLayer):
         home = (rows, lp.home_rows) if self.own_kv else None
         norm = (self.norm_w, s.kv_rank, self.eps, self._table(plan), plan.positions)
         tensor_cores = x.is_cuda and x.dtype == torch.bfloat16
-        if not plan.decode and tensor_cores and ops.latent_prefill_supported(self.d, self.r, self.dv):
+        if not plan.decode and tensor_cores and ops.latent_prefill_supported(self.d, self.r, self.dv, s.scale):
             return self.linear(self._expanded(z, gate, plan, lp, rows, home, norm), self.wo)
         q = ops.latent_absorb(z, self.uk_t, self.r, *norm, home)
-        if plan.decode and tensor_cores and ops.latent_decode_supported(self.R, self.r):
+        if plan.decode and tensor_cores and ops.latent_decode_supported(self.R, self.r, s.scale):
             o, ml = ops.latent_decode(q, rows, plan.slots, lp.kv_lens, self.R, s.scale)
         else:
             o, ml = ops.latent_attention(q, rows, lp.row0, lp.n_keys, self.R, s.scale), None
@@ -83,17 +83,19 @@ class TP_LatentAttn(TPLayer):
     def _expanded(self, z, gate, plan, lp, rows, home, norm):
         norm_w, R_real, eps, table, pos = norm
         W = self.R + self.r
-        ctx = None
-        if self.own_kv:
+        ctx = None if self.own_kv else plan.contexts.get(self.source)
+        fresh = ctx is None
+        if fresh:
             ctx = torch.zeros(lp.ctx_len, W, dtype=z.dtype, device=z.device)
             if lp.carry_src is not None:
                 ctx[lp.carry_dst] = rows.view(-1, W)[lp.carry_src]
-            if self.shared:
-                plan.contexts[self.index] = ctx
+            if self.shared or not self.own_kv:
+                plan.contexts[self.source] = ctx
         ops.latent_rotate(z, self.heads, self.d, self.r, norm_w, self.R, R_real, eps, table, pos, home,
-                          None if ctx is None else (ctx, lp.ctx_rows))
-        if ctx is None:
-            ctx = plan.contexts[self.source]
+                          (ctx, lp.ctx_rows) if self.own_kv else None)
+        if fresh and not self.own_kv:              # the layer that owns the rows ran in the other form
+            ctx[lp.ctx_rows] = rows.view(-1, W)[lp.home_rows]
         k = self.linear(ctx[:, :self.R], self.uk)
         vt = self.linear(self.uv.view(-1, self.R), ctx[:, :self.R])
-        return ops.latent_prefill(z, k, ctx, vt, plan.cu, lp, self.heads, self.d, self.r, self.R, self.dv, self.spec.scale, gate)
+        return ops.latent_prefill(z, k, ctx, vt, plan.cu, lp.q_pos0, lp.kv_lens, lp.ctx0, lp.max_q, self.heads, self.d, self.r,
+                                  self.dv, self.spec.scale, gate)
