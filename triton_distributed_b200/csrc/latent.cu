@@ -121,7 +121,12 @@ TDB_DEVICE void head_blocks(float (&c)[4], const __nv_bfloat16* as, int pitch, c
   }
 }
 TDB_DEVICE int head_pitch(int K) { return (K + 31) / 32 * 32 + 32; }
-inline size_t head_smem(int K, bool f32) { return static_cast<size_t>(kTok) * ((K + 31) / 32 * 32 + 32) * (f32 ? 4 : 2); }
+__host__ __device__ inline size_t head_smem(int K, bool f32) { return static_cast<size_t>(kTok) * ((K + 31) / 32 * 32 + 32) * (f32 ? 4 : 2); }
+
+// Groups of threads that share the partials of a token in latent_out_kernel.
+__host__ __device__ inline int merge_groups(int n_tok, int splits) {
+  return n_tok > 2 || splits < 8 ? 1 : n_tok == 2 ? 2 : 4;
+}
 
 // The map itself.  `stage` fills as[16][pitch] (after the previous kernel's results are visible), `put(token, column, value)`
 // takes the products; w [n_cols, K] are the head's weights.
@@ -254,21 +259,46 @@ __global__ void __launch_bounds__(kThreads) latent_out_kernel(const LatentOutArg
             if (lane + 32 * j < p.splits) wsplit[i][lane + 32 * j] = l > 0.f ? w[j] / l : 0.f;
         }
         __syncthreads();
-        for (int i = threadIdx.x; i < kTok * (pitch / 8); i += kThreads) {
-          const int r = i / (pitch / 8), c = (i % (pitch / 8)) * 8;
+        // few tokens: the partials of a token are dealt out to groups of threads, so that all loads are in flight together
+        const int per_row = pitch / 8, groups = merge_groups(n_tok, p.splits);
+        float* part = reinterpret_cast<float*>(smem + head_smem(p.R, sizeof(T) == 4));      // [groups][n_tok][R]
+        const int n_items = (groups > 1 ? n_tok : kTok) * per_row;
+        for (int i = threadIdx.x; i < n_items * groups; i += kThreads) {
+          const int grp = i / n_items, r = (i % n_items) / per_row, c = (i % per_row) * 8;
           float acc[8] = {};
           if (r < n_tok && c < p.R) {
             const float* o = p.o + ((t0 + r) * p.H + h) * static_cast<int64_t>(p.splits) * p.R + c;
-            for (int s = 0; s < p.splits; ++s) {
-              const float w = wsplit[r][s];
-              if (w == 0.f) continue;       // an empty partial was never written
-              float f[8];
-              load8(o + static_cast<int64_t>(s) * p.R, f);
+            for (int s0 = grp; s0 < p.splits; s0 += groups * 4) {
+              float f[4][8], w[4];
 #pragma unroll
-              for (int j = 0; j < 8; ++j) acc[j] = fmaf(w, f[j], acc[j]);
+              for (int u = 0; u < 4; ++u) {
+                const int s = s0 + u * groups;
+                w[u] = s < p.splits ? wsplit[r][s] : 0.f;
+                if (w[u] != 0.f) load8(o + static_cast<int64_t>(s) * p.R, f[u]);      // an empty partial was never written
+              }
+#pragma unroll
+              for (int u = 0; u < 4; ++u)
+                if (w[u] != 0.f)
+#pragma unroll
+                  for (int j = 0; j < 8; ++j) acc[j] = fmaf(w[u], f[u][j], acc[j]);
             }
           }
-          store8(as + r * pitch + c, acc);
+          if (groups == 1) store8(as + r * pitch + c, acc);
+          else if (c < p.R) store8(part + (grp * n_tok + r) * p.R + c, acc);
+        }
+        if (groups > 1) {
+          __syncthreads();
+          for (int i = threadIdx.x; i < kTok * per_row; i += kThreads) {
+            const int r = i / per_row, c = (i % per_row) * 8;
+            float acc[8] = {}, f[8];
+            if (r < n_tok && c < p.R)
+              for (int g = 0; g < groups; ++g) {
+                load8(part + (g * n_tok + r) * p.R + c, f);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) acc[j] += f[j];
+              }
+            store8(as + r * pitch + c, acc);
+          }
         }
       },
       [&](int r, int n, float v) {
@@ -307,7 +337,8 @@ cudaError_t launch_latent_absorb(const LatentPrepArgs& a, cudaStream_t s) {
 }
 
 cudaError_t launch_latent_out(const LatentOutArgs& a, cudaStream_t s) {
-  const size_t smem = head_smem(a.R, a.is_f32);
+  // (a tail of one or two tokens behind full tiles merges in groups as well: room for the largest case)
+  const size_t smem = head_smem(a.R, a.is_f32) + static_cast<size_t>(a.splits < 8 ? 0 : 4) * a.R * 4;
   const int64_t tiles = (a.T + kTok - 1) / kTok;
   if (a.R % 8 != 0 || a.dv < 1 || a.H < 1 || a.splits < 1 || a.splits > kMaxSplits || (a.ml == nullptr && a.splits != 1) ||
       smem > 200 * 1024 || tiles > 65535)

@@ -3,16 +3,18 @@
 // latent_prefill_kernel   prompts, expanded form.  One CTA = 256 query rows of one head as two 128-row tiles that share every
 //                         block of 64 keys, as in the two-tile form of attn_sm100.cu (same softmax warps).  A key is
 //                         [unrotated | rotated] from two tensors: the head's keys and the rotated part in the packed rows, which
-//                         all heads share; queries likewise.  Values arrive transposed from their GEMM.  Head sizes that are no
-//                         multiple of 64 are zero-filled by the TMA boxes.
+//                         all heads share; queries likewise.  Values arrive transposed from their GEMM.  Keys and values have
+//                         rings of their own: scores run a block ahead, so a key buffer is free a block earlier than the values
+//                         beside it.  Head sizes that are no multiple of 64 are zero-filled by the TMA boxes.
 // latent_decode_kernel    decoding, absorbed form: split-KV, one CTA per (split, 32 heads, sequence).  The cached rows are both
-//                         keys and values, so a tile of 128 tokens is loaded once and multiplied twice:
-//                           S^T[token, head]  = row . q'            M = 128 tokens, N = 32 heads, K = rank + rotated
-//                           O^T[latent, head] += row^T . P^T        M = 128 latents, N = 32 heads, K = 128 tokens
+//                         keys and values, so a tile of 64 tokens is loaded once and multiplied twice:
+//                           S^T[token, head]  = row . q'            M = 64 tokens, N = 32 heads, K = rank + rotated
+//                           O^T[latent, head] += row^T . P^T        M = 128 latents, N = 32 heads, K = 64 tokens
 //                         (the second product takes the same shared-memory tile as an MN-major A operand).  Few heads cost few
-//                         columns, not idle rows.  A softmax thread owns a token; maxima over tokens are butterfly-transposed
-//                         so that lane h of every warp keeps head h's reference maximum.  Partials are merged by
-//                         latent_out_kernel.
+//                         columns, not idle rows.  The ring holds more than two tiles, so S^T of the next tile runs during the
+//                         exponentials and loads never stop.  A softmax thread holds 2 tokens x 8 heads; maxima over tokens are
+//                         butterfly-transposed, after which lane h of every warp keeps head h's reference maximum.  Partials
+//                         are merged by latent_out_kernel.
 //
 // Every wait is bounded; a timeout is recorded, the CTA runs through without further waiting, frees its TMEM and returns.
 #include <cuda.h>
@@ -64,7 +66,7 @@ struct PfLay {
   static constexpr int kOffV = kOffK + kStages * kK;
   static constexpr int kOffP = kOffV + kStages * kV;
   static constexpr int kOffBar = kOffP + 2 * kP;
-  static constexpr int kSmem = kOffBar + (2 * kStages + 12) * 8 + 64 + 1024;
+  static constexpr int kSmem = kOffBar + (4 * kStages + 10) * 8 + 64 + 1024;
 };
 static_assert(PfLay<3, 128>::kSmem <= 227 * 1024 && PfLay<2, 128>::kSmem <= 227 * 1024, "prompt kernel must fit one SM");
 
@@ -84,9 +86,11 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tq, const __grid_const
   uint64_t* s_free = bars + 3;
   uint64_t* p_full = bars + 5;
   uint64_t* pv_full = bars + 7;
-  uint64_t* kv_full = bars + 9;                 // [kStages]
-  uint64_t* kv_empty = kv_full + kStages;       // [kStages]
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(kv_empty + kStages);
+  uint64_t* k_full = bars + 9;                  // [kStages] each
+  uint64_t* k_empty = k_full + kStages;
+  uint64_t* v_full = k_empty + kStages;
+  uint64_t* v_empty = v_full + kStages;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(v_empty + kStages);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int b = blockIdx.z, head = blockIdx.y;
@@ -102,13 +106,15 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tq, const __grid_const
     nblk_t[t] = rows_t[t] > 0 ? (kv_end + kBN - 1) / kBN : 0;
   }
   const int nblk = max(nblk_t[0], nblk_t[1]);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;      // warp-uniform
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
     for (int i = 0; i < kStages; ++i) {
-      mbar_init(&kv_full[i], 1);
-      mbar_init(&kv_empty[i], 1);
+      mbar_init(&k_full[i], 1);
+      mbar_init(&k_empty[i], 1);
+      mbar_init(&v_full[i], 1);
+      mbar_init(&v_empty[i], 1);
     }
     for (int t = 0; t < 2; ++t) {
       mbar_init(&s_full[t], 1);
@@ -139,74 +145,91 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tq, const __grid_const
         for (int c = 0; c < NC - 1; ++c) tma_load_3d(sq + c * kQChunk, &tq, q_full, c * 64, q_begin + row0 + t * kBM, head);
         tma_load_3d(sq + (NC - 1) * kQChunk, &tqr, q_full, 0, q_begin + row0 + t * kBM, head);
       }
-      int issued = 0;
-      for (int j = 0; j < nblk; ++j, ++issued) {
+      auto load_k = [&](int j) -> bool {
         const int s = j % kStages;
-        if (!mbar_wait(&kv_empty[s], ((j / kStages) & 1) ^ 1, abort_flag, kWaitNs)) {
-          *abort_flag = 1;
-          break;
-        }
-        mbar_arrive_expect_tx(&kv_full[s], L::kK + L::kV);
+        if (!mbar_wait(&k_empty[s], ((j / kStages) & 1) ^ 1, abort_flag, kWaitNs)) return false;
+        mbar_arrive_expect_tx(&k_full[s], L::kK);
         uint8_t* sk = smem + L::kOffK + s * L::kK;
 #pragma unroll
-        for (int c = 0; c < NC - 1; ++c) tma_load_3d(sk + c * kKChunk, &tk, &kv_full[s], c * 64, base + j * kBN, head);
-        tma_load_2d(sk + (NC - 1) * kKChunk, &tkr, &kv_full[s], 0, base + j * kBN);
-        tma_load_3d(smem + L::kOffV + s * L::kV, &tv, &kv_full[s], base + j * kBN, 0, head);
+        for (int c = 0; c < NC - 1; ++c) tma_load_3d(sk + c * kKChunk, &tk, &k_full[s], c * 64, base + j * kBN, head);
+        tma_load_2d(sk + (NC - 1) * kKChunk, &tkr, &k_full[s], 0, base + j * kBN);
+        return true;
+      };
+      int nk = 0, nv = 0;              // blocks requested so far
+      bool ok = nblk == 0 || load_k(nk++);
+      for (int j = 0; j < nblk && ok; ++j) {
+        if (j + 1 < nblk) {            // keys a block ahead of the values
+          ok = load_k(j + 1);
+          if (!ok) break;
+          ++nk;
+        }
+        const int s = j % kStages;
+        ok = mbar_wait(&v_empty[s], ((j / kStages) & 1) ^ 1, abort_flag, kWaitNs);
+        if (!ok) break;
+        mbar_arrive_expect_tx(&v_full[s], L::kV);
+        tma_load_3d(smem + L::kOffV + s * L::kV, &tv, &v_full[s], base + j * kBN, 0, head);
+        ++nv;
       }
-      if (*abort_flag != 0)            // own copies land before the CTA's shared memory goes away
-        for (int j = max(0, issued - kStages); j < issued; ++j) mbar_wait(&kv_full[j % kStages], (j / kStages) & 1, nullptr, kWaitNs);
+      if (!ok) {                       // own copies land before the CTA's shared memory goes away
+        *abort_flag = 1;
+        mbar_wait(q_full, 0, nullptr, kWaitNs);
+        for (int j = max(0, nk - kStages); j < nk; ++j) mbar_wait(&k_full[j % kStages], (j / kStages) & 1, nullptr, kWaitNs);
+        for (int j = max(0, nv - kStages); j < nv; ++j) mbar_wait(&v_full[j % kStages], (j / kStages) & 1, nullptr, kWaitNs);
+      }
     }
   } else if (warp == 1) {
-    if (lane == 0) {
-      constexpr uint32_t idesc_s = make_idesc(1u, kBM, kBN);
-      constexpr uint32_t idesc_pv = make_idesc(1u, kBM, DV);
-      bool ok = mbar_wait(q_full, 0, abort_flag, kWaitNs);
-      auto issue_s = [&](int t, int j) -> bool {
-        const int s = j % kStages;
-        if (!mbar_wait(&kv_full[s], (j / kStages) & 1, abort_flag, kWaitNs)) return false;
-        if (j > 0 && !mbar_wait(&s_free[t], (j - 1) & 1, abort_flag, kWaitNs)) return false;
-        tc_fence_after_sync();
-        const uint32_t sq = smem_u32(smem + t * L::kQ);
-        const uint32_t sk = smem_u32(smem + L::kOffK + s * L::kK);
-        uint32_t acc = 0;
+    constexpr uint32_t idesc_s = make_idesc(1u, kBM, kBN);
+    constexpr uint32_t idesc_pv = make_idesc(1u, kBM, DV);
+    bool ok = mbar_wait(q_full, 0, abort_flag, kWaitNs);
+    // the last tile that block j is multiplied with: the second one sees at least the blocks of the first, unless it is empty
+    auto last_tile = [&](int j) { return j < nblk_t[1] ? 1 : 0; };
+    auto issue_s = [&](int t, int j) -> bool {
+      const int s = j % kStages;
+      if (!mbar_wait(&k_full[s], (j / kStages) & 1, abort_flag, kWaitNs)) return false;
+      if (j > 0 && !mbar_wait(&s_free[t], (j - 1) & 1, abort_flag, kWaitNs)) return false;
+      tc_fence_after_sync();
+      const uint32_t sq = smem_u32(smem + t * L::kQ);
+      const uint32_t sk = smem_u32(smem + L::kOffK + s * L::kK);
+      uint32_t acc = 0;
 #pragma unroll
-        for (int c = 0; c < NC; ++c) {
-          const int cols = c < NC - 1 ? pp.d - c * 64 : pp.r;
+      for (int c = 0; c < NC; ++c) {
+        const int cols = c < NC - 1 ? pp.d - c * 64 : pp.r;
 #pragma unroll
-          for (int k = 0; k < 4; ++k) {
-            if (k * kUmmaK >= cols) break;
-            umma_f16(tmem_base + t * 256, make_smem_desc_sw128(sq + c * kQChunk) + 2 * k, make_smem_desc_sw128(sk + c * kKChunk) + 2 * k,
-                     idesc_s, acc);
-            acc = 1;
-          }
+        for (int k = 0; k < 4; ++k) {
+          if (k * kUmmaK >= cols) break;
+          umma_f16_elect(tmem_base + t * 256, make_smem_desc_sw128(sq + c * kQChunk) + 2 * k, make_smem_desc_sw128(sk + c * kKChunk) + 2 * k,
+                   idesc_s, acc);
+          acc = 1;
         }
-        umma_commit(&s_full[t]);
-        return true;
-      };
-      auto issue_pv = [&](int t, int j) -> bool {
-        if (!mbar_wait(&p_full[t], j & 1, abort_flag, kWaitNs)) return false;
-        tc_fence_after_sync();
-        const uint32_t sp = smem_u32(smem + L::kOffP + t * L::kP);
-        const uint32_t sv = smem_u32(smem + L::kOffV + (j % kStages) * L::kV);
-#pragma unroll
-        for (int k = 0; k < kBN / kUmmaK; ++k)
-          umma_f16(tmem_base + t * 256 + 64, make_smem_desc_sw128(sp) + 2 * k, make_smem_desc_sw128(sv) + 2 * k, idesc_pv,
-                   (j > 0 || k > 0) ? 1u : 0u);
-        umma_commit(&pv_full[t]);
-        return true;
-      };
-      for (int t = 0; t < 2 && ok; ++t)
-        if (nblk_t[t] > 0) ok = issue_s(t, 0);
-      for (int j = 0; j < nblk && ok; ++j) {
-        // per tile: S of the next block as soon as this block's S has been read, then this block's P V
-        for (int t = 0; t < 2 && ok; ++t) {
-          if (j + 1 < nblk_t[t]) ok = issue_s(t, j + 1);
-          if (ok && j < nblk_t[t]) ok = issue_pv(t, j);
-        }
-        if (ok) umma_commit(&kv_empty[j % kStages]);   // every product that reads this stage has been issued before
       }
-      if (!ok) *abort_flag = 1;
+      umma_commit_elect(&s_full[t]);
+      if (t == last_tile(j)) umma_commit_elect(&k_empty[s]);      // both tiles' scores against this block have been issued
+      return true;
+    };
+    auto issue_pv = [&](int t, int j) -> bool {
+      if (!mbar_wait(&v_full[j % kStages], (j / kStages) & 1, abort_flag, kWaitNs)) return false;
+      if (!mbar_wait(&p_full[t], j & 1, abort_flag, kWaitNs)) return false;
+      tc_fence_after_sync();
+      const uint32_t sp = smem_u32(smem + L::kOffP + t * L::kP);
+      const uint32_t sv = smem_u32(smem + L::kOffV + (j % kStages) * L::kV);
+#pragma unroll
+      for (int k = 0; k < kBN / kUmmaK; ++k)
+        umma_f16_elect(tmem_base + t * 256 + 64, make_smem_desc_sw128(sp) + 2 * k, make_smem_desc_sw128(sv) + 2 * k, idesc_pv,
+                 (j > 0 || k > 0) ? 1u : 0u);
+      umma_commit_elect(&pv_full[t]);
+      if (t == last_tile(j)) umma_commit_elect(&v_empty[j % kStages]);
+      return true;
+    };
+    for (int t = 0; t < 2 && ok; ++t)
+      if (nblk_t[t] > 0) ok = issue_s(t, 0);
+    for (int j = 0; j < nblk && ok; ++j) {
+      // per tile: S of the next block as soon as this block's S has been read, then this block's P V
+      for (int t = 0; t < 2 && ok; ++t) {
+        if (j + 1 < nblk_t[t]) ok = issue_s(t, j + 1);
+        if (ok && j < nblk_t[t]) ok = issue_pv(t, j);
+      }
     }
+    if (!ok) *abort_flag = 1;
   } else {
     const int t = (warp - 2) >> 2;
     TileCtx c;
@@ -253,20 +276,20 @@ bool encode2(CUtensorMap* m, const void* base, uint64_t rows, uint64_t cols, uin
 // Decoding
 // ------------------------------------------------------------------------------------------------------------------
 constexpr int kNH = 32;                       // heads of a CTA
-constexpr int kTile = 128;                    // tokens of a tile
-constexpr int kChunk = kTile * 128;           // 128 tokens x 64 columns: 16 KB
+constexpr int kTile = 64;                     // tokens of a tile
+constexpr int kChunk = kTile * 128;           // 64 tokens x 64 columns: 8 KB
 constexpr int kPair = 2 * kChunk;             // 128 latent columns: the M of one O^T block
-constexpr int kSlots = 5;                     // ring of pairs; rank 512 takes four per tile
+constexpr int kSlots = 10;                    // ring of pairs; rank 512 takes four per tile
 constexpr int kDecThreads = 192;              // warp 0 TMA, warp 1 MMA, warps 2-5 softmax
-constexpr int kOffRot = kSlots * kPair;
-constexpr int kOffQ = kOffRot + kChunk;       // [up to 9 chunks][32 heads x 128 bytes]
+constexpr int kOffRot = kSlots * kPair;       // two rotated parts
+constexpr int kOffQ = kOffRot + 2 * kChunk;   // [up to 9 chunks][32 heads x 128 bytes]
 constexpr int kQChunkD = kNH * 128;
-constexpr int kOffP = kOffQ + 9 * kQChunkD;   // [2 halves of 64 tokens][32 heads x 128 bytes]
-constexpr int kOffRed = kOffP + 2 * kQChunkD; // fp32 [3][4 warps][32]: tile maxima, reference maxima, rescale factors
-constexpr int kOffBar = kOffRed + 3 * 4 * 32 * 4;
-constexpr int kDecSmem = kOffBar + (2 * kSlots + 8) * 8 + 64 + 1024;
+constexpr int kOffP = kOffQ + 9 * kQChunkD;   // P^T: [32 heads][64 tokens]
+constexpr int kOffRed = kOffP + kQChunkD;     // fp32 [4][4 warps][32]: tile maxima (even / odd tiles), reference maxima, rescale factors
+constexpr int kOffBar = kOffRed + 4 * 4 * 32 * 4;
+constexpr int kDecSmem = kOffBar + (2 * kSlots + 10) * 8 + 64 + 1024;
 static_assert(kDecSmem <= 227 * 1024, "decode kernel must fit one SM");
-constexpr int kTmemO = 32;                    // S^T: columns [0, 32); O^T block p: [32 + 32 p, 64 + 32 p)
+constexpr int kTmemO = 2 * kNH;               // S^T of even / odd tiles: columns [0, 32) / [32, 64); O^T block p: [64 + 32 p, 96 + 32 p)
 constexpr int kTmemCols = 256;
 
 struct DecodeParams {
@@ -281,16 +304,16 @@ struct DecodeParams {
 
 __device__ __forceinline__ void softmax_warps_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 
-// Lane l's v[h] over heads h -> the reduction over lanes of head l, in lane l.
+// v[k] of the lanes with the same lane % 4 -> the reduction over those lanes of element k = lane / 4, in that lane.
 template <typename Op>
-__device__ __forceinline__ float reduce_transposed(float (&v)[32], int lane, Op op) {
+__device__ __forceinline__ float reduce_transposed(float (&v)[8], int lane, Op op) {
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
+  for (int o = 4; o > 0; o >>= 1) {
+    const bool up = ((lane >> 2) & o) != 0;
 #pragma unroll
     for (int i = 0; i < o; ++i) {
-      const bool up = (lane & o) != 0;
       const float keep = up ? v[i + o] : v[i], send = up ? v[i] : v[i + o];
-      v[i] = op(keep, __shfl_xor_sync(0xffffffffu, send, o));
+      v[i] = op(keep, __shfl_xor_sync(0xffffffffu, send, 4 * o));
     }
   }
   return v[0];
@@ -304,26 +327,28 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tq, const __grid_consta
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + kOffBar);
   uint64_t* q_full = bars;
-  uint64_t* rot_full = bars + 1;
-  uint64_t* rot_empty = bars + 2;
-  uint64_t* s_full = bars + 3;
-  uint64_t* p_full = bars + 4;
-  uint64_t* pv_full = bars + 5;
-  uint64_t* pair_full = bars + 6;               // [kSlots]
+  uint64_t* p_full = bars + 1;
+  uint64_t* pv_full = bars + 2;
+  uint64_t* rot_full = bars + 3;                // [2] each, even / odd tiles
+  uint64_t* rot_empty = bars + 5;
+  uint64_t* s_full = bars + 7;
+  uint64_t* pair_full = bars + 9;               // [kSlots]
   uint64_t* pair_empty = pair_full + kSlots;    // [kSlots]
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(pair_empty + kSlots);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   const int split = blockIdx.x, h0 = blockIdx.y * kNH, b = blockIdx.z;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;      // warp-uniform
   const int n_chunks = (p.R + 63) / 64, n_pairs = (n_chunks + 1) / 2;
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
-    mbar_init(rot_full, 1);
-    mbar_init(rot_empty, 1);
-    mbar_init(s_full, 1);
     mbar_init(p_full, 128);
     mbar_init(pv_full, 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&rot_full[i], 1);
+      mbar_init(&rot_empty[i], 1);
+      mbar_init(&s_full[i], 1);
+    }
     for (int i = 0; i < kSlots; ++i) {
       mbar_init(&pair_full[i], 1);
       mbar_init(&pair_empty[i], 1);
@@ -352,7 +377,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tq, const __grid_consta
       tma_load_3d(smem + kOffQ + n_chunks * kQChunkD, &tqr, q_full, 0, h0, b);
       int slot_row = p.slots[b];
       if (slot_row < 0 || slot_row >= p.num_slots) slot_row = 0;
-      int it = 0;
+      int it = 0, rots = 0;
       bool ok = true;
       for (int n = 0; n < n_tiles && ok; ++n) {
         const int tok = (first + n) * kTile;
@@ -365,27 +390,32 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tq, const __grid_consta
           tma_load_3d(smem + s * kPair + kChunk, &tc, &pair_full[s], q * 128 + 64, tok, slot_row);
           ++it;
         }
-        if (ok) ok = mbar_wait(rot_empty, (n & 1) ^ 1, abort_flag, kWaitNs);
+        const int e = n & 1;
+        if (ok) ok = mbar_wait(&rot_empty[e], ((n >> 1) & 1) ^ 1, abort_flag, kWaitNs);
         if (!ok) break;
-        mbar_arrive_expect_tx(rot_full, kChunk);
-        tma_load_3d(smem + kOffRot, &tr, rot_full, 0, tok, slot_row);
+        mbar_arrive_expect_tx(&rot_full[e], kChunk);
+        tma_load_3d(smem + kOffRot + e * kChunk, &tr, &rot_full[e], 0, tok, slot_row);
+        ++rots;
       }
       if (!ok) {
         *abort_flag = 1;
+        mbar_wait(q_full, 0, nullptr, kWaitNs);
         for (int i = max(0, it - kSlots); i < it; ++i) mbar_wait(&pair_full[i % kSlots], (i / kSlots) & 1, nullptr, kWaitNs);
+        for (int i = max(0, rots - 2); i < rots; ++i) mbar_wait(&rot_full[i & 1], (i >> 1) & 1, nullptr, kWaitNs);
       }
     }
   } else if (warp == 1) {
-    if (lane == 0 && n_tiles > 0) {
+    if (n_tiles > 0) {
       constexpr uint32_t idesc_s = make_idesc(1u, kTile, kNH);
       constexpr uint32_t idesc_pv = make_idesc(1u, 128, kNH) | kMajorA;
-      const uint32_t sq = smem_u32(smem + kOffQ), sp = smem_u32(smem + kOffP), srot = smem_u32(smem + kOffRot);
-      bool ok = mbar_wait(q_full, 0, abort_flag, kWaitNs);
-      for (int n = 0; n < n_tiles && ok; ++n) {
-        for (int q = 0; q < n_pairs && ok; ++q) {
+      const uint32_t sq = smem_u32(smem + kOffQ), sp = smem_u32(smem + kOffP);
+      // S^T of tile n; its columns were read before P of tile n - 2 was waited for
+      auto issue_s = [&](int n) -> bool {
+        const int e = n & 1;
+        const uint32_t d = tmem + e * kNH, srot = smem_u32(smem + kOffRot + e * kChunk);
+        for (int q = 0; q < n_pairs; ++q) {
           const int it = n * n_pairs + q, s = it % kSlots;
-          ok = mbar_wait(&pair_full[s], (it / kSlots) & 1, abort_flag, kWaitNs);
-          if (!ok) break;
+          if (!mbar_wait(&pair_full[s], (it / kSlots) & 1, abort_flag, kWaitNs)) return false;
           tc_fence_after_sync();
           const uint32_t sc = smem_u32(smem + s * kPair);
 #pragma unroll
@@ -394,18 +424,22 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tq, const __grid_consta
             if (c >= n_chunks) break;
 #pragma unroll
             for (int k = 0; k < 4; ++k)
-              umma_f16(tmem, make_smem_desc_sw128(sc + half * kChunk) + 2 * k, make_smem_desc_sw128(sq + c * kQChunkD) + 2 * k, idesc_s,
+              umma_f16_elect(d, make_smem_desc_sw128(sc + half * kChunk) + 2 * k, make_smem_desc_sw128(sq + c * kQChunkD) + 2 * k, idesc_s,
                        (c > 0 || k > 0) ? 1u : 0u);
           }
         }
-        if (ok) ok = mbar_wait(rot_full, n & 1, abort_flag, kWaitNs);
-        if (!ok) break;
+        if (!mbar_wait(&rot_full[e], (n >> 1) & 1, abort_flag, kWaitNs)) return false;
         tc_fence_after_sync();
         for (int k = 0; k * kUmmaK < p.r; ++k)
-          umma_f16(tmem, make_smem_desc_sw128(srot) + 2 * k, make_smem_desc_sw128(sq + n_chunks * kQChunkD) + 2 * k, idesc_s, 1u);
-        umma_commit(rot_empty);
-        umma_commit(s_full);
-        ok = mbar_wait(p_full, n & 1, abort_flag, kWaitNs);
+          umma_f16_elect(d, make_smem_desc_sw128(srot) + 2 * k, make_smem_desc_sw128(sq + n_chunks * kQChunkD) + 2 * k, idesc_s, 1u);
+        umma_commit_elect(&rot_empty[e]);
+        umma_commit_elect(&s_full[e]);
+        return true;
+      };
+      bool ok = mbar_wait(q_full, 0, abort_flag, kWaitNs) && issue_s(0);
+      for (int n = 0; n < n_tiles && ok; ++n) {
+        if (n + 1 < n_tiles) ok = issue_s(n + 1);
+        if (ok) ok = mbar_wait(p_full, n & 1, abort_flag, kWaitNs);
         if (!ok) break;
         tc_fence_after_sync();
         for (int q = 0; q < n_pairs; ++q) {
@@ -413,42 +447,51 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tq, const __grid_consta
           const uint32_t sc = smem_u32(smem + s * kPair);
 #pragma unroll
           for (int k = 0; k < kTile / kUmmaK; ++k)
-            umma_f16(tmem + kTmemO + q * kNH, make_smem_desc_sw128_mn(sc + k * 2048, kChunk),
-                     make_smem_desc_sw128(sp + (k / 4) * kQChunkD) + 2 * (k % 4), idesc_pv, (n > 0 || k > 0) ? 1u : 0u);
-          umma_commit(&pair_empty[s]);
+            umma_f16_elect(tmem + kTmemO + q * kNH, make_smem_desc_sw128_mn(sc + k * 2048, kChunk), make_smem_desc_sw128(sp) + 2 * k, idesc_pv,
+                     (n > 0 || k > 0) ? 1u : 0u);
+          umma_commit_elect(&pair_empty[s]);
         }
-        umma_commit(pv_full);
+        umma_commit_elect(pv_full);
       }
       if (!ok) *abort_flag = 1;
     }
   } else {
     float* red = reinterpret_cast<float*>(smem + kOffRed);
-    float* red_max = red;                 // [4][32]
     const int qd = warp & 3;              // TMEM lane quarter of this warp
-    float* my_m = red + 128 + qd * 32;
-    float* my_alpha = red + 256 + qd * 32;
+    float* my_m = red + 256 + qd * 32;
+    float* my_alpha = red + 384 + qd * 32;
     const uint32_t lane_off = static_cast<uint32_t>(qd * 32) << 16;
     constexpr float kRescaleStep = 8.f;
-    const int t = qd * 32 + lane;         // token inside the tile
+    const int t0 = qd * 16 + (lane >> 2); // this thread's tokens inside the tile: t0, t0 + 8
+    const int h0t = 2 * (lane & 3);       // its heads: element k is head 8 (k / 2) + h0t + k % 2
+    const int my_head = 8 * (lane >> 3) + h0t + ((lane >> 2) & 1);     // the head a transposed reduction leaves in this lane
     float m = -INFINITY;                  // reference maximum of head h0 + lane (the same in all four warps)
-    float l[kNH];                         // this thread's share of the heads' sums
+    float l[8];                           // this thread's share of its heads' sums
 #pragma unroll
-    for (int h = 0; h < kNH; ++h) l[h] = 0.f;
+    for (int k = 0; k < 8; ++k) l[k] = 0.f;
     auto mx = [](float a, float c) { return fmaxf(a, c); };
     // After a timeout the waits return at once and the loop runs through: the warps meet at barriers, so none may leave.
     for (int n = 0; n < n_tiles; ++n) {
-      if (!mbar_wait(s_full, n & 1, abort_flag, kWaitNs)) *abort_flag = 1;
+      const int e = n & 1;
+      if (!mbar_wait(&s_full[e], (n >> 1) & 1, abort_flag, kWaitNs)) *abort_flag = 1;
       __syncwarp();
       tc_fence_after_sync();
-      uint32_t s[kNH];
-      tmem_ld_32x32(tmem + lane_off, s);
+      uint32_t s[16];
+      tmem_ld_16x256b_x4(tmem + e * kNH + lane_off, s);
       tmem_ld_wait();
       tc_fence_before_sync();
-      const bool seen = (first + n) * kTile + t < kv_len;
-      float x[kNH], v[kNH];
+      const int tok = (first + n) * kTile + t0;
+      const bool seen0 = tok < kv_len, seen1 = tok + 8 < kv_len;
+      float x[16], v[8];                  // x[2 k + i]: head element k, token t0 + 8 i
 #pragma unroll
-      for (int h = 0; h < kNH; ++h) v[h] = x[h] = seen ? __uint_as_float(s[h]) * p.scale_log2 : -INFINITY;
-      red_max[qd * 32 + lane] = reduce_transposed(v, lane, mx);
+      for (int k = 0; k < 8; ++k) {
+        const int at = 4 * (k >> 1) + (k & 1);
+        x[2 * k] = seen0 ? __uint_as_float(s[at]) * p.scale_log2 : -INFINITY;
+        x[2 * k + 1] = seen1 ? __uint_as_float(s[at + 2]) * p.scale_log2 : -INFINITY;
+        v[k] = fmaxf(x[2 * k], x[2 * k + 1]);
+      }
+      float* red_max = red + e * 128;     // a fast warp may be at the next tile while a slow one still reads this one's
+      red_max[qd * 32 + my_head] = reduce_transposed(v, lane, mx);
       softmax_warps_sync();
       const float top = fmaxf(fmaxf(red_max[lane], red_max[32 + lane]), fmaxf(red_max[64 + lane], red_max[96 + lane]));
       float alpha = 1.f;
@@ -482,26 +525,28 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tq, const __grid_consta
         tmem_st_wait();
         tc_fence_before_sync();
 #pragma unroll
-        for (int h = 0; h < kNH; ++h) l[h] *= my_alpha[h];
+        for (int k = 0; k < 8; ++k) l[k] *= my_alpha[8 * (k >> 1) + h0t + (k & 1)];
       }
-      // P^T: head rows of 64 tokens (128 bytes, swizzled in 16-byte pieces), two halves
-      uint8_t* prow = smem + kOffP + (t >> 6) * kQChunkD + (t & 7) * 2;
-      const int piece = (t & 63) >> 3;
+      // P^T: a head's row of 64 tokens is 128 bytes, swizzled in 16-byte pieces
+      uint8_t* prow = smem + kOffP + (t0 & 7) * 2;
+      const int piece = t0 >> 3;          // of token t0; token t0 + 8 is in the next one
 #pragma unroll
-      for (int h = 0; h < kNH; ++h) {
-        const float e = ex2(x[h] - my_m[h]);
-        l[h] += e;
-        *reinterpret_cast<__nv_bfloat16*>(prow + h * 128 + ((piece ^ (h & 7)) << 4)) = __float2bfloat16(e);
+      for (int k = 0; k < 8; ++k) {
+        const int h = 8 * (k >> 1) + h0t + (k & 1);
+        const float mh = my_m[h], e0 = ex2(x[2 * k] - mh), e1 = ex2(x[2 * k + 1] - mh);
+        l[k] += e0 + e1;
+        *reinterpret_cast<__nv_bfloat16*>(prow + h * 128 + ((piece ^ (h & 7)) << 4)) = __float2bfloat16(e0);
+        *reinterpret_cast<__nv_bfloat16*>(prow + h * 128 + (((piece + 1) ^ (h & 7)) << 4)) = __float2bfloat16(e1);
       }
       fence_proxy_async_smem();
       mbar_arrive(p_full);
     }
     // sums over tokens, then the output columns
     softmax_warps_sync();
-    red_max[qd * 32 + lane] = reduce_transposed(l, lane, [](float a, float c) { return a + c; });
+    red[qd * 32 + my_head] = reduce_transposed(l, lane, [](float a, float c) { return a + c; });
     softmax_warps_sync();
     if (qd == 0 && h0 + lane < p.H) {
-      const float sum = red_max[lane] + red_max[32 + lane] + red_max[64 + lane] + red_max[96 + lane];
+      const float sum = red[lane] + red[32 + lane] + red[64 + lane] + red[96 + lane];
       p.ml[(static_cast<int64_t>(b) * p.H + h0 + lane) * p.splits + split] = make_float2(m, sum);
     }
     if (n_tiles > 0) {

@@ -141,7 +141,7 @@ def latent_prefill(z: torch.Tensor, k: torch.Tensor, ctx: torch.Tensor, vt: torc
                                              ctx.shape[1] - int(r), int(dv), float(scale), gate, _error_flag(z.device))
 
 
-DECODE_TILE, DECODE_HEADS = 128, 32     # tokens per tile and heads per CTA of the decode kernel
+DECODE_TILE, DECODE_HEADS = 64, 32     # tokens per tile and heads per CTA of the decode kernel
 
 
 def pick_latent_splits(batch: int, heads: int, rows: int, num_sms: int = 148) -> int:
