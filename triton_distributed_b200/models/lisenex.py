@@ -186,10 +186,19 @@ class LisenexLayer:
             self.norm2 = pad_rows(get(p + "norm2").float(), w8).to(device)
             self.mlp.load(get, p + "mlp.", width, dtype, device)
 
-    def sublayers(self, h1, h2, plan, storage):
-        """(mixer output or None, feed-forward pieces or None): what the layer adds to the stream, summed over the ranks."""
+    def sublayers(self, h1, h2, plan, storage, side=None):
+        """(mixer output, feed-forward pieces or None): what this rank's part of the layer adds to the stream.  Neither reads the
+        other: with ``side`` (a stream) the feed-forward runs beside the mixer."""
+        if self.mlp is None or side is None:
+            return self.mixer(h1, plan, storage), (self.mlp(h2) if self.mlp is not None else None)
+        # Tensors of either stream's pool are only reused by that stream, which has waited for the other by then: both wait for
+        # each other once a layer.
+        main = torch.cuda.current_stream()
+        side.wait_stream(main)
+        with torch.cuda.stream(side), ops.scratch_lane(1):
+            ff = self.mlp(h2)
         mix = self.mixer(h1, plan, storage)
-        ff = self.mlp(h2) if self.mlp is not None else None
+        main.wait_stream(side)
         return mix, ff
 
 
@@ -197,12 +206,19 @@ class LisenexLLM(LayeredLLM):
     """See :class:`LayeredLLM`.  On several ranks a layer costs one all-reduce: the partial sums of mixer and feed-forward travel
     together, in fp32."""
 
+    _side = None
+
     def make_layers(self):
         layers = [LisenexLayer(i, s, self.rank, self.world_size, self.group) for i, s in enumerate(self.arch.layers)]
         for l in layers:
             if not l.mixer.own_kv:
                 layers[l.mixer.source].mixer.shared = True
         return layers
+
+    def side_stream(self):
+        if self._side is None:
+            self._side = torch.cuda.Stream(device=self.device)
+        return self._side
 
     def load_head(self, get):
         self.embed_tokens = self.lm_head = self.table(get, "embed")
@@ -216,9 +232,11 @@ class LisenexLLM(LayeredLLM):
             w = (None, None) if nxt is None else (nxt.norm1, nxt.norm2)
             return ops.parallel_add(x, mix, ff, *w, a.hidden_size, a.rms_norm_eps, self.dtype)
 
+        # decode steps are bound by latency and weight streaming: mixer and feed-forward overlap
+        side = self.side_stream() if plan.decode and x.is_cuda else None
         h1, h2 = add(None, None, self.layers[0])
         for i, l in enumerate(self.layers):
-            mix, ff = l.sublayers(h1, h2, plan, plan.cache.layers[i])
+            mix, ff = l.sublayers(h1, h2, plan, plan.cache.layers[i], side)
             if self.world_size > 1:
                 mix, ff = None, ops.FeedForward(l.mixer.reduce(ops.parallel_sum(x, mix, ff)))
             h1, h2 = add(mix, ff, self.layers[i + 1] if i + 1 < len(self.layers) else None)

@@ -10,6 +10,7 @@ large-tile GEMM followed by the all-reduce library.  CPU / reference path: ``mat
 """
 from __future__ import annotations
 
+import contextlib
 from dataclasses import dataclass
 from typing import Dict, Optional, Tuple
 
@@ -32,12 +33,13 @@ def _bulk_exchange() -> int:
     return 1 if os.environ.get("TDB200_SKINNY_EXCHANGE", SKINNY_EXCHANGE) == "bulk" else 0
 
 _SCRATCH: Dict[Tuple[int, int], Tuple[torch.Tensor, torch.Tensor]] = {}
+_LANE = 0      # which scratch calls use: concurrent streams need one each
 _UNFIT_TABLE_SHAPES: set = set()   # (token pad, N, K, tile width, cluster size) from the tuned table that did not fit here
 
 
 def _scratch(device, need_acc: int, need_tiles: int):
     """Per-device split-K scratch (fp32 accumulator + tile counters); the kernel leaves both zeroed."""
-    key = (device.index if device.index is not None else torch.cuda.current_device(), 0)
+    key = (device.index if device.index is not None else torch.cuda.current_device(), _LANE)
     cur = _SCRATCH.get(key)
     if cur is None or cur[0].numel() < need_acc or cur[1].numel() < need_tiles:
         acc = torch.zeros(max(need_acc, 1 << 20), dtype=torch.float32, device=device)
@@ -45,6 +47,17 @@ def _scratch(device, need_acc: int, need_tiles: int):
         _SCRATCH[key] = (acc, cnt)
         cur = _SCRATCH[key]
     return cur
+
+
+@contextlib.contextmanager
+def scratch_lane(lane: int):
+    """GEMMs launched inside use scratch of their own, so that they may run beside those of another stream."""
+    global _LANE
+    old, _LANE = _LANE, lane
+    try:
+        yield
+    finally:
+        _LANE = old
 
 
 def _mpad(m: int) -> int:
