@@ -9,6 +9,8 @@
   python benchmarks/ncu_case.py gdn       # chunk-parallel gated delta rule, 8192 tokens x 16 heads
   python benchmarks/ncu_case.py gla       # chunk-parallel gated linear attention, 8192 tokens x 16 heads, 128 x 128 states
   python benchmarks/ncu_case.py tied      # tied-KV block decode attention, 64 seqs x 4096 positions, 32 q heads / 4 kv heads
+  python benchmarks/ncu_case.py latent_decode   # latent decode attention, 64 seqs x 4096 tokens, 32 heads, rows of 512 + 64
+  python benchmarks/ncu_case.py latent_prefill  # latent prompt attention, 8192 tokens, 8 heads of 128 + 64 / 128
 """
 import sys
 
@@ -83,6 +85,23 @@ def main():
         sink = torch.zeros(Hq, device="cuda")
         for _ in range(3):
             ops.tied_attn_decode(q, k, scale, bt, lens, L, ops.pick_tied_splits(B, Hkv, 1, L), sink)
+    elif case == "latent_decode":
+        B, H, R, r, L = 64, 32, 512, 64, 4096
+        cache = torch.randn(B, L, R + r, device="cuda", dtype=torch.bfloat16)
+        q = torch.randn(B, H, R + r, device="cuda", dtype=torch.bfloat16)
+        slots, lens = torch.arange(B, dtype=torch.int32, device="cuda"), torch.full((B,), L, dtype=torch.int32, device="cuda")
+        for _ in range(3):
+            ops.latent_decode(q, cache, slots, lens, R, (R + r) ** -0.5)
+        ops.check_latent_errors()
+    elif case == "latent_prefill":
+        T, H, d, r, dv, R = 8192, 8, 128, 64, 128, 512
+        z = torch.randn(T, H * (d + r + dv), device="cuda", dtype=torch.bfloat16)
+        k, vt = (torch.randn(*s, device="cuda", dtype=torch.bfloat16) for s in ((T, H * d), (H * dv, T)))
+        ctx = torch.randn(T, R + r, device="cuda", dtype=torch.bfloat16)
+        i32 = lambda *v: torch.tensor(v, dtype=torch.int32, device="cuda")   # noqa: E731
+        for _ in range(3):
+            ops.latent_prefill(z, k, ctx, vt, i32(0, T), i32(0), i32(T), i32(0), T, H, d, r, dv, (d + r) ** -0.5, z[:, H * (d + r):])
+        ops.check_latent_errors()
     elif case == "decode":
         B, Hq, Hkv, D, L = 16, 8, 1, 128, 4096
         k = torch.randn(B, L, Hkv, D, device="cuda", dtype=torch.bfloat16)

@@ -93,9 +93,10 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tq, const __grid_const
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(v_empty + kStages);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
-  const int b = blockIdx.z, head = blockIdx.y;
+  const int b = blockIdx.z, head = blockIdx.x;
   const int q_begin = p.cu_seqlens_q[b], q_len = p.cu_seqlens_q[b + 1] - q_begin;
-  const int row0 = static_cast<int>(gridDim.x - 1 - blockIdx.x) * (2 * kBM);      // long causal tiles first
+  // the long causal tiles of all heads first (blocks are handed out in order of blockIdx.x, then y): no long tile in the last wave
+  const int row0 = static_cast<int>(gridDim.y - 1 - blockIdx.y) * (2 * kBM);
   if (row0 >= q_len) return;                      // whole CTA, before any barrier or TMEM use
   const int kv_len = p.kv_lens[b], pos0 = p.q_pos0[b], base = pp.ctx0[b];
   int rows_t[2], nblk_t[2];
@@ -612,7 +613,7 @@ cudaError_t launch_latent_prefill(const LatentPrefillArgs& a, cudaStream_t s) {
   p.ctx0 = a.ctx0;
   p.d = a.d;
   p.r = a.r;
-  const dim3 grid((a.max_q + 2 * kBM - 1) / (2 * kBM), a.H, a.B);
+  const dim3 grid(a.H, (a.max_q + 2 * kBM - 1) / (2 * kBM), a.B);
   if (nc == 3) return DV == 128 ? launch_prefill_t<3, 128>(m, p, grid, s) : launch_prefill_t<3, 64>(m, p, grid, s);
   return DV == 128 ? launch_prefill_t<2, 128>(m, p, grid, s) : launch_prefill_t<2, 64>(m, p, grid, s);
 }

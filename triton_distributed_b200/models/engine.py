@@ -173,6 +173,12 @@ class Engine:
         self.step_cache.advance(slots, lens)
         return logits
 
+    def check_errors(self):
+        """Raise if a bounded wait of any kernel launched so far gave up (synchronises)."""
+        self.rt.check_status(sync=True)
+        ops.check_attention_errors()
+        ops.check_latent_errors()
+
     def end(self, request_ids: Sequence):
         """Requests that are finished: their cache rows and states go back."""
         for rid in request_ids:
@@ -248,4 +254,6 @@ class Engine:
         if self.verbose and self.rt.rank == 0:
             logger.info(f"decode: {self.last_decode_ms:.3f} ms/step over {n_timed} steps (backend {self.backend})")
         self.rt.check_status(sync=False)
+        ops.check_attention_errors()
+        ops.check_latent_errors()
         return torch.stack(out, dim=1)

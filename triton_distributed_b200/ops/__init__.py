@@ -18,7 +18,7 @@ from .elementwise import (rmsnorm, silu_mul, residual_add, qk_norm_rope_kv, embe
 from .attention import (flash_attn_varlen, gqa_fwd_batch_decode, gqa_fwd_batch_decode_intra_rank,  # noqa: F401
                         gqa_fwd_batch_decode_persistent, attention_reference, merge_attention_partials,
                         dense_block_table, decode_workspace, pick_kv_splits, tied_attention_simple, tied_attn_varlen,
-                        tied_attn_decode, pick_tied_splits, TIED_TENSOR_CORE_DIMS)
+                        tied_attn_decode, pick_tied_splits, TIED_TENSOR_CORE_DIMS, check_attention_errors)
 from .gemv import (GemvARContext, create_gemv_ar_context, gemv_fused, gemv_reference, gemv_supported,  # noqa: F401
                    GEMV_FAST_M, GEMV_MAX_M)
 from .gemm_ar import (GemmARContext, LLGemmARContext, create_gemm_ar_context, create_ll_gemm_ar_context,  # noqa: F401
