@@ -409,30 +409,31 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tq, const __grid_consta
     if (n_tiles > 0) {
       constexpr uint32_t idesc_s = make_idesc(1u, kTile, kNH);
       constexpr uint32_t idesc_pv = make_idesc(1u, 128, kNH) | kMajorA;
-      const uint32_t sq = smem_u32(smem + kOffQ), sp = smem_u32(smem + kOffP);
+      // descriptors advance by plain additions (the address field counts 16-byte units and never overflows)
+      const uint64_t dq = make_smem_desc_sw128(smem_u32(smem + kOffQ)), dp = make_smem_desc_sw128(smem_u32(smem + kOffP));
+      const uint64_t drot = make_smem_desc_sw128(smem_u32(smem + kOffRot));
+      const uint64_t dk = make_smem_desc_sw128(smem_u32(smem)), dv = make_smem_desc_sw128_mn(smem_u32(smem), kChunk);
+      int s_slot = 0, s_phase = 0, v_slot = 0;       // ring positions of the score and of the value products
       // S^T of tile n; its columns were read before P of tile n - 2 was waited for
       auto issue_s = [&](int n) -> bool {
         const int e = n & 1;
-        const uint32_t d = tmem + e * kNH, srot = smem_u32(smem + kOffRot + e * kChunk);
+        const uint32_t d = tmem + e * kNH;
         for (int q = 0; q < n_pairs; ++q) {
-          const int it = n * n_pairs + q, s = it % kSlots;
-          if (!mbar_wait(&pair_full[s], (it / kSlots) & 1, abort_flag, kWaitNs)) return false;
+          if (!mbar_wait(&pair_full[s_slot], s_phase, abort_flag, kWaitNs)) return false;
           tc_fence_after_sync();
-          const uint32_t sc = smem_u32(smem + s * kPair);
+          const uint64_t a = dk + s_slot * (kPair >> 4), b = dq + 2 * q * (kQChunkD >> 4);
 #pragma unroll
-          for (int half = 0; half < 2; ++half) {
-            const int c = 2 * q + half;
-            if (c >= n_chunks) break;
+          for (int k = 0; k < 4; ++k) umma_f16_elect(d, a + 2 * k, b + 2 * k, idesc_s, (q > 0 || k > 0) ? 1u : 0u);
+          if (2 * q + 1 < n_chunks) {
 #pragma unroll
-            for (int k = 0; k < 4; ++k)
-              umma_f16_elect(d, make_smem_desc_sw128(sc + half * kChunk) + 2 * k, make_smem_desc_sw128(sq + c * kQChunkD) + 2 * k, idesc_s,
-                       (c > 0 || k > 0) ? 1u : 0u);
+            for (int k = 0; k < 4; ++k) umma_f16_elect(d, a + (kChunk >> 4) + 2 * k, b + (kQChunkD >> 4) + 2 * k, idesc_s, 1u);
           }
+          if (++s_slot == kSlots) s_slot = 0, s_phase ^= 1;
         }
         if (!mbar_wait(&rot_full[e], (n >> 1) & 1, abort_flag, kWaitNs)) return false;
         tc_fence_after_sync();
         for (int k = 0; k * kUmmaK < p.r; ++k)
-          umma_f16_elect(d, make_smem_desc_sw128(srot) + 2 * k, make_smem_desc_sw128(sq + n_chunks * kQChunkD) + 2 * k, idesc_s, 1u);
+          umma_f16_elect(d, drot + e * (kChunk >> 4) + 2 * k, dq + n_chunks * (kQChunkD >> 4) + 2 * k, idesc_s, 1u);
         umma_commit_elect(&rot_empty[e]);
         umma_commit_elect(&s_full[e]);
         return true;
@@ -444,13 +445,12 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tq, const __grid_consta
         if (!ok) break;
         tc_fence_after_sync();
         for (int q = 0; q < n_pairs; ++q) {
-          const int s = (n * n_pairs + q) % kSlots;
-          const uint32_t sc = smem_u32(smem + s * kPair);
+          const uint64_t a = dv + v_slot * (kPair >> 4);
 #pragma unroll
           for (int k = 0; k < kTile / kUmmaK; ++k)
-            umma_f16_elect(tmem + kTmemO + q * kNH, make_smem_desc_sw128_mn(sc + k * 2048, kChunk), make_smem_desc_sw128(sp) + 2 * k, idesc_pv,
-                     (n > 0 || k > 0) ? 1u : 0u);
-          umma_commit_elect(&pair_empty[s]);
+            umma_f16_elect(tmem + kTmemO + q * kNH, a + k * (2048 >> 4), dp + 2 * k, idesc_pv, (n > 0 || k > 0) ? 1u : 0u);
+          umma_commit_elect(&pair_empty[v_slot]);
+          if (++v_slot == kSlots) v_slot = 0;
         }
         umma_commit_elect(pv_full);
       }
