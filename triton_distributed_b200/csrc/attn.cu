@@ -1,5 +1,5 @@
 #include <atomic>
-// Attention kernels over a paged KV cache (bf16, GQA, head dim 64 or 128):
+// Attention kernels over a paged KV cache (bf16, GQA, head dim 64, 128 or 256):
 //
 //   flash_fwd_kernel         var-len causal prefill / context-parallel attention: one CTA = 64 query rows of one
 //                            head (4 warps x 16 rows), KV streamed in 64-token blocks through double-buffered
@@ -538,7 +538,7 @@ cudaError_t launch_flash_fwd(const FlashFwdArgs& a, cudaStream_t stream) {
     kernel<<<grid, kAttnThreads, smem, stream>>>(p);
     return cudaGetLastError();
   };
-  static SmemOptIn s128, s64, t32, t64, t128, t256;
+  static SmemOptIn s256, s128, s64, t32, t64, t128, t256;
   if (tied) {
     switch (a.head_dim) {
       case 32: return launch(flash_fwd_kernel<32, true>, 2 * Tiles<32>::kTiedStage, &t32);
@@ -551,6 +551,7 @@ cudaError_t launch_flash_fwd(const FlashFwdArgs& a, cudaStream_t stream) {
   switch (a.head_dim) {
     case 64: return launch(flash_fwd_kernel<64, false>, Tiles<64>::kSmem, &s64);
     case 128: return launch(flash_fwd_kernel<128, false>, Tiles<128>::kSmem, &s128);
+    case 256: return launch(flash_fwd_kernel<256, false>, Tiles<256>::kSmem, &s256);
     default: return cudaErrorInvalidValue;
   }
 }
@@ -564,7 +565,7 @@ namespace {
 cudaError_t launch_splitkv_impl(const DecodeArgs& a, const DistTail* tail, cudaStream_t stream) {
   const bool tied = a.kv.k_scale != nullptr;
   if (tied && a.kv.max_pages != 1) return cudaErrorInvalidValue;
-  if (!tied && a.head_dim != 64 && a.head_dim != 128) return cudaErrorInvalidValue;
+  if (!tied && a.head_dim != 64 && a.head_dim != 128 && (a.head_dim != 256 || tail != nullptr)) return cudaErrorInvalidValue;
   if (a.num_q_heads % a.kv.num_kv_heads != 0 || a.splits < 1) return cudaErrorInvalidValue;
   // the epilogue belongs to the fused combine; the distributed tail has neither it nor the tied form
   const bool plain = !tied && a.epi.sink == nullptr && a.epi.gate == nullptr && a.chunk == 0;
@@ -632,7 +633,8 @@ cudaError_t launch_splitkv_impl(const DecodeArgs& a, const DistTail* tail, cudaS
       default: return cudaErrorInvalidValue;
     }
   }
-  static SmemOptIn set128_2, set128_4, set64_2, set64_4;
+  static SmemOptIn set256_2, set128_2, set128_4, set64_2, set64_4;
+  if (a.head_dim == 256) return launch(decode_splitkv_kernel<256, 2>, Tiles<256>::kSmem, &set256_2);
   if (a.head_dim == 128) {
     return deep ? launch(decode_splitkv_kernel<128, 4>, 2 * Tiles<128>::kSmem, &set128_4)
                 : launch(decode_splitkv_kernel<128, 2>, Tiles<128>::kSmem, &set128_2);

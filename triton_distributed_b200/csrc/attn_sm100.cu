@@ -115,7 +115,7 @@ __global__ void __launch_bounds__(256) attn_pack_kv_kernel(const PackParams p) {
 // ------------------------------------------------------------------------------------------------------------------
 // Main kernel
 // ------------------------------------------------------------------------------------------------------------------
-template <int kStages, int kCtasPerSm>
+template <int kStages, int kCtasPerSm, bool CAP>
 __global__ void __launch_bounds__(kThreads, kCtasPerSm)
 flash_fwd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                        const __grid_constant__ CUtensorMap tmap_vt, const FwdParams p) {
@@ -250,7 +250,7 @@ flash_fwd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
     t.tmem_s = tmem_s; t.tmem_pv = tmem_pv;
     t.p_smem = smem + kOffP;
     t.row0 = row0; t.rows_here = rows_here; t.nblk = nblk;
-    softmax_tile<kD>(p, t, warp, lane, q_begin, head, kv_len, pos0, abort_flag);
+    softmax_tile<kD, CAP>(p, t, warp, lane, q_begin, head, kv_len, pos0, abort_flag);
   }
 
   // ------------------------------------------------------------ teardown
@@ -280,7 +280,7 @@ struct LayPP {
 };
 static_assert(LayPP<3>::kSmem + 1024 <= 227 * 1024, "the two-tile prefill kernel must fit one SM");
 
-template <int kStages>
+template <int kStages, bool CAP>
 __global__ void __launch_bounds__(kPPThreads, 1)
 flash_fwd_sm100_pp_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                           const __grid_constant__ CUtensorMap tmap_vt, const FwdParams p) {
@@ -420,7 +420,7 @@ flash_fwd_sm100_pp_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
     c.tmem_s = tmem_base + t * 256; c.tmem_pv = tmem_base + t * 256 + 64;
     c.p_smem = smem + kOffP + t * kPBytes;
     c.row0 = row0 + t * kBM; c.rows_here = rows_t[t]; c.nblk = nblk_t[t];
-    softmax_tile<kD>(p, c, warp, lane, q_begin, head, kv_len, pos0, abort_flag);
+    softmax_tile<kD, CAP>(p, c, warp, lane, q_begin, head, kv_len, pos0, abort_flag);
   }
 
   tc_fence_before_sync();
@@ -482,6 +482,9 @@ cudaError_t launch_flash_fwd_sm100(const FlashFwdSm100Args& a, cudaStream_t stre
   p.causal = a.causal;
   p.dv = kD;
   p.scale_log2 = a.scale * 1.4426950408889634f;
+  if (a.softcap < 0.f) return cudaErrorInvalidValue;
+  p.cap_log2 = a.softcap * 1.4426950408889634f;
+  p.to_cap = a.softcap > 0.f ? a.scale / a.softcap : 0.f;
   p.total_q = a.total_q;
   p.error_flag = a.error_flag;
   p.epi = a.epi;
@@ -499,24 +502,24 @@ cudaError_t launch_flash_fwd_sm100(const FlashFwdSm100Args& a, cudaStream_t stre
     const char* e = std::getenv("TDB200_ATTN_FORM");
     return e != nullptr ? std::atoi(e) : 2;
   }();
+  auto launch = [&](auto kernel, SmemOptIn& opt, dim3 g, int threads, int smem) -> cudaError_t {
+    const cudaError_t err = opt.ensure(kernel, smem);
+    if (err != cudaSuccess) return err;
+    kernel<<<g, threads, smem, stream>>>(mq, mk, mv, p);
+    return cudaGetLastError();
+  };
+  static SmemOptIn opt1, opt2, opt3, cap1, cap2, cap3;
+  const bool cap = a.softcap > 0.f;
   if (form == 3) {
-    static SmemOptIn opt3;
-    e = opt3.ensure(flash_fwd_sm100_pp_kernel<3>, LayPP<3>::kSmem + 1024);
-    if (e != cudaSuccess) return e;
-    dim3 grid2((a.max_q_len + 2 * kBM - 1) / (2 * kBM), a.num_q_heads, a.batch);
-    flash_fwd_sm100_pp_kernel<3><<<grid2, kPPThreads, LayPP<3>::kSmem + 1024, stream>>>(mq, mk, mv, p);
-  } else if (form == 1) {
-    static SmemOptIn opt1;
-    e = opt1.ensure(flash_fwd_sm100_kernel<5, 1>, Lay<5>::kSmem);
-    if (e != cudaSuccess) return e;
-    flash_fwd_sm100_kernel<5, 1><<<grid, kThreads, Lay<5>::kSmem, stream>>>(mq, mk, mv, p);
-  } else {
-    static SmemOptIn opt2;
-    e = opt2.ensure(flash_fwd_sm100_kernel<2, 2>, Lay<2>::kSmem);
-    if (e != cudaSuccess) return e;
-    flash_fwd_sm100_kernel<2, 2><<<grid, kThreads, Lay<2>::kSmem, stream>>>(mq, mk, mv, p);
+    const dim3 grid2((a.max_q_len + 2 * kBM - 1) / (2 * kBM), a.num_q_heads, a.batch);
+    return cap ? launch(flash_fwd_sm100_pp_kernel<3, true>, cap3, grid2, kPPThreads, LayPP<3>::kSmem + 1024)
+               : launch(flash_fwd_sm100_pp_kernel<3, false>, opt3, grid2, kPPThreads, LayPP<3>::kSmem + 1024);
   }
-  return cudaGetLastError();
+  if (form == 1)
+    return cap ? launch(flash_fwd_sm100_kernel<5, 1, true>, cap1, grid, kThreads, Lay<5>::kSmem)
+               : launch(flash_fwd_sm100_kernel<5, 1, false>, opt1, grid, kThreads, Lay<5>::kSmem);
+  return cap ? launch(flash_fwd_sm100_kernel<2, 2, true>, cap2, grid, kThreads, Lay<2>::kSmem)
+             : launch(flash_fwd_sm100_kernel<2, 2, false>, opt2, grid, kThreads, Lay<2>::kSmem);
 }
 
 }  // namespace tdb

@@ -108,7 +108,7 @@ std::vector<at::Tensor> flash_fwd_sm100(const at::Tensor& q, const at::Tensor& k
                                         const at::Tensor& block_table, const at::Tensor& cu_seqlens_q, const at::Tensor& kv_lens,
                                         c10::optional<at::Tensor> q_pos0, int64_t max_q_len, int64_t max_kv_len, bool causal,
                                         double scale, c10::optional<at::Tensor> lse, c10::optional<at::Tensor> k_scale,
-                                        c10::optional<at::Tensor> sink, c10::optional<at::Tensor> gate) {
+                                        c10::optional<at::Tensor> sink, c10::optional<at::Tensor> gate, double softcap) {
   TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && q.scalar_type() == at::kBFloat16 && q.size(2) == 128,
               "flash_fwd_sm100: q must be contiguous bf16 [T, Hq, 128]");
   TORCH_CHECK(k_cache.scalar_type() == at::kBFloat16 && v_cache.scalar_type() == at::kBFloat16 && k_cache.is_contiguous() &&
@@ -145,6 +145,7 @@ std::vector<at::Tensor> flash_fwd_sm100(const at::Tensor& q, const at::Tensor& k
   a.total_q = q.size(0);
   a.causal = causal ? 1 : 0;
   a.scale = scale;
+  a.softcap = softcap;
   TORCH_CHECK(max_kv_len >= 1, "flash_fwd_sm100: max_kv_len must be positive");
   a.Lp = static_cast<int>((max_kv_len + 63) / 64 * 64);
   at::Tensor kd = at::empty({a.batch * a.num_kv_heads, a.Lp, 128}, q.options());
@@ -248,7 +249,7 @@ int64_t dist_decode_attn(SymmHeap& h, const at::Tensor& q, const at::Tensor& k_c
 // Attention of every token over rows [row0, row0 + n_keys) of a tied cache, fp32 arithmetic (fp32 or bf16 tensors).
 at::Tensor tied_attn_simple(const at::Tensor& q, const at::Tensor& k, c10::optional<at::Tensor> k_scale, const at::Tensor& row0,
                             const at::Tensor& n_keys, c10::optional<at::Tensor> sink, c10::optional<at::Tensor> gate, double scale,
-                            int64_t dv, bool out_f32) {
+                            int64_t dv, bool out_f32, c10::optional<at::Tensor> v, double softcap) {
   TORCH_CHECK(q.is_cuda() && q.dim() == 3 && q.is_contiguous() && (q.scalar_type() == at::kFloat || q.scalar_type() == at::kBFloat16),
               "tied_attn_simple: contiguous q [T, Hq, D], fp32 or bf16");
   TORCH_CHECK(k.dim() >= 3 && k.is_contiguous() && k.scalar_type() == q.scalar_type() && k.size(-1) == q.size(2),
@@ -267,6 +268,12 @@ at::Tensor tied_attn_simple(const at::Tensor& q, const at::Tensor& k, c10::optio
   tdb::TiedSimpleArgs a;
   a.q = q.data_ptr();
   a.k = k.data_ptr();
+  if (v.has_value()) {
+    TORCH_CHECK(v->is_cuda() && v->is_contiguous() && v->scalar_type() == q.scalar_type() && v->dim() == k.dim() && v->size(-1) == Dv &&
+                    v->numel() / Dv == k.numel() / k.size(-1), "tied_attn_simple: contiguous v [..., Hkv, dv] with the rows of k");
+    a.v = v->data_ptr();
+  }
+  a.softcap = softcap;
   a.k_scale = k_scale.has_value() ? k_scale->data_ptr<float>() : nullptr;
   a.row0 = row0.data_ptr<int64_t>();
   a.n_keys = n_keys.data_ptr<int32_t>();
@@ -294,14 +301,14 @@ void bind_attn(py::module_& m) {
   m.def("flash_fwd_sm100", &flash_fwd_sm100, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_table"),
         py::arg("cu_seqlens_q"), py::arg("kv_lens"), py::arg("q_pos0"), py::arg("max_q_len"), py::arg("max_kv_len"),
         py::arg("causal"), py::arg("scale"), py::arg("lse"), py::arg("k_scale") = py::none(), py::arg("sink") = py::none(),
-        py::arg("gate") = py::none());
+        py::arg("gate") = py::none(), py::arg("softcap") = 0.0);
   m.def("decode_attn", &decode_attn, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("block_table"),
         py::arg("kv_lens"), py::arg("workspace"), py::arg("splits"), py::arg("scale"), py::arg("softcap"), py::arg("out"),
         py::arg("out_lse"), py::arg("out_f32"), py::arg("counters"), py::arg("k_scale") = py::none(),
         py::arg("sink") = py::none(), py::arg("gate") = py::none(), py::arg("chunk") = 0);
   m.def("tied_attn_simple", &tied_attn_simple, py::arg("q"), py::arg("k"), py::arg("k_scale"), py::arg("row0"), py::arg("n_keys"),
         py::arg("sink") = py::none(), py::arg("gate") = py::none(), py::arg("scale") = 1.0, py::arg("dv") = 0,
-        py::arg("out_f32") = false);
+        py::arg("out_f32") = false, py::arg("v") = py::none(), py::arg("softcap") = 0.0);
   m.def("dist_decode_attn", &dist_decode_attn, py::arg("heap"), py::arg("q"), py::arg("k_cache"), py::arg("v_cache"),
         py::arg("block_table"), py::arg("kv_lens"), py::arg("workspace"), py::arg("splits"), py::arg("scale"),
         py::arg("softcap"), py::arg("out"), py::arg("staging"), py::arg("ctx"), py::arg("timeout_s"),

@@ -3,8 +3,10 @@
 #include <c10/cuda/CUDAGuard.h>
 #include <torch/extension.h>
 
+#include "tdb/delta.h"
 #include "tdb/hybrid.h"
 #include "tdb/latent.h"
+#include "tdb/streams.h"
 
 namespace py = pybind11;
 using OptTensor = c10::optional<at::Tensor>;
@@ -530,6 +532,164 @@ at::Tensor gla_forward(const at::Tensor& qkvg, const at::Tensor& lowrank, const 
   return out;
 }
 
+// ---- several residual streams
+// One pass between two sublayers (see tdb/streams.h).  ids / table: the streams start; y: what the last sublayer adds; in_w / w: the next
+// one's input, which is returned (an empty tensor without them).
+at::Tensor hyper_step(at::Tensor& x, const OptTensor& ids, const OptTensor& table, const OptTensor& y, const OptTensor& y2, const OptTensor& y_w,
+                      const OptTensor& y2_w, const OptTensor& mix, const OptTensor& out_w, const OptTensor& in_w, const OptTensor& w,
+                      const OptTensor& rows, int64_t n_real, double eps, bool act_is_f32) {
+  TORCH_CHECK(x.dim() == 3, "hyper_step: x [T, streams, W]");
+  tdb::HyperArgs a = {};
+  a.T = x.size(0); a.S = x.size(1); a.W = x.size(2);
+  a.x = f32(x, a.T * a.S * static_cast<int64_t>(a.W), "x");
+  a.is_f32 = act_is_f32 ? 1 : 0;
+  a.n_real = n_real;
+  a.eps = eps;
+  a.n = rows.has_value() ? rows->numel() : a.T;
+  a.store = rows.has_value() ? 0 : 1;
+  c10::cuda::CUDAGuard guard(x.device());
+  const auto act = x.options().dtype(act_is_f32 ? at::kFloat : at::kBFloat16);
+  auto in = [&](const at::Tensor& t, const char* name) -> const void* {
+    TORCH_CHECK(t.is_cuda() && t.scalar_type() == act.dtype() && t.is_contiguous() && t.size(-1) == a.W, name, ": contiguous [.., W] of the activation dtype");
+    return t.data_ptr();
+  };
+  if (rows.has_value()) a.rows = i64(*rows, a.n, "rows");
+  if (ids.has_value()) {
+    TORCH_CHECK(table.has_value(), "hyper_step: table missing");
+    a.ids = i64(*ids, a.T, "ids");
+    a.table = in(*table, "table");
+    a.vocab = table->size(0);
+  }
+  if (y.has_value()) {
+    TORCH_CHECK(mix.has_value() && out_w.has_value() && y->numel() == a.T * a.W, "hyper_step: y [T, W] with its weights");
+    a.y = in(*y, "y");
+    a.mix = f32(*mix, a.S * a.S, "mix");
+    a.out = f32(*out_w, a.S, "out");
+  }
+  if (y2.has_value()) {
+    TORCH_CHECK(y.has_value() && y_w.has_value() && y2_w.has_value() && y2->numel() == a.T * a.W, "hyper_step: second branch");
+    a.y2 = in(*y2, "y2");
+    a.y_w = f32(*y_w, a.W, "y_w");
+    a.y2_w = f32(*y2_w, a.W, "y2_w");
+  }
+  at::Tensor h = at::empty({in_w.has_value() ? a.n : 0, a.W}, act);
+  if (in_w.has_value()) {
+    TORCH_CHECK(w.has_value(), "hyper_step: norm weight missing");
+    a.in = f32(*in_w, a.S, "in");
+    a.w = f32(*w, a.W, "w");
+    a.h = h.data_ptr();
+  }
+  check_cuda(tdb::launch_hyper_step(a, cur_stream()), "launch_hyper_step");
+  return h;
+}
+
+at::Tensor head_prep(const at::Tensor& z, int64_t H, int64_t G, int64_t D, int64_t d_real, const OptTensor& q_w, const OptTensor& k_w, bool unit,
+                     double eps, const at::Tensor& cos_sin, int64_t rot, bool interleaved, const at::Tensor& pos, at::Tensor& k_cache,
+                     at::Tensor& v_cache, const at::Tensor& rows) {
+  tdb::HeadPrepArgs a = {};
+  a.is_f32 = act_f32(z, "z");
+  TORCH_CHECK(z.dim() == 2 && z.stride(1) == 1 && z.size(1) >= (H + 2 * G) * D, "head_prep: z [T, >= (H + 2 G) D]");
+  check_same(k_cache, z, "k_cache");
+  check_same(v_cache, z, "v_cache");
+  TORCH_CHECK(k_cache.numel() % (G * D) == 0 && v_cache.numel() == k_cache.numel(), "head_prep: caches [rows, G, D]");
+  TORCH_CHECK(cos_sin.dim() == 2, "head_prep: cos_sin [positions, width]");
+  a.z = z.data_ptr(); a.ld = z.stride(0); a.T = z.size(0);
+  a.H = H; a.G = G; a.D = D; a.d_real = d_real;
+  if (q_w.has_value()) a.q_w = f32(*q_w, D, "q_w");
+  if (k_w.has_value()) a.k_w = f32(*k_w, D, "k_w");
+  a.n_pos = cos_sin.size(0);
+  a.rot_ld = cos_sin.size(1);
+  a.cos_sin = f32(cos_sin, 0, "cos_sin");
+  a.rot = rot; a.interleaved = interleaved ? 1 : 0; a.unit = unit ? 1 : 0;
+  a.eps = eps;
+  a.pos = i64(pos, a.T, "pos");
+  a.rows = i64(rows, a.T, "rows");
+  a.cap = k_cache.numel() / (G * D);
+  a.k_cache = k_cache.data_ptr();
+  a.v_cache = v_cache.data_ptr();
+  c10::cuda::CUDAGuard guard(z.device());
+  at::Tensor q = at::empty({a.T, H, D}, z.options());
+  a.q_out = q.data_ptr();
+  check_cuda(tdb::launch_head_prep(a, cur_stream()), "launch_head_prep");
+  return q;
+}
+
+at::Tensor gated_act(const at::Tensor& in, int64_t act) {
+  const int fp = act_f32(in, "in");
+  TORCH_CHECK(in.dim() == 2 && in.is_contiguous() && in.size(1) % 2 == 0, "gated_act: contiguous [rows, 2 F]");
+  c10::cuda::CUDAGuard guard(in.device());
+  at::Tensor out = at::empty({in.size(0), in.size(1) / 2}, in.options());
+  check_cuda(tdb::launch_gated_act(in.data_ptr(), out.data_ptr(), in.size(0), in.size(1) / 2, act, fp, cur_stream()), "launch_gated_act");
+  return out;
+}
+
+// Gated delta rule, serving form.  form: 0 decode (one token per sequence), 1 recurrent, 2 chunk-parallel
+at::Tensor delta_forward(const at::Tensor& z, const at::Tensor& ab, const at::Tensor& conv_w, const at::Tensor& a_log, const at::Tensor& dt_bias,
+                         const at::Tensor& norm_w, at::Tensor& state, at::Tensor& conv, const at::Tensor& slots, const at::Tensor& pos0,
+                         const OptTensor& cu, int64_t G, int64_t dv_real, double q_scale, double unit_eps, double eps, int64_t form,
+                         const OptTensor& chunk_seq, const OptTensor& chunk_t0, const OptTensor& seq_chunk0) {
+  tdb::DeltaArgs a = {};
+  a.is_f32 = act_f32(z, "z");
+  TORCH_CHECK(z.dim() == 2 && z.stride(1) == 1, "delta: z [T, ld]");
+  TORCH_CHECK(state.dim() == 4 && conv.dim() == 3, "delta: state [slots, H, dk, dv], conv [slots, taps, C]");
+  a.T = z.size(0); a.ld = z.stride(0);
+  a.G = G; a.H = state.size(1); a.dk = state.size(2); a.dv = state.size(3);
+  a.taps = conv.size(1);
+  const int64_t Gk = G * a.dk, Hv = static_cast<int64_t>(a.H) * a.dv, C = 2 * Gk + Hv;
+  TORCH_CHECK(z.size(1) >= C + Hv && conv.size(2) == C && conv.size(0) == state.size(0), "delta: shapes of z and conv");
+  TORCH_CHECK(conv_w.dim() == 2 && conv_w.size(0) == C && conv_w.size(1) == a.taps, "delta: conv_w [C, taps]");
+  check_same(conv, z, "conv");
+  a.z = z.data_ptr();
+  a.ab = f32(ab, a.T * 2 * a.H, "ab");
+  a.conv_w = f32(conv_w, C * a.taps, "conv_w");
+  a.a_log = f32(a_log, a.H, "a_log");
+  a.dt_bias = f32(dt_bias, a.H, "dt_bias");
+  a.norm_w = f32(norm_w, a.dv, "norm_w");
+  a.state = f32(state, 0, "state");
+  a.conv = conv.data_ptr();
+  a.N = slots.numel();
+  a.slots = i32(slots, a.N, "slots");
+  a.pos0 = i64(pos0, a.N, "pos0");
+  if (cu.has_value()) a.cu = i32(*cu, a.N + 1, "cu");
+  a.dv_real = dv_real; a.q_scale = q_scale; a.unit_eps = unit_eps; a.eps = eps;
+  c10::cuda::CUDAGuard guard(z.device());
+  at::Tensor out = at::empty({a.T, Hv}, z.options());
+  a.out = out.data_ptr();
+  if (form == 0) {
+    TORCH_CHECK(a.T == a.N, "delta decode: one token per sequence");
+    check_cuda(tdb::launch_delta_decode(a, cur_stream()), "launch_delta_decode");
+    return out;
+  }
+  TORCH_CHECK(cu.has_value() && chunk_seq.has_value() && chunk_t0.has_value() && seq_chunk0.has_value(), "delta prompt: tables missing");
+  a.NC = chunk_seq->numel();
+  a.chunk_seq = i32(*chunk_seq, a.NC, "chunk_seq");
+  a.chunk_t0 = i32(*chunk_t0, a.NC, "chunk_t0");
+  a.seq_chunk0 = i32(*seq_chunk0, a.N + 1, "seq_chunk0");
+  const auto fo = z.options().dtype(at::kFloat), bo = z.options().dtype(at::kBFloat16);
+  at::Tensor gb = at::empty({2, a.T, a.H}, fo);
+  a.log_g = gb.data_ptr<float>();
+  a.beta = a.log_g + a.T * a.H;
+  if (form == 1) {
+    at::Tensor qk = at::empty({2, a.T, Gk}, fo), v = at::empty({2, a.T, Hv}, fo);
+    a.q = qk.data_ptr<float>();
+    a.k = qk.data_ptr<float>() + a.T * Gk;
+    a.v = v.data_ptr<float>();
+    a.o_raw = v.data_ptr<float>() + a.T * Hv;
+    check_cuda(tdb::launch_delta_recurrent(a, cur_stream()), "launch_delta_recurrent");
+    return out;
+  }
+  at::Tensor qk = at::empty({4, a.T, Gk}, bo), v = at::empty({a.T, Hv}, bo);
+  a.q = qk[0].data_ptr(); a.q_lo = qk[1].data_ptr(); a.k = qk[2].data_ptr(); a.k_lo = qk[3].data_ptr();
+  a.v = v.data_ptr();
+  const int64_t NH = static_cast<int64_t>(a.NC) * a.H;
+  at::Tensor trans = at::empty({NH, a.dk, a.dk}, fo), inject = at::empty({NH, a.dk, a.dv}, fo), read = at::empty({NH, 64, a.dk}, fo);
+  at::Tensor local = at::empty({NH, 64, a.dv}, fo), states = at::empty({NH, a.dk, a.dv}, fo), decay = at::empty({NH}, fo);
+  a.trans = trans.data_ptr(); a.inject = inject.data_ptr<float>(); a.read = read.data_ptr();
+  a.local = local.data_ptr<float>(); a.states = states.data_ptr(); a.decay = decay.data_ptr<float>();
+  check_cuda(tdb::launch_delta_chunk(a, cur_stream()), "launch_delta_chunk");
+  return out;
+}
+
 }  // namespace
 
 void bind_hybrid(py::module_& m) {
@@ -553,5 +713,10 @@ void bind_hybrid(py::module_& m) {
   m.def("latent_prefill", &latent_prefill);
   m.def("latent_decode", &latent_decode);
   m.def("gla_forward", &gla_forward);
+  m.def("hyper_step", &hyper_step);
+  m.def("head_prep", &head_prep);
+  m.def("gated_act", &gated_act);
+  m.def("delta_forward", &delta_forward);
+  m.def("delta_chunk_supported", &tdb::delta_chunk_supported);
   m.def("gla_chunk_supported", &tdb::gla_chunk_supported);
 }

@@ -23,6 +23,7 @@
 #include "tdb/gemv.h"
 #include "tdb/launch.cuh"
 #include "tdb/symm_device.cuh"
+#include "tdb/vec.cuh"
 
 namespace tdb {
 
@@ -43,7 +44,7 @@ struct GemvParams {
   int64_t ld_out;
   const __nv_bfloat16* norm_w;
   float eps;
-  int silu_mul;
+  int gated;
   const __nv_bfloat16* residual;
   int64_t ld_res;
   int rows_per_cta;
@@ -150,18 +151,19 @@ __global__ void __launch_bounds__(kGemvThreads, 1) gemv_kernel(const GemvParams 
       for (int i = 0; i < MB; ++i) {
         const int m = m0 + i;
         v[i] = (m < p.M) ? ld_v4(p.x + static_cast<int64_t>(m) * p.ldx + c * 8) : make_uint4(0u, 0u, 0u, 0u);
-        if (p.silu_mul)
+        if (p.gated)
           u[i] = (m < p.M) ? ld_v4(p.x + static_cast<int64_t>(m) * p.ldx + p.K + c * 8) : make_uint4(0u, 0u, 0u, 0u);
       }
 #pragma unroll
       for (int i = 0; i < MB; ++i) {
         const int m = m0 + i;
-        if (p.silu_mul) {
+        if (p.gated) {
           float gg[8], h[8];
           unpack8(v[i], gg);
           unpack8(u[i], h);
 #pragma unroll
-          for (int j = 0; j < 8; ++j) gg[j] = gg[j] / (1.f + __expf(-gg[j])) * h[j];
+          for (int j = 0; j < 8; ++j)
+            gg[j] = (p.gated == 1 ? gg[j] / (1.f + __expf(-gg[j])) : gelu_tanh_f32(gg[j])) * h[j];
           v[i] = pack8(gg);
         } else if (p.norm_w != nullptr) {
           float a[8];
@@ -352,7 +354,7 @@ cudaError_t launch_gemv(const GemvArgs& a, cudaStream_t stream) {
   if (a.M < 1 || a.M > 16 || a.K % 8 != 0 || a.K > gemv_max_k(a.M)) return cudaErrorInvalidValue;
   if (a.ldw % 8 != 0 || a.ldx % 8 != 0) return cudaErrorInvalidValue;
   if ((reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.x)) & 15u) return cudaErrorInvalidValue;
-  if (a.norm_w != nullptr && a.silu_mul) return cudaErrorInvalidValue;
+  if (a.norm_w != nullptr && a.gated) return cudaErrorInvalidValue;
   GemvParams p;
   p.M = a.M; p.N = a.N; p.K = a.K;
   p.x = reinterpret_cast<const __nv_bfloat16*>(a.x);
@@ -363,7 +365,7 @@ cudaError_t launch_gemv(const GemvArgs& a, cudaStream_t stream) {
   p.ld_out = a.ld_out;
   p.norm_w = reinterpret_cast<const __nv_bfloat16*>(a.norm_w);
   p.eps = a.eps;
-  p.silu_mul = a.silu_mul;
+  p.gated = a.gated;
   p.residual = reinterpret_cast<const __nv_bfloat16*>(a.residual);
   p.ld_res = a.ld_res;
   p.all_reduce = a.all_reduce;

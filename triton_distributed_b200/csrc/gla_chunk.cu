@@ -21,6 +21,7 @@
 // The state and everything that enters it count as fp32, so the tensor cores (mma.sync bf16, fp32 accumulate) get every
 // fp32 operand as a high and a low bf16 part: two products where one side is bf16 anyway (v), three where both are fp32.
 #include "tdb/attn_device.cuh"
+#include "tdb/chunk.cuh"
 #include "tdb/gla.cuh"
 #include "tdb/hybrid.h"
 #include "tdb/launch.cuh"
@@ -36,42 +37,18 @@ using attn::cp_async_wait;
 using attn::ldmatrix_x4_trans;
 using attn::mma_bf16;
 
-constexpr int kC = 64;            // tokens per chunk
+using chunk::ChunkPos;
+using chunk::HiLo;
+using chunk::chunk_pos;
+using chunk::kC;
+using chunk::ld2;
+using chunk::ldmatrix_x4;
+using chunk::split2;
+
 constexpr int kThreads = 256;
 
-struct HiLo {
-  uint32_t hi, lo;
-};
-// Two fp32 values as packed bf16 high parts and packed bf16 remainders.
-TDB_DEVICE HiLo split2(float a, float b) {
-  HiLo r;
-  r.hi = pack_bf16x2(a, b);
-  const float2 h = unpack_bf16x2(r.hi);
-  r.lo = pack_bf16x2(a - h.x, b - h.y);
-  return r;
-}
-TDB_DEVICE float2 ld2(const __nv_bfloat16* p) { return unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p)); }
-
-struct ChunkPos {
-  int64_t t0;
-  int n;       // tokens of the chunk
-};
-TDB_DEVICE ChunkPos chunk_pos(const GlaArgs& p, int chunk) {
-  ChunkPos r;
-  r.t0 = p.chunk_t0[chunk];
-  const int64_t end = p.cu[p.chunk_seq[chunk] + 1];
-  r.n = static_cast<int>(min(static_cast<int64_t>(kC), end - r.t0));
-  return r;
-}
-
-// Rows [0, 64) of `cols` bf16 columns starting at src (row stride ld) into smem with row pitch `pitch` elements; rows >= n
-// are zero.
 TDB_DEVICE void load_tile(__nv_bfloat16* dst, int pitch, const __nv_bfloat16* src, int64_t ld, int cols, int n) {
-  const int vec = cols >> 3;
-  for (int i = threadIdx.x; i < kC * vec; i += kThreads) {
-    const int r = i / vec, c = i - r * vec;
-    cp_async16(dst + r * pitch + c * 8, src + (r < n ? r * ld : 0) + c * 8, r < n);
-  }
+  chunk::load_tile(dst, pitch, src, ld, cols, n, kThreads);
 }
 
 // The chunk's cumulative log decays of one head into G [64][dk + 8] (asynchronous, 16-byte copies) ...
@@ -373,12 +350,6 @@ TDB_DEVICE void triangle_scores(const GlaArgs& p, const __nv_bfloat16* qs, const
     acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], 2);
     if (part == 0) A[tt[i] * kAp + jj[i]] = acc[i];
   }
-}
-
-TDB_DEVICE void ldmatrix_x4(uint32_t (&r)[4], const void* smem_row) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(smem_u32(smem_row)));
 }
 
 template <int TW>     // 8-column tiles per warp: dv <= 64 TW

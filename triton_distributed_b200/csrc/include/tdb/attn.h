@@ -59,6 +59,7 @@ struct FlashFwdSm100Args {
   int64_t total_q;
   int causal;
   float scale;
+  float softcap = 0.f;
   int Lp;
   void* k_dense;
   void* vt_dense;
@@ -82,12 +83,13 @@ struct DecodeArgs {
   int chunk = 0;                       // > 0: block-local attention, see DecodeParams
 };
 
-// Attention in plain fp32 arithmetic over the tied form, for any head dim up to 1024 and fp32 or bf16 tensors: one warp
-// per (token, head).  Token t sees the rows [row0[t], row0[t] + n_keys[t]) of k (viewed as [rows, Hkv, D]); its value is the
-// first Dv elements of a row (a row may end in a part that is key only).
+// Attention in plain fp32 arithmetic, for any head dim up to 1024 and fp32 or bf16 tensors: one warp per (token, head).
+// Token t sees the rows [row0[t], row0[t] + n_keys[t]) of k (viewed as [rows, Hkv, D]); its value is a row of v, or in the tied
+// form the first Dv elements of a row of k (a row may end in a part that is key only).
 struct TiedSimpleArgs {
   const void* q;               // [T, Hq, D]
   const void* k;               // [rows, Hkv, D]
+  const void* v = nullptr;     // [rows, Hkv, Dv] values of their own; null = tied
   const float* k_scale;        // [rows], null = 1
   const int64_t* row0;         // [T]
   const int32_t* n_keys;       // [T]
@@ -95,6 +97,7 @@ struct TiedSimpleArgs {
   int64_t T;
   int Hq, Hkv, D, Dv;
   float scale;                 // of the scores, beside k_scale
+  float softcap = 0.f;         // score -> softcap * tanh(score / softcap), 0 = none
   int is_f32;                  // dtype of q / k / gate
   int out_f32;                 // dtype of out
   AttnEpilogue epi;

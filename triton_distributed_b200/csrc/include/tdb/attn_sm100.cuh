@@ -29,6 +29,8 @@ struct FwdParams {
   int Hq, Hkv, group, causal;
   int dv;                      // columns of an output row
   float scale_log2;            // scale * log2(e)
+  float cap_log2 = 0.f;        // soft cap * log2(e), 0 = none: the score s becomes cap * tanh(s * scale / cap)
+  float to_cap = 0.f;          // scale / cap
   int64_t total_q;
   int* error_flag;             // device int, set on a timeout
   AttnEpilogue epi;            // sink / output gate of the rows
@@ -45,8 +47,43 @@ struct TileCtx {
   int row0, rows_here, nblk;
 };
 
-// DV: columns of the output accumulator (a multiple of 32); the rows written have p.dv <= DV columns, a multiple of 8.
-template <int DV>
+// Scores -> cap_log2 * tanh(to_cap * score), exact to fp32 rounding of the cap.  The power series of tanh takes the place of the
+// exponential and the division while all 32 arguments of the warp's rows are small: those two share the unit that the softmax keeps
+// busy.  Masked scores (minus infinity) stay what they are.
+__device__ __forceinline__ void cap_scores(uint32_t (&s)[32], float to_cap, float cap_log2) {
+  float big = 0.f;
+#pragma unroll
+  for (int c = 0; c < 32; ++c) {
+    const float x = __uint_as_float(s[c]) * to_cap;
+    s[c] = __float_as_uint(x);
+    big = fmaxf(big, x == -INFINITY ? 0.f : fabsf(x));
+  }
+  if (__all_sync(0xffffffffu, big < 0.3f)) {
+    // x (1 - x^2/3 + 2 x^4/15 - 17 x^6/315 + 62 x^8/2835): the next term is below 1e-8 here
+#pragma unroll
+    for (int c = 0; c < 32; ++c) {
+      const float x = __uint_as_float(s[c]);
+      const float q = x * x;
+      float f = fmaf(q, 62.f / 2835.f, -17.f / 315.f);
+      f = fmaf(q, f, 2.f / 15.f);
+      f = fmaf(q, f, -1.f / 3.f);
+      const float y = cap_log2 * fmaf(x * q, f, x);
+      s[c] = x == -INFINITY ? 0xff800000u : __float_as_uint(y);
+    }
+    return;
+  }
+#pragma unroll
+  for (int c = 0; c < 32; ++c) {
+    const float x = __uint_as_float(s[c]);
+    // tanh x = 1 - 2 / (e^{2x} + 1); the exponent is clamped where fp32 tanh has long been 1
+    const float y = 1.f - __fdividef(2.f, ex2(fminf(x * 2.8853900817779268f, 60.f)) + 1.f);
+    s[c] = x == -INFINITY ? 0xff800000u : __float_as_uint(cap_log2 * y);
+  }
+}
+
+// DV: columns of the output accumulator (a multiple of 32); the rows written have p.dv <= DV columns, a multiple of 8.  CAP: with
+// soft cap.
+template <int DV, bool CAP = false>
 __device__ __forceinline__ void softmax_tile(const FwdParams& p, const TileCtx& t, int warp, int lane, int q_begin, int head,
                                              int kv_len, int pos0, volatile int* abort_flag) {
   uint64_t* s_full = t.s_full;
@@ -87,10 +124,15 @@ __device__ __forceinline__ void softmax_tile(const FwdParams& p, const TileCtx& 
         if (t0 + 32 + c >= lim) s1[c] = 0xff800000u;
       }
     }
+    if constexpr (CAP) {
+      cap_scores(s0, p.to_cap, p.cap_log2);
+      cap_scores(s1, p.to_cap, p.cap_log2);
+    }
     float mx = -INFINITY;
 #pragma unroll
     for (int c = 0; c < 32; ++c) mx = fmaxf(mx, fmaxf(__uint_as_float(s0[c]), __uint_as_float(s1[c])));
-    mx *= p.scale_log2;                                   // scale > 0: the maximum commutes with it
+    const float scale_log2 = CAP ? 1.f : p.scale_log2;    // capped scores are in the log2 domain already
+    mx *= scale_log2;                                     // scale > 0: the maximum commutes with it
     // raise the reference only when the row maximum has outgrown it by more than the step (or there is none yet)
     float alpha = 1.f;
     bool raise = false;
@@ -129,8 +171,8 @@ __device__ __forceinline__ void softmax_tile(const FwdParams& p, const TileCtx& 
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int c = c8 * 8 + 2 * e;
-        const float x0 = ex2(fmaf(__uint_as_float(c < 32 ? s0[c] : s1[c - 32]), p.scale_log2, -m_use));
-        const float x1 = ex2(fmaf(__uint_as_float(c + 1 < 32 ? s0[c + 1] : s1[c + 1 - 32]), p.scale_log2, -m_use));
+        const float x0 = ex2(fmaf(__uint_as_float(c < 32 ? s0[c] : s1[c - 32]), scale_log2, -m_use));
+        const float x1 = ex2(fmaf(__uint_as_float(c + 1 < 32 ? s0[c + 1] : s1[c + 1 - 32]), scale_log2, -m_use));
         sum += x0 + x1;
         pk[e] = pack_bf16x2(x0, x1);
       }

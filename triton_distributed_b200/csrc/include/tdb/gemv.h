@@ -7,7 +7,7 @@ namespace tdb {
 
 struct GemvArgs {
   int M, N, K;
-  const void* x;        // bf16 [M, ldx]; with silu_mul: [M, 2K] as gate | up
+  const void* x;        // bf16 [M, ldx]; gated: [M, 2K] as gate | up
   int64_t ldx;
   const void* w;        // bf16 [N, ldw], K contiguous
   int64_t ldw;
@@ -15,7 +15,7 @@ struct GemvArgs {
   int64_t ld_out;
   const void* norm_w;   // bf16 [K] or null: f(x) = rmsnorm(x) * norm_w
   float eps;
-  int silu_mul;         // f(x) = silu(x[:, :K]) * x[:, K:]
+  int gated;            // f(x) = act(x[:, :K]) * x[:, K:], 1: silu, 2: gelu (tanh form); 0: not gated
   const void* residual; // bf16 [M, ld_res] or null, added to the result; may be `out` itself
   int64_t ld_res;
   int num_ctas;

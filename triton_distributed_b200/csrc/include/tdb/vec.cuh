@@ -46,5 +46,6 @@ TDB_DEVICE float block_reduce_sum(float v, float* red) {
 }
 
 TDB_DEVICE float sigmoid_f32(float z) { return 1.f / (1.f + expf(-z)); }
+TDB_DEVICE float gelu_tanh_f32(float z) { return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
 
 }  // namespace tdb

@@ -123,6 +123,15 @@ __global__ void __launch_bounds__(128) tied_attn_simple_kernel(const TiedSimpleA
       s = fmaf(qf[i], kf[i], s);
     }
     s = warp_sum(s) * (p.k_scale != nullptr ? p.k_scale[row0 + j] * p.scale : p.scale);
+    if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
+    if (p.v != nullptr) {
+      const T* vr = reinterpret_cast<const T*>(p.v) + ((row0 + j) * p.Hkv + hkv) * p.Dv;
+#pragma unroll
+      for (int i = 0; i < kPer; ++i) {
+        const int d = lane + 32 * i;
+        kf[i] = (i < per && d < p.Dv) ? to_f32(vr[d]) : 0.f;
+      }
+    }
     const float mn = fmaxf(m, s);
     const float corr = expf(m - mn), e = expf(s - mn);   // m = -inf -> 0
     l = l * corr + e;
@@ -180,7 +189,7 @@ cudaError_t launch_qk_sumsq(const QkNormArgs& a, float* out, cudaStream_t s) {
 }
 
 cudaError_t launch_tied_attn_simple(const TiedSimpleArgs& a, cudaStream_t s) {
-  if (a.D < 1 || a.D > kSimpleMaxD || a.Dv < 1 || a.Dv > a.D || a.Hkv < 1 || a.Hq % a.Hkv != 0) return cudaErrorInvalidValue;
+  if (a.D < 1 || a.D > kSimpleMaxD || a.Dv < 1 || a.Dv > a.D || a.softcap < 0.f || a.Hkv < 1 || a.Hq % a.Hkv != 0) return cudaErrorInvalidValue;
   if (a.T == 0) return cudaSuccess;
   if (a.is_f32) return launch_simple<float, float>(a, s);
   return a.out_f32 ? launch_simple<__nv_bfloat16, float>(a, s) : launch_simple<__nv_bfloat16, __nv_bfloat16>(a, s);

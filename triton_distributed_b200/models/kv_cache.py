@@ -147,9 +147,47 @@ class LatentSpec:
 
 
 @dataclass(frozen=True)
+class KVSpec:
+    """A layer that caches a key and a value per token and KV head, both of ``head_dim`` elements."""
+    kv_heads: int
+    head_dim: int
+
+
+@dataclass(frozen=True)
+class DeltaSpec:
+    """A recurrent layer behind short convolutions: fp32 state [heads, dk, dv] and the convolutions' last inputs, a ring of ``taps``
+    rows (position p at row ``p % taps``) of ``channels`` elements."""
+    heads: int
+    dk: int
+    dv: int
+    channels: int
+    taps: int
+
+
+@dataclass(frozen=True)
+class GroupSpec:
+    """A layer of several mixers side by side, each with its own storage under its own names."""
+    parts: tuple
+
+
+@dataclass(frozen=True)
 class SharedSpec:
     """A layer without storage of its own: it reads that of layer ``source``."""
     source: int
+
+
+@dataclass
+class KVPlan:
+    """What layers with a key and a value per token need to know about a step (see ``StepPlan.kv``): a sequence's rows are one page of
+    ``max_length`` rows, the page of its slot."""
+    home_rows: torch.Tensor                         # int64 [T] cache row of every token
+    row0: torch.Tensor                              # int64 [T] cache row of the sequence's first token
+    n_keys: torch.Tensor                            # int32 [T]
+    kv_lens: torch.Tensor                           # int32 [sequences]
+    block_table: torch.Tensor                       # int32 [sequences, 1]
+    q_pos0: Optional[torch.Tensor] = None           # int32 [sequences] (prompts)
+    max_q: int = 1
+    max_kv: int = 0                                 # longest sequence after the step (prompts)
 
 
 @dataclass
@@ -203,6 +241,7 @@ class StepPlan:
         self._blocks: Dict[int, BlockPlan] = {}
         self._chunks = None
         self._latent: Optional[LatentPlan] = None
+        self._kv: Optional[KVPlan] = None
         self.contexts: Dict[int, torch.Tensor] = {}  # packed rows of the layers that later layers of the step read as well
         if not self.decode:
             cu = [0]
@@ -213,10 +252,26 @@ class StepPlan:
             self.last_rows = torch.tensor([c - 1 for c in cu[1:]], dtype=torch.int64).to(slots.device)
 
     def chunk_tables(self):
-        """Chunks of the gated-linear-attention kernels (None for a decode step)."""
+        """Chunks of the recurrent layers' kernels (None for a decode step)."""
         if self._chunks is None and not self.decode:
             self._chunks = gla_chunk_tables(self.cu_host, self.slots.device)
         return self._chunks
+
+    def kv(self) -> KVPlan:
+        if self._kv is None:
+            M = self.cache.max_length
+            pages = self.slots.unsqueeze(1).contiguous()
+            n = (self.positions + 1).to(torch.int32)
+            if self.decode:
+                row0 = self.slots.to(torch.int64) * M
+                self._kv = KVPlan(row0 + self.positions, row0, n, n, pages)
+            else:
+                slots, starts, lens = self.host
+                row0 = torch.cat([torch.full((k,), s * M, dtype=torch.int64) for s, k in zip(slots, lens)]).to(self.slots.device)
+                ends = [a + k for a, k in zip(starts, lens)]
+                small = torch.tensor(ends + list(starts), dtype=torch.int32).to(self.slots.device)
+                self._kv = KVPlan(row0 + self.positions, row0, n, small[:len(lens)], pages, small[len(lens):], max(lens), max(ends))
+        return self._kv
 
     def latent(self) -> LatentPlan:
         if self._latent is None:
@@ -300,8 +355,8 @@ class StepPlan:
 
 
 class HybridCache:
-    """Cache of a layered decoder: one storage per layer (``TiedKVSpec``, ``LatentSpec`` or ``StateSpec``; ``SharedSpec`` layers
-    share another layer's), indexed by a sequence's slot.
+    """Cache of a layered decoder: one storage per layer run (``KVSpec``, ``TiedKVSpec``, ``LatentSpec``, ``StateSpec``, ``DeltaSpec``, or a
+    ``GroupSpec`` of several; ``SharedSpec`` layers share another layer's), indexed by a sequence's slot.
 
     Slots are handed out by ``alloc`` and given back by ``free``; nothing is cleared in between, because a sequence that
     starts at position 0 neither reads its state row nor any row it has not written.  ``kv_offset`` (device) and ``lens``
@@ -336,18 +391,31 @@ class HybridCache:
                 if not 0 <= spec.source < i or isinstance(self.specs[spec.source], SharedSpec):
                     raise ValueError(f"layer {i} cannot share the cache of layer {spec.source}")
                 self.layers[i] = self.layers[spec.source]
-            elif isinstance(spec, LatentSpec):
-                st["latent"] = widen(st.get("latent"), self.max_length, spec.rank + spec.rot, dtype=self.dtype)
-            elif isinstance(spec, TiedKVSpec):
-                rows = spec.rows(self.max_length)
-                st["k"] = widen(st.get("k"), rows, spec.kv_heads, spec.head_dim, dtype=self.dtype)
-                st["scale"] = widen(st.get("scale"), rows, dtype=torch.float32)
-            else:
-                st["state"] = widen(st.get("state"), spec.heads, spec.dk, spec.dv, dtype=torch.float32)
+                continue
+            parts = spec.parts if isinstance(spec, GroupSpec) else (spec,)
+            names = [n for s in parts for n in self._tensors(s)]
+            if len(set(names)) != len(names):
+                raise ValueError(f"layer {i}: mixers side by side need storage of different names")
+            for s in parts:
+                for name, (shape, dtype) in self._tensors(s).items():
+                    st[name] = widen(st.get(name), *shape, dtype=dtype)
         self.kv_offset = widen(self.kv_offset, dtype=torch.int32)
         self._free = list(range(capacity - 1, self.capacity - 1, -1)) + self._free
         self.lens += [0] * (capacity - self.capacity)
         self.capacity = capacity
+
+    def _tensors(self, spec) -> Dict[str, tuple]:
+        """Storage of one slot: name -> (shape, dtype)."""
+        M, act = self.max_length, self.dtype
+        if isinstance(spec, LatentSpec):
+            return {"latent": ((M, spec.rank + spec.rot), act)}
+        if isinstance(spec, TiedKVSpec):
+            rows = spec.rows(M)
+            return {"k": ((rows, spec.kv_heads, spec.head_dim), act), "scale": ((rows,), torch.float32)}
+        if isinstance(spec, KVSpec):
+            return {n: ((M, spec.kv_heads, spec.head_dim), act) for n in ("k", "v")}
+        state = {"state": ((spec.heads, spec.dk, spec.dv), torch.float32)}
+        return {**state, "conv": ((spec.taps, spec.channels), act)} if isinstance(spec, DeltaSpec) else state
 
     def alloc(self) -> int:
         """A slot for a new sequence (the storage doubles when none is free; captured graphs do not survive that)."""
@@ -412,8 +480,8 @@ class HybridCache:
         self.lens = [0] * self.capacity
 
     def snapshot(self):
-        """Copies of what a decode step changes besides the row it writes (recurrent states): a step run for warm-up must
-        not count."""
+        """Copies of what a decode step changes besides the rows it writes (recurrent states): a step run for warm-up must
+        not count.  (Writing a row again, of a ring as well, writes the same values.)"""
         return [st["state"].clone() if "state" in st else None for st in self.layers]
 
     def restore(self, snap):

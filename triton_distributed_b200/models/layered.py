@@ -1,4 +1,4 @@
-"""Common part of the decoders whose configuration lists the layers one by one (Vasolix, Lisenex): loading, execution modes,
+"""Common part of the decoders whose configuration lists the layers one by one (Vasolix, Lisenex, Tazitar): loading, execution modes,
 cache, packed steps, the engine's rectangular interface, random weights by tensor name.
 
 A model is a list of layers with ``parts()`` (tensor-parallel mixers / feed-forwards) and ``load``; a subclass builds them and runs
@@ -66,9 +66,17 @@ class LayeredLLM:
     def make_layers(self) -> list:
         raise NotImplementedError
 
-    def hidden(self, ids: torch.Tensor, plan: StepPlan, streams: Optional[List[torch.Tensor]]) -> torch.Tensor:
-        """The residual stream [T, W] after the last layer; ``streams`` collects it after every layer."""
+    def hidden(self, ids: torch.Tensor, plan: StepPlan, streams: Optional[List[torch.Tensor]]):
+        """The residual stream [T, W] after the last layer (or what ``final_hidden`` takes); ``streams`` collects it after every layer."""
         raise NotImplementedError
+
+    def final_hidden(self, x, rows: Optional[torch.Tensor]) -> torch.Tensor:
+        """What the output projection reads: the normed rows of what ``hidden`` returned."""
+        return ops.stream_norm(x, self.final_norm_w, self.arch.hidden_size, self.arch.rms_norm_eps, self.dtype, rows)
+
+    def cache_specs(self) -> list:
+        """Storage of every layer in the order in which they run."""
+        return [l.mixer.cache_spec() for l in self.layers]
 
     # -- parameters -------------------------------------------------------------------------------------------
     def table(self, get, name: str) -> torch.Tensor:
@@ -119,7 +127,7 @@ class LayeredLLM:
                 part.ar_ctx = part.gemm_ar_ctx = None
 
     def new_cache(self, batch_size: int, max_length: int, allocate: bool = True) -> HybridCache:
-        return HybridCache([l.mixer.cache_spec() for l in self.layers], batch_size, max_length, self.dtype, self.device, allocate)
+        return HybridCache(self.cache_specs(), batch_size, max_length, self.dtype, self.device, allocate)
 
     # -- forward ----------------------------------------------------------------------------------------------
     @torch.no_grad()
@@ -128,8 +136,7 @@ class LayeredLLM:
         """One step over packed tokens ``ids`` [T]: fp32 logits [len(rows), vocab] of the given token rows (None: all), or
         the normed hidden rows.  The caller advances the cache.  ``streams`` collects the residual stream after every
         layer (a debugging aid)."""
-        x = self.hidden(ids, plan, streams)
-        h = ops.stream_norm(x, self.final_norm_w, self.arch.hidden_size, self.arch.rms_norm_eps, self.dtype, rows)
+        h = self.final_hidden(self.hidden(ids, plan, streams), rows)
         if wo_lm_head:
             return h
         logits = torch.matmul(h, self.lm_head.t()) if self.mode == "torch" else ops.gemm(h, self.lm_head)

@@ -13,12 +13,12 @@ from .allgather import (AllGatherMethod, get_auto_all_gather_method, FastAllGath
                         create_fast_allgather_context, fast_allgather, all_gather_ll, all_gather,
                         cp_engine_producer_all_gather_intra_node,
                         cp_engine_producer_all_gather_inter_node)
-from .elementwise import (rmsnorm, silu_mul, residual_add, qk_norm_rope_kv, embedding, argmax, sample_token,  # noqa: F401
+from .elementwise import (rmsnorm, silu_mul, gated_act, residual_add, qk_norm_rope_kv, embedding, argmax, sample_token,  # noqa: F401
                           abs_sum)
 from .attention import (flash_attn_varlen, gqa_fwd_batch_decode, gqa_fwd_batch_decode_intra_rank,  # noqa: F401
                         gqa_fwd_batch_decode_persistent, attention_reference, merge_attention_partials,
-                        dense_block_table, decode_workspace, pick_kv_splits, tied_attention_simple, tied_attn_varlen,
-                        tied_attn_decode, pick_tied_splits, TIED_TENSOR_CORE_DIMS, check_attention_errors)
+                        dense_block_table, decode_workspace, pick_kv_splits, attention_simple, tied_attention_simple, tied_attn_varlen,
+                        tied_attn_decode, TENSOR_CORE_DIMS, pick_tied_splits, TIED_TENSOR_CORE_DIMS, check_attention_errors)
 from .gemv import (GemvARContext, create_gemv_ar_context, gemv_fused, gemv_reference, gemv_supported,  # noqa: F401
                    GEMV_FAST_M, GEMV_MAX_M)
 from .gemm_ar import (GemmARContext, LLGemmARContext, create_gemm_ar_context, create_ll_gemm_ar_context,  # noqa: F401
@@ -40,10 +40,12 @@ from .fp8 import (ag_gemm_fp8, dequantize_act_1x128, dequantize_weight_128x128, 
 from .moe import (tile_arrival_order, tile_schedule, sort_topk_ids_staged, group_gemm_gather,  # noqa: F401,E402
                   MoESort, MoEAgScatterGroupGemmContext, MoEReduceRSContext)
 from .stream import (embed_stream, postnorm_add, combine_rows, stream_norm, qk_sumsq, qk_norm_tied, FeedForward,  # noqa: F401,E402
-                     parallel_add, parallel_sum)
+                     parallel_add, parallel_sum, HyperWeights, SublayerOutput, hyper_step)
+from .rotary import rope_table, YarnScaling, head_prep  # noqa: F401,E402
+from .delta import gated_delta_rule, DELTA_MAX_DIM  # noqa: F401,E402
 from .gla import gated_linear_attention, gla_chunk_tables, GLA_CHUNK  # noqa: F401,E402
 from .moe import (narrow_linear, sigmoid_router, softmax_router, relu2, relu2_experts_gemv, gated_experts_gemv,  # noqa: F401,E402
                   EXPERT_GEMV_MAX_T)
-from .latent import (rope_table, latent_rotate, latent_absorb, latent_out, latent_attention, latent_prefill,  # noqa: F401,E402
+from .latent import (latent_rotate, latent_absorb, latent_out, latent_attention, latent_prefill,  # noqa: F401,E402
                      latent_decode, latent_prefill_supported, latent_decode_supported, pick_latent_splits,
                      check_latent_errors)

@@ -33,7 +33,7 @@ def _gather_kv(k_cache, v_cache, block_table, b: int, n: int):
 
 
 def attention_reference(q, k_cache, v_cache, block_table, cu_seqlens_q, kv_lens, q_pos0=None, causal=True,
-                        scale=None, softcap: float = 0.0, return_lse: bool = False):
+                        scale=None, softcap: float = 0.0, return_lse: bool = False, sink=None):
     """fp32 softmax attention, one sequence at a time.  q [T, Hq, D] packed by ``cu_seqlens_q``."""
     T, Hq, D = q.shape
     Hkv = k_cache.shape[2]
@@ -59,7 +59,8 @@ def attention_reference(q, k_cache, v_cache, block_table, cu_seqlens_q, kv_lens,
             kpos = torch.arange(n, device=q.device)
             s = s.masked_fill(kpos[None, None, :] > qpos[None, :, None], float("-inf"))
         l = torch.logsumexp(s, dim=-1)
-        p = torch.exp(s - l.unsqueeze(-1))
+        d = l if sink is None else torch.logaddexp(l, sink.float()[:, None])
+        p = torch.exp(s - d.unsqueeze(-1))
         p = torch.nan_to_num(p, nan=0.0)
         out[qs:qe] = torch.einsum("hqk,khd->qhd", p, vf)
         lse[:, qs:qe] = l
@@ -68,6 +69,7 @@ def attention_reference(q, k_cache, v_cache, block_table, cu_seqlens_q, kv_lens,
     return out.to(q.dtype)
 
 
+TENSOR_CORE_DIMS = (64, 128, 256)      # head dims of the mma.sync kernels (tcgen05: 128)
 SM100_PREFILL_MIN_Q = 128      # below this the 64-row mma.sync kernel has less padding and no KV packing pass
 _PENDING_ERRORS = []            # error flags of tcgen05 prefill launches that have not been looked at yet
 
@@ -86,36 +88,37 @@ def flash_attn_varlen(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
                       cu_seqlens_q: torch.Tensor, kv_lens: torch.Tensor, max_q_len: int,
                       q_pos0: Optional[torch.Tensor] = None, causal: bool = True, scale: Optional[float] = None,
                       softcap: float = 0.0, return_lse: bool = False, max_kv_len: Optional[int] = None,
-                      impl: str = "auto"):
+                      impl: str = "auto", sink: Optional[torch.Tensor] = None):
     """Prefill / context attention.  ``q`` [T, Hq, D] packed; query row i of sequence b has absolute position
     ``q_pos0[b] + i`` (default: the queries are the last ``q_len`` positions of the ``kv_lens[b]`` visible tokens).
 
-    ``impl``: "auto" picks the tcgen05 kernel (head dim 128, no soft cap, at least ``SM100_PREFILL_MIN_Q`` query rows per
+    ``impl``: "auto" picks the tcgen05 kernel (head dim 128, positive scale, at least ``SM100_PREFILL_MIN_Q`` query rows per
     sequence) and otherwise the ``mma.sync`` kernel; "sm100" / "mma" force one.  ``max_kv_len`` (an upper bound of
-    ``kv_lens``) saves the tcgen05 path a device-to-host read."""
+    ``kv_lens``) saves the tcgen05 path a device-to-host read.  ``softcap``: scores become ``softcap * tanh(score / softcap)``.
+    ``sink`` fp32 [Hq]: exp(sink) joins every denominator (the LSE that is returned is that of the keys alone)."""
     D = q.shape[-1]
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
-    if _native.use_native(q, k_cache, v_cache) and q.dtype == torch.bfloat16 and D in (64, 128):
+    if _native.use_native(q, k_cache, v_cache) and q.dtype == torch.bfloat16 and D in TENSOR_CORE_DIMS:
         lib = _native.load(True)
         lse = torch.empty((q.shape[1], q.shape[0]), dtype=torch.float32, device=q.device) if return_lse else None
-        sm100_ok = D == 128 and softcap == 0.0 and k_cache.dtype == torch.bfloat16 and os.environ.get("TDB200_ATTN_SM100", "1") != "0"
+        sm100_ok = D == 128 and scale > 0 and k_cache.dtype == torch.bfloat16 and os.environ.get("TDB200_ATTN_SM100", "1") != "0"
         if impl == "sm100" and not sm100_ok:
-            raise ValueError("flash_attn_varlen: the tcgen05 kernel needs head dim 128, bf16 caches and no soft cap")
+            raise ValueError("flash_attn_varlen: the tcgen05 kernel needs head dim 128, bf16 caches and a positive scale")
         if impl == "sm100" or (impl == "auto" and sm100_ok and max_q_len >= SM100_PREFILL_MIN_Q):
             if max_kv_len is None:
                 max_kv_len = int(kv_lens.max().item())
             out, err = lib.flash_fwd_sm100(q.contiguous(), k_cache.contiguous(), v_cache.contiguous(), block_table.contiguous(),
                                            cu_seqlens_q, kv_lens, q_pos0, int(max_q_len), max(int(max_kv_len), 1),
-                                           bool(causal), float(scale), lse)
+                                           bool(causal), float(scale), lse, None, sink, None, float(softcap))
             _PENDING_ERRORS.append(err)
             if len(_PENDING_ERRORS) > 64:
                 check_attention_errors()
             return (out, lse) if return_lse else out
         out = lib.flash_fwd(q.contiguous(), k_cache, v_cache, block_table, cu_seqlens_q, kv_lens, q_pos0, int(max_q_len),
-                            bool(causal), float(scale), float(softcap), lse)
+                            bool(causal), float(scale), float(softcap), lse, None, sink)
         return (out, lse) if return_lse else out
     return attention_reference(q, k_cache, v_cache, block_table, cu_seqlens_q, kv_lens, q_pos0, causal, scale, softcap,
-                               return_lse)
+                               return_lse, sink)
 
 
 def pick_kv_splits(batch: int, num_kv_heads: int, head_dim_chunks: int, max_kv_len: int, num_sms: int = 148) -> int:
@@ -154,11 +157,14 @@ def _decode_counters(device, n: int) -> torch.Tensor:
 def gqa_fwd_batch_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                          workspace: Optional[torch.Tensor], q_lens, kv_lens: torch.Tensor, block_table: torch.Tensor,
                          scale: Optional[float] = None, soft_cap: float = 0.0, output_split=None, output_combine=None,
-                         kv_split: int = -1, return_lse: bool = False):
-    """Decode attention, one query token per sequence.  ``q`` [B, Hq, D] -> [B, Hq, D] (and the LSE [B, Hq])."""
+                         kv_split: int = -1, return_lse: bool = False, sink: Optional[torch.Tensor] = None):
+    """Decode attention, one query token per sequence.  ``q`` [B, Hq, D] -> [B, Hq, D] (and the LSE [B, Hq]).
+    ``sink`` fp32 [Hq]: exp(sink) joins every denominator (not together with ``return_lse``)."""
+    if sink is not None and return_lse:
+        raise ValueError("gqa_fwd_batch_decode: the sink belongs to the merge, which does not return the LSE")
     B, Hq, D = q.shape
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
-    if _native.use_native(q, k_cache, v_cache) and q.dtype == torch.bfloat16 and D in (64, 128):
+    if _native.use_native(q, k_cache, v_cache) and q.dtype == torch.bfloat16 and D in TENSOR_CORE_DIMS:
         lib = _native.load(True)
         Hkv = k_cache.shape[2]
         group = Hq // Hkv
@@ -170,13 +176,13 @@ def gqa_fwd_batch_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
         out = output_combine if output_combine is not None else torch.empty_like(q)
         lse = torch.empty((B, Hq), dtype=torch.float32, device=q.device) if return_lse else None
         # without the LSE the last split CTA of every (sequence, KV head) merges the partials: one launch
-        counters = None if (return_lse or splits > FUSED_COMBINE_MAX_SPLITS) else \
+        counters = None if (return_lse or (splits > FUSED_COMBINE_MAX_SPLITS and sink is None)) else \
             _decode_counters(q.device, B * Hkv * ((group + 15) // 16))
         lib.decode_attn(q.contiguous(), k_cache, v_cache, block_table, kv_lens, workspace, int(splits), float(scale),
-                        float(soft_cap), out, lse, None, counters)
+                        float(soft_cap), out, lse, None, counters, None, sink)
         return (out, lse) if return_lse else out
     cu = torch.arange(B + 1, dtype=torch.int32, device=q.device)
-    res = attention_reference(q, k_cache, v_cache, block_table, cu, kv_lens, None, False, scale, soft_cap, return_lse)
+    res = attention_reference(q, k_cache, v_cache, block_table, cu, kv_lens, None, False, scale, soft_cap, return_lse, sink)
     return res
 
 
@@ -198,20 +204,24 @@ def merge_attention_partials(outs: torch.Tensor, lses: torch.Tensor) -> torch.Te
 TIED_TENSOR_CORE_DIMS = (32, 64, 128, 256)      # head dims of the mma.sync / tcgen05 kernels in tied form
 
 
-def _tied_attention_restatement(q, k, k_scale, row0, n_keys, sink, gate, scale=1.0, dv=0):
+def _tied_attention_restatement(q, k, k_scale, row0, n_keys, sink, gate, scale=1.0, dv=0, v=None, softcap=0.0):
     T, Hq, D = q.shape
     Hkv = k.shape[-2]
     kf = k.reshape(-1, Hkv, D)
     sf = torch.full((kf.shape[0],), float(scale)) if k_scale is None else k_scale.reshape(-1) * scale
     dv = dv or D
+    vf = kf[..., :dv] if v is None else v.reshape(-1, Hkv, dv)
     out = torch.empty(T, Hq, dv)
     for t in range(T):
         lo, hi = int(row0[t]), int(row0[t]) + int(n_keys[t])
         kk = kf[lo:hi].float().repeat_interleave(Hq // Hkv, dim=1)
         s = torch.einsum("hd,nhd->hn", q[t].float(), kk) * sf[lo:hi]
+        if softcap > 0:
+            s = softcap * torch.tanh(s / softcap)
         if sink is not None:
             s = torch.cat([s, sink.float().unsqueeze(1)], dim=1)
-        out[t] = torch.einsum("hn,nhd->hd", torch.softmax(s, dim=-1)[:, :hi - lo], kk[..., :dv])
+        out[t] = torch.einsum("hn,nhd->hd", torch.softmax(s, dim=-1)[:, :hi - lo],
+                              vf[lo:hi].float().repeat_interleave(Hq // Hkv, dim=1))
     if gate is not None:
         out *= torch.sigmoid(gate.float()).reshape(T, Hq, D)
     return out.to(q.dtype)
@@ -225,6 +235,14 @@ def tied_attention_simple(q, k, k_scale, row0, n_keys, sink=None, gate=None, sca
         return _native.load(True).tied_attn_simple(q, k, k_scale, row0, n_keys, sink, gate, float(scale), int(dv), bool(out_f32))
     o = _tied_attention_restatement(q, k, k_scale, row0, n_keys, sink, gate, scale, dv)
     return o.float() if out_f32 else o
+
+
+def attention_simple(q, k, v, row0, n_keys, sink=None, scale: float = 1.0, softcap: float = 0.0):
+    """fp32-arithmetic attention for any head dim up to 1024 and bf16 or fp32 tensors: token t sees rows ``row0[t] .. + n_keys[t]`` of
+    ``k`` and ``v`` (viewed as [rows, Hkv, D]): fp32 models, head dims beyond the tensor-core kernels, and the check of those."""
+    if _native.use_native(q, k, v):
+        return _native.load(True).tied_attn_simple(q, k, None, row0, n_keys, sink, None, float(scale), int(v.shape[-1]), False, v, float(softcap))
+    return _tied_attention_restatement(q, k, None, row0, n_keys, sink, None, scale, v.shape[-1], v, softcap)
 
 
 def tied_attn_varlen(q: torch.Tensor, k: torch.Tensor, k_scale: torch.Tensor, block_table: torch.Tensor,

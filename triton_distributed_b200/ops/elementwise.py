@@ -80,6 +80,22 @@ def silu_mul(x: torch.Tensor) -> torch.Tensor:
     return silu_mul_reference(x)
 
 
+GATED_ACTS = {"silu": 0, "gelu": 1}      # gelu: the tanh form
+
+
+def gated_act_reference(x: torch.Tensor, act: str) -> torch.Tensor:
+    g, u = x.float().chunk(2, dim=-1)
+    a = torch.nn.functional.silu(g) if act == "silu" else torch.nn.functional.gelu(g, approximate="tanh")
+    return (a * u).to(x.dtype)
+
+
+def gated_act(x: torch.Tensor, act: str = "silu") -> torch.Tensor:
+    """``act(x[:, :F]) * x[:, F:]`` for the output [rows, 2 F] of a fused gate / up projection, bf16 or fp32."""
+    if _native.use_native(x):
+        return _native.load(True).gated_act(x, GATED_ACTS[act])
+    return gated_act_reference(x, act)
+
+
 def residual_add(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
     if _native.use_native(a, b) and a.dtype == torch.bfloat16 and a.numel() % 8 == 0 and a.is_contiguous() and b.is_contiguous():
         return _native.load(True).add(a, b)

@@ -1,6 +1,6 @@
 """Decode GEMV with its layer neighbours fused in (``gemv_fused``): for up to sixteen tokens
 
-    out = [residual +] [all_reduce(] f(x) @ w^T [)],   f = identity | RMSNorm(x) * norm_weight | SiLU(gate) * up
+    out = [residual +] [all_reduce(] f(x) @ w^T [)],   f = identity | RMSNorm(x) * norm_weight | act(gate) * up
 
 in one launch of ``csrc/gemv.cu``.  With these a decoder layer at decode time is four launches plus attention, where
 the reference's layer runs rmsnorm, linear, all-reduce, add and activation kernels one after the other
@@ -18,6 +18,7 @@ import torch
 from .. import _native
 from ..runtime import Runtime, get_runtime
 from .common import new_ctx_dev, sm_count
+from .elementwise import GATED_ACTS, gated_act_reference
 
 GEMV_MAX_M = 16    # what the kernel accepts
 GEMV_FAST_M = 8    # up to here it beats the tcgen05 weight-streaming kernel (two MMA tiles of tokens are mma.sync-bound)
@@ -66,12 +67,11 @@ def create_gemv_ar_context(N: int, rt: Optional[Runtime] = None, use_multimem: b
 
 def gemv_reference(x: torch.Tensor, w: torch.Tensor, norm_weight: Optional[torch.Tensor] = None, eps: float = 1e-6,
                    silu_mul: bool = False, residual: Optional[torch.Tensor] = None, group=None,
-                   all_reduce: bool = False) -> torch.Tensor:
+                   all_reduce: bool = False, act: str = "silu") -> torch.Tensor:
     """fp32 reference of the fused op (all-reduce through torch.distributed when asked for)."""
     xf = x.float()
     if silu_mul:
-        k = w.shape[1]
-        xf = torch.nn.functional.silu(xf[..., :k]) * xf[..., k:]
+        xf = gated_act_reference(xf, act)
     elif norm_weight is not None:
         xf = xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * norm_weight.float()
     y = xf @ w.float().t()
@@ -93,30 +93,32 @@ def gemv_supported(M: int, K: int) -> bool:
 
 def gemv_fused(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None,
                norm_weight: Optional[torch.Tensor] = None, eps: float = 1e-6, silu_mul: bool = False,
-               residual: Optional[torch.Tensor] = None, ar_ctx: Optional[GemvARContext] = None) -> torch.Tensor:
+               residual: Optional[torch.Tensor] = None, ar_ctx: Optional[GemvARContext] = None, act: str = "silu") -> torch.Tensor:
     """``x`` [M<=16, K] (or [M, 2K] with ``silu_mul``), ``w`` [N, K] -> [M, N].  ``residual`` may be ``out`` itself.
+    ``act``: what ``silu_mul`` applies to the gate columns ("silu", "gelu").
     With ``ar_ctx`` of a multi-rank runtime the per-rank results are summed over the ranks before the residual."""
     M = x.shape[0]
     N, K = w.shape
     do_ar = ar_ctx is not None and ar_ctx.world_size > 1
     if not (_native.use_native(x, w) and x.dtype == torch.bfloat16 and gemv_supported(M, K)):
         res = gemv_reference(x, w, norm_weight, eps, silu_mul, residual,
-                             group=ar_ctx.rt.group if do_ar else None, all_reduce=do_ar)
+                             group=ar_ctx.rt.group if do_ar else None, all_reduce=do_ar, act=act)
         if out is not None:
             out.copy_(res)
             return out
         return res
     lib = _native.load(True)
+    gated = 1 + GATED_ACTS[act] if silu_mul else 0
     if out is None:
         out = torch.empty((M, N), dtype=x.dtype, device=x.device)
     if do_ar:
         if N != ar_ctx.N:
             raise ValueError(f"gemv_fused: N={N} differs from the context's N={ar_ctx.N}")
         rt = ar_ctx.rt
-        lib.gemv_ar_bf16(rt.heap, x, w, out, norm_weight, float(eps), bool(silu_mul), residual, ar_ctx.partial,
+        lib.gemv_ar_bf16(rt.heap, x, w, out, norm_weight, float(eps), gated, residual, ar_ctx.partial,
                          ar_ctx.flags, ar_ctx.ctx_dev, ar_ctx.m_cap, ar_ctx.max_ctas, 0,
                          bool(ar_ctx.use_multimem and rt.has_multicast), rt.config.wait_timeout_s)
         ar_ctx.calls += 1
     else:
-        lib.gemv_bf16(x, w, out, norm_weight, float(eps), bool(silu_mul), residual, 0)
+        lib.gemv_bf16(x, w, out, norm_weight, float(eps), gated, residual, 0)
     return out

@@ -20,22 +20,7 @@ import torch
 from .. import _native
 from .attention import tied_attention_simple
 
-_TABLES = {}
 _FLAGS = {}         # one error flag per device, set by a tcgen05 launch whose waits gave up
-
-
-def rope_table(base: float, dims: int, width: int, positions: int, device) -> torch.Tensor:
-    """fp32 [positions, width]: cos and sin of ``p * base^(-2 i / dims)`` for the pair (2 i, 2 i + 1), computed in fp64; columns
-    from ``dims`` on (padding) are zero.  One table per (base, dims) and device, grown when more positions are needed."""
-    key = (float(base), int(dims), int(width), str(device))
-    t = _TABLES.get(key)
-    if t is None or t.shape[0] < positions:
-        f = float(base) ** (-torch.arange(0, dims, 2, dtype=torch.float64) / dims)
-        a = torch.arange(positions, dtype=torch.float64)[:, None] * f
-        t = torch.zeros(positions, width, dtype=torch.float32)
-        t[:, :dims] = torch.stack([a.cos(), a.sin()], dim=-1).reshape(positions, dims).float()
-        t = _TABLES[key] = t.to(device)
-    return t
 
 
 def _rotate(x: torch.Tensor, cs: torch.Tensor) -> torch.Tensor:

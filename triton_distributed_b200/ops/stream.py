@@ -108,6 +108,55 @@ def _parallel(x, mix, ff, w1, w2, n_real, eps, dtype, sum_only):
     return [(r * w).to(dtype) for w in (w1, w2) if w is not None]
 
 
+# ------------------------------------------------------------------ several streams
+@dataclass
+class HyperWeights:
+    """What joins a sublayer to S streams, fp32: its input is ``sum_s inp[s] x_s``; then ``x_t <- sum_s mix[s, t] x_s + out[t] y``."""
+    inp: torch.Tensor
+    out: torch.Tensor
+    mix: torch.Tensor
+
+
+@dataclass
+class SublayerOutput:
+    """``y``, or with a second branch ``(RMSNorm(y) * y_w + RMSNorm(y2) * y2_w) / 2`` (weights fp32)."""
+    y: torch.Tensor
+    y2: Optional[torch.Tensor] = None
+    y_w: Optional[torch.Tensor] = None
+    y2_w: Optional[torch.Tensor] = None
+
+
+def hyper_step(x: torch.Tensor, last: Optional[Tuple[HyperWeights, SublayerOutput]], nxt: Optional[Tuple[torch.Tensor, torch.Tensor]],
+               n_real: int, eps: float, dtype: torch.dtype, rows: Optional[torch.Tensor] = None,
+               start: Optional[Tuple[torch.Tensor, torch.Tensor]] = None) -> Optional[torch.Tensor]:
+    """One pass over the streams ``x`` [T, S, W] (fp32, in place) between two sublayers: adds the output of the ``last`` one and
+    returns the normed input ``RMSNorm(sum_s inp[s] x_s) * w`` of the next, ``nxt = (inp, w)``, in ``dtype``.  ``start = (ids, table)``
+    sets all streams to the tokens' rows first.  With ``rows`` (int64) only these tokens are computed and ``x`` stays as it is."""
+    if _native.use_native(x):
+        ids, table = start if start is not None else (None, None)
+        hw, o = last if last is not None else (None, None)
+        h = _native.load(True).hyper_step(x, ids, table, *((o.y, o.y2, o.y_w, o.y2_w, hw.mix, hw.out) if o is not None else (None,) * 6),
+                                          *(nxt if nxt is not None else (None, None)), rows, int(n_real), float(eps), dtype == torch.float32)
+        return h if nxt is not None else None
+    if start is not None:
+        x.copy_(start[1][start[0].long()].float().unsqueeze(1).expand_as(x))
+    v = x if rows is None else x[rows]
+    if last is not None:
+        hw, o = last
+        y, y2 = (t if t is None or rows is None else t[rows] for t in (o.y, o.y2))
+        y = y.float()
+        if y2 is not None:
+            y2 = y2.float()
+            y = 0.5 * (y * _rms_factor(y, n_real, eps) * o.y_w + y2 * _rms_factor(y2, n_real, eps) * o.y2_w)
+        v = torch.einsum("st,nsw->ntw", hw.mix, v) + hw.out[:, None] * y.unsqueeze(1)
+        if rows is None:
+            x.copy_(v)
+    if nxt is None:
+        return None
+    u = torch.einsum("s,nsw->nw", nxt[0], v)
+    return (u * _rms_factor(u, n_real, eps) * nxt[1]).to(dtype)
+
+
 def combine_rows(y: torch.Tensor, T: int, rows_per_token: int, shared: Optional[torch.Tensor] = None,
                  shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The sum of :func:`postnorm_add` alone, [T, W] in the dtype of ``y`` (what tensor-parallel ranks exchange)."""

@@ -8,7 +8,10 @@ from .tp_block_attn import TP_BlockAttn  # noqa: F401
 from .tp_gla import TP_GLA  # noqa: F401
 from .tp_sigmoid_moe import TP_SigmoidMoE  # noqa: F401
 from .tp_latent_attn import TP_LatentAttn  # noqa: F401
-from .tp_routed_ff import TP_DenseFF, TP_RoutedMoE  # noqa: F401
+from .tp_routed_ff import TP_DenseFF, TP_GatedFF, TP_RoutedMoE  # noqa: F401
+from .tp_rotary_attn import TP_RotaryAttn  # noqa: F401
+from .tp_delta import TP_DeltaRule  # noqa: F401
+from .tp_twin import TP_TwinMixer  # noqa: F401
 from .ep_layer import EPAll2AllLayer, EP_MoE  # noqa: F401
 from .sp_flash_decode import SpGQAFlashDecodeAttention  # noqa: F401
 from .sp_attention import (SPAllGatherAttentionContextIntraNode, create_sp_ag_attention_context_intra_node,  # noqa: F401

@@ -1,8 +1,8 @@
-"""Tensor-parallel feed-forwards of parallel layers: dense squared-ReLU with biases, and a mixture of gated (SiLU) experts with a
+"""Tensor-parallel feed-forwards of layered decoders: dense gated; and of parallel layers: dense squared-ReLU with biases, and a mixture of gated (SiLU) experts with a
 softmax router, a choice correction, expert groups, identity experts and a shared expert.  Intermediate dimensions are split over
 the ranks, the router is replicated.
 
-Both return their contribution in pieces (``ops.FeedForward``): the layer's one addition to the stream sums them together with
+The latter two return their contribution in pieces (``ops.FeedForward``): the layer's one addition to the stream sums them together with
 the mixer's.  What is not split (biases, identity experts) is added by rank 0 alone.
 """
 from __future__ import annotations
@@ -30,6 +30,29 @@ class TP_DenseFF(TPLayer):
     def __call__(self, x: torch.Tensor) -> ops.FeedForward:
         y = self.linear(ops.relu2(self.linear(x, self.up), None, self.up_b), self.down)
         return ops.FeedForward(y, bias=self.down_b)
+
+
+class TP_GatedFF(TPLayer):
+    """``W_down (act(W_gate x) * W_up x)`` with ``act`` one of ``ops.GATED_ACTS``; ``spec.ff`` is the intermediate size.  Decode steps of
+    a few tokens apply the activation inside the down projection's launch."""
+
+    def __init__(self, spec, act: str, rank: int = 0, world_size: int = 1, group=None):
+        super().__init__(rank, world_size, group)
+        self.spec, self.act = spec, act
+
+    def load(self, get, prefix: str, width: int, dtype, device):
+        w8 = pad8(width)
+        gate, up = (shard(get(prefix + n), self.rank, self.world_size) for n in ("gate", "up"))
+        ff = pad8(up.shape[0])
+        self.gate_up = torch.cat([pad_rows(gate, ff, w8), pad_rows(up, ff, w8)]).to(dtype).to(device).contiguous()
+        self.down = pad_rows(shard(get(prefix + "down"), self.rank, self.world_size, 1), w8, ff).to(dtype).to(device).contiguous()
+
+    def __call__(self, x: torch.Tensor) -> ops.SublayerOutput:
+        h = self.linear(x, self.gate_up)
+        few = x.shape[0] <= ops.GEMV_FAST_M and ops.gemv_supported(x.shape[0], self.down.shape[1])
+        if few and self.mode != "torch" and self.world_size == 1 and x.is_cuda and x.dtype == torch.bfloat16:
+            return ops.SublayerOutput(ops.gemv_fused(h, self.down, silu_mul=True, act=self.act))
+        return ops.SublayerOutput(self.out_linear(ops.gated_act(h, self.act), self.down))
 
 
 class TP_RoutedMoE(TPLayer):
