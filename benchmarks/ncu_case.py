@@ -8,6 +8,8 @@
   python benchmarks/ncu_case.py moe       # grouped GEMM with in-kernel row gather: 8192 tokens, top-2 of 16 experts, 2048 x 2048
   python benchmarks/ncu_case.py gdn       # chunk-parallel gated delta rule, 8192 tokens x 16 heads
   python benchmarks/ncu_case.py gla       # chunk-parallel gated linear attention, 8192 tokens x 16 heads, 128 x 128 states
+  python benchmarks/ncu_case.py delta     # chunk-parallel gated delta rule with convolutions, 8192 tokens x 16 heads, 128 x 128 states
+  python benchmarks/ncu_case.py hyper     # pass over 4 residual streams between two sublayers, 8192 tokens, width 2048
   python benchmarks/ncu_case.py tied      # tied-KV block decode attention, 64 seqs x 4096 positions, 32 q heads / 4 kv heads
   python benchmarks/ncu_case.py latent_decode   # latent decode attention, 64 seqs x 4096 tokens, 32 heads, rows of 512 + 64
   python benchmarks/ncu_case.py latent_prefill  # latent prompt attention, 8192 tokens, 8 heads of 128 + 64 / 128
@@ -76,6 +78,25 @@ def main():
         tabs = ops.gla_chunk_tables([0, T], "cuda")
         for _ in range(2):
             ops.gated_linear_attention(qkvg, low, a2, bias, 16.0, norm, state, slot, pos0, cu, dv, dk ** -0.5, 1e-5, tabs)
+    elif case == "delta":
+        T, H, dk, dv, taps = 8192, 16, 128, 128, 4
+        C = H * (2 * dk + dv)
+        z, ab = torch.randn(T, C + H * dv, device="cuda", dtype=torch.bfloat16), torch.randn(T, 2 * H, device="cuda")
+        conv_w, norm = torch.randn(C, taps, device="cuda"), torch.ones(dv, device="cuda")
+        alog, dt = torch.zeros(H, device="cuda"), torch.full((H,), -2.0, device="cuda")
+        state, ring = torch.zeros(1, H, dk, dv, device="cuda"), torch.zeros(1, taps, C, device="cuda", dtype=torch.bfloat16)
+        slot, pos0 = torch.zeros(1, dtype=torch.int32, device="cuda"), torch.zeros(1, dtype=torch.int64, device="cuda")
+        cu = torch.tensor([0, T], dtype=torch.int32, device="cuda")
+        tabs = ops.gla_chunk_tables([0, T], "cuda")
+        for _ in range(2):
+            ops.gated_delta_rule(z, ab, conv_w, alog, dt, norm, state, ring, slot, pos0, cu, H, dv, dk ** -0.5, 1e-5, tabs)
+    elif case == "hyper":
+        T, S, W = 8192, 4, 2048
+        x, y = torch.randn(T, S, W, device="cuda"), torch.randn(T, W, device="cuda", dtype=torch.bfloat16)
+        one = torch.ones(S, device="cuda")
+        hc = ops.HyperWeights(one / S, one, torch.eye(S, device="cuda"))
+        for _ in range(3):
+            ops.hyper_step(x, (hc, ops.SublayerOutput(y)), (hc.inp, torch.ones(W, device="cuda")), W, 1e-5, torch.bfloat16)
     elif case == "tied":
         B, Hq, Hkv, D, L = 64, 32, 4, 128, 4096
         k = torch.randn(B, L, Hkv, D, device="cuda", dtype=torch.bfloat16)

@@ -28,7 +28,6 @@ TDB_DEVICE float delta_log_decay(const DeltaArgs& p, float a, int h) {
 }
 
 // ---------------------------------------------------------------------------------------------------- decode
-constexpr int kDecodeThreads = 512;
 
 // Convolution of channel c at the sequence's newest token, followed by silu.
 template <typename T>
@@ -40,8 +39,9 @@ TDB_DEVICE float conv_now(const DeltaArgs& p, const T* zrow, const T* ring, int6
   return silu_f32(acc);
 }
 
-template <typename T>
-__global__ void __launch_bounds__(kDecodeThreads, 1) delta_decode_kernel(const DeltaArgs p) {
+// U rows of the state per thread are in flight (or held in registers, when that is all of them).
+template <typename T, int THREADS, int U>
+__global__ void __launch_bounds__(THREADS) delta_decode_kernel(const DeltaArgs p) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[3][32];
   float* s_q = sm;                 // [dk]
@@ -53,12 +53,11 @@ __global__ void __launch_bounds__(kDecodeThreads, 1) delta_decode_kernel(const D
   pdl_wait();
   pdl_launch_dependents();
   const int dv4 = p.dv >> 2;
-  const int groups = kDecodeThreads / dv4;           // rows processed side by side
+  const int groups = THREADS / dv4;           // rows processed side by side
   const int c4 = threadIdx.x % dv4, rg = threadIdx.x / dv4;
   const int64_t pos = p.pos0[n], slot = p.slots[n];
   const bool fresh = pos == 0;
   float4* S = reinterpret_cast<float4*>(p.state + ((slot * p.H + h) * p.dk) * p.dv) + c4;
-  constexpr int U = 8;
   float4 s[U];
   auto fetch = [&](int r0) {
 #pragma unroll
@@ -75,14 +74,14 @@ __global__ void __launch_bounds__(kDecodeThreads, 1) delta_decode_kernel(const D
   T* ring = reinterpret_cast<T*>(p.conv) + slot * p.taps * C;
   T* keep = ring + (pos % p.taps) * C;
   float qq = 0.f, kk = 0.f, qk = 0.f;
-  for (int i = threadIdx.x; i < 2 * p.dk + p.dv; i += kDecodeThreads) {
+  for (int i = threadIdx.x; i < 2 * p.dk + p.dv; i += THREADS) {
     const bool is_v = i >= 2 * p.dk;
     const int c = is_v ? 2 * Gk + h * p.dv + i - 2 * p.dk : (i < p.dk ? g * p.dk + i : Gk + g * p.dk + i - p.dk);
     sm[i] = conv_now(p, zrow, ring, pos, C, c);
     if (is_v || h % share == 0) keep[c] = zrow[c];
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < p.dk; i += kDecodeThreads) {
+  for (int i = threadIdx.x; i < p.dk; i += THREADS) {
     const float q = s_q[i], k = s_k[i];
     qq += q * q; kk += k * k; qk += q * k;
   }
@@ -111,7 +110,7 @@ __global__ void __launch_bounds__(kDecodeThreads, 1) delta_decode_kernel(const D
   }
   __syncthreads();
   float ss = 0.f;
-  for (int c = threadIdx.x; c < p.dv; c += kDecodeThreads) {
+  for (int c = threadIdx.x; c < p.dv; c += THREADS) {
     float a = 0.f, b = 0.f;
     for (int i = 0; i < groups; ++i) {
       a += s_p[(2 * i) * p.dv + c];
@@ -141,84 +140,170 @@ __global__ void __launch_bounds__(kDecodeThreads, 1) delta_decode_kernel(const D
     }
   }
   T* out = reinterpret_cast<T*>(p.out) + static_cast<int64_t>(n) * Hv + h * p.dv;
-  for (int c = threadIdx.x; c < p.dv; c += kDecodeThreads)
+  for (int c = threadIdx.x; c < p.dv; c += THREADS)
     out[c] = from_f32<T>(s_o[c] * inv * p.norm_w[c] * silu_f32(to_f32(zrow[C + h * p.dv + c])));
 }
 
 // ---------------------------------------------------------------------------------------------------- inputs of prompts
-constexpr int kPrepTok = 16;      // tokens per CTA
+constexpr int kPrepTok = 32;      // tokens per CTA
 constexpr int kPrepThreads = 256;
 
-TDB_DEVICE void store_split(__nv_bfloat16* hi, __nv_bfloat16* lo, const float (&f)[8]) {
-  float h[8], l[8];
+// V = 4 or 8 neighbouring elements.
+TDB_DEVICE void load_n(const __nv_bfloat16* p, float (&f)[8]) { load8(p, f); }
+TDB_DEVICE void load_n(const float* p, float (&f)[8]) { load8(p, f); }
+TDB_DEVICE void load_n(const __nv_bfloat16* p, float (&f)[4]) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y);
+  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+}
+TDB_DEVICE void load_n(const float* p, float (&f)[4]) {
+  const float4 v = *reinterpret_cast<const float4*>(p);
+  f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+}
+TDB_DEVICE void store_n(__nv_bfloat16* p, const float (&f)[8]) { store8(p, f); }
+TDB_DEVICE void store_n(float* p, const float (&f)[8]) { store8(p, f); }
+TDB_DEVICE void store_n(__nv_bfloat16* p, const float (&f)[4]) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
+}
+TDB_DEVICE void store_n(float* p, const float (&f)[4]) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+
+template <int V>
+TDB_DEVICE void store_split(__nv_bfloat16* hi, __nv_bfloat16* lo, const float (&f)[V]) {
+  float l[V];
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
-    h[i] = __bfloat162float(__float2bfloat16(f[i]));
-    l[i] = f[i] - h[i];
-  }
-  store8(hi, h);
-  store8(lo, l);
+  for (int i = 0; i < V; ++i) l[i] = f[i] - __bfloat162float(__float2bfloat16(f[i]));
+  store_n(hi, f);
+  store_n(lo, l);
 }
 
-// P lanes (a power of two) share a unit, one head of q, k or v: eight channels per lane.
-template <typename T, bool SPLIT>
+// P lanes (a power of two) share a unit, one head of q, k or v: V channels per lane.  TAPS > 0: convolutions of at most TAPS taps,
+// weights and the last inputs in registers; 0: any number.
+template <typename T, bool SPLIT, int TAPS, int V>
 __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const DeltaArgs p, int P) {
   pdl_wait();
   pdl_launch_dependents();
   const int per_block = kPrepThreads / P, units = 2 * p.G + p.H;
   const int unit = blockIdx.y * per_block + threadIdx.x / P, lane = threadIdx.x % P;
   const int n = p.chunk_seq[blockIdx.x];
-  const int64_t c0 = p.chunk_t0[blockIdx.x], begin = p.cu[n], end = p.cu[n + 1];
+  const int64_t c0 = p.chunk_t0[blockIdx.x], begin = p.cu[n], end = p.cu[n + 1], before = p.pos0[n] - begin;
   const int64_t t0 = c0 + blockIdx.z * kPrepTok, t1 = min(min(t0 + kPrepTok, c0 + 64), end);
+  if (t0 >= t1) return;
   const int Gk = p.G * p.dk, C = 2 * Gk + p.H * p.dv;
   const bool live = unit < units;
   const int kind = unit < p.G ? 0 : unit < 2 * p.G ? 1 : 2;
   const int dim = kind == 2 ? p.dv : p.dk;
   const int head = unit - kind * p.G;
-  const int d = lane * 8, c = (kind == 2 ? 2 * Gk + head * p.dv : kind * Gk + head * p.dk) + d;
+  const int d = lane * V, c = (kind == 2 ? 2 * Gk + head * p.dv : kind * Gk + head * p.dk) + d;
   const bool ok = live && d < dim;
   const T* z = reinterpret_cast<const T*>(p.z);
   const T* ring = reinterpret_cast<const T*>(p.conv) + static_cast<int64_t>(p.slots[n]) * p.taps * C;
-  for (int64_t t = t0; t < t1; ++t) {
-    const int64_t pos = p.pos0[n] + t - begin;
-    float acc[8] = {};
-    if (ok) {
-      for (int j = 0; j < p.taps; ++j) {
-        if (pos - j < 0) break;
-        float f[8];
-        if (t - j >= begin) load8(z + (t - j) * p.ld + c, f);
-        else load8(ring + ((pos - j) % p.taps) * C + c, f);
-        const float* w = p.conv_w + static_cast<int64_t>(c) * p.taps + p.taps - 1 - j;
+  // input of channel group c at (packed) token t, zero before the sequence
+  auto input = [&](int64_t t, float (&f)[V]) {
+    const int64_t pos = before + t;
+    if (t >= begin) {
+      load_n(z + t * p.ld + c, f);
+    } else if (pos >= 0) {
+      load_n(ring + (pos % p.taps) * C + c, f);
+    } else {
 #pragma unroll
-        for (int i = 0; i < 8; ++i) acc[i] = fmaf(w[i * p.taps], f[i], acc[i]);
-      }
-#pragma unroll
-      for (int i = 0; i < 8; ++i) acc[i] = silu_f32(acc[i]);
+      for (int i = 0; i < V; ++i) f[i] = 0.f;
     }
+  };
+  constexpr int kWin = TAPS > 0 ? TAPS : 1;
+  constexpr int kBatch = 4;           // tokens whose inputs are requested together
+  float w[kWin][V], x[kWin + kBatch - 1][V];       // x[j]: input of token (first of the batch) + kBatch - 1 - j
+#pragma unroll
+  for (int j = 0; j < kWin + kBatch - 1; ++j)
+#pragma unroll
+    for (int i = 0; i < V; ++i) x[j][i] = 0.f;
+  if (TAPS > 0 && ok) {
+#pragma unroll
+    for (int j = 0; j < kWin; ++j) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) w[j][i] = j < p.taps ? p.conv_w[static_cast<int64_t>(c + i) * p.taps + p.taps - 1 - j] : 0.f;
+      if (j + 1 < p.taps && j + 1 < kWin) input(t0 - 1 - j, x[j]);          // shifted into place below
+    }
+  }
+  auto finish = [&](int64_t t, float (&acc)[V]) {
     float ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) ss += acc[i] * acc[i];
+    for (int i = 0; i < V; ++i) {
+      acc[i] = __fdividef(acc[i], 1.f + __expf(-acc[i]));
+      ss += ok ? acc[i] * acc[i] : 0.f;
+    }
     for (int o = P >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    if (!ok) continue;
+    if (!ok || t >= t1) return;
     if (kind == 2) {
-      if (SPLIT) store8(reinterpret_cast<__nv_bfloat16*>(p.v) + (t * p.H + head) * p.dv + d, acc);
-      else store8(reinterpret_cast<float*>(p.v) + (t * p.H + head) * p.dv + d, acc);
-      if (lane == 0) {
-        p.log_g[t * p.H + head] = delta_log_decay(p, p.ab[t * 2 * p.H + head], head);
-        p.beta[t * p.H + head] = sigmoid_f32(p.ab[t * 2 * p.H + p.H + head]);
-      }
-      continue;
+      if (SPLIT) store_n(reinterpret_cast<__nv_bfloat16*>(p.v) + (t * p.H + head) * p.dv + d, acc);
+      else store_n(reinterpret_cast<float*>(p.v) + (t * p.H + head) * p.dv + d, acc);
+      return;
     }
     const float f = rsqrtf(ss + p.unit_eps) * (kind == 0 ? p.q_scale : 1.f);
 #pragma unroll
-    for (int i = 0; i < 8; ++i) acc[i] *= f;
+    for (int i = 0; i < V; ++i) acc[i] *= f;
     const int64_t at = (t * p.G + head) * p.dk + d;
     void* dst = kind == 0 ? p.q : p.k;
     if (SPLIT)
-      store_split(reinterpret_cast<__nv_bfloat16*>(dst) + at, reinterpret_cast<__nv_bfloat16*>(kind == 0 ? p.q_lo : p.k_lo) + at, acc);
+      store_split<V>(reinterpret_cast<__nv_bfloat16*>(dst) + at, reinterpret_cast<__nv_bfloat16*>(kind == 0 ? p.q_lo : p.k_lo) + at, acc);
     else
-      store8(reinterpret_cast<float*>(dst) + at, acc);
+      store_n(reinterpret_cast<float*>(dst) + at, acc);
+  };
+  for (int64_t b = t0; b < t1; b += kBatch) {
+    if constexpr (TAPS > 0) {
+      if (ok) {
+#pragma unroll
+        for (int j = kWin - 2; j >= 0; --j)
+#pragma unroll
+          for (int i = 0; i < V; ++i) x[j + kBatch][i] = x[j][i];
+#pragma unroll
+        for (int j = 0; j < kBatch; ++j)
+          if (b + j < t1) load_n(z + (b + j) * p.ld + c, x[kBatch - 1 - j]);
+      }
+#pragma unroll
+      for (int k = 0; k < kBatch; ++k) {
+        float acc[V] = {};
+#pragma unroll
+        for (int j = 0; j < kWin; ++j)
+#pragma unroll
+          for (int i = 0; i < V; ++i) acc[i] = fmaf(w[j][i], x[kBatch - 1 - k + j][i], acc[i]);
+        finish(b + k, acc);
+      }
+    } else {
+      for (int k = 0; k < kBatch; ++k) {
+        float acc[V] = {};
+        if (ok && b + k < t1)
+          for (int j = 0; j < p.taps; ++j) {
+            float f[V];
+            input(b + k - j, f);
+            const float* wj = p.conv_w + static_cast<int64_t>(c) * p.taps + p.taps - 1 - j;
+#pragma unroll
+            for (int i = 0; i < V; ++i) acc[i] = fmaf(wj[i * p.taps], f[i], acc[i]);
+          }
+        finish(b + k, acc);
+      }
+    }
   }
+  if (blockIdx.y == 0)                 // decays and step sizes of these tokens
+    for (int64_t i = threadIdx.x; i < (t1 - t0) * p.H; i += kPrepThreads) {
+      const int64_t t = t0 + i / p.H;
+      const int h = static_cast<int>(i % p.H);
+      p.log_g[t * p.H + h] = delta_log_decay(p, p.ab[t * 2 * p.H + h], h);
+      p.beta[t * p.H + h] = sigmoid_f32(p.ab[t * 2 * p.H + p.H + h]);
+    }
+}
+template <typename T, bool SPLIT, int V>
+cudaError_t launch_prepare_v(const DeltaArgs& a, cudaStream_t s) {
+  int P = 1;
+  while (P * V < a.dk || P * V < a.dv) P *= 2;
+  const int per_block = kPrepThreads / P, units = 2 * a.G + a.H;
+  const dim3 grid(a.NC, (units + per_block - 1) / per_block, 64 / kPrepTok), block(kPrepThreads);
+  return a.taps <= 2   ? launch_pdl(delta_prepare_kernel<T, SPLIT, 2, V>, grid, block, 0, s, a, P)
+         : a.taps <= 4 ? launch_pdl(delta_prepare_kernel<T, SPLIT, 4, V>, grid, block, 0, s, a, P)
+                       : launch_pdl(delta_prepare_kernel<T, SPLIT, 0, V>, grid, block, 0, s, a, P);
+}
+template <typename T, bool SPLIT>
+cudaError_t launch_prepare(const DeltaArgs& a, cudaStream_t s) {
+  return a.dk <= 128 && a.dv <= 128 ? launch_prepare_v<T, SPLIT, 4>(a, s) : launch_prepare_v<T, SPLIT, 8>(a, s);
 }
 
 template <typename T>
@@ -340,6 +425,15 @@ cudaError_t launch_rec(const DeltaArgs& a, cudaStream_t s) {
                     static_cast<size_t>(smem), s, a);
 }
 
+template <int THREADS, int U>
+cudaError_t launch_decode(const DeltaArgs& a, cudaStream_t s) {
+  const int groups = THREADS / (a.dv / 4);
+  const size_t smem = static_cast<size_t>(2 * a.dk + 2 * a.dv + 2 * groups * a.dv) * 4;
+  const dim3 grid(a.H, a.N), block(THREADS);
+  return a.is_f32 ? launch_pdl(delta_decode_kernel<float, THREADS, U>, grid, block, smem, s, a)
+                  : launch_pdl(delta_decode_kernel<__nv_bfloat16, THREADS, U>, grid, block, smem, s, a);
+}
+
 bool args_ok(const DeltaArgs& a) {
   return a.N >= 0 && a.G >= 1 && a.H >= 1 && a.H % a.G == 0 && a.dk >= 8 && a.dk % 8 == 0 && a.dk <= 256 && a.dv >= 8 && a.dv % 8 == 0 &&
          a.dv <= 256 && a.dv_real >= 1 && a.taps >= 1 && a.ld % 8 == 0 && a.H <= 65535 && a.N <= 65535;
@@ -350,23 +444,15 @@ bool args_ok(const DeltaArgs& a) {
 cudaError_t launch_delta_decode(const DeltaArgs& a, cudaStream_t s) {
   if (!args_ok(a)) return cudaErrorInvalidValue;
   if (a.N == 0) return cudaSuccess;
-  const int groups = kDecodeThreads / (a.dv / 4);
-  const size_t smem = static_cast<size_t>(2 * a.dk + 2 * a.dv + 2 * groups * a.dv) * 4;
-  const dim3 grid(a.H, a.N), block(kDecodeThreads);
-  return a.is_f32 ? launch_pdl(delta_decode_kernel<float>, grid, block, smem, s, a)
-                  : launch_pdl(delta_decode_kernel<__nv_bfloat16>, grid, block, smem, s, a);
+  // the small form holds states of up to 8192 elements in registers, the large one of up to 16384
+  return a.dk * a.dv <= 8192 ? launch_decode<256, 8>(a, s) : launch_decode<512, 8>(a, s);
 }
 
 cudaError_t launch_delta_prepare(const DeltaArgs& a, bool split, cudaStream_t s) {
   if (!args_ok(a) || a.cu == nullptr || (split && a.is_f32)) return cudaErrorInvalidValue;
   if (a.NC == 0) return cudaSuccess;
-  int P = 1;
-  while (P * 8 < a.dk || P * 8 < a.dv) P *= 2;
-  const int per_block = kPrepThreads / P, units = 2 * a.G + a.H;
-  const dim3 grid(a.NC, (units + per_block - 1) / per_block, 64 / kPrepTok), block(kPrepThreads);
-  if (a.is_f32) return launch_pdl(delta_prepare_kernel<float, false>, grid, block, 0, s, a, P);
-  return split ? launch_pdl(delta_prepare_kernel<__nv_bfloat16, true>, grid, block, 0, s, a, P)
-               : launch_pdl(delta_prepare_kernel<__nv_bfloat16, false>, grid, block, 0, s, a, P);
+  if (a.is_f32) return launch_prepare<float, false>(a, s);
+  return split ? launch_prepare<__nv_bfloat16, true>(a, s) : launch_prepare<__nv_bfloat16, false>(a, s);
 }
 
 cudaError_t launch_delta_keep(const DeltaArgs& a, cudaStream_t s) {

@@ -38,17 +38,24 @@ constexpr int kFp = kC + 4;       // pitch of fp32 [64][64] matrices
 constexpr int kSp = kC + 8;       // pitch of bf16 [64][64] slabs
 
 // ---------------------------------------------------------------------------------------------------- chunk-local matrices
+// Lower 16 x 16 block (bi, bj) of a 64 x 64 matrix.
+TDB_DEVICE constexpr int lower_block(int bi, int bj) { return bi * (bi + 1) / 2 + bj; }
+constexpr int kFrags = 10 * 64;    // uint4 of a lower triangular matrix as A fragments: ten blocks, high and low parts of 32 lanes
+
 struct LocalSmem {
   int kp;                          // pitch of K / Q
   __nv_bfloat16 *kh, *kl, *qh, *ql, *sh, *sl, *vs;
-  float *A, *P, *gc, *beta;
+  uint4 *pf, *uf, *wf;             // fragments of P, of A beta and of A beta e^{gc}
+  float *A, *gc, *beta;
   __device__ LocalSmem(uint8_t* base, int dk) {
     kp = dk + 8;
     kh = reinterpret_cast<__nv_bfloat16*>(base);
     kl = kh + kC * kp;
-    A = reinterpret_cast<float*>(kl + kC * kp);
-    P = A + kC * kFp;
-    gc = P + kC * kFp;
+    pf = reinterpret_cast<uint4*>(kl + kC * kp);
+    uf = pf + kFrags;
+    wf = uf + kFrags;
+    A = reinterpret_cast<float*>(uf);                     // until its fragments take its place
+    gc = reinterpret_cast<float*>(wf + kFrags);
     beta = gc + kC;
     qh = reinterpret_cast<__nv_bfloat16*>(beta + kC);     // only until the scores are there; then the slabs
     ql = qh + kC * kp;
@@ -57,31 +64,48 @@ struct LocalSmem {
     vs = sl + kC * kSp;
   }
 };
+static_assert(kC * kFp * 4 <= 2 * kFrags * 16, "the fp32 matrix must fit where its fragments go");
 size_t local_smem(int dk) {
   const size_t q = 2 * static_cast<size_t>(kC) * (dk + 8) * 2, slabs = 3 * static_cast<size_t>(kC) * kSp * 2;
-  return 2 * static_cast<size_t>(kC) * (dk + 8) * 2 + 2 * static_cast<size_t>(kC) * kFp * 4 + 2 * kC * 4 + (q > slabs ? q : slabs);
+  return 2 * static_cast<size_t>(kC) * (dk + 8) * 2 + 3 * kFrags * 16 + 2 * kC * 4 + (q > slabs ? q : slabs);
 }
 
 // 16 x 16 block (bi, bj) of X K^T with X as (xh, xl): two tiles of eight columns.
 TDB_DEVICE void score_block(const LocalSmem& s, const __nv_bfloat16* xh, const __nv_bfloat16* xl, int dk, int bi, int bj, float (&acc)[2][4]) {
   const int lane = threadIdx.x & 31, mat = lane >> 3, mr = lane & 7;
+  float lo[2][4];
 #pragma unroll
-  for (int j = 0; j < 2; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+  for (int j = 0; j < 2; ++j) {
+    acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+    lo[j][0] = lo[j][1] = lo[j][2] = lo[j][3] = 0.f;
+  }
   const int arow = (bi * 16 + (mat & 1) * 8 + mr) * s.kp + (mat >> 1) * 8;
   const int brow = (bj * 16 + (mat >> 1) * 8 + mr) * s.kp + (mat & 1) * 8;
+#pragma unroll 2
   for (int k0 = 0; k0 < dk; k0 += 16) {
     uint32_t ah[4], al[4], bh[4], bl[4];
     ldmatrix_x4(ah, xh + arow + k0);
-    ldmatrix_x4(al, xl + arow + k0);
     ldmatrix_x4(bh, s.kh + brow + k0);
     ldmatrix_x4(bl, s.kl + brow + k0);
+    ldmatrix_x4(al, xl + arow + k0);
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       mma_bf16(acc[j], ah, bh[2 * j], bh[2 * j + 1]);
-      mma_bf16(acc[j], ah, bl[2 * j], bl[2 * j + 1]);
-      mma_bf16(acc[j], al, bh[2 * j], bh[2 * j + 1]);
+      mma_bf16(lo[j], ah, bl[2 * j], bl[2 * j + 1]);
+      mma_bf16(lo[j], al, bh[2 * j], bh[2 * j + 1]);
     }
   }
+#pragma unroll
+  for (int j = 0; j < 2; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[j][e] += lo[j][e];
+}
+
+// Two neighbouring accumulator tiles are one A fragment: high and low parts to dst[0] and dst[32].
+TDB_DEVICE void store_a_fragment(uint4* dst, const float (&a)[4], const float (&b)[4]) {
+  const HiLo r0 = split2(a[0], a[1]), r1 = split2(a[2], a[3]), r2 = split2(b[0], b[1]), r3 = split2(b[2], b[3]);
+  dst[0] = make_uint4(r0.hi, r1.hi, r2.hi, r3.hi);
+  dst[32] = make_uint4(r0.lo, r1.lo, r2.lo, r3.lo);
 }
 
 // A <- (I + A)^-1 for the strictly lower triangular A (blocks above the diagonal are scratch).
@@ -108,73 +132,107 @@ TDB_DEVICE void invert_unit_lower(float* A) {
     }
   }
   __syncthreads();
-  // blocks below the diagonal, 16 then 32: A21 = -A22 (L21 A11); the product in brackets goes to the block above the diagonal
+  // blocks below the diagonal, 16 then 32: A21 = -A22 (L21 A11); the product in brackets goes to the block above the diagonal.
+  // A thread owns four neighbouring columns of a row.
 #pragma unroll
   for (int n = 16; n <= 32; n *= 2) {
-    const int pairs = 32 / n, per = n * n;
-    for (int i = tid; i < pairs * per; i += kThreads) {
-      const int b = (i / per) * 2 * n, r = (i % per) / n, c = i % n;
-      float a = 0.f;
-      for (int m = c & ~15; m < n; ++m) a = fmaf(A[(b + n + r) * kFp + b + m], A[(b + m) * kFp + b + c], a);
-      A[(b + r) * kFp + b + n + c] = a;
+    const int per = n * n / 4, all = 32 / n * per;
+    for (int i = tid; i < all; i += kThreads) {
+      const int b = (i / per) * 2 * n, r = (i % per) / (n / 4), c = (i % (n / 4)) * 4;
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+      for (int m = c & ~15; m < n; ++m) {
+        const float l = A[(b + n + r) * kFp + b + m];
+        const float4 v = *reinterpret_cast<const float4*>(A + (b + m) * kFp + b + c);
+        a.x = fmaf(l, v.x, a.x); a.y = fmaf(l, v.y, a.y); a.z = fmaf(l, v.z, a.z); a.w = fmaf(l, v.w, a.w);
+      }
+      *reinterpret_cast<float4*>(A + (b + r) * kFp + b + n + c) = a;
     }
     __syncthreads();
-    for (int i = tid; i < pairs * per; i += kThreads) {
-      const int b = (i / per) * 2 * n, r = (i % per) / n, c = i % n;
-      float a = 0.f;
-      for (int m = 0; m < (r & ~15) + 16; ++m) a = fmaf(A[(b + n + r) * kFp + b + n + m], A[(b + m) * kFp + b + n + c], a);
-      A[(b + n + r) * kFp + b + c] = -a;
+    for (int i = tid; i < all; i += kThreads) {
+      const int b = (i / per) * 2 * n, r = (i % per) / (n / 4), c = (i % (n / 4)) * 4;
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+      for (int m = 0; m < (r & ~15) + 16; ++m) {
+        const float l = -A[(b + n + r) * kFp + b + n + m];
+        const float4 v = *reinterpret_cast<const float4*>(A + (b + m) * kFp + b + n + c);
+        a.x = fmaf(l, v.x, a.x); a.y = fmaf(l, v.y, a.y); a.z = fmaf(l, v.z, a.z); a.w = fmaf(l, v.w, a.w);
+      }
+      *reinterpret_cast<float4*>(A + (b + n + r) * kFp + b + c) = a;
     }
     __syncthreads();
   }
 }
 
-// acc += X[rows of block rb, tokens 0 .. 16 rb + 15] B[those tokens, 32 columns from col], X fp32 [64][64] lower triangular with
-// optional factors per column, B bf16 in one or two parts (row pitch bp).  Tiles from `tiles` on are left out.
+// Fragments of A beta and A beta e^{gc} take the place of A.
+TDB_DEVICE void split_inverse(const LocalSmem& s) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
+  float x[2][8], f[2][4];
+#pragma unroll
+  for (int u = 0; u < 2; ++u) {
+    const int i = warp + 8 * u;
+    if (i >= 10) break;
+    const int bi = i < 1 ? 0 : i < 3 ? 1 : i < 6 ? 2 : 3, bj = i - lower_block(bi, 0);
+    const int c = bj * 16 + 2 * t4;
+    const float* a = s.A + (bi * 16 + g) * kFp + c;
+    const float* b = a + 8 * kFp;
+    const float b0 = s.beta[c], b1 = s.beta[c + 1], b2 = s.beta[c + 8], b3 = s.beta[c + 9];
+    x[u][0] = a[0] * b0; x[u][1] = a[1] * b1; x[u][2] = b[0] * b0; x[u][3] = b[1] * b1;
+    x[u][4] = a[8] * b2; x[u][5] = a[9] * b3; x[u][6] = b[8] * b2; x[u][7] = b[9] * b3;
+    f[u][0] = __expf(s.gc[c]); f[u][1] = __expf(s.gc[c + 1]); f[u][2] = __expf(s.gc[c + 8]); f[u][3] = __expf(s.gc[c + 9]);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int u = 0; u < 2; ++u) {
+    const int i = warp + 8 * u;
+    if (i >= 10) break;
+    const float a[4] = {x[u][0], x[u][1], x[u][2], x[u][3]}, b[4] = {x[u][4], x[u][5], x[u][6], x[u][7]};
+    store_a_fragment(s.uf + i * 64 + lane, a, b);
+    const float c[4] = {a[0] * f[u][0], a[1] * f[u][1], a[2] * f[u][0], a[3] * f[u][1]};
+    const float d[4] = {b[0] * f[u][2], b[1] * f[u][3], b[2] * f[u][2], b[3] * f[u][3]};
+    store_a_fragment(s.wf + i * 64 + lane, c, d);
+  }
+  __syncthreads();
+}
+
+// Row blocks rb and 3 - rb of (lower triangular X as fragments) x (64 tokens x 16 columns from col of B, bf16 in one or two parts):
+// the two together have the same length for every rb.  Columns beyond the tensor yield numbers that nobody uses.
 template <bool SPLIT_B>
-TDB_DEVICE void lower_product(float (&acc)[4][4], const float* X, const float* f, const float* gc, int rb, const __nv_bfloat16* bh,
-                              const __nv_bfloat16* bl, int bp, int col, int tiles) {
-  const int lane = threadIdx.x & 31, mat = lane >> 3, mr = lane & 7, g = lane >> 2, t4 = lane & 3;
+TDB_DEVICE void lower_product(float (&acc)[2][2][4], const uint4* xf, int rb, const __nv_bfloat16* bh, const __nv_bfloat16* bl, int bp, int col) {
+  const int lane = threadIdx.x & 31, mat = lane >> 3, mr = lane & 7;
+  float lo[2][2][4];
 #pragma unroll
-  for (int kb = 0; kb < 4; ++kb) {
-    if (kb > rb) break;
-    const float* x0 = X + (rb * 16 + g) * kFp + kb * 16 + 2 * t4;
-    const float* x1 = x0 + 8 * kFp;
-    float s0 = 1.f, s1 = 1.f, s2 = 1.f, s3 = 1.f;
-    if (f != nullptr) {
-      const int c = kb * 16 + 2 * t4;
-      s0 = f[c]; s1 = f[c + 1]; s2 = f[c + 8]; s3 = f[c + 9];
-      if (gc != nullptr) {
-        s0 *= __expf(gc[c]); s1 *= __expf(gc[c + 1]); s2 *= __expf(gc[c + 8]); s3 *= __expf(gc[c + 9]);
-      }
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
+      lo[i][j][0] = lo[i][j][1] = lo[i][j][2] = lo[i][j][3] = 0.f;
     }
-    const HiLo w0 = split2(x0[0] * s0, x0[1] * s1), w1 = split2(x1[0] * s0, x1[1] * s1);
-    const HiLo w2 = split2(x0[8] * s2, x0[9] * s3), w3 = split2(x1[8] * s2, x1[9] * s3);
-    const uint32_t ah[4] = {w0.hi, w1.hi, w2.hi, w3.hi}, al[4] = {w0.lo, w1.lo, w2.lo, w3.lo};
+  auto row = [&](int i, int kb, const uint32_t (&b)[4], const uint32_t (&c)[4]) {
+    const uint4* x = xf + lower_block(i == 0 ? rb : 3 - rb, kb) * 64 + lane;
+    const uint4 h = x[0], l = x[32];
+    const uint32_t ah[4] = {h.x, h.y, h.z, h.w}, al[4] = {l.x, l.y, l.z, l.w};
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      mma_bf16(acc[i][j], ah, b[2 * j], b[2 * j + 1]);
+      mma_bf16(lo[i][j], al, b[2 * j], b[2 * j + 1]);
+      if constexpr (SPLIT_B) mma_bf16(lo[i][j], ah, c[2 * j], c[2 * j + 1]);
+    }
+  };
+  for (int kb = 0; kb <= 3 - rb; ++kb) {
     const int brow = (kb * 16 + (mat & 1) * 8 + mr) * bp + col + (mat >> 1) * 8;
-#pragma unroll
-    for (int j = 0; j < 4; j += 2) {
-      if (j >= tiles) break;
-      uint32_t b[4];
-      ldmatrix_x4_trans(b, bh + brow + j * 8);
-      mma_bf16(acc[j], ah, b[0], b[1]);
-      mma_bf16(acc[j + 1], ah, b[2], b[3]);
-      mma_bf16(acc[j], al, b[0], b[1]);
-      mma_bf16(acc[j + 1], al, b[2], b[3]);
-      if constexpr (SPLIT_B) {
-        ldmatrix_x4_trans(b, bl + brow + j * 8);
-        mma_bf16(acc[j], ah, b[0], b[1]);
-        mma_bf16(acc[j + 1], ah, b[2], b[3]);
-      }
-    }
+    uint32_t b[4], c[4] = {};
+    ldmatrix_x4_trans(b, bh + brow);
+    if constexpr (SPLIT_B) ldmatrix_x4_trans(c, bl + brow);
+    row(1, kb, b, c);
+    if (kb <= rb) row(0, kb, b, c);
   }
-}
-
-// Two neighbouring accumulator tiles are one A fragment: high and low parts to dst[0] and dst[32].
-TDB_DEVICE void store_a_fragment(uint4* dst, const float (&a)[4], const float (&b)[4]) {
-  const HiLo r0 = split2(a[0], a[1]), r1 = split2(a[2], a[3]), r2 = split2(b[0], b[1]), r3 = split2(b[2], b[3]);
-  dst[0] = make_uint4(r0.hi, r1.hi, r2.hi, r3.hi);
-  dst[32] = make_uint4(r0.lo, r1.lo, r2.lo, r3.lo);
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[i][j][e] += lo[i][j][e];
 }
 
 __global__ void __launch_bounds__(kThreads, 2) delta_local_kernel(const DeltaArgs p) {
@@ -219,7 +277,7 @@ __global__ void __launch_bounds__(kThreads, 2) delta_local_kernel(const DeltaArg
   for (int u = warp; u < 20; u += kThreads / 32) {
     const bool is_q = u >= 10;
     const int i = is_q ? u - 10 : u;
-    const int bi = i < 1 ? 0 : i < 3 ? 1 : i < 6 ? 2 : 3, bj = i - bi * (bi + 1) / 2;
+    const int bi = i < 1 ? 0 : i < 3 ? 1 : i < 6 ? 2 : 3, bj = i - lower_block(bi, 0);
     float acc[2][4];
     score_block(s, is_q ? s.qh : s.kh, is_q ? s.ql : s.kl, p.dk, bi, bj, acc);
 #pragma unroll
@@ -227,15 +285,16 @@ __global__ void __launch_bounds__(kThreads, 2) delta_local_kernel(const DeltaArg
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int r = bi * 16 + g + 8 * (e >> 1), c = bj * 16 + j * 8 + 2 * t4 + (e & 1);
-        const float d = r >= c ? acc[j][e] * __expf(s.gc[r] - s.gc[c]) : 0.f;
-        if (is_q) s.P[r * kFp + c] = d;
-        else s.A[r * kFp + c] = r > c ? d * s.beta[r] : 0.f;
+        acc[j][e] = r >= c ? acc[j][e] * __expf(s.gc[r] - s.gc[c]) : 0.f;
+        if (!is_q) s.A[r * kFp + c] = r > c ? acc[j][e] * s.beta[r] : 0.f;
       }
+    if (is_q) store_a_fragment(s.pf + i * 64 + lane, acc[0], acc[1]);
   }
   __syncthreads();                      // Q is no longer needed: its place takes the slabs
   load_tile(s.vs, kSp, v_g, Hv, min(64, p.dv), cp.n, kThreads);
   cp_async_commit();
   invert_unit_lower(s.A);
+  split_inverse(s);
 
   const int64_t ch = static_cast<int64_t>(chunk) * p.H + h;
   const int ksteps = p.dk >> 4, vtiles = p.dv >> 3;
@@ -243,114 +302,136 @@ __global__ void __launch_bounds__(kThreads, 2) delta_local_kernel(const DeltaArg
   uint4* read = reinterpret_cast<uint4*>(p.read) + ch * 4 * ksteps * 64 + lane;
   float4* inject = reinterpret_cast<float4*>(p.inject) + ch * ksteps * vtiles * 32 + lane;
   float4* local = reinterpret_cast<float4*>(p.local) + ch * 4 * vtiles * 32 + lane;
-  const int rb = warp >> 1, half = (warp & 1) * 32;
+  // a warp owns 16 columns of a slab of 64 for two of the four row blocks
+  const int rb = warp >> 2, col = (warp & 3) * 16, rows[2] = {rb, 3 - rb};
+  const float gl = s.gc[kC - 1];
   const int wslabs = (p.dk + 63) / 64, slabs = wslabs + (p.dv + 63) / 64;
   for (int sl = 0; sl < slabs; ++sl) {
     const bool is_w = sl < wslabs;
     const int col0 = (is_w ? sl : sl - wslabs) * 64, dim = is_w ? p.dk : p.dv;
-    const int tiles = (min(dim - col0 - half, 32)) >> 3;      // this warp's tiles of eight columns (<= 0: none)
-    float acc[4][4];
-#pragma unroll
-    for (int j = 0; j < 4; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+    const bool live = col0 + col < dim;
+    float acc[2][2][4];
     if (is_w) {
-      lower_product<true>(acc, s.A, s.beta, s.gc, rb, s.kh, s.kl, s.kp, col0 + half, tiles);
+      lower_product<true>(acc, s.wf, rb, s.kh, s.kl, s.kp, live ? col0 + col : 0);
     } else {
       cp_async_wait<0>();
       __syncthreads();
-      lower_product<false>(acc, s.A, s.beta, nullptr, rb, s.vs, nullptr, kSp, half, tiles);
+      lower_product<false>(acc, s.uf, rb, s.vs, nullptr, kSp, col);
     }
-    auto put = [&](float f0, float f1) {
+    auto put = [&](bool decayed) {
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        if (j >= tiles) break;
-        const HiLo a = split2(acc[j][0] * f0, acc[j][1] * f0), b = split2(acc[j][2] * f1, acc[j][3] * f1);
-        const int at = (rb * 16 + g) * kSp + half + j * 8 + 2 * t4;
-        *reinterpret_cast<uint32_t*>(s.sh + at) = a.hi;
-        *reinterpret_cast<uint32_t*>(s.sl + at) = a.lo;
-        *reinterpret_cast<uint32_t*>(s.sh + at + 8 * kSp) = b.hi;
-        *reinterpret_cast<uint32_t*>(s.sl + at + 8 * kSp) = b.lo;
+      for (int i = 0; i < 2; ++i) {
+        const int r = rows[i] * 16 + g;
+        const float f0 = decayed ? __expf(gl - s.gc[r]) : 1.f, f1 = decayed ? __expf(gl - s.gc[r + 8]) : 1.f;
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          const HiLo a = split2(acc[i][j][0] * f0, acc[i][j][1] * f0), b = split2(acc[i][j][2] * f1, acc[i][j][3] * f1);
+          const int at = r * kSp + col + j * 8 + 2 * t4;
+          *reinterpret_cast<uint32_t*>(s.sh + at) = a.hi;
+          *reinterpret_cast<uint32_t*>(s.sl + at) = a.lo;
+          *reinterpret_cast<uint32_t*>(s.sh + at + 8 * kSp) = b.hi;
+          *reinterpret_cast<uint32_t*>(s.sl + at + 8 * kSp) = b.lo;
+        }
       }
     };
-    put(1.f, 1.f);
+    put(false);
     __syncthreads();
     if (!is_w && sl + 1 < slabs) {      // every warp is done with this slab of v
       load_tile(s.vs, kSp, v_g + col0 + 64, Hv, min(64, p.dv - col0 - 64), cp.n, kThreads);
       cp_async_commit();
     }
-    {
-      float o[4][4];
+    if (live) {
+      float o[2][2][4];
+      lower_product<true>(o, s.pf, rb, s.sh, s.sl, kSp, col);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
-      lower_product<true>(o, s.P, nullptr, nullptr, rb, s.sh, s.sl, kSp, half, tiles);
-      if (is_w) {
-        const int r0 = rb * 16 + g, r1 = r0 + 8;
-        const float e0 = __expf(s.gc[r0]), e1 = __expf(s.gc[r1]);
+      for (int i = 0; i < 2; ++i) {
+        if (is_w) {
+          const int r0 = rows[i] * 16 + g, r1 = r0 + 8;
+          const float e0 = __expf(s.gc[r0]), e1 = __expf(s.gc[r1]);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          if (j >= tiles) break;
-          const int c = col0 + half + j * 8 + 2 * t4;
-          float2 q0 = make_float2(0.f, 0.f), q1 = q0;
-          if (r0 < cp.n) {
-            const float2 a = ld2(qh_g + r0 * Gk + c), b = ld2(ql_g + r0 * Gk + c);
-            q0 = make_float2(a.x + b.x, a.y + b.y);
+          for (int j = 0; j < 2; ++j) {
+            const int c = col0 + col + j * 8 + 2 * t4;
+            float2 q0 = make_float2(0.f, 0.f), q1 = q0;
+            if (r0 < cp.n) {
+              const float2 a = ld2(qh_g + r0 * Gk + c), b = ld2(ql_g + r0 * Gk + c);
+              q0 = make_float2(a.x + b.x, a.y + b.y);
+            }
+            if (r1 < cp.n) {
+              const float2 a = ld2(qh_g + r1 * Gk + c), b = ld2(ql_g + r1 * Gk + c);
+              q1 = make_float2(a.x + b.x, a.y + b.y);
+            }
+            o[i][j][0] = fmaf(q0.x, e0, -o[i][j][0]); o[i][j][1] = fmaf(q0.y, e0, -o[i][j][1]);
+            o[i][j][2] = fmaf(q1.x, e1, -o[i][j][2]); o[i][j][3] = fmaf(q1.y, e1, -o[i][j][3]);
           }
-          if (r1 < cp.n) {
-            const float2 a = ld2(qh_g + r1 * Gk + c), b = ld2(ql_g + r1 * Gk + c);
-            q1 = make_float2(a.x + b.x, a.y + b.y);
-          }
-          o[j][0] = fmaf(q0.x, e0, -o[j][0]); o[j][1] = fmaf(q0.y, e0, -o[j][1]);
-          o[j][2] = fmaf(q1.x, e1, -o[j][2]); o[j][3] = fmaf(q1.y, e1, -o[j][3]);
+          store_a_fragment(read + (rows[i] * ksteps + (col0 + col) / 16) * 64, o[i][0], o[i][1]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 2; ++j)
+            local[(rows[i] * vtiles + (col0 + col) / 8 + j) * 32] = make_float4(o[i][j][0], o[i][j][1], o[i][j][2], o[i][j][3]);
         }
-#pragma unroll
-        for (int j = 0; j < 4; j += 2)
-          if (j < tiles) store_a_fragment(read + (rb * ksteps + (col0 + half) / 16 + j / 2) * 64, o[j], o[j + 1]);
-      } else {
-#pragma unroll
-        for (int j = 0; j < 4; ++j)
-          if (j < tiles) local[(rb * vtiles + (col0 + half) / 8 + j) * 32] = make_float4(o[j][0], o[j][1], o[j][2], o[j][3]);
       }
     }
     __syncthreads();
-    put(__expf(s.gc[kC - 1] - s.gc[rb * 16 + g]), __expf(s.gc[kC - 1] - s.gc[rb * 16 + g + 8]));
+    put(true);
     __syncthreads();
-    for (int u = warp; u < 2 * ksteps; u += kThreads / 32) {
-      const int kb = u >> 1, hf = (u & 1) * 32, nt = (min(dim - col0 - hf, 32)) >> 3;
-      float o[4][4];
+    // K^T times the decayed slab: a warp computes 32 x 32 (two row blocks, four tiles)
+    for (int u = warp; u < ((ksteps + 1) >> 1) * 2; u += kThreads / 32) {
+      const int kb = (u >> 1) * 2, hf = (u & 1) * 32;
+      const bool two = kb + 1 < ksteps;
+      if (col0 + hf >= dim) continue;
+      float o[2][4][4];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.f;
 #pragma unroll
       for (int ks = 0; ks < 4; ++ks) {
-        uint32_t ah[4], al[4];
+        uint32_t ah[2][4], al[2][4];
         const int arow = (ks * 16 + (mat >> 1) * 8 + mr) * s.kp + kb * 16 + (mat & 1) * 8;
-        ldmatrix_x4_trans(ah, s.kh + arow);
-        ldmatrix_x4_trans(al, s.kl + arow);
+        ldmatrix_x4_trans(ah[0], s.kh + arow);
+        ldmatrix_x4_trans(al[0], s.kl + arow);
+        ldmatrix_x4_trans(ah[1], s.kh + arow + (two ? 16 : 0));
+        ldmatrix_x4_trans(al[1], s.kl + arow + (two ? 16 : 0));
         const int brow = (ks * 16 + (mat & 1) * 8 + mr) * kSp + hf + (mat >> 1) * 8;
 #pragma unroll
         for (int j = 0; j < 4; j += 2) {
-          if (j >= nt) break;
           uint32_t bh[4], bl[4];
           ldmatrix_x4_trans(bh, s.sh + brow + j * 8);
           ldmatrix_x4_trans(bl, s.sl + brow + j * 8);
-          mma_bf16(o[j], ah, bh[0], bh[1]);
-          mma_bf16(o[j + 1], ah, bh[2], bh[3]);
-          mma_bf16(o[j], ah, bl[0], bl[1]);
-          mma_bf16(o[j + 1], ah, bl[2], bl[3]);
-          mma_bf16(o[j], al, bh[0], bh[1]);
-          mma_bf16(o[j + 1], al, bh[2], bh[3]);
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            mma_bf16(o[i][j], ah[i], bh[0], bh[1]);
+            mma_bf16(o[i][j + 1], ah[i], bh[2], bh[3]);
+          }
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            mma_bf16(o[i][j], ah[i], bl[0], bl[1]);
+            mma_bf16(o[i][j + 1], ah[i], bl[2], bl[3]);
+          }
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            mma_bf16(o[i][j], al[i], bh[0], bh[1]);
+            mma_bf16(o[i][j + 1], al[i], bh[2], bh[3]);
+          }
         }
       }
-      if (is_w) {
+      const int pairs = min(dim - col0 - hf, 32) >> 4;           // of tiles
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
+      for (int i = 0; i < 2; ++i) {
+        if (i == 1 && !two) break;
+        if (is_w) {
 #pragma unroll
-          for (int e = 0; e < 4; ++e) o[j][e] = -o[j][e];
+          for (int j = 0; j < 4; ++j)
 #pragma unroll
-        for (int j = 0; j < 4; j += 2)
-          if (j < nt) store_a_fragment(trans + (kb * ksteps + (col0 + hf) / 16 + j / 2) * 64, o[j], o[j + 1]);
-      } else {
+            for (int e = 0; e < 4; ++e) o[i][j][e] = -o[i][j][e];
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-          if (j < nt) inject[(kb * vtiles + (col0 + hf) / 8 + j) * 32] = make_float4(o[j][0], o[j][1], o[j][2], o[j][3]);
+          for (int j = 0; j < 4; j += 2)
+            if (j / 2 < pairs) store_a_fragment(trans + ((kb + i) * ksteps + (col0 + hf) / 16 + j / 2) * 64, o[i][j], o[i][j + 1]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            if (j / 2 < pairs) inject[((kb + i) * vtiles + (col0 + hf) / 8 + j) * 32] = make_float4(o[i][j][0], o[i][j][1], o[i][j][2], o[i][j][3]);
+        }
       }
     }
     __syncthreads();
@@ -358,13 +439,14 @@ __global__ void __launch_bounds__(kThreads, 2) delta_local_kernel(const DeltaArg
 }
 
 // ---------------------------------------------------------------------------------------------------- sequential part
-// KS: 16-row blocks of dk (a warp each), at least dk / 16; NT: tiles of eight columns per CTA.
+// KS: 16-row blocks of dk, a warp each; NT: tiles of eight columns per CTA.
 template <int KS, int NT>
 __global__ void __launch_bounds__(32 * KS, 1) delta_state_kernel(const DeltaArgs p) {
   extern __shared__ __align__(16) uint8_t smem[];
   constexpr int kPitch = NT * 8 + 8;
   constexpr bool kAhead = KS <= 8;          // the next chunk's operands wait in registers
-  const int ksteps = p.dk >> 4, vtiles = p.dv >> 3;
+  constexpr int ksteps = KS;
+  const int vtiles = p.dv >> 3;
   const int tile0 = blockIdx.x * NT, h = blockIdx.y, n = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3, mat = lane >> 3, mr = lane & 7;
   const int tiles = min(NT, vtiles - tile0);
@@ -396,11 +478,10 @@ __global__ void __launch_bounds__(32 * KS, 1) delta_state_kernel(const DeltaArgs
     nd = p.decay[ch];
     if constexpr (kAhead) {
 #pragma unroll
-      for (int ks = 0; ks < KS; ++ks)
-        if (ks < ksteps) {
-          nh[ks] = trans[ch * tr_step + ks * 64];
-          nl[ks] = trans[ch * tr_step + ks * 64 + 32];
-        }
+      for (int ks = 0; ks < KS; ++ks) {
+        nh[ks] = trans[ch * tr_step + ks * 64];
+        nl[ks] = trans[ch * tr_step + ks * 64 + 32];
+      }
     }
 #pragma unroll
     for (int j = 0; j < NT; ++j)
@@ -421,12 +502,13 @@ __global__ void __launch_bounds__(32 * KS, 1) delta_state_kernel(const DeltaArgs
       *reinterpret_cast<uint32_t*>(lo + at + 8 * kPitch) = b.lo;
     }
     uint4 th[kAhead ? KS : 1], tl[kAhead ? KS : 1];
-    float acc[NT][4], part2[NT][4];
+    float acc[NT][4], lo1[NT][4], lo2[NT][4];
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
       acc[j][0] = fmaf(nd, S[j][0], ni[j].x); acc[j][1] = fmaf(nd, S[j][1], ni[j].y);
       acc[j][2] = fmaf(nd, S[j][2], ni[j].z); acc[j][3] = fmaf(nd, S[j][3], ni[j].w);
-      part2[j][0] = part2[j][1] = part2[j][2] = part2[j][3] = 0.f;
+      lo1[j][0] = lo1[j][1] = lo1[j][2] = lo1[j][3] = 0.f;
+      lo2[j][0] = lo2[j][1] = lo2[j][2] = lo2[j][3] = 0.f;
     }
     if constexpr (kAhead) {
 #pragma unroll
@@ -439,7 +521,6 @@ __global__ void __launch_bounds__(32 * KS, 1) delta_state_kernel(const DeltaArgs
     __syncthreads();       // the other buffer is free as well: its readers have passed this barrier
 #pragma unroll
     for (int ks = 0; ks < KS; ++ks) {
-      if (ks >= ksteps) break;
       uint4 fh, fl;
       if constexpr (kAhead) {
         fh = th[ks];
@@ -457,10 +538,10 @@ __global__ void __launch_bounds__(32 * KS, 1) delta_state_kernel(const DeltaArgs
         ldmatrix_x4_trans(bl, lo + brow + j * 8);
         mma_bf16(acc[j], ah, bh[0], bh[1]);
         mma_bf16(acc[j + 1], ah, bh[2], bh[3]);
-        mma_bf16(part2[j], ah, bl[0], bl[1]);
-        mma_bf16(part2[j + 1], ah, bl[2], bl[3]);
-        mma_bf16(part2[j], al, bh[0], bh[1]);
-        mma_bf16(part2[j + 1], al, bh[2], bh[3]);
+        mma_bf16(lo1[j], ah, bl[0], bl[1]);
+        mma_bf16(lo1[j + 1], ah, bl[2], bl[3]);
+        mma_bf16(lo2[j], al, bh[0], bh[1]);
+        mma_bf16(lo2[j + 1], al, bh[2], bh[3]);
         if (ks == warp) {          // a warp writes its own rows of the state before this chunk, as B fragments of the read-out
           if (j < tiles) states[ch * in_step + j * 32] = make_uint4(bh[0], bh[1], bl[0], bl[1]);
           if (j + 1 < tiles) states[ch * in_step + (j + 1) * 32] = make_uint4(bh[2], bh[3], bl[2], bl[3]);
@@ -470,7 +551,7 @@ __global__ void __launch_bounds__(32 * KS, 1) delta_state_kernel(const DeltaArgs
 #pragma unroll
     for (int j = 0; j < NT; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) S[j][e] = acc[j][e] + part2[j][e];
+      for (int e = 0; e < 4; ++e) S[j][e] = acc[j][e] + (lo1[j][e] + lo2[j][e]);
   }
 #pragma unroll
   for (int j = 0; j < NT; ++j) {
@@ -481,8 +562,14 @@ __global__ void __launch_bounds__(32 * KS, 1) delta_state_kernel(const DeltaArgs
 }
 
 // ---------------------------------------------------------------------------------------------------- outputs
+// Operands come in stages of kOutSteps k-steps (64 rows of the state) through shared memory, two stages in flight; all of it is
+// stored in fragment order, so a stage is a plain copy.
+constexpr int kOutSteps = 4;
+size_t out_stage(int dv) { return static_cast<size_t>(kOutSteps) * (dv / 8 * 32 + 4 * 64) * 16; }
+
 template <int TW>     // tiles of eight columns per warp: dv <= 16 TW
-__global__ void __launch_bounds__(kThreads) delta_out_kernel(const DeltaArgs p) {
+__global__ void __launch_bounds__(kThreads, TW <= 8 ? 2 : 1) delta_out_kernel(const DeltaArgs p) {
+  extern __shared__ __align__(16) uint8_t smem[];
   __shared__ float ssq[2][kC];
   const int chunk = blockIdx.x, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
@@ -492,9 +579,26 @@ __global__ void __launch_bounds__(kThreads) delta_out_kernel(const DeltaArgs p) 
   pdl_launch_dependents();
   const ChunkPos cp = chunk_pos(p, chunk);
   const int64_t ch = static_cast<int64_t>(chunk) * p.H + h;
-  const uint4* read = reinterpret_cast<const uint4*>(p.read) + (ch * 4 + rb) * ksteps * 64 + lane;
-  const uint4* states = reinterpret_cast<const uint4*>(p.states) + (ch * ksteps * vtiles + tile0) * 32 + lane;
+  const uint4* read = reinterpret_cast<const uint4*>(p.read) + ch * 4 * ksteps * 64;
+  const uint4* states = reinterpret_cast<const uint4*>(p.states) + ch * ksteps * vtiles * 32;
   const float4* local = reinterpret_cast<const float4*>(p.local) + ((ch * 4 + rb) * vtiles + tile0) * 32 + lane;
+  uint4* bufs = reinterpret_cast<uint4*>(smem);
+  const int b_size = kOutSteps * vtiles * 32, stage = b_size + kOutSteps * 4 * 64;     // uint4 of a stage: states, then rows to read with
+  const int stages = (ksteps + kOutSteps - 1) / kOutSteps;
+  auto fetch = [&](int st) {
+    if (st < stages) {
+      const int k0 = st * kOutSteps, kn = min(kOutSteps, ksteps - k0);
+      uint4* dst = bufs + (st & 1) * stage;
+      for (int i = threadIdx.x; i < kn * vtiles * 32; i += kThreads) attn::cp_async16(dst + i, states + k0 * vtiles * 32 + i, true);
+      for (int i = threadIdx.x; i < 4 * kn * 64; i += kThreads) {
+        const int r = i / (kn * 64), c = i - r * kn * 64;
+        attn::cp_async16(dst + b_size + r * kOutSteps * 64 + c, read + (r * ksteps + k0) * 64 + c, true);
+      }
+    }
+    cp_async_commit();
+  };
+  fetch(0);
+  fetch(1);
   float acc[TW][4];
 #pragma unroll
   for (int j = 0; j < TW; ++j) {
@@ -502,21 +606,36 @@ __global__ void __launch_bounds__(kThreads) delta_out_kernel(const DeltaArgs p) 
     if (j < tiles) f = local[j * 32];
     acc[j][0] = f.x; acc[j][1] = f.y; acc[j][2] = f.z; acc[j][3] = f.w;
   }
-  if (rb * 16 < cp.n) {
-#pragma unroll 2
-    for (int ks = 0; ks < ksteps; ++ks) {
-      const uint4 fh = read[ks * 64], fl = read[ks * 64 + 32];
-      const uint32_t ah[4] = {fh.x, fh.y, fh.z, fh.w}, al[4] = {fl.x, fl.y, fl.z, fl.w};
+  for (int st = 0; st < stages; ++st) {
+    cp_async_wait<1>();
+    __syncthreads();
+    const uint4* B = bufs + (st & 1) * stage + tile0 * 32 + lane;
+    const uint4* A = bufs + (st & 1) * stage + b_size + rb * kOutSteps * 64 + lane;
+    const int kn = min(kOutSteps, ksteps - st * kOutSteps);
+    if (rb * 16 < cp.n) {
+      for (int ks = 0; ks < kn; ++ks) {
+        const uint4 fh = A[ks * 64], fl = A[ks * 64 + 32];
+        const uint32_t ah[4] = {fh.x, fh.y, fh.z, fh.w}, al[4] = {fl.x, fl.y, fl.z, fl.w};
 #pragma unroll
-      for (int j = 0; j < TW; ++j) {
-        if (j >= tiles) break;
-        const uint4 b = states[(ks * vtiles + j) * 32];
-        mma_bf16(acc[j], ah, b.x, b.y);
-        mma_bf16(acc[j], ah, b.z, b.w);
-        mma_bf16(acc[j], al, b.x, b.y);
+        for (int j0 = 0; j0 < TW; j0 += 4) {
+          uint4 b[4];
+#pragma unroll
+          for (int j = 0; j < 4; ++j) b[j] = B[(ks * vtiles + min(j0 + j, tiles - 1)) * 32];       // tiles beyond the last: unused copies
+#pragma unroll
+          for (int j = 0; j < 4; ++j) mma_bf16(acc[j0 + j], ah, b[j].x, b[j].y);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) mma_bf16(acc[j0 + j], ah, b[j].z, b[j].w);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) mma_bf16(acc[j0 + j], al, b[j].x, b[j].y);
+        }
       }
     }
+    __syncthreads();
+    fetch(st + 2);
   }
+#pragma unroll
+  for (int j = 0; j < TW; ++j)
+    if (j >= tiles) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
   float q0 = 0.f, q1 = 0.f;
 #pragma unroll
   for (int j = 0; j < TW; ++j) {
@@ -561,17 +680,33 @@ cudaError_t launch_state(const DeltaArgs& a, cudaStream_t s) {
 }
 template <int NT>
 cudaError_t launch_state_nt(const DeltaArgs& a, cudaStream_t s) {
-  return a.dk <= 32 ? launch_state<2, NT>(a, s) : a.dk <= 64 ? launch_state<4, NT>(a, s) : a.dk <= 128 ? launch_state<8, NT>(a, s)
-                                                                                                   : launch_state<16, NT>(a, s);
+  switch (a.dk / 16) {
+    case 1: return launch_state<1, NT>(a, s);
+    case 2: return launch_state<2, NT>(a, s);
+    case 3: return launch_state<3, NT>(a, s);
+    case 4: return launch_state<4, NT>(a, s);
+    case 5: return launch_state<5, NT>(a, s);
+    case 6: return launch_state<6, NT>(a, s);
+    case 8: return launch_state<8, NT>(a, s);
+    case 12: return launch_state<12, NT>(a, s);
+    case 16: return launch_state<16, NT>(a, s);
+    default: return cudaErrorInvalidValue;
+  }
 }
 template <int TW>
 cudaError_t launch_out(const DeltaArgs& a, cudaStream_t s) {
-  return launch_pdl(delta_out_kernel<TW>, dim3(a.NC, a.H), dim3(kThreads), 0, s, a);
+  static SmemOptIn opt;
+  cudaError_t e = opt.ensure(delta_out_kernel<TW>, static_cast<int>(2 * out_stage(16 * TW)));
+  if (e != cudaSuccess) return e;
+  return launch_pdl(delta_out_kernel<TW>, dim3(a.NC, a.H), dim3(kThreads), 2 * out_stage(a.dv), s, a);
 }
 
 }  // namespace
 
-bool delta_chunk_supported(int dk, int dv) { return dk % 16 == 0 && dv % 16 == 0 && dk <= 256 && dv <= 256 && dk >= 16 && dv >= 16; }
+bool delta_chunk_supported(int dk, int dv) {
+  const int ks = dk / 16;        // the state kernel is compiled for these numbers of row blocks
+  return dk % 16 == 0 && dv % 16 == 0 && dv >= 16 && dv <= 256 && ((ks >= 1 && ks <= 6) || ks == 8 || ks == 12 || ks == 16);
+}
 
 cudaError_t launch_delta_chunk(const DeltaArgs& a, cudaStream_t s) {
   if (a.is_f32 || !delta_chunk_supported(a.dk, a.dv) || a.cu == nullptr || a.trans == nullptr) return cudaErrorInvalidValue;
@@ -584,8 +719,11 @@ cudaError_t launch_delta_chunk(const DeltaArgs& a, cudaStream_t s) {
   if (e != cudaSuccess) return e;
   e = launch_pdl(delta_local_kernel, dim3(a.NC, a.H), dim3(kThreads), local_smem(a.dk), s, a);
   if (e != cudaSuccess) return e;
-  // narrow column tiles only while the grid is small: every CTA of a head reads the same operands
-  e = static_cast<int64_t>(a.N) * a.H * ((a.dv + 31) / 32) < 64 ? launch_state_nt<2>(a, s) : launch_state_nt<4>(a, s);
+  // every CTA of a head reads the same operands: narrow column tiles only while they still fit one wave
+  int dev = 0, sms = 0;
+  cudaGetDevice(&dev);
+  cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+  e = static_cast<int64_t>(a.N) * a.H * ((a.dv + 15) / 16) <= sms ? launch_state_nt<2>(a, s) : launch_state_nt<4>(a, s);
   if (e != cudaSuccess) return e;
   if (a.dv <= 64) return launch_out<4>(a, s);
   if (a.dv <= 128) return launch_out<8>(a, s);

@@ -112,6 +112,34 @@ TDB_DEVICE void load_kv_block(const PagedKV& kv, int b, int h, int t0, int kv_en
   }
 }
 
+// Soft cap: scores -> cap * tanh(to_cap * score), to fp32 accuracy of the cap.  While all arguments of the warp are small the power
+// series of tanh takes the place of an exponential and a division, which the softmax's own exponentials would have to share a unit
+// with.  Executed by whole warps.
+template <int N>
+TDB_DEVICE void cap_scores(float (&s)[N], float to_cap, float cap) {
+  float big = 0.f;
+#pragma unroll
+  for (int i = 0; i < N; ++i) big = fmaxf(big, fabsf(s[i]));
+  if (__all_sync(0xffffffffu, big * to_cap < 0.2f)) {
+    // x - x^3/3 + 2 x^5/15 - 17 x^7/315: the next term is below 6e-8 of x here
+    const float c0 = cap * to_cap, t2 = to_cap * to_cap;
+    const float c1 = c0 * t2 * (-1.f / 3.f), c2 = c0 * t2 * t2 * (2.f / 15.f), c3 = c0 * t2 * t2 * t2 * (-17.f / 315.f);
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const float q = s[i] * s[i];
+      s[i] *= fmaf(q, fmaf(q, fmaf(q, c3, c2), c1), c0);
+    }
+    return;
+  }
+  const float twice = to_cap * 2.8853900817779268f, mcap = -2.f * cap;
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    // tanh x = 1 - 2 / (e^{2x} + 1); the exponent is clamped where fp32 tanh has long been 1
+    const float e = exp2f(fminf(s[i] * twice, 60.f)) + 1.f;
+    s[i] = fmaf(mcap, __fdividef(1.f, e), cap);
+  }
+}
+
 // Per-warp state of a 16-row attention tile.
 template <int D>
 struct WarpTile {
@@ -161,14 +189,23 @@ struct WarpTile {
     }
     // scale, soft-cap, mask; row maxima
     float mx[2] = {-INFINITY, -INFINITY};
+    if (softcap > 0.f) {
+      if constexpr (TIED) {
+#pragma unroll
+        for (int j = 0; j < NT; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[j][e] *= tok_scale[tok_in_block + 8 * j + c + (e & 1)];
+      }
+      cap_scores(reinterpret_cast<float (&)[NT * 4]>(s), scale / softcap, softcap);
+    }
+    const float f = softcap > 0.f ? 1.f : scale;
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int tok = t0 + tok_in_block + 8 * j + c + (e & 1);
-        float v = s[j][e] * scale;
-        if constexpr (TIED) v *= tok_scale[tok_in_block + 8 * j + c + (e & 1)];
-        if (softcap > 0.f) v = softcap * tanhf(v / softcap);
+        float v = s[j][e] * f;
+        if constexpr (TIED) v *= softcap > 0.f ? 1.f : tok_scale[tok_in_block + 8 * j + c + (e & 1)];
         v *= kLog2e;
         const int lim = (e < 2) ? limit_lo : limit_hi;
         v = (tok < lim) ? v : -INFINITY;

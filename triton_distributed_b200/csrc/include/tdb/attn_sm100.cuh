@@ -4,6 +4,7 @@
 #include <cuda_bf16.h>
 
 #include "attn.h"
+#include "attn_device.cuh"
 #include "ptx.cuh"
 
 namespace tdb {
@@ -47,40 +48,6 @@ struct TileCtx {
   int row0, rows_here, nblk;
 };
 
-// Scores -> cap_log2 * tanh(to_cap * score), exact to fp32 rounding of the cap.  The power series of tanh takes the place of the
-// exponential and the division while all 32 arguments of the warp's rows are small: those two share the unit that the softmax keeps
-// busy.  Masked scores (minus infinity) stay what they are.
-__device__ __forceinline__ void cap_scores(uint32_t (&s)[32], float to_cap, float cap_log2) {
-  float big = 0.f;
-#pragma unroll
-  for (int c = 0; c < 32; ++c) {
-    const float x = __uint_as_float(s[c]) * to_cap;
-    s[c] = __float_as_uint(x);
-    big = fmaxf(big, x == -INFINITY ? 0.f : fabsf(x));
-  }
-  if (__all_sync(0xffffffffu, big < 0.3f)) {
-    // x (1 - x^2/3 + 2 x^4/15 - 17 x^6/315 + 62 x^8/2835): the next term is below 1e-8 here
-#pragma unroll
-    for (int c = 0; c < 32; ++c) {
-      const float x = __uint_as_float(s[c]);
-      const float q = x * x;
-      float f = fmaf(q, 62.f / 2835.f, -17.f / 315.f);
-      f = fmaf(q, f, 2.f / 15.f);
-      f = fmaf(q, f, -1.f / 3.f);
-      const float y = cap_log2 * fmaf(x * q, f, x);
-      s[c] = x == -INFINITY ? 0xff800000u : __float_as_uint(y);
-    }
-    return;
-  }
-#pragma unroll
-  for (int c = 0; c < 32; ++c) {
-    const float x = __uint_as_float(s[c]);
-    // tanh x = 1 - 2 / (e^{2x} + 1); the exponent is clamped where fp32 tanh has long been 1
-    const float y = 1.f - __fdividef(2.f, ex2(fminf(x * 2.8853900817779268f, 60.f)) + 1.f);
-    s[c] = x == -INFINITY ? 0xff800000u : __float_as_uint(cap_log2 * y);
-  }
-}
-
 // DV: columns of the output accumulator (a multiple of 32); the rows written have p.dv <= DV columns, a multiple of 8.  CAP: with
 // soft cap.
 template <int DV, bool CAP = false>
@@ -117,16 +84,16 @@ __device__ __forceinline__ void softmax_tile(const FwdParams& p, const TileCtx& 
     // a sequence) skip the masking; the scale is folded into the exponent (one FMA per element), so an element
     // costs a max, an FMA, an ex2, an add and half a pack.
     const bool full = __all_sync(0xffffffffu, t0 + kBN <= lim);
+    if constexpr (CAP) {
+      attn::cap_scores(reinterpret_cast<float (&)[32]>(s0), p.to_cap, p.cap_log2);
+      attn::cap_scores(reinterpret_cast<float (&)[32]>(s1), p.to_cap, p.cap_log2);
+    }
     if (!full) {
 #pragma unroll
       for (int c = 0; c < 32; ++c) {
         if (t0 + c >= lim) s0[c] = 0xff800000u;          // -inf
         if (t0 + 32 + c >= lim) s1[c] = 0xff800000u;
       }
-    }
-    if constexpr (CAP) {
-      cap_scores(s0, p.to_cap, p.cap_log2);
-      cap_scores(s1, p.to_cap, p.cap_log2);
     }
     float mx = -INFINITY;
 #pragma unroll

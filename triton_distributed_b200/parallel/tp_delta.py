@@ -9,6 +9,11 @@ from .tp_gla import pad16
 from .tp_layer import TPLayer, pad8, pad_heads, pad_rows, shard
 
 
+def pad_key_dim(n: int) -> int:
+    """Key dim the weights are padded to: one the chunk kernels are compiled for."""
+    return next((d for d in (16, 32, 48, 64, 80, 96, 128, 192, 256) if d >= n), pad16(n))
+
+
 class TP_DeltaRule(TPLayer):
     """``spec``: heads, kv_heads (of q and k), dim, vdim, conv (taps)."""
 
@@ -18,7 +23,7 @@ class TP_DeltaRule(TPLayer):
             raise ValueError(f"{spec.kv_heads} key heads cannot be split over {world_size} ranks")
         self.spec = spec
         self.heads, self.kv_heads = spec.heads // world_size, spec.kv_heads // world_size
-        self.dk, self.dv = pad16(spec.dim), pad16(spec.vdim)
+        self.dk, self.dv = pad_key_dim(spec.dim), pad16(spec.vdim)
         if max(self.dk, self.dv) > ops.DELTA_MAX_DIM:
             raise ValueError(f"delta rule: heads of at most {ops.DELTA_MAX_DIM} elements")
         self.channels = 2 * self.kv_heads * self.dk + self.heads * self.dv
