@@ -6,7 +6,7 @@ with the source tree.  Nothing is compiled at import time: ``python -m triton_di
 (or ``build()`` below) is the only entry point that runs a compiler.
 
 ``build("decoder")`` compiles a subset into ``_C_decoder.so``: what a layered decoder needs on one GPU (no collectives, expert
-parallelism, megakernel, fp8 or gated-delta-rule kernels); ``ensure`` builds it when no library is there yet.
+parallelism, megakernel, fp8 or bare gated-delta-rule kernels); ``ensure`` builds it when no library is there yet.
 
 Stands in for the reference's CMake + setup.py build of its plugin and ``csrc`` library
 (CMakeLists.txt:183-227, python/setup.py); here there is no compiler plugin to build, only kernels.

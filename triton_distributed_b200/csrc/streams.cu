@@ -123,7 +123,9 @@ cudaError_t launch_s(const HyperArgs& a, cudaStream_t s) {
     if (e != cudaSuccess) return e;
   }
   const int vec = a.W / 8;
-  const int threads = vec >= 256 ? 256 : vec >= 128 ? 128 : 64;
+  // few tokens: as many loads in flight per token as a block allows
+  const int most = a.n <= 148 && MAXS <= 4 ? 512 : 256;
+  const int threads = vec >= most ? most : vec >= 256 ? 256 : vec >= 128 ? 128 : 64;
   return launch_pdl(hyper_step_kernel<T, MAXS>, dim3(static_cast<unsigned>(a.n)), dim3(threads), smem, s, a);
 }
 template <typename T>
