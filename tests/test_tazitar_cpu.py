@@ -147,7 +147,7 @@ def test_registry_presets_and_limits(rt):
         TP_DeltaRule(DeltaRuleSpec(2, 2, 300, 16, 4))
     with pytest.raises(ValueError, match="1024"):
         TP_RotaryAttn(RotaryAttnSpec(2, 2, 1100, 16, 1.0, 1e4, 8))
-    dims = [TP_RotaryAttn(RotaryAttnSpec(2, 2, d, v, 1.0, 1e4, 8)).head_dim for d, v in ((8, 8), (48, 80), (64, 64), (200, 16), (64, 300))]
+    dims = [TP_RotaryAttn(RotaryAttnSpec(2, 2, d, v, 1.0, 1e4, 8)).head_dim for d, v in ((8, 8), (44, 72), (64, 64), (200, 16), (64, 300))]
     assert dims == [64, 128, 64, 256, 512]
     assert [TP_DeltaRule(DeltaRuleSpec(2, 2, d, 16, 4)).dk for d in (9, 48, 100, 130, 200)] == [16, 48, 128, 192, 256]
 

@@ -316,7 +316,7 @@ class Rule:
             close(self.state[self.slots[s].item()][:, :self.dk, :self.dv], S, self.dtype, scale)
 
 
-RULES = [(4, 2, 128, 128, 4), (6, 3, 48, 80, 3), (2, 2, 64, 64, 1), (2, 1, 256, 250, 2), (3, 3, 10, 20, 7), (4, 4, 96, 160, 4), (1, 1, 100, 16, 12)]
+RULES = [(4, 2, 128, 128, 4), (6, 3, 40, 72, 3), (2, 2, 64, 64, 1), (2, 1, 256, 250, 2), (3, 3, 10, 20, 7), (4, 4, 96, 160, 4), (1, 1, 100, 16, 12)]
 
 
 @pytest.mark.parametrize("shape", RULES)
