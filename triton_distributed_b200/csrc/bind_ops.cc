@@ -339,11 +339,13 @@ void bind_moe(py::module_& m);
 void bind_ep(py::module_& m);
 void bind_mega(py::module_& m);
 void bind_hybrid(py::module_& m);
+void bind_window(py::module_& m);
 
 void bind_more(py::module_& m) {
   bind_attn(m);
   bind_moe(m);
   bind_hybrid(m);
+  bind_window(m);
 #ifndef TDB_DECODER_ONLY
   bind_ep(m);
   bind_mega(m);

@@ -51,6 +51,27 @@ struct ParallelAddArgs {
   float eps;
 };
 cudaError_t launch_parallel_add(const ParallelAddArgs& a, cudaStream_t s);
+// A sublayer between two norms: x += rmsnorm(y) * post, then h = rmsnorm(x) * pre, the input of the next one.
+struct SandwichArgs {
+  float* x;               // [T, W]
+  const int64_t* ids;     // [T] start: x = scale * table[id] instead of reading it; null = x as it is
+  const void* table;      // [vocab, W]
+  int64_t vocab;
+  float scale;
+  const void* y;          // [T, W], null = nothing is added
+  const float* post;      // [post_n]; one number for all coordinates (post_n = 1) or one each (post_n = W)
+  int post_n;
+  const float* pre;
+  int pre_n;
+  void* h;                // [n, W], null = stream only
+  const int64_t* rows;    // [n] tokens, null = all
+  int store;              // write x
+  int64_t n;
+  int W, n_real;          // W a multiple of 8, columns from n_real on are zero and do not count
+  float eps;
+  int is_f32;             // dtype of table, y, h
+};
+cudaError_t launch_sandwich(const SandwichArgs& a, cudaStream_t s);
 cudaError_t launch_stream_norm(const float* x, const int64_t* rows, const float* w, void* out, int64_t n, int W, int n_real,
                                float eps, int out_f32, cudaStream_t s);
 

@@ -187,6 +187,75 @@ __global__ void parallel_add_kernel(const ParallelAddArgs p) {
   }
 }
 
+// One block per row; a thread keeps its NCH groups of eight columns in registers through both norms.
+template <typename T, int NCH>
+__global__ void __launch_bounds__(512) sandwich_kernel(const SandwichArgs p) {
+  __shared__ float red[2][32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t i = blockIdx.x, t = p.rows != nullptr ? p.rows[i] : i;
+  float x[NCH][8], y[NCH][8];
+  float ss = 0.f;
+  int64_t id = 0;
+  if (p.ids != nullptr) {
+    id = p.ids[t];
+    if (id < 0 || id >= p.vocab) id = 0;
+  }
+#pragma unroll
+  for (int k = 0; k < NCH; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * 8;
+    if (c >= p.W) continue;
+    if (p.ids != nullptr) {
+      load8(reinterpret_cast<const T*>(p.table) + id * p.W + c, x[k]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[k][e] *= p.scale;
+    } else {
+      load8(p.x + t * p.W + c, x[k]);
+    }
+    if (p.y != nullptr) {
+      load8(reinterpret_cast<const T*>(p.y) + t * p.W + c, y[k]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += y[k][e] * y[k][e];
+    }
+  }
+  auto weight = [&](const float* w, int n, int c, float (&f)[8]) {
+    if (n > 1) {
+      load8(w + c, f);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[e] = w[0];
+    }
+  };
+  const float inv_y = p.y != nullptr ? 1.f / sqrtf(block_reduce_sum(ss, red[0]) / p.n_real + p.eps) : 0.f;
+  ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < NCH; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * 8;
+    if (c >= p.W) continue;
+    if (p.y != nullptr) {
+      float w[8];
+      weight(p.post, p.post_n, c, w);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[k][e] += y[k][e] * inv_y * w[e];
+    }
+    if (p.store) store8(p.x + t * p.W + c, x[k]);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss += x[k][e] * x[k][e];
+  }
+  if (p.h == nullptr) return;
+  const float inv_x = 1.f / sqrtf(block_reduce_sum(ss, red[1]) / p.n_real + p.eps);
+#pragma unroll
+  for (int k = 0; k < NCH; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * 8;
+    if (c >= p.W) continue;
+    float w[8];
+    weight(p.pre, p.pre_n, c, w);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[k][e] *= inv_x * w[e];
+    store8(reinterpret_cast<T*>(p.h) + i * p.W + c, x[k]);
+  }
+}
+
 int row_threads(int W) {
   const int vec = W / 8;
   return vec >= 512 ? 512 : vec >= 256 ? 256 : vec >= 128 ? 128 : 64;
@@ -249,6 +318,26 @@ cudaError_t launch_parallel_add(const ParallelAddArgs& a, cudaStream_t s) {
   return a.act_f32 ? launch_pdl(parallel_add_kernel<float, float>, grid, block, smem, s, a)
          : a.y_f32 ? launch_pdl(parallel_add_kernel<__nv_bfloat16, float>, grid, block, smem, s, a)
                    : launch_pdl(parallel_add_kernel<__nv_bfloat16, __nv_bfloat16>, grid, block, smem, s, a);
+}
+
+namespace {
+template <typename T>
+cudaError_t launch_sandwich_t(const SandwichArgs& a, cudaStream_t s) {
+  const dim3 grid(static_cast<unsigned>(a.n));
+  const int vec = a.W / 8;
+  if (vec <= 512) return launch_pdl(sandwich_kernel<T, 1>, grid, dim3((vec + 31) / 32 * 32), 0, s, a);
+  if (vec <= 1024) return launch_pdl(sandwich_kernel<T, 2>, grid, dim3(512), 0, s, a);
+  return launch_pdl(sandwich_kernel<T, 8>, grid, dim3(512), 0, s, a);
+}
+}  // namespace
+
+cudaError_t launch_sandwich(const SandwichArgs& a, cudaStream_t s) {
+  auto weight_ok = [&](const float* w, int n) { return w != nullptr && (n == 1 || n == a.W); };
+  if (a.W % 8 != 0 || a.W < 8 || a.W > 32768 || a.n_real < 1 || (a.y != nullptr && !weight_ok(a.post, a.post_n)) || (a.h != nullptr && !weight_ok(a.pre, a.pre_n)) ||
+      (a.ids != nullptr && a.table == nullptr))
+    return cudaErrorInvalidValue;
+  if (a.n == 0) return cudaSuccess;
+  return a.is_f32 ? launch_sandwich_t<float>(a, s) : launch_sandwich_t<__nv_bfloat16>(a, s);
 }
 
 cudaError_t launch_stream_norm(const float* x, const int64_t* rows, const float* w, void* out, int64_t n, int W, int n_real,

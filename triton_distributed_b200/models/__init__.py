@@ -1,22 +1,24 @@
 """Models, KV caches, weight loading and the serving engine (the reference's ``triton_dist.models``)."""
 from .config import ArchConfig, ModelConfig, PRESETS  # noqa: F401
 from .kv_cache import (DeltaSpec, GroupSpec, HybridCache, KV_Cache, KVSpec, LatentSpec, PagedKVCache, SharedSpec, StateSpec,  # noqa: F401
-                       StepPlan, TiedKVSpec)
+                       StepPlan, TiedKVSpec, WindowKVSpec)
 from .safetensors_io import SafetensorsFile, ShardedCheckpoint, save_file  # noqa: F401
 from .dense import DenseLLM, DenseLLMLayer  # noqa: F401
 from .engine import Engine  # noqa: F401
 from .qwen_moe import Qwen3MoE, Qwen3MoELayer  # noqa: F401
+from .bagasun import BAGASUN_PRESETS, BagasunConfig, BagasunLLM  # noqa: F401
 from .lisenex import LISENEX_PRESETS, LisenexConfig, LisenexLLM  # noqa: F401
 from .tazitar import TAZITAR_PRESETS, TazitarConfig, TazitarLLM  # noqa: F401
 from .vasolix import VASOLIX_PRESETS, VasolixConfig, VasolixLLM  # noqa: F401
 
 # "architecture" of a config.json -> (configuration class, model class); configurations without that key are read as
 # Hugging Face ones (DenseLLM / Qwen3MoE).
-ARCHITECTURES = {"Vasolix": (VasolixConfig, VasolixLLM), "Lisenex": (LisenexConfig, LisenexLLM), "Tazitar": (TazitarConfig, TazitarLLM)}
+ARCHITECTURES = {"Vasolix": (VasolixConfig, VasolixLLM), "Lisenex": (LisenexConfig, LisenexLLM), "Tazitar": (TazitarConfig, TazitarLLM),
+                 "Bagasun": (BagasunConfig, BagasunLLM)}
 
 
 def all_presets() -> dict:
-    return {**PRESETS, **VASOLIX_PRESETS, **LISENEX_PRESETS, **TAZITAR_PRESETS}
+    return {**PRESETS, **VASOLIX_PRESETS, **LISENEX_PRESETS, **TAZITAR_PRESETS, **BAGASUN_PRESETS}
 
 
 class AutoLLM:
@@ -41,7 +43,7 @@ def smoke_decode():
     from ..runtime import get_runtime
 
     rt = get_runtime()
-    for name in ("tiny-dense", "tiny-vasolix", "tiny-lisenex", "tiny-tazitar"):
+    for name in ("tiny-dense", "tiny-vasolix", "tiny-lisenex", "tiny-tazitar", "tiny-bagasun"):
         cfg = ModelConfig(model_name=name, max_length=64, rank=rt.rank, world_size=rt.world_size)
         eng = Engine(cfg)
         eng.backend = "triton_dist_gemm_ar"

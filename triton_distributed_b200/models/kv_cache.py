@@ -154,6 +154,19 @@ class KVSpec:
 
 
 @dataclass(frozen=True)
+class WindowKVSpec:
+    """A layer that caches a key of ``key_dim`` and a value of ``value_dim`` elements per token and KV head.  ``window`` > 0: position i sees
+    the positions j with i - j < window, so a sequence keeps ``window`` rows, position p at row ``p % window``."""
+    kv_heads: int
+    key_dim: int
+    value_dim: int
+    window: int = 0
+
+    def rows(self, max_length: int) -> int:
+        return min(self.window, max_length) if self.window > 0 else max_length
+
+
+@dataclass(frozen=True)
 class DeltaSpec:
     """A recurrent layer behind short convolutions: fp32 state [heads, dk, dv] and the convolutions' last inputs, a ring of ``taps``
     rows (position p at row ``p % taps``) of ``channels`` elements."""
@@ -188,6 +201,56 @@ class KVPlan:
     q_pos0: Optional[torch.Tensor] = None           # int32 [sequences] (prompts)
     max_q: int = 1
     max_kv: int = 0                                 # longest sequence after the step (prompts)
+
+
+class WindowPlan:
+    """What a layer with a window needs to know about a step (see ``StepPlan.window``); ``rows`` is the length of its rings.  A decode step
+    reads the rings; a prompt reads packed rows: per sequence, what the ring held of earlier steps and is still visible, then the
+    new tokens."""
+
+    def __init__(self, plan: "StepPlan", window: int, rows: int):
+        self.plan, self.window, self.rows = plan, window, rows
+        self._visible = None
+        base = plan.slots.to(torch.int64) * rows
+        if plan.decode:
+            self.row0 = base
+            self.home_rows = base + plan.positions % rows            # int64 [T] cache row of every token, -1 = not kept after the step
+            return
+        slots, starts, lens = plan.host
+        home, packed, src, dst, shift, at = [], [], [], [], [], 0
+        for slot, start, n in zip(slots, starts, lens):
+            first = max(0, start - window + 1) if window > 0 else 0  # oldest position that the step still sees
+            p = torch.arange(start, start + n)
+            home.append(torch.where(p >= start + n - rows, p % rows + slot * rows, -1))
+            packed.append(p - first + at)
+            if start > first:
+                old = torch.arange(first, start)
+                src.append(old % rows + slot * rows)
+                dst.append(old - first + at)
+            shift.append(at - first)
+            at += start + n - first
+        dev, T, N = plan.slots.device, plan.num_tokens, len(lens)
+        nc = sum(int(t.numel()) for t in src)
+        big = torch.cat(home + packed + src + dst).to(torch.int64).to(dev)
+        small = torch.tensor(list(starts) + shift, dtype=torch.int32).to(dev)
+        self.home_rows, self.packed_rows = big[:T], big[T:2 * T]      # packed_rows int64 [T]
+        self.carry_src = big[2 * T:2 * T + nc] if nc else None        # cache rows of earlier steps ...
+        self.carry_dst = big[2 * T + nc:] if nc else None             # ... and their packed rows
+        self.q_pos0, self.shift = small[:N], small[N:]                # int32 [sequences]; position p is packed row p + shift
+        self.total, self.max_q = at, max(lens)
+
+    def visible(self):
+        """Per token: first row it sees (int64; cache rows in a decode step, else packed rows), number of rows, and its own row among
+        them (int32)."""
+        if self._visible is None:
+            pos = self.plan.positions
+            if self.plan.decode:
+                n = (pos + 1).clamp(max=self.rows)
+                self._visible = (self.row0, n.to(torch.int32), (pos % self.rows).to(torch.int32))
+            else:
+                n = (pos + 1).clamp(max=self.window) if self.window > 0 else pos + 1
+                self._visible = (self.packed_rows - n + 1, n.to(torch.int32), (n - 1).to(torch.int32))
+        return self._visible
 
 
 @dataclass
@@ -242,6 +305,7 @@ class StepPlan:
         self._chunks = None
         self._latent: Optional[LatentPlan] = None
         self._kv: Optional[KVPlan] = None
+        self._windows: Dict[int, WindowPlan] = {}
         self.contexts: Dict[int, torch.Tensor] = {}  # packed rows of the layers that later layers of the step read as well
         if not self.decode:
             cu = [0]
@@ -272,6 +336,11 @@ class StepPlan:
                 small = torch.tensor(ends + list(starts), dtype=torch.int32).to(self.slots.device)
                 self._kv = KVPlan(row0 + self.positions, row0, n, small[:len(lens)], pages, small[len(lens):], max(lens), max(ends))
         return self._kv
+
+    def window(self, spec: WindowKVSpec) -> WindowPlan:
+        if spec.window not in self._windows:
+            self._windows[spec.window] = WindowPlan(self, spec.window, spec.rows(self.cache.max_length))
+        return self._windows[spec.window]
 
     def latent(self) -> LatentPlan:
         if self._latent is None:
@@ -355,7 +424,7 @@ class StepPlan:
 
 
 class HybridCache:
-    """Cache of a layered decoder: one storage per layer run (``KVSpec``, ``TiedKVSpec``, ``LatentSpec``, ``StateSpec``, ``DeltaSpec``, or a
+    """Cache of a layered decoder: one storage per layer run (``KVSpec``, ``WindowKVSpec``, ``TiedKVSpec``, ``LatentSpec``, ``StateSpec``, ``DeltaSpec``, or a
     ``GroupSpec`` of several; ``SharedSpec`` layers share another layer's), indexed by a sequence's slot.
 
     Slots are handed out by ``alloc`` and given back by ``free``; nothing is cleared in between, because a sequence that
@@ -414,6 +483,9 @@ class HybridCache:
             return {"k": ((rows, spec.kv_heads, spec.head_dim), act), "scale": ((rows,), torch.float32)}
         if isinstance(spec, KVSpec):
             return {n: ((M, spec.kv_heads, spec.head_dim), act) for n in ("k", "v")}
+        if isinstance(spec, WindowKVSpec):
+            rows = spec.rows(M)
+            return {"k": ((rows, spec.kv_heads, spec.key_dim), act), "v": ((rows, spec.kv_heads, spec.value_dim), act)}
         state = {"state": ((spec.heads, spec.dk, spec.dv), torch.float32)}
         return {**state, "conv": ((spec.taps, spec.channels), act)} if isinstance(spec, DeltaSpec) else state
 

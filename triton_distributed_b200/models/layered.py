@@ -1,4 +1,4 @@
-"""Common part of the decoders whose configuration lists the layers one by one (Vasolix, Lisenex, Tazitar): loading, execution modes,
+"""Common part of the decoders whose configuration lists the layers one by one (Vasolix, Lisenex, Tazitar, Bagasun): loading, execution modes,
 cache, packed steps, the engine's rectangular interface, random weights by tensor name.
 
 A model is a list of layers with ``parts()`` (tensor-parallel mixers / feed-forwards) and ``load``; a subclass builds them and runs
@@ -87,6 +87,10 @@ class LayeredLLM:
         """Embedding table and output projection."""
         raise NotImplementedError
 
+    def final_norm(self, get) -> torch.Tensor:
+        """fp32 weight of the norm before the output projection."""
+        return pad_rows(get("final.norm").float(), pad8(self.arch.hidden_size)).to(self.device)
+
     def init_parameters(self):
         a, mc = self.arch, self.model_config
         if mc.checkpoint_dir:
@@ -95,7 +99,7 @@ class LayeredLLM:
         else:
             ckpt, get = None, self.random_weights(a, mc.seed, self.device)
         self.load_head(get)
-        self.final_norm_w = pad_rows(get("final.norm").float(), pad8(a.hidden_size)).to(self.device)
+        self.final_norm_w = self.final_norm(get)
         for l in self.layers:
             l.load(get, a.hidden_size, a.rms_norm_eps, self.dtype, self.device)
         if ckpt is not None:

@@ -40,9 +40,12 @@ from .fp8 import (ag_gemm_fp8, dequantize_act_1x128, dequantize_weight_128x128, 
 from .moe import (tile_arrival_order, tile_schedule, sort_topk_ids_staged, group_gemm_gather,  # noqa: F401,E402
                   MoESort, MoEAgScatterGroupGemmContext, MoEReduceRSContext)
 from .stream import (embed_stream, postnorm_add, combine_rows, stream_norm, qk_sumsq, qk_norm_tied, FeedForward,  # noqa: F401,E402
-                     parallel_add, parallel_sum, HyperWeights, SublayerOutput, hyper_step)
-from .rotary import rope_table, YarnScaling, head_prep  # noqa: F401,E402
+                     parallel_add, parallel_sum, HyperWeights, SublayerOutput, hyper_step, sandwich_step)
+from .rotary import rope_table, YarnScaling, BandScaling, head_prep  # noqa: F401,E402
 from .delta import gated_delta_rule, DELTA_MAX_DIM  # noqa: F401,E402
+from .window import (SigmoidWeights, DifferentialWeights, distance_table, qkv_prep, window_attention_simple,  # noqa: F401,E402
+                     window_attention_decode, window_attention_prompt, window_tensor_cores, pick_window_splits, WINDOW_DIMS, WINDOW_MAX_DIM)
+from .ssd import SsdWeights, state_space, gated_group_norm, SSD_MAX_DIM  # noqa: F401,E402
 from .gla import gated_linear_attention, gla_chunk_tables, GLA_CHUNK  # noqa: F401,E402
 from .moe import (narrow_linear, sigmoid_router, softmax_router, relu2, relu2_experts_gemv, gated_experts_gemv,  # noqa: F401,E402
                   EXPERT_GEMV_MAX_T)

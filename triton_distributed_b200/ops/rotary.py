@@ -1,10 +1,10 @@
-"""Rotary positions: tables of cos and sin (optionally with YaRN scaling), and the per-head preparation of queries and keys (norm with
+"""Rotary positions: tables of cos and sin (optionally with scaled frequencies), and the per-head preparation of queries and keys (norm with
 a weight, rotation, norm without one, cache write) in one launch of ``csrc/rotary.cu``.  CPU tensors run the restatement here."""
 from __future__ import annotations
 
 import math
 from dataclasses import dataclass
-from typing import Optional
+from typing import Optional, Union
 
 import torch
 
@@ -41,7 +41,30 @@ class YarnScaling:
         return 0.1 * math.log(self.factor) + 1.0
 
 
-def rope_table(base: float, dims: int, width: int, positions: int, device, scaling: Optional[YarnScaling] = None) -> torch.Tensor:
+@dataclass(frozen=True)
+class BandScaling:
+    """Frequencies whose wavelength is longer than ``original / low`` are divided by ``factor``, those below ``original / high`` are kept;
+    between the two bounds the scaled and the kept frequency are mixed linearly in ``original / wavelength``.  cos and sin keep their size."""
+    factor: float
+    original: float
+    low: float
+    high: float
+    amplitude = 1.0
+
+    @staticmethod
+    def from_json(c: Optional[dict]) -> Optional["BandScaling"]:
+        return BandScaling(*(float(c[n]) for n in ("factor", "original", "low", "high"))) if c else None
+
+    def apply(self, freqs: torch.Tensor, base: float, dims: int) -> torch.Tensor:
+        turns = self.original * freqs / (2 * math.pi)         # within the original length
+        keep = (turns > self.high).to(freqs.dtype)
+        if self.high > self.low:
+            keep = ((turns - self.low) / (self.high - self.low)).clamp(0, 1)
+        return (1 - keep) * freqs / self.factor + keep * freqs
+
+
+def rope_table(base: float, dims: int, width: int, positions: int, device,
+               scaling: Union[YarnScaling, BandScaling, None] = None) -> torch.Tensor:
     """fp32 [positions, width]: cos and sin of ``p * base^(-2 i / dims)`` for pair i at columns (2 i, 2 i + 1), computed in fp64;
     columns from ``dims`` on (padding) are zero.  One table per rotation and device, grown when more positions are needed."""
     key = (float(base), int(dims), int(width), str(device), scaling)

@@ -1,4 +1,4 @@
-"""fp32 residual stream of layered decoders: embedding, ``x += RMSNorm(y) * w`` (norm on a sublayer's output) or ``x += mixer +
+"""fp32 residual stream of layered decoders: embedding, ``x += RMSNorm(y) * w`` (norm on a sublayer's output), sublayers between two norms or ``x += mixer +
 feed-forward`` with the next layer's norms (parallel layers), the norm before the head, and the whole-projection q / k norm that
 writes a tied KV cache.
 
@@ -155,6 +155,30 @@ def hyper_step(x: torch.Tensor, last: Optional[Tuple[HyperWeights, SublayerOutpu
         return None
     u = torch.einsum("s,nsw->nw", nxt[0], v)
     return (u * _rms_factor(u, n_real, eps) * nxt[1]).to(dtype)
+
+
+# ------------------------------------------------------------------ a sublayer between two norms
+def sandwich_step(x: torch.Tensor, last: Optional[Tuple[torch.Tensor, torch.Tensor]], pre: Optional[torch.Tensor], n_real: int, eps: float,
+                  dtype: torch.dtype, rows: Optional[torch.Tensor] = None,
+                  start: Optional[Tuple[torch.Tensor, torch.Tensor, float]] = None) -> Optional[torch.Tensor]:
+    """One pass over the stream ``x`` [T, W] (fp32, in place) between two sublayers: ``x += RMSNorm(y) * post`` with ``last = (y, post)``,
+    then the next one's input ``RMSNorm(x) * pre`` in ``dtype``.  ``post`` and ``pre`` are fp32 weights, one number for all coordinates
+    or one each.  ``start = (ids, table, scale)`` sets x to the tokens' scaled rows first.  With ``rows`` (int64) only these tokens
+    are computed and ``x`` stays as it is."""
+    if _native.use_native(x):
+        ids, table, scale = start if start is not None else (None, None, 1.0)
+        h = _native.load(True).sandwich(x, ids, table, float(scale), *(last if last is not None else (None, None)), pre, rows, int(n_real), float(eps),
+                                        dtype == torch.float32)
+        return h if pre is not None else None
+    if start is not None:
+        x.copy_(start[1][start[0].long()].float() * start[2])
+    v = x if rows is None else x[rows]
+    if last is not None:
+        y = (last[0] if rows is None else last[0][rows]).float()
+        v = v + y * _rms_factor(y, n_real, eps) * last[1]
+        if rows is None:
+            x.copy_(v)
+    return None if pre is None else (v * _rms_factor(v, n_real, eps) * pre).to(dtype)
 
 
 def combine_rows(y: torch.Tensor, T: int, rows_per_token: int, shared: Optional[torch.Tensor] = None,

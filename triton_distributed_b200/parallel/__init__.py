@@ -11,6 +11,8 @@ from .tp_latent_attn import TP_LatentAttn  # noqa: F401
 from .tp_routed_ff import TP_DenseFF, TP_GatedFF, TP_RoutedMoE  # noqa: F401
 from .tp_rotary_attn import TP_RotaryAttn  # noqa: F401
 from .tp_delta import TP_DeltaRule  # noqa: F401
+from .tp_window_attn import TP_DifferentialAttn, TP_SigmoidAttn  # noqa: F401
+from .tp_ssd import TP_StateSpace  # noqa: F401
 from .tp_twin import TP_TwinMixer  # noqa: F401
 from .ep_layer import EPAll2AllLayer, EP_MoE  # noqa: F401
 from .sp_flash_decode import SpGQAFlashDecodeAttention  # noqa: F401
