@@ -13,8 +13,8 @@ Arms:
                     needs the patched Triton submodule, which is empty in the mounted checkout), so this arm
                     prints an "unavailable" line
 
-``--workload hybrid``, ``--workload latent`` and ``--workload streams`` run other measurements instead (see
-benchmarks/bench_hybrid.py, benchmarks/bench_latent.py and benchmarks/bench_streams.py).
+``--workload hybrid``, ``latent``, ``streams`` and ``windows`` run other measurements instead (see
+benchmarks/bench_hybrid.py, bench_latent.py, bench_streams.py and bench_windows.py).
 
 Prints ONE JSON line on rank 0.  Device times come from CUDA events around exactly --steps steps, max over ranks.
 """
@@ -44,11 +44,12 @@ def parse():
     ap.add_argument("--e2e-return", default="metric", choices=["metric", "full"],
                     help="what the host reads back every step: the 4-byte checksum of the output (default), or the "
                          "whole output tensor as well (PCIe-bound at small N: 128 MB per step and direction at N=1)")
-    ap.add_argument("--workload", default="tp_mlp", choices=["tp_mlp", "hybrid", "latent", "streams"],
+    ap.add_argument("--workload", default="tp_mlp", choices=["tp_mlp", "hybrid", "latent", "streams", "windows"],
                     help="tp_mlp: the headline above (default); hybrid: prefill and decode throughput of the layered decoder "
                          "(Vasolix) beside Qwen3-MoE at equal layer sizes, one GPU, one JSON line per measurement; latent: the same "
-                         "for Lisenex beside Vasolix; streams: the same for Tazitar beside Qwen3 (dense)")
-    ap.add_argument("--hybrid-size", default=None, help="sizes of the hybrid / latent (30b-a3b,1b) and streams (8b,1b) workloads; default: all")
+                         "for Lisenex beside Vasolix; streams: the same for Tazitar beside Qwen3 (dense); windows: "
+                         "for Bagasun beside Qwen3 (dense)")
+    ap.add_argument("--hybrid-size", default=None, help="sizes of the hybrid / latent (30b-a3b,1b) and streams / windows (8b,1b) workloads; default: all")
     ap.add_argument("--hybrid-parts", default="prefill,decode,kernels")
     return ap.parse_args()
 
@@ -62,7 +63,7 @@ def reference_unavailable():
 
 def layered_workload(args):
     import triton_distributed_b200 as tdb
-    from benchmarks import bench_hybrid, bench_latent, bench_streams
+    from benchmarks import bench_hybrid, bench_latent, bench_streams, bench_windows
     from triton_distributed_b200.utils import ClockSampler
 
     if args.impl != "ours":
@@ -72,7 +73,7 @@ def layered_workload(args):
     sampler = ClockSampler(gpu_index=tdb.get_runtime().local_rank).start()
     sampler.wait_first_sample(5.0)
     sampler.begin_window()
-    bench = {"hybrid": bench_hybrid, "latent": bench_latent, "streams": bench_streams}[args.workload]
+    bench = {"hybrid": bench_hybrid, "latent": bench_latent, "streams": bench_streams, "windows": bench_windows}[args.workload]
     recs = bench.run(args.hybrid_size.split(",") if args.hybrid_size else list(bench.SIZES), args.hybrid_parts.split(","))
     sampler.end_window()
     for r in recs:

@@ -10,6 +10,11 @@
   python benchmarks/ncu_case.py gla       # chunk-parallel gated linear attention, 8192 tokens x 16 heads, 128 x 128 states
   python benchmarks/ncu_case.py delta     # chunk-parallel gated delta rule with convolutions, 8192 tokens x 16 heads, 128 x 128 states
   python benchmarks/ncu_case.py hyper     # pass over 4 residual streams between two sublayers, 8192 tokens, width 2048
+  python benchmarks/ncu_case.py ssd       # chunk-parallel state space layer with convolutions, 8192 tokens x 64 heads, 128 x 64 states
+  python benchmarks/ncu_case.py sandwich  # sublayer between two norms, 8192 tokens, width 4096
+  python benchmarks/ncu_case.py sigmoid   # sigmoid prompt attention, 8192 tokens, window 4096, 32 heads / 8 kv heads of 128
+  python benchmarks/ncu_case.py differential  # differential prompt attention, 8192 tokens, window 4096, 32 heads / 8 kv heads of 2 x 64 / 128
+  python benchmarks/ncu_case.py window_decode  # sigmoid decode attention over full rings, 64 seqs x 4096 positions, 32 heads / 8 kv heads of 128
   python benchmarks/ncu_case.py tied      # tied-KV block decode attention, 64 seqs x 4096 positions, 32 q heads / 4 kv heads
   python benchmarks/ncu_case.py latent_decode   # latent decode attention, 64 seqs x 4096 tokens, 32 heads, rows of 512 + 64
   python benchmarks/ncu_case.py latent_prefill  # latent prompt attention, 8192 tokens, 8 heads of 128 + 64 / 128
@@ -97,6 +102,38 @@ def main():
         hc = ops.HyperWeights(one / S, one, torch.eye(S, device="cuda"))
         for _ in range(3):
             ops.hyper_step(x, (hc, ops.SublayerOutput(y)), (hc.inp, torch.ones(W, device="cuda")), W, 1e-5, torch.bfloat16)
+    elif case == "ssd":
+        T, H, G, N, dv, taps = 8192, 64, 8, 128, 64, 4
+        C = H * dv + 2 * G * N
+        z = torch.randn(T, C + H, device="cuda", dtype=torch.bfloat16)
+        w = ops.SsdWeights(torch.randn(C, taps, device="cuda"), torch.randn(C, device="cuda"), torch.zeros(H, device="cuda"), torch.full((H,), -2.0, device="cuda"),
+                           torch.ones(H, device="cuda"))
+        state, ring = torch.zeros(1, H, N, dv, device="cuda"), torch.zeros(1, taps, C, device="cuda", dtype=torch.bfloat16)
+        slot, pos0 = torch.zeros(1, dtype=torch.int32, device="cuda"), torch.zeros(1, dtype=torch.int64, device="cuda")
+        cu = torch.tensor([0, T], dtype=torch.int32, device="cuda")
+        tabs = ops.gla_chunk_tables([0, T], "cuda")
+        for _ in range(2):
+            ops.state_space(z, C, w, state, ring, slot, pos0, cu, G, tabs)
+    elif case == "sandwich":
+        T, W = 8192, 4096
+        x, y, one = torch.randn(T, W, device="cuda"), torch.randn(T, W, device="cuda", dtype=torch.bfloat16), torch.ones(1, device="cuda")
+        for _ in range(3):
+            ops.sandwich_step(x, (y, one), one, W, 1e-5, torch.bfloat16)
+    elif case in ("sigmoid", "differential", "window_decode"):
+        T, H, G, window = (64 if case == "window_decode" else 8192), 32, 8, 4096
+        m, dk, dv = (2, 64, 128) if case == "differential" else (1, 128, 128)
+        w = ops.DifferentialWeights(0.6, 0.5, 1e-5, dv)
+        if m == 1:
+            w = ops.SigmoidWeights(ops.distance_table(torch.full((H,), 0.3), torch.full((H,), 0.5), torch.full((H,), -3.0), window).cuda())
+        rows = (T, window) if case == "window_decode" else (T,)
+        q, k, v = (torch.randn(*s, device="cuda", dtype=torch.bfloat16) for s in ((T, H * m, dk), (*rows, G * m, dk), (*rows, G, dv)))
+        i32 = lambda *v: torch.tensor(v, dtype=torch.int32, device="cuda")   # noqa: E731
+        for _ in range(3):
+            if case == "window_decode":
+                ops.window_attention_decode(q, k, v, w, dk ** -0.5, None, i32(*range(T)), torch.full((T,), 3 * window, dtype=torch.int64, device="cuda"))
+            else:
+                ops.window_attention_prompt(q, k, v, w, dk ** -0.5, None, i32(0, T), i32(0), i32(0), T, window)
+        ops.check_attention_errors()
     elif case == "tied":
         B, Hq, Hkv, D, L = 64, 32, 4, 128, 4096
         k = torch.randn(B, L, Hkv, D, device="cuda", dtype=torch.bfloat16)

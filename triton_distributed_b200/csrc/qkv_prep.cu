@@ -80,18 +80,34 @@ __global__ void qkv_prep_kernel(const QkvPrepArgs p) {
     }
     const int d0 = cw % p.dk;
     if (d0 < p.rot) {
+      auto turn = [&](int i, float other, int pair, bool second) {
+        const float co = cs[2 * pair], si = cs[2 * pair + 1];
+        f[i] = second ? f[i] * co + other * si : f[i] * co - other * si;
+      };
+      if (half % 8 == 0) {                        // the eight partners are neighbours as well
+        const bool second = d0 >= half;
+        const int off = second ? -half : half;
+        float o[8];
+        load_biased(z + c + off, p.bias != nullptr ? p.bias + c + off : nullptr, o);
+        if (w != nullptr) {
+          float g[8];
+          load8(w + cw + off, g);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        const int d = d0 + i;
-        if (d < p.rot) {
+          for (int i = 0; i < 8; ++i) o[i] *= n * g[i];
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) turn(i, o[i], d0 + i - (second ? half : 0), second);
+      } else {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const int d = d0 + i;
+          if (d >= p.rot) continue;
           const bool second = d >= half;
           const int off = second ? -half : half;
           float other = to_f32(z[c + i + off]);
           if (p.bias != nullptr) other += p.bias[c + i + off];
           if (w != nullptr) other *= n * w[cw + i + off];
-          const int pair = second ? d - half : d;
-          const float co = cs[2 * pair], si = cs[2 * pair + 1];
-          f[i] = second ? f[i] * co + other * si : f[i] * co - other * si;
+          turn(i, other, second ? d - half : d, second);
         }
       }
     }

@@ -111,9 +111,24 @@ __global__ void __launch_bounds__(kDecThreads) ssd_decode_kernel(const SsdArgs p
 // ---------------------------------------------------------------------------------------------------- inputs of prompts
 constexpr int kPrepTok = 32;      // tokens per CTA
 constexpr int kPrepThreads = 128;
-constexpr int kBatch = 4;         // tokens whose inputs are requested together
+constexpr int kBatch = 8;         // tokens whose inputs are requested together
+constexpr int kV = 4;             // channels of a thread
 
-// A thread owns eight channels.  TAPS > 0: convolutions of at most TAPS taps, weights and the last inputs in registers; 0: any number.
+TDB_DEVICE void load_v(const __nv_bfloat16* p, float (&f)[kV]) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y);
+  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+}
+TDB_DEVICE void load_v(const float* p, float (&f)[kV]) {
+  const float4 v = *reinterpret_cast<const float4*>(p);
+  f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+}
+TDB_DEVICE void store_v(__nv_bfloat16* p, const float (&f)[kV]) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
+}
+TDB_DEVICE void store_v(float* p, const float (&f)[kV]) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+
+// A thread owns kV channels.  TAPS > 0: convolutions of at most TAPS taps, weights and the last inputs in registers; 0: any number.
 // The last row of blocks takes the step sizes and decays.
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(kPrepThreads) ssd_prepare_kernel(const SsdArgs p) {
@@ -136,34 +151,34 @@ __global__ void __launch_bounds__(kPrepThreads) ssd_prepare_kernel(const SsdArgs
     return;
   }
   const int64_t t0 = c0 + blockIdx.z * kPrepTok, t1 = min(t0 + kPrepTok, end), before = p.pos0[n] - begin;
-  const int c = (blockIdx.y * kPrepThreads + threadIdx.x) * 8;
+  const int c = (blockIdx.y * kPrepThreads + threadIdx.x) * kV;
   if (t0 >= t1 || c >= C) return;
   const T* z = reinterpret_cast<const T*>(p.z);
   const T* ring = reinterpret_cast<const T*>(p.conv) + static_cast<int64_t>(p.slots[n]) * p.taps * C;
-  auto input = [&](int64_t t, float (&f)[8]) {           // of (packed) token t, zero before the sequence
+  auto input = [&](int64_t t, float (&f)[kV]) {           // of (packed) token t, zero before the sequence
     const int64_t pos = before + t;
     if (t >= begin) {
-      load8(z + t * p.ld + c, f);
+      load_v(z + t * p.ld + c, f);
     } else if (pos >= 0) {
-      load8(ring + (pos % p.taps) * C + c, f);
+      load_v(ring + (pos % p.taps) * C + c, f);
     } else {
 #pragma unroll
-      for (int i = 0; i < 8; ++i) f[i] = 0.f;
+      for (int i = 0; i < kV; ++i) f[i] = 0.f;
     }
   };
-  float bias[8];
-  load8(p.conv_b + c, bias);
-  auto finish = [&](int64_t t, float (&acc)[8]) {
+  float bias[kV];
+  load_v(p.conv_b + c, bias);
+  auto finish = [&](int64_t t, float (&acc)[kV]) {
 #pragma unroll
-    for (int i = 0; i < 8; ++i) acc[i] = __fdividef(acc[i], 1.f + __expf(-acc[i]));
-    store8(reinterpret_cast<T*>(p.xbc) + t * C + c, acc);
+    for (int i = 0; i < kV; ++i) acc[i] = __fdividef(acc[i], 1.f + __expf(-acc[i]));
+    store_v(reinterpret_cast<T*>(p.xbc) + t * C + c, acc);
   };
   if constexpr (TAPS > 0) {
-    float w[TAPS][8], x[TAPS + kBatch - 1][8];           // x[j]: input of token (first of the batch) + kBatch - 1 - j
+    float w[TAPS][kV], x[TAPS + kBatch - 1][kV];           // x[j]: input of token (first of the batch) + kBatch - 1 - j
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) {
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
+      for (int i = 0; i < kV; ++i) {
         w[j][i] = j < p.taps ? p.conv_w[static_cast<int64_t>(c + i) * p.taps + p.taps - 1 - j] : 0.f;
         x[j][i] = 0.f;
       }
@@ -173,40 +188,40 @@ __global__ void __launch_bounds__(kPrepThreads) ssd_prepare_kernel(const SsdArgs
 #pragma unroll
       for (int j = TAPS - 2; j >= 0; --j)
 #pragma unroll
-        for (int i = 0; i < 8; ++i) x[j + kBatch][i] = x[j][i];
+        for (int i = 0; i < kV; ++i) x[j + kBatch][i] = x[j][i];
 #pragma unroll
       for (int j = 0; j < kBatch; ++j) {
         if (b + j < t1) {
-          load8(z + (b + j) * p.ld + c, x[kBatch - 1 - j]);
+          load_v(z + (b + j) * p.ld + c, x[kBatch - 1 - j]);
         } else {
 #pragma unroll
-          for (int i = 0; i < 8; ++i) x[kBatch - 1 - j][i] = 0.f;
+          for (int i = 0; i < kV; ++i) x[kBatch - 1 - j][i] = 0.f;
         }
       }
 #pragma unroll
       for (int k = 0; k < kBatch; ++k) {
         if (b + k >= t1) break;
-        float acc[8];
+        float acc[kV];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) acc[i] = bias[i];
+        for (int i = 0; i < kV; ++i) acc[i] = bias[i];
 #pragma unroll
         for (int j = 0; j < TAPS; ++j)
 #pragma unroll
-          for (int i = 0; i < 8; ++i) acc[i] = fmaf(w[j][i], x[kBatch - 1 - k + j][i], acc[i]);
+          for (int i = 0; i < kV; ++i) acc[i] = fmaf(w[j][i], x[kBatch - 1 - k + j][i], acc[i]);
         finish(b + k, acc);
       }
     }
   } else {
     for (int64_t t = t0; t < t1; ++t) {
-      float acc[8];
+      float acc[kV];
 #pragma unroll
-      for (int i = 0; i < 8; ++i) acc[i] = bias[i];
+      for (int i = 0; i < kV; ++i) acc[i] = bias[i];
       for (int j = 0; j < p.taps; ++j) {
-        float f[8];
+        float f[kV];
         input(t - j, f);
         const float* wj = p.conv_w + static_cast<int64_t>(c) * p.taps + p.taps - 1 - j;
 #pragma unroll
-        for (int i = 0; i < 8; ++i) acc[i] = fmaf(wj[i * p.taps], f[i], acc[i]);
+        for (int i = 0; i < kV; ++i) acc[i] = fmaf(wj[i * p.taps], f[i], acc[i]);
       }
       finish(t, acc);
     }
@@ -215,7 +230,7 @@ __global__ void __launch_bounds__(kPrepThreads) ssd_prepare_kernel(const SsdArgs
 
 template <typename T>
 cudaError_t launch_prepare(const SsdArgs& a, cudaStream_t s) {
-  const dim3 grid(a.NC, (ssd_channels(a) / 8 + kPrepThreads - 1) / kPrepThreads + 1, 64 / kPrepTok), block(kPrepThreads);
+  const dim3 grid(a.NC, (ssd_channels(a) / kV + kPrepThreads - 1) / kPrepThreads + 1, 64 / kPrepTok), block(kPrepThreads);
   return a.taps <= 2   ? launch_pdl(ssd_prepare_kernel<T, 2>, grid, block, 0, s, a)
          : a.taps <= 4 ? launch_pdl(ssd_prepare_kernel<T, 4>, grid, block, 0, s, a)
                        : launch_pdl(ssd_prepare_kernel<T, 0>, grid, block, 0, s, a);

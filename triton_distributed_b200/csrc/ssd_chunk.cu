@@ -11,9 +11,9 @@
 // Contributions and states are stored tile by tile in the order in which the lanes of a warp hold the B fragments of m16n8k16, as in
 // gla_chunk.cu: the scan turns each value into its bf16 high and low part, the output kernel loads ready fragments.
 //
-// Exponentials are of differences that cannot be positive.  The decay being one number per token and head, it multiplies rows of x, of the
-// scores and of the first product's result, so B, C and x enter the tensor cores as the bf16 numbers they are; what counts as fp32
-// (states, scaled x, scaled scores) enters as a high and a low part: two products each.
+// Exponentials are of differences that cannot be positive.  The decay being one number per token and head, it multiplies B, the scores and
+// rows of the first product's result, so C and x enter the tensor cores as the bf16 numbers they are; what counts as fp32 (states, scaled
+// B, scaled scores) enters as a high and a low part: two products each.
 #include "tdb/attn_device.cuh"
 #include "tdb/chunk.cuh"
 #include "tdb/launch.cuh"
@@ -41,15 +41,14 @@ constexpr int kThreads = 256;
 __host__ __device__ __forceinline__ int channels(const SsdArgs& p) { return p.H * p.dv + 2 * p.G * p.dk; }
 
 // ---------------------------------------------------------------------------------------------------- contributions
-size_t inject_smem(int dk, int dv) { return static_cast<size_t>(kC) * (dk + 8) * 2 + 2 * static_cast<size_t>(kC) * (dv + 8) * 2 + kC * 4; }
+size_t inject_smem(int dk, int dv) { return static_cast<size_t>(kC) * (dk + 8) * 2 + 2 * (static_cast<size_t>(kC) * (dv + 8) * 2 + kC * 4); }
 
 __global__ void __launch_bounds__(kThreads) inject_kernel(const SsdArgs p, int heads) {
   extern __shared__ __align__(16) uint8_t smem[];
   const int kp = p.dk + 8, vp = p.dv + 8;
   __nv_bfloat16* bs = reinterpret_cast<__nv_bfloat16*>(smem);     // [64][kp]
-  __nv_bfloat16* xh = bs + kC * kp;                               // [64][vp] inputs, then their scaled high parts in place
-  __nv_bfloat16* xl = xh + kC * vp;
-  float* f = reinterpret_cast<float*>(xl + kC * vp);              // [64] factor of a token
+  __nv_bfloat16* xs = bs + kC * kp;                               // [2][64][vp] inputs of this head and the next
+  float* fs = reinterpret_cast<float*>(xs + 2 * kC * vp);         // [2][64] factors of the tokens
   const int chunk = blockIdx.x, h0 = blockIdx.y * heads, g = h0 / (p.H / p.G);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_wait();
@@ -58,28 +57,27 @@ __global__ void __launch_bounds__(kThreads) inject_kernel(const SsdArgs p, int h
   const int C = channels(p), Hv = p.H * p.dv;
   const __nv_bfloat16* base = reinterpret_cast<const __nv_bfloat16*>(p.xbc) + cp.t0 * C;
   chunk::load_tile(bs, kp, base + Hv + g * p.dk, C, p.dk, cp.n, kThreads);
-  const int nb = (p.dv + 63) / 64, units = (p.dk / 16) * nb;
-  const int mat = lane >> 3, mr = lane & 7, gr = lane >> 2, t4 = lane & 3;
-  for (int h = h0; h < h0 + heads; ++h) {
-    chunk::load_tile(xh, vp, base + h * p.dv, C, p.dv, cp.n, kThreads);
+  auto load_head = [&](int h) {
+    const int s = (h - h0) & 1;
+    chunk::load_tile(xs + s * kC * vp, vp, base + h * p.dv, C, p.dv, cp.n, kThreads);
+    cp_async_commit();
     if (threadIdx.x < kC) {
       const int64_t at = cp.t0 * p.H + h;
       const float last = p.log_g[at + static_cast<int64_t>(cp.n - 1) * p.H];
       const int64_t mine = at + static_cast<int64_t>(min(static_cast<int>(threadIdx.x), cp.n - 1)) * p.H;
-      f[threadIdx.x] = static_cast<int>(threadIdx.x) < cp.n ? __expf(last - p.log_g[mine]) * p.dt[mine] : 0.f;
+      fs[s * kC + threadIdx.x] = static_cast<int>(threadIdx.x) < cp.n ? __expf(last - p.log_g[mine]) * p.dt[mine] : 0.f;
     }
-    cp_async_commit();
+  };
+  load_head(h0);
+  const int nb = (p.dv + 63) / 64, units = (p.dk / 16) * nb;
+  const int mat = lane >> 3, mr = lane & 7, gr = lane >> 2, t4 = lane & 3;
+  for (int h = h0; h < h0 + heads; ++h) {
     cp_async_wait<0>();
     __syncthreads();
-    for (int i = threadIdx.x; i < kC * (p.dv / 2); i += kThreads) {
-      const int t = i / (p.dv / 2), c = (i - t * (p.dv / 2)) * 2;
-      const float2 x = ld2(xh + t * vp + c);
-      const HiLo s = split2(x.x * f[t], x.y * f[t]);
-      *reinterpret_cast<uint32_t*>(xh + t * vp + c) = s.hi;
-      *reinterpret_cast<uint32_t*>(xl + t * vp + c) = s.lo;
-    }
-    __syncthreads();
-    // units of 16 rows x 64 columns of the state; A = B^T (read transposed)
+    if (h + 1 < h0 + heads) load_head(h + 1);      // into the buffers that were read before the barrier
+    const __nv_bfloat16* x = xs + ((h - h0) & 1) * kC * vp;
+    const float* f = fs + ((h - h0) & 1) * kC;
+    // units of 16 rows x 64 columns of the state; A = B^T (read transposed), scaled by the tokens' factors and cut into two parts
     float4* out = reinterpret_cast<float4*>(p.inject) + (static_cast<int64_t>(chunk) * p.H + h) * p.dk * (p.dv / 4);
     for (int u = warp; u < units; u += kThreads / 32) {
       const int c0 = (u / nb) * 16, n0 = (u % nb) * 64;
@@ -88,19 +86,25 @@ __global__ void __launch_bounds__(kThreads) inject_kernel(const SsdArgs p, int h
       for (int i = 0; i < 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
 #pragma unroll
       for (int ks = 0; ks < kC / 16; ++ks) {
-        uint32_t a[4];
+        uint32_t a[4], ah[4], al[4];
         ldmatrix_x4_trans(a, bs + (ks * 16 + (mat >> 1) * 8 + mr) * kp + c0 + (mat & 1) * 8);
+        const float2 f0 = *reinterpret_cast<const float2*>(f + ks * 16 + 2 * t4), f1 = *reinterpret_cast<const float2*>(f + ks * 16 + 8 + 2 * t4);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float2 b = unpack_bf16x2(a[i]);
+          const HiLo v = split2(b.x * (i < 2 ? f0.x : f1.x), b.y * (i < 2 ? f0.y : f1.y));
+          ah[i] = v.hi;
+          al[i] = v.lo;
+        }
 #pragma unroll
         for (int j = 0; j < 8; j += 2) {
           if (n0 + j * 8 >= p.dv) break;
-          uint32_t vh[4], vl[4];
-          const int at = (ks * 16 + (mat & 1) * 8 + mr) * vp + n0 + j * 8 + (mat >> 1) * 8;
-          ldmatrix_x4_trans(vh, xh + at);
-          ldmatrix_x4_trans(vl, xl + at);
-          mma_bf16(acc[j], a, vh[0], vh[1]);
-          mma_bf16(acc[j], a, vl[0], vl[1]);
-          mma_bf16(acc[j + 1], a, vh[2], vh[3]);
-          mma_bf16(acc[j + 1], a, vl[2], vl[3]);
+          uint32_t v[4];
+          ldmatrix_x4_trans(v, x + (ks * 16 + (mat & 1) * 8 + mr) * vp + n0 + j * 8 + (mat >> 1) * 8);
+          mma_bf16(acc[j], ah, v[0], v[1]);
+          mma_bf16(acc[j], al, v[0], v[1]);
+          mma_bf16(acc[j + 1], ah, v[2], v[3]);
+          mma_bf16(acc[j + 1], al, v[2], v[3]);
         }
       }
       // accumulator layout (row g, columns 2t, 2t + 1; row g + 8) -> B-fragment layout (rows 2t, 2t + 1, + 8; column g)
@@ -120,7 +124,6 @@ __global__ void __launch_bounds__(kThreads) inject_kernel(const SsdArgs p, int h
         out[((c0 / 16) * (p.dv / 8) + n0 / 8 + j) * 32 + lane] = v;
       }
     }
-    __syncthreads();                                // the next head's inputs overwrite these
   }
 }
 

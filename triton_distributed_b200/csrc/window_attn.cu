@@ -180,14 +180,26 @@ __global__ void __launch_bounds__(kAttnThreads) window_decode_kernel(const Windo
     if (j < nblk) load(j);
     cp_async_commit();
   }
+  const bool upper = group - hc * kHeads > 8;            // rows 8-15 hold heads (sigmoid form)
   for (int i = 0; i < nblk; ++i) {
     if (i + S - 1 < nblk) load(i + S - 1);
     cp_async_commit();
+    const int tb = warp * 16, t0 = (blk0 + i) * kBlockN + tb;      // each warp takes 16 of the 64 tokens
+    float bias[2][4];                                    // on its way while the block arrives
+    if constexpr (!kSoft) {
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int tok = t0 + 8 * j + c2 + (e & 1);
+          const int dist = newest - tok + (newest < tok ? p.ring : 0);
+          bias[j][e] = tok < n && (e < 2 || upper) ? __ldg((e < 2 ? bias_lo : bias_hi) + min(static_cast<int64_t>(dist), p.bias_n - 1)) : 0.f;
+        }
+    }
     cp_async_wait<S - 1>();
     __syncthreads();
     const uint8_t* sk = smem + (i % S) * L::kStage;
     const uint8_t* sv = sk + L::kK;
-    const int tb = warp * 16, t0 = (blk0 + i) * kBlockN + tb;      // each warp takes 16 of the 64 tokens
     float s[2][4];
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
@@ -231,10 +243,8 @@ __global__ void __launch_bounds__(kAttnThreads) window_decode_kernel(const Windo
       for (int j = 0; j < 2; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int tok = t0 + 8 * j + c2 + (e & 1);
-          const int dist = newest - tok + (newest < tok ? p.ring : 0);
-          const float y = fmaf(s[j][e], p.scale, tok < n ? __ldg((e < 2 ? bias_lo : bias_hi) + min(static_cast<int64_t>(dist), p.bias_n - 1)) : 0.f);
-          s[j][e] = tok < n ? __fdividef(1.f, 1.f + exp2f(fminf(-y * kLog2e, 100.f))) : 0.f;
+          const float y = fmaf(s[j][e], p.scale, bias[j][e]);
+          s[j][e] = t0 + 8 * j + c2 + (e & 1) < n && (e < 2 || upper) ? __fdividef(1.f, 1.f + exp2f(fminf(-y * kLog2e, 100.f))) : 0.f;
         }
     }
     uint32_t pa[4];

@@ -176,8 +176,8 @@ def sandwich_stack(name: str, vocab: int, width: int, pattern: str, attention: S
 BAGASUN_PRESETS = {
     # layers of the size of Qwen3-8B's (width, heads, feed-forward)
     "bagasun-8b": sandwich_stack("bagasun-8b", 151936, 4096, "MDMA" * 9, SigmoidAttnSpec(32, 8, 128, 128, 128 ** -0.5, 4096),
-                                 DifferentialAttnSpec(32, 8, 64, 128, 0.125, 0.6, 5e5, 64, ops.BandScaling(4.0, 8192, 1.0, 4.0), 4096),
-                                 StateSpaceSpec(128, 8, 128, 64, 4, 8), 12288, embed_scale=12.0),
+                                 DifferentialAttnSpec(32, 8, 64, 128, 0.125, 0.8, 1e6, 64, ops.BandScaling(4.0, 8192, 1.0, 4.0), 4096),
+                                 StateSpaceSpec(128, 8, 128, 64, 4, 8), 12288),
     "bagasun-1b": sandwich_stack("bagasun-1b", 65536, 1536, "MDMA" * 3, SigmoidAttnSpec(24, 4, 64, 64, 0.125, 1024),
                                  DifferentialAttnSpec(12, 4, 64, 128, 0.125, 0.5, 1e5, 32, ops.BandScaling(8.0, 4096, 1.0, 4.0), 1024),
                                  StateSpaceSpec(48, 1, 128, 64, 4, 1), 4096, repeats=2, embed_scale=8.0),

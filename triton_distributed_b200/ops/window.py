@@ -131,11 +131,14 @@ def window_tensor_cores(q: torch.Tensor, v: torch.Tensor, scale: float) -> bool:
 
 
 def pick_window_splits(batch: int, units: int, rows: int, num_sms: int = 148) -> int:
-    """KV splits of :func:`window_attention_decode`; ``units``: CTAs per sequence and split.  As in ``pick_kv_splits``: about sqrt(8 x blocks)
-    while all CTAs are resident, two per SM."""
-    blocks = max(1, (rows + 63) // 64)
-    one_wave = max(1, (2 * num_sms) // max(1, batch * units))
-    return int(max(1, min(math.ceil(math.sqrt(8.0 * blocks)), one_wave, blocks, 64)))
+    """KV splits of :func:`window_attention_decode`; ``units``: CTAs per sequence and split.  The number of 64-token blocks that one CTA slot
+    of the device walks (three CTAs per SM, as many waves as it takes) plus what the merge of a split costs, in blocks; at most 32."""
+    blocks, ctas = max(1, (rows + 63) // 64), max(1, batch * units)
+
+    def cost(splits):
+        return math.ceil(splits * ctas / (3 * num_sms)) * math.ceil(blocks / splits) + 0.15 * splits
+
+    return min(range(1, min(blocks, 32) + 1), key=cost)
 
 
 def window_attention_decode(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, weights: Weights, scale: float, gate: Optional[torch.Tensor],
