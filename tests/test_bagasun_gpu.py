@@ -229,16 +229,20 @@ def test_window_decode(rt, kind, H, G, dk, dv, R):
     close(ops.window_attention_simple(f(qd), f(kd), f(vd), h.weights(), scale, f(wide), *seen), want, torch.float32)
 
 
+# (lengths, start positions) of the portions of a step
+STEPS = [([150], [0]), ([300, 1], [0, 0]), ([1, 130, 64, 257], [0, 0, 0, 0]), ([2, 140, 7, 1], [63, 500, 210, 0])]
+# every window with every step for the largest heads, some of them for the other sizes
+PROMPTS = [(SHAPES[-1], w, s) for w in (0, 1, 2, 63, 65, 129, 200, 700) for s in STEPS] + \
+    [(shape, w, s) for shape in SHAPES[:-1] for w in (0, 1, 65, 129, 700) for s in STEPS if len(s[0]) != 2]
+
+
 @pytest.mark.parametrize("kind", KINDS)
-@pytest.mark.parametrize("H,G,dk,dv", SHAPES)
-@pytest.mark.parametrize("window", [0, 1, 2, 63, 65, 129, 200, 700])
-@pytest.mark.parametrize("lens,starts", [([150], [0]), ([300, 1], [0, 0]), ([1, 130, 64, 257], [0, 0, 0, 0]), ([2, 140, 7, 1], [63, 500, 210, 0])])
-def test_window_prompts(rt, kind, H, G, dk, dv, window, lens, starts):
+@pytest.mark.parametrize("shape,window,step", PROMPTS)
+def test_window_prompts(rt, kind, shape, window, step):
     """Prompts and portions of prompts; keys just inside and outside the window of some queries, at block and tile edges stand out."""
     from triton_distributed_b200 import ops
 
-    if (H, G, dk, dv) != SHAPES[-1] and (window in (2, 63, 200) or len(lens) == 2):
-        pytest.skip("covered by the other shapes")
+    (H, G, dk, dv), (lens, starts) = shape, step
     dt, T = torch.bfloat16, sum(lens)
     h = Heads(kind, H, dv, 3, window or 1000)
     m, scale, share = h.maps, h.scale(dk), H // G

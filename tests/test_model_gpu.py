@@ -17,8 +17,8 @@ def test_backends_agree_and_graph_replays(rt):
     from triton_distributed_b200.models import Engine, ModelConfig
 
     cfg = ModelConfig(model_name="tiny-dense", max_length=128, rank=rt.rank, world_size=rt.world_size)
-    ids = torch.randint(0, 1000, (4, 17), device=rt.device)
-    ref = None
+    ids = torch.randint(0, 1000, (4, 17), generator=torch.Generator().manual_seed(0)).to(rt.device)
+    ref = ref_toks = None
     for backend, graph in [("torch", False), ("triton_dist_AR", False), ("triton_dist_gemm_ar", True),
                            ("triton_dist", True)]:
         eng = Engine(cfg)
@@ -28,10 +28,13 @@ def test_backends_agree_and_graph_replays(rt):
         logits = eng._logits.float().clone()
         assert toks.shape == (4, 6)
         if ref is None:
-            ref = logits
+            ref, ref_toks = logits, toks
         else:
             # bf16 model, different kernels: logits agree to bf16 accuracy
-            assert (logits - ref).abs().max().item() < 0.15 * ref.abs().max().item() + 0.05, backend
+            # (of the sequences that continued alike: a near tie may pick another token, and the rest follows from it)
+            same = (toks[:, :-1] == ref_toks[:, :-1]).all(dim=1)
+            assert int(same.sum()) >= 3, backend
+            assert (logits - ref)[same].abs().max().item() < 0.15 * ref.abs().max().item() + 0.05, backend
 
 
 def test_smoke_entry(rt):

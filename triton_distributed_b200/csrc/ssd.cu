@@ -21,6 +21,18 @@ namespace {
 
 TDB_DEVICE float softplus_f32(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 TDB_DEVICE float silu_f32(float z) { return z * sigmoid_f32(z); }
+// silu of an activation of type T: to fp32 accuracy where that is what comes out.
+template <typename T>
+TDB_DEVICE float silu_act(float z) {
+  if constexpr (sizeof(T) == 4) return silu_f32(z);
+  else return __fdividef(z, 1.f + __expf(-z));
+}
+// exp(-exp(a_log) dt).  An error of the rate counts once per token for as long as the state lives, so the 32-bit path rounds once, at the end.
+template <typename T>
+TDB_DEVICE float decay_of(float a_log, float dt) {
+  if constexpr (sizeof(T) == 4) return static_cast<float>(exp(-exp(static_cast<double>(a_log)) * dt));
+  else return expf(-expf(a_log) * dt);
+}
 __host__ __device__ __forceinline__ int ssd_channels(const SsdArgs& p) { return p.H * p.dv + 2 * p.G * p.dk; }
 template <typename T>
 TDB_DEVICE float step_size(const SsdArgs& p, int64_t t, int h) {
@@ -70,7 +82,7 @@ __global__ void __launch_bounds__(kDecThreads) ssd_decode_kernel(const SsdArgs p
   const T* zrow = reinterpret_cast<const T*>(p.z) + n * p.ld;
   T* ring = reinterpret_cast<T*>(p.conv) + slot * p.taps * C;
   T* keep = ring + (pos % p.taps) * C;
-  const float dt = step_size<T>(p, n, h), decay = expf(-expf(p.a_log[h]) * dt);
+  const float dt = step_size<T>(p, n, h), decay = decay_of<T>(p.a_log[h], dt);
   for (int i = threadIdx.x; i < 2 * p.dk + p.dv; i += kDecThreads) {
     const bool is_x = i >= 2 * p.dk;
     const int c = is_x ? h * p.dv + i - 2 * p.dk : Hv + (i < p.dk ? g * p.dk + i : Gk + g * p.dk + i - p.dk);
@@ -170,7 +182,7 @@ __global__ void __launch_bounds__(kPrepThreads) ssd_prepare_kernel(const SsdArgs
   load_v(p.conv_b + c, bias);
   auto finish = [&](int64_t t, float (&acc)[kV]) {
 #pragma unroll
-    for (int i = 0; i < kV; ++i) acc[i] = __fdividef(acc[i], 1.f + __expf(-acc[i]));
+    for (int i = 0; i < kV; ++i) acc[i] = silu_act<T>(acc[i]);
     store_v(reinterpret_cast<T*>(p.xbc) + t * C + c, acc);
   };
   if constexpr (TAPS > 0) {
@@ -272,7 +284,7 @@ __global__ void __launch_bounds__(4 * kRecCols) ssd_recurrent_kernel(const SsdAr
   const int g = h / (p.H / p.G), Hv = p.H * p.dv, Gk = p.G * p.dk, C = ssd_channels(p);
   const int64_t tb = p.cu[n], te = p.cu[n + 1];
   const bool col_ok = v0 + col < p.dv, fresh = p.pos0[n] == 0;
-  const float rate = -expf(p.a_log[h]), skip = p.skip[h];
+  const float a_log = p.a_log[h], skip = p.skip[h];
   const T* xbc = reinterpret_cast<const T*>(p.xbc);
   float* st = p.state + ((static_cast<int64_t>(p.slots[n]) * p.H + h) * p.dk) * p.dv + v0 + col;
   float S[KP];
@@ -297,7 +309,7 @@ __global__ void __launch_bounds__(4 * kRecCols) ssd_recurrent_kernel(const SsdAr
     if (threadIdx.x < nt) {
       const float dt = p.dt[(t0 + threadIdx.x) * p.H + h];
       s_d[threadIdx.x] = dt;
-      s_g[threadIdx.x] = expf(rate * dt);
+      s_g[threadIdx.x] = decay_of<T>(a_log, dt);
     }
     __syncthreads();
     for (int j = 0; j < nt; ++j) {
@@ -359,7 +371,7 @@ __global__ void __launch_bounds__(512) gated_norm_kernel(const GatedNormArgs p) 
       load8(gate + part * size + e, g);
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
-        f[k][i] *= __fdividef(g[i], 1.f + __expf(-g[i]));
+        f[k][i] *= silu_act<T>(g[i]);
         ss += f[k][i] * f[k][i];
       }
     }
@@ -378,7 +390,7 @@ __global__ void __launch_bounds__(512) gated_norm_kernel(const GatedNormArgs p) 
     auto at = [&](int e) { return (e / p.dv_real) * p.dv + e % p.dv_real; };
     auto gated = [&](int c) {
       const float g = to_f32(gate[c]);
-      return to_f32(y[c]) * g * sigmoid_f32(g);
+      return to_f32(y[c]) * silu_f32(g);
     };
     for (int e = threadIdx.x; e < size; e += blockDim.x) {
       const float f = gated(at(part * size + e));

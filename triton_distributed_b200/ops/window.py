@@ -131,12 +131,13 @@ def window_tensor_cores(q: torch.Tensor, v: torch.Tensor, scale: float) -> bool:
 
 
 def pick_window_splits(batch: int, units: int, rows: int, num_sms: int = 148) -> int:
-    """KV splits of :func:`window_attention_decode`; ``units``: CTAs per sequence and split.  The number of 64-token blocks that one CTA slot
-    of the device walks (three CTAs per SM, as many waves as it takes) plus what the merge of a split costs, in blocks; at most 32."""
+    """KV splits of :func:`window_attention_decode`; ``units``: CTAs per sequence and split.  Makes the longest way of a CTA slot short, in
+    64-token blocks: waves of three CTAs per SM, each with its blocks and what starting and merging cost (about one and a half blocks per
+    CTA, and a little per split); at most 32."""
     blocks, ctas = max(1, (rows + 63) // 64), max(1, batch * units)
 
     def cost(splits):
-        return math.ceil(splits * ctas / (3 * num_sms)) * math.ceil(blocks / splits) + 0.15 * splits
+        return math.ceil(splits * ctas / (3 * num_sms)) * (math.ceil(blocks / splits) + 1.5) + 0.15 * splits
 
     return min(range(1, min(blocks, 32) + 1), key=cost)
 
